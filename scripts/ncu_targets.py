@@ -1,6 +1,6 @@
 """Launch each hot kernel a few times so that `ncu --set full -k regex:<name> -s 3 -c 1` can capture it in isolation.
 
-    ncu --set full --clock-control none --import-source on -k regex:gemm_fp8_kernel -s 3 -c 1 -o gpurun_out/ncu_fp8 \
+    ncu --set full --clock-control none -k regex:gemm_fp8_kernel -s 3 -c 1 -o gpurun_out/ncu_fp8 \
         python scripts/ncu_targets.py fp8
 """
 import sys
