@@ -6,7 +6,9 @@ Reference: vllm/config/model.py (``ModelConfig``), transformers_utils/config.py.
 """
 from __future__ import annotations
 
+import copy
 import json
+import math
 import os
 from dataclasses import dataclass, field
 from typing import Any, Optional
@@ -749,6 +751,28 @@ PRESETS: dict[str, dict[str, Any]] = {
         tie_word_embeddings=False),
 }
 
+def pomipel_config(*, vocab: int, width: int, layers: int, heads: int, dim: int, vdim: int, q_rank: int, kv_rank: int, ff: int,
+                   experts: int, top: int, groups: int, keep: int, max_positions: int, share_every: int = 0, **kw) -> dict[str, Any]:
+    """A Pomipel config.json with like layers; ``share_every`` n > 0: of every n layers the first owns the latent."""
+    out = []
+    for i in range(layers):
+        m = dict(heads=heads, dim=dim, vdim=vdim, q_rank=q_rank, kv_rank=kv_rank, scale=dim ** -0.5)
+        if share_every and i % share_every:
+            m["kv_from"] = i - i % share_every
+        out.append(dict(type="latent_attention", mixer=m, mlp=dict(
+            kind="moe", expert=dict(ff=ff), router=dict(experts=experts, top=top, groups=dict(count=groups, keep=keep)))))
+    return dict(dict(architecture="Pomipel", vocab=vocab, width=width, max_positions=max_positions, layers=out,
+                     embedding=dict(scale=width ** 0.5), norm=dict(eps=1e-6), logit_scale=1.0), **kw)
+
+
+PRESETS.update({
+    "pomipel-tiny": pomipel_config(vocab=320, width=80, layers=3, heads=2, dim=24, vdim=40, q_rank=56, kv_rank=48, ff=56, experts=6,
+                                   top=2, groups=3, keep=2, max_positions=512, share_every=2, torch_dtype="float32"),
+    # the layer sizes of "deepseek-small", for side-by-side measurements
+    "pomipel-small": pomipel_config(vocab=4096, width=1024, layers=3, heads=16, dim=128, vdim=128, q_rank=384, kv_rank=512, ff=512,
+                                    experts=16, top=4, groups=4, keep=2, max_positions=4096, share_every=3, torch_dtype="bfloat16"),
+})
+
 _ALIASES = {
     "facebook/opt-125m": "opt-125m",
     "meta-llama/meta-llama-3-8b": "llama-3-8b", "meta-llama/meta-llama-3-8b-instruct": "llama-3-8b",
@@ -766,11 +790,32 @@ def get_preset_hf_config(name: str) -> Optional[dict[str, Any]]:
     key = name.lower()
     key = _ALIASES.get(key, key)
     cfg = PRESETS.get(key)
-    return dict(cfg) if cfg is not None else None
+    return copy.deepcopy(cfg) if cfg is not None else None
 
 
 def _flatten_nested_config(c: dict) -> None:
     """Families whose config.json nests or renames the fields the engine sizes the KV cache from."""
+    if c.get("architecture") == "Pomipel":
+        layers = c["layers"]
+        mixers = [l["mixer"] for l in layers]
+        moes = [l["mlp"]["router"] for l in layers if l.get("mlp")]
+        c.setdefault("architectures", ["PomipelForCausalLM"])
+        c.setdefault("model_type", "pomipel")
+        c.setdefault("vocab_size", c["vocab"])
+        c.setdefault("hidden_size", c["width"])
+        c.setdefault("num_hidden_layers", len(layers))
+        c.setdefault("max_position_embeddings", c["max_positions"])
+        # layers may differ: tensor parallelism must divide every head count
+        c.setdefault("num_attention_heads", math.gcd(*(m["heads"] for m in mixers)))
+        c.setdefault("kv_lora_rank", max(m["kv_rank"] for m in mixers))
+        c.setdefault("qk_rope_head_dim", 0)
+        if moes:
+            c.setdefault("num_experts", max(r["experts"] for r in moes))
+            c.setdefault("num_experts_per_tok", max(r["top"] for r in moes))
+        for i, m in enumerate(mixers):
+            j = m.get("kv_from")
+            if j is not None and not (0 <= j < i and mixers[j].get("kv_from") is None and mixers[j]["kv_rank"] == m["kv_rank"]):
+                raise ValueError(f"layer {i}: kv_from {j} must name an earlier layer with a latent of its own and the same kv_rank")
     if c.get("model_type") == "dbrx":
         a, f = c.get("attn_config") or {}, c.get("ffn_config") or {}
         c.setdefault("hidden_size", c.get("d_model"))

@@ -223,6 +223,15 @@ class Request:
         if self._hash_fn is not None:
             self.block_hashes.extend(self._hash_fn(self))
 
+    def append_prompt_token_ids(self, token_ids: list[int]) -> None:
+        """More of a prompt that is fed in portions (before anything is generated)."""
+        assert not self._output_token_ids
+        self.prompt_token_ids = self.prompt_token_ids + list(token_ids)
+        self.num_prompt_tokens = len(self.prompt_token_ids)
+        self._all_token_ids.extend(token_ids)
+        if self._hash_fn is not None:
+            self.block_hashes.extend(self._hash_fn(self))
+
     @property
     def output_token_ids(self) -> list[int]:
         return self._output_token_ids

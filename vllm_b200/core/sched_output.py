@@ -54,6 +54,8 @@ class SchedulerOutput:
     grammar_bitmask: Any = None  # np.ndarray [n_structured, ceil(V/32)] int32
     kv_connector_metadata: Any = None
     preempted_req_ids: set[str] = field(default_factory=set)
+    # a step that wants logits instead of samples: request id → places among the tokens it runs in this step
+    logits_positions: Optional[dict[str, list[int]]] = None
     step_id: int = 0
 
     @property
@@ -82,6 +84,7 @@ class ModelRunnerOutput:
     logprobs: Optional[LogprobsTensors] = None
     prompt_logprobs_dict: dict[str, Optional[LogprobsTensors]] = field(default_factory=dict)
     pooler_output: list[Any] = field(default_factory=list)
+    logits: Optional[dict[str, Any]] = None  # request id → [places, vocab] fp32 (steps with ``logits_positions``)
     spec_token_ids: Optional[list[list[int]]] = None  # drafts for the next step
     kv_connector_output: Any = None
     num_nans_in_logits: Optional[dict[str, int]] = None

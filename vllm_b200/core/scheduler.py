@@ -386,6 +386,59 @@ class Scheduler:
         self._last_sched_ms = (time.perf_counter() - t0) * 1e3
         return out
 
+    def schedule_given(self, entries: list[tuple[str, list[int]]], logits_positions: dict[str, list[int]],
+                       sampling_params: Any = None) -> SchedulerOutput:
+        """A step whose content the caller prescribes: every entry brings a request's next tokens (an unknown id is admitted),
+        all of them run, and the logits at ``logits_positions`` (request → places among its tokens) come back instead of
+        samples.  Slots come from the same cache manager as ``schedule``'s; a pool that is too small is an error, not a
+        preemption.  Requests end through ``finish_requests``."""
+        kv = self.kv_cache_manager
+        if len({rid for rid, _ in entries}) != len(entries) or not all(toks for _, toks in entries):
+            raise ValueError("a step names each request once and brings at least one token for it")
+        total = sum(len(toks) for _, toks in entries)
+        if total > self.max_num_scheduled_tokens:
+            raise ValueError(f"step of {total} tokens exceeds max_num_batched_tokens {self.max_num_scheduled_tokens}")
+        c = CachedRequestData()
+        new_data, num_sched = [], {}
+        for rid, toks in entries:
+            req = self.requests.get(rid)
+            fresh = req is None
+            if fresh:
+                if len(self.running) >= self.max_num_running_reqs:
+                    raise ValueError(f"more than {self.max_num_running_reqs} live requests")
+                req = Request(rid, list(toks), sampling_params, block_hasher=self.get_block_hasher())
+                req.status = RequestStatus.RUNNING
+                req.num_cached_tokens = 0
+                self.requests[rid] = req
+                self.running.append(req)
+            else:
+                req.append_prompt_token_ids(toks)
+            if req.num_tokens > self.max_model_len:
+                raise ValueError(f"request {rid!r}: {req.num_tokens} tokens exceed max_model_len {self.max_model_len}")
+            blocks = kv.allocate_slots(req, len(toks))
+            if blocks is None:
+                raise RuntimeError(f"the KV cache has no room for {len(toks)} more tokens of request {rid!r}")
+            if fresh:
+                new_data.append(NewRequestData(req_id=rid, prompt_token_ids=req.prompt_token_ids, sampling_params=sampling_params,
+                                               pooling_params=None, block_ids=kv.get_blocks(rid).get_block_ids(),
+                                               num_computed_tokens=0))
+            else:
+                c.req_ids.append(rid)
+                c.resumed_from_preemption.append(False)
+                c.new_token_ids.append(list(toks))
+                c.new_block_ids.append(blocks.get_block_ids() if blocks is not kv.empty_blocks() else None)
+                c.num_computed_tokens.append(req.num_computed_tokens)
+                c.num_output_tokens.append(0)
+            num_sched[rid] = len(toks)
+        self._step += 1
+        out = SchedulerOutput(scheduled_new_reqs=new_data, scheduled_cached_reqs=c, num_scheduled_tokens=num_sched,
+                              total_num_scheduled_tokens=total, num_common_prefix_blocks=[0] * kv.num_groups,
+                              finished_req_ids=self.finished_req_ids, logits_positions=logits_positions, step_id=self._step)
+        for rid, n in num_sched.items():
+            self.requests[rid].num_computed_tokens += n
+        self.finished_req_ids = set()
+        return out
+
     def _make_cached(self, running, resumed, num_sched, spec_sched, new_blocks_of) -> CachedRequestData:
         c = CachedRequestData()
         pp = self.vllm_config.parallel_config.pipeline_parallel_size > 1

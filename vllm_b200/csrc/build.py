@@ -2,12 +2,19 @@
 
 Plain nvcc (cross-compiles without a GPU): one object per .cu in parallel, then one
 shared library.  The .so is loaded with ctypes (ops/cuda.py) — no torch headers are
-needed, so a full rebuild takes well under a minute.
+needed, so a full rebuild takes a minute or two.
+
+``build_sources`` compiles single sources into libraries of their own (``vllm_b200/_C_<source>.so``): what a checkout
+without the full library does for the kernels a model needs.
 """
 from __future__ import annotations
 
+import contextlib
+import fcntl
+import functools
 import hashlib
 import os
+import re
 import shutil
 import subprocess
 import sys
@@ -79,6 +86,59 @@ def build(force: bool = False, verbose: bool = False) -> str:
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
     return OUT
+
+
+@functools.lru_cache(maxsize=None)
+def _export_map() -> dict[str, str]:
+    """C symbol → source (name without suffix) that defines it."""
+    out = {}
+    for f in sorted(os.listdir(HERE)):
+        if f.endswith(".cu"):
+            with open(os.path.join(HERE, f)) as fh:
+                for name in re.findall(r"^EXPORT\s+\w+\s+(vb_\w+)\s*\(", fh.read(), re.M):
+                    out.setdefault(name, f[:-3])
+    return out
+
+
+def source_of(symbol: str) -> str:
+    src = _export_map().get(symbol)
+    if src is None:
+        raise RuntimeError(f"no source in {HERE} exports {symbol}")
+    return src
+
+
+@contextlib.contextmanager
+def _locked(path: str):
+    with open(path, "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        yield
+
+
+def build_source(name: str) -> str:
+    """``vllm_b200/_C_<name>.so`` from one source; concurrent processes build it once."""
+    out = os.path.join(PKG, f"_C_{name}.so")
+    os.makedirs(OBJ_DIR, exist_ok=True)
+    hdrs = sorted(os.path.join(HERE, f) for f in os.listdir(HERE) if f.endswith((".cuh", ".h")))
+    sig = _sig(os.path.join(HERE, name + ".cu"), hdrs)
+    sig_file = os.path.join(OBJ_DIR, f"{name}.lib.sig")
+    with _locked(os.path.join(OBJ_DIR, f"{name}.lock")):
+        if os.path.exists(out) and os.path.exists(sig_file) and open(sig_file).read() == sig:
+            return out
+        tmp = f"{out[:-3]}.{os.getpid()}.so"
+        r = subprocess.run([_nvcc(), "-shared", *ARCH, *FLAGS, os.path.join(HERE, name + ".cu"), "-o", tmp, "-lcudart"],
+                           capture_output=True, text=True)
+        if r.returncode != 0:
+            raise RuntimeError(f"nvcc failed for {name}.cu:\n{r.stdout}\n{r.stderr}")
+        os.replace(tmp, out)
+        with open(sig_file, "w") as f:
+            f.write(sig)
+    return out
+
+
+def build_sources(names) -> list[str]:
+    names = list(names)
+    with ThreadPoolExecutor(max_workers=max(1, min(os.cpu_count() or 1, len(names)))) as ex:
+        return list(ex.map(build_source, names))
 
 
 if __name__ == "__main__":

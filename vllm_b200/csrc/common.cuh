@@ -129,6 +129,23 @@ VB_DEVICE void mbar_wait(uint64_t* bar, uint32_t parity) {
   while (!mbar_try_wait(bar, parity)) {}
 }
 
+// Bounded wait: gives up after MBAR_TRIES polls (each poll suspends in hardware, so this is seconds — no valid wait
+// comes near it) or as soon as another thread of the CTA gave up (`give_up` in shared memory).  A kernel that gets
+// `false` drains its own copies, frees its TMEM, raises its error flag and returns.
+constexpr uint32_t MBAR_TRIES = 1u << 20;
+VB_DEVICE bool mbar_wait_lim(uint64_t* bar, uint32_t parity, volatile int* give_up) {
+  for (uint32_t i = 0; i < MBAR_TRIES; ++i) {
+    if (mbar_try_wait(bar, parity)) return true;
+    if (*give_up) return false;
+  }
+  *give_up = 1;
+  return false;
+}
+// the same for a whole warp that goes on in step: every lane gets the same answer
+VB_DEVICE bool mbar_wait_warp(uint64_t* bar, uint32_t parity, volatile int* give_up) {
+  return __all_sync(0xffffffffu, mbar_wait_lim(bar, parity, give_up)) != 0;
+}
+
 // ------------------------------------------------- PTX: bulk / tensor copies
 // 1-D bulk copy global → shared, completion counted on an mbarrier (bytes % 16 == 0)
 VB_DEVICE void bulk_g2s(void* dst_smem, const void* src_gmem, uint32_t bytes, uint64_t* bar) {

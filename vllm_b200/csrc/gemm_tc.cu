@@ -33,12 +33,14 @@ struct Params {
   int M, N, K;
   int k_blocks_per_split;  // BK blocks handled by one CTA
   int splits;
-  int act;                 // 0 none, 1 silu-mul over interleaved (gate,up) feature pairs (SWAP only)
+  int act;                 // 0 none, 1 silu-mul over interleaved (gate,up) feature pairs (SWAP only), 2 squared ReLU (grouped)
   int pf;                  // L2 prefetch ahead of the smem ring (SWAP)
   // grouped (MoE) mode, SWAP only: grid.y = n_experts * chunks; expert e multiplies the rows
   // [expert_offs[e], expert_offs[e+1]) of X (tokens sorted by expert) with W[e] = rows [e*N, (e+1)*N) of the weight
   const int* expert_offs;
   int n_experts;
+  int flat;                // grouped: grid.y enumerates the (expert, chunk) pairs that exist (bound: R / BN + experts)
+                           // instead of every chunk an expert could have
   // grouped mode, fused MoE combine (+ cross-rank reduce-scatter): instead of storing Y, every output element is scaled
   // by its pair's routing weight and ADDED (red.add.f32, system scope, straight over NVLink) into the fp32 accumulator
   // row of the rank that OWNS the token (row owner = token / red_per, the same sharding the fused all-reduce kernels use
@@ -93,8 +95,34 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
   if constexpr (SWAP) {
     if (p.expert_offs) {
       pdl_wait();                           // the offsets come from the routing kernels just before us
-      const int chunks = gridDim.y / p.n_experts;
-      const int e = blockIdx.y / chunks, chunk = blockIdx.y % chunks;
+      int e, chunk;
+      if (p.flat) {
+        // flat index → (expert, chunk): every warp walks the chunk counts, 32 experts at a time
+        int target = blockIdx.y;
+        e = -1; chunk = 0;
+        for (int base = 0; base < p.n_experts && e < 0; base += 32) {
+          int nt = 0;
+          if (base + lane < p.n_experts) nt = (p.expert_offs[base + lane + 1] - p.expert_offs[base + lane] + BN - 1) / BN;
+          int inc = nt;
+#pragma unroll
+          for (int o = 1; o < 32; o <<= 1) {
+            const int v = __shfl_up_sync(0xffffffffu, inc, o);
+            if (lane >= o) inc += v;
+          }
+          const unsigned hit = __ballot_sync(0xffffffffu, target < inc);
+          if (hit) {
+            const int l = __ffs(hit) - 1;
+            chunk = target - __shfl_sync(0xffffffffu, inc - nt, l);
+            e = base + l;
+          } else {
+            target -= __shfl_sync(0xffffffffu, inc, 31);
+          }
+        }
+        if (e < 0) return;                  // more CTAs than chunks
+      } else {
+        const int chunks = gridDim.y / p.n_experts;
+        e = blockIdx.y / chunks; chunk = blockIdx.y % chunks;
+      }
       b_row0 = p.expert_offs[e] + chunk * BN;
       m_lim = p.expert_offs[e + 1] - b_row0;
       if (m_lim <= 0) return;               // no token of this chunk routed to expert e: nothing to stream
@@ -122,11 +150,12 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
       // PDL: the weight operand does not depend on the preceding kernel, so the first ring of weight tiles is
       // requested BEFORE griddepcontrol.wait — the weight stream starts while the previous kernel is still
       // draining; only the activation operand waits for it.
+      const uint64_t w_policy = p.flat ? L2_EVICT_NORMAL : L2_EVICT_FIRST;   // prefill chunks of an expert share its weights
       const int pre = SWAP ? min(nkb, STAGES) : 0;
       for (int kb = 0; kb < pre; ++kb) {
         unsigned char* a_dst = stage_base + kb * L::STAGE_BYTES;
         mbar_expect_tx(&full[kb], L::STAGE_BYTES);
-        tma_load_2d_hint(a_dst, &tmap_a, (kb0 + kb) * BK, a_row0, &full[kb], L2_EVICT_FIRST);
+        tma_load_2d_hint(a_dst, &tmap_a, (kb0 + kb) * BK, a_row0, &full[kb], w_policy);
       }
       // the smem ring alone (STAGES x 16 KB of weights) cannot cover the HBM latency-bandwidth product of one
       // SM's share when few CTAs stream a lot each: run an L2 prefetch PF k-blocks ahead of the ring
@@ -147,7 +176,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
         unsigned char* b_dst = a_dst + L::A_BYTES;
         mbar_expect_tx(&full[s], L::STAGE_BYTES);
         const int kc = (kb0 + kb) * BK;
-        tma_load_2d_hint(a_dst, &tmap_a, kc, a_row0, &full[s], SWAP ? L2_EVICT_FIRST : L2_EVICT_LAST);
+        tma_load_2d_hint(a_dst, &tmap_a, kc, a_row0, &full[s], SWAP ? w_policy : L2_EVICT_LAST);
         tma_load_2d_hint(b_dst, &tmap_b, kc, b_row0, &full[s], SWAP ? L2_EVICT_LAST : L2_EVICT_FIRST);
       }
     }
@@ -239,7 +268,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
               }
             }
           }
-        } else if (SWAP && p.act) {
+        } else if (SWAP && p.act == 1) {
           // rows interleave (gate_i, up_i): even lane holds gate, odd lane up → y[tok, i] = silu(gate) * up
           const int n = a_tile * TM + row;
           const int m0 = b_row0 + c;
@@ -259,7 +288,11 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
             const int m0 = b_row0 + c;
 #pragma unroll
             for (int j = 0; j < CH; ++j)
-              if (c + j < m_lim) y[(size_t)(m0 + j) * p.N + n] = from_f32<T>(v[j] + bias);
+              if (c + j < m_lim) {
+                float o = v[j] + bias;
+                if (p.act == 2) { o = fmaxf(o, 0.f); o *= o; }
+                y[(size_t)(m0 + j) * p.N + n] = from_f32<T>(o);
+              }
           }
         } else {
           const int m = a_tile * TM + row;
@@ -479,12 +512,12 @@ EXPORT int vb_gemm_tc2(const void* x, const void* w, const void* bias, void* y, 
                        int swap, int bn, int splits, float* ws, unsigned* counters, int act, int dtype, cudaStream_t st) {
   using namespace gemm;
   if (dtype == DT_F32 || K % 8 != 0) return -1;
-  if (act && (!swap || bias || (N & 3))) return -1;
+  if (act && (act != 1 || !swap || bias || (N & 3))) return -1;
   const bool bf16 = dtype == DT_BF16;
   CUtensorMap ta, tb;
   Params p;
   p.trace = g_trace;
-  p.expert_offs = nullptr; p.n_experts = 0; p.red_acc = nullptr; p.row_pair = nullptr; p.pair_w = nullptr; p.red_k = 1; p.red_H = 0; p.red_world = 1; p.red_per = 1;
+  p.expert_offs = nullptr; p.n_experts = 0; p.flat = 0; p.red_acc = nullptr; p.row_pair = nullptr; p.pair_w = nullptr; p.red_k = 1; p.red_H = 0; p.red_world = 1; p.red_per = 1;
   { static int pf = -1; if (pf < 0) { const char* e = std::getenv("VLLM_B200_GEMM_PF"); pf = (e && e[0] == '1') ? 1 : 0; } p.pf = pf; }
   p.y = y; p.bias = bias; p.ws = ws; p.counters = counters; p.M = M; p.N = N; p.K = K; p.splits = splits; p.act = act;
   const int kb = (K + BK - 1) / BK;
@@ -539,6 +572,15 @@ EXPORT int vb_gemm_tc_grouped_red(const void* x, const void* w, void* y, const i
                                   float* red_acc, void* const* red_peers, int64_t red_off, int red_world, int red_per,
                                   const int* row_pair, const float* pair_w, int red_k, int red_H, int dtype,
                                   cudaStream_t st);
+static int grouped_impl(const void* x, const void* w, void* y, const int* offs, int R, int N, int K, int E, int bn, int act,
+                        int flat, float* red_acc, void* const* red_peers, int64_t red_off, int red_world, int red_per,
+                        const int* row_pair, const float* pair_w, int red_k, int red_H, int dtype, cudaStream_t st);
+// act 2: y = relu(x w^T)^2.  flat: size the grid by the rows there are (prefill: R may be large), not by R chunks per expert
+EXPORT int vb_gemm_tc_grouped2(const void* x, const void* w, void* y, const int* offs, int R, int N, int K, int E, int bn,
+                               int act, int flat, int dtype, cudaStream_t st) {
+  if (act != 0 && act != 2) return -1;
+  return grouped_impl(x, w, y, offs, R, N, K, E, bn, act, flat, nullptr, nullptr, 0, 1, 1, nullptr, nullptr, 1, 0, dtype, st);
+}
 EXPORT int vb_gemm_tc_grouped(const void* x, const void* w, void* y, const int* offs, int R, int N, int K, int E, int bn,
                               int dtype, cudaStream_t st) {
   return vb_gemm_tc_grouped_red(x, w, y, offs, R, N, K, E, bn, nullptr, nullptr, 0, 1, 1, nullptr, nullptr, 1, 0, dtype, st);
@@ -550,14 +592,20 @@ EXPORT int vb_gemm_tc_grouped_red(const void* x, const void* w, void* y, const i
                                   float* red_acc, void* const* red_peers, int64_t red_off, int red_world, int red_per,
                                   const int* row_pair, const float* pair_w, int red_k, int red_H, int dtype,
                                   cudaStream_t st) {
+  return grouped_impl(x, w, y, offs, R, N, K, E, bn, 0, 0, red_acc, red_peers, red_off, red_world, red_per, row_pair, pair_w,
+                      red_k, red_H, dtype, st);
+}
+static int grouped_impl(const void* x, const void* w, void* y, const int* offs, int R, int N, int K, int E, int bn, int act,
+                        int flat, float* red_acc, void* const* red_peers, int64_t red_off, int red_world, int red_per,
+                        const int* row_pair, const float* pair_w, int red_k, int red_H, int dtype, cudaStream_t st) {
   using namespace gemm;
   if (dtype == DT_F32 || K % 8 != 0 || bn > 128 || bn % 16) return -1;
   const bool bf16 = dtype == DT_BF16;
   CUtensorMap ta, tb;
   Params p;
   p.trace = nullptr; p.pf = 0;
-  p.y = y; p.bias = nullptr; p.ws = nullptr; p.counters = nullptr; p.M = R; p.N = N; p.K = K; p.splits = 1; p.act = 0;
-  p.expert_offs = offs; p.n_experts = E;
+  p.y = y; p.bias = nullptr; p.ws = nullptr; p.counters = nullptr; p.M = R; p.N = N; p.K = K; p.splits = 1; p.act = act;
+  p.expert_offs = offs; p.n_experts = E; p.flat = flat;
   p.red_acc = red_acc; p.row_pair = row_pair; p.pair_w = pair_w; p.red_k = red_k; p.red_H = red_H;
   p.red_world = red_world; p.red_per = red_per < 1 ? 1 : red_per;
   for (int i = 0; i < 8; ++i)
@@ -568,7 +616,8 @@ EXPORT int vb_gemm_tc_grouped_red(const void* x, const void* w, void* y, const i
   if ((rc = make_tmap(&ta, w, (uint64_t)E * N, K, K, TM, bf16))) return rc;
   if ((rc = make_tmap(&tb, x, R, K, K, bn, bf16))) return rc;
   const int chunks = (R + bn - 1) / bn;
-  dim3 grid((N + TM - 1) / TM, E * chunks, 1);
+  dim3 grid((N + TM - 1) / TM, flat ? R / bn + (E < R ? E : R) : E * chunks, 1);
+  if (grid.y > 65535) return -6;
 #define GOG(BNV, ST2)                                                                    \
     if (bf16) return launch<__nv_bfloat16, BNV, ST2, true>(ta, tb, p, grid, st);         \
     else return launch<__half, BNV, ST2, true>(ta, tb, p, grid, st);

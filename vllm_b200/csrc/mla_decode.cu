@@ -1,9 +1,9 @@
 // Multi-head latent attention (MLA) decode on tcgen05: MQA over the paged latent cache, the latent tile shared by all
 // heads of the CTA and by BOTH matrix products.
 //
-//   cache row (one per token, all heads share it):  [ c_kv : 512 | k_rope : 64 ]  (bf16 / fp16)
-//   S^T[tok, h] = Kc[tok, 0:576] · Q[h, 0:576]^T      A = latent tile [128 tok x 64-dim k-blocks] K-major (TMA, SW128)
-//                                                     B = Q           [N heads x 576]
+//   cache row (one per token, all heads share it):  [ c_kv : R | k_rope : 0 or 64 ]  (bf16 / fp16)
+//   S^T[tok, h] = Kc[tok, :] · Q[h, :]^T              A = latent tile [128 tok x 64-dim k-blocks] K-major (TMA, SW128)
+//                                                     B = Q           [N heads x (R + rope)]
 //   O^T[d, h]  += Kc[tok, d]^T · P^T[tok, h]          A = THE SAME shared-memory bytes read as an MN-major operand
 //                                                         (d contiguous inside a 128-byte swizzle row, tokens along K)
 //                                                     B = P           [N heads x 128 tok]
@@ -11,7 +11,11 @@
 // for O, the heads are the MMA N (16 or 32 per CTA; 128-head models run 4 head groups per sequence) — and each latent
 // byte is fetched from HBM once and from shared memory by two tcgen05.mma streams, never transposed, never copied.
 //
-// A tile is 64 KV tokens (9 k-blocks of [64 tok x 64 dims] = 72 KB); two tiles are resident.  Every k-block has its own
+// R is any multiple of 8 up to 512: NL k-blocks of 64 dims (TMA zero-fills the tail of the last one), and ceil(NL / 2)
+// output chunks of 128 dims — the second half of an odd last chunk multiplies whatever block follows in shared memory,
+// into TMEM lanes that are never stored.
+//
+// A tile is 64 KV tokens (R = 512 with rope: 9 k-blocks of [64 tok x 64 dims] = 72 KB); 2-4 tiles are resident.  Every k-block has its own
 // full / empty mbarrier: QK starts on the first k-block that lands (rope first), the rope block is released when QK
 // retires and each pair of latent blocks when the PV product of its 128 output dims retires — so the TMA stream of
 // tile j+2 starts under the PV of tile j instead of after it (ncu of the whole-tile version: softmax warps spent 70 %
@@ -26,25 +30,30 @@
 
 namespace mla {
 
-constexpr int DL = 512, DR = 64, DK = DL + DR;
-constexpr int NKB = DK / 64;          // 9 k-blocks of 64 dims
+constexpr int DR = 64;                // width of the rope part, where there is one
 constexpr int TILE = 64;
 constexpr int KB_BYTES = TILE * 128;  // 8 KB: one k-block [64 tok x 64 dims]
-constexpr int STAGE_BYTES = NKB * KB_BYTES;   // 72 KB
-constexpr int STAGES = 2;
+// tile geometry of a latent of NL 64-dim blocks with (ROPE = 1) or without a rope block behind it
+template <int NL, int ROPE> struct Geo {
+  static constexpr int NKB = NL + ROPE;
+  static constexpr int STAGE_BYTES = NKB * KB_BYTES;
+  static constexpr int STAGES = NKB >= 7 ? 2 : (NKB >= 4 ? 3 : 4);
+  static constexpr int NC = (NL + 1) / 2;         // 128-dim output chunks
+};
 constexpr int NUM_THREADS = 192;
 constexpr int MAX_IDS_SMEM = 1024;
 
 struct Params {
   const int* block_table;
   const int* seq_lens;
-  void* out;            // [B, H, 512]
-  float* part_out;      // [B, H, splits, 512]
+  void* out;            // [B, H, R]
+  float* part_out;      // [B, H, splits, R]
   float* part_lse;      // [B, H, splits]
   float* lse_out;       // optional [B, H] (natural log)
   int64_t out_stride;   // elements between batch rows of out
   int bt_stride;
-  int H, BS, num_splits;
+  int H, BS, num_splits, R;
+  int* error;           // raised when a wait ran into its limit
   float scale_log2;
 };
 
@@ -78,16 +87,18 @@ VB_HOST_DEVICE uint32_t idesc_f16_a_mn(int M, int N, bool bf16) {
   return umma_idesc_f16(M, N, bf16) | (1u << 15);     // bit 15: A operand is MN-major
 }
 
-template <typename T, int N>
+template <typename T, int N, int NL, int ROPE>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_constant__ CUtensorMap tmap_qr,
                   const __grid_constant__ CUtensorMap tmap_kv, const Params p) {
-  constexpr int Q_BYTES = NKB * N * 128;     // 9 k-blocks of [N x 64]
+  constexpr int NKB = Geo<NL, ROPE>::NKB, STAGE_BYTES = Geo<NL, ROPE>::STAGE_BYTES, STAGES = Geo<NL, ROPE>::STAGES;
+  constexpr int NC = Geo<NL, ROPE>::NC;
+  constexpr int Q_BYTES = NKB * N * 128;     // k-blocks of [N x 64]
   constexpr int P_BYTES = N * 128;           // [N x 64 tok]
   constexpr int CH = 16;                     // TMEM columns moved per tcgen05.ld/st
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  unsigned char* kv_smem = smem;                                // STAGES x 72 KB
+  unsigned char* kv_smem = smem;                                // STAGES tiles
   unsigned char* q_smem = kv_smem + STAGES * STAGE_BYTES;       // (also what QK's padding rows of the last k-block read)
   unsigned char* p_smem = q_smem + Q_BYTES;
   uint64_t* bars = reinterpret_cast<uint64_t*>(p_smem + (P_BYTES < 8192 ? 8192 : P_BYTES));
@@ -101,6 +112,8 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 1);
   float* wred = reinterpret_cast<float*>(tmem_slot + 2);        // [4][N]
   int* blk_ids = reinterpret_cast<int*>(wred + 4 * N);          // [MAX_IDS_SMEM]
+  __shared__ int give_up_s;
+  volatile int* give_up = &give_up_s;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int split = blockIdx.x, hg = blockIdx.y, b = blockIdx.z;
@@ -119,7 +132,9 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
     tile_hi = min(tile_hi, tile_lo + per);
   }
   const int n_tiles = max(tile_hi - tile_lo, 0);
-  constexpr uint32_t TMEM_COLS = 6 * N <= 128 ? 128 : 256;
+  constexpr uint32_t TMEM_USE = (2 + NC) * N;
+  constexpr uint32_t TMEM_COLS = TMEM_USE <= 64 ? 64 : (TMEM_USE <= 128 ? 128 : 256);
+  if (threadIdx.x == 0) give_up_s = 0;
 
   if (warp == 0 && lane == 0) {
     tma_prefetch_desc(&tmap_qn); tma_prefetch_desc(&tmap_qr); tma_prefetch_desc(&tmap_kv);
@@ -138,7 +153,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
     const int n16 = (STAGES * STAGE_BYTES + Q_BYTES + (P_BYTES < 8192 ? 8192 : P_BYTES)) / 16;
     for (int i = threadIdx.x; i < n16; i += NUM_THREADS) s4[i] = z;
   }
-  // token row (in the [num_blocks * BS, 576] view of the cache) of every TMA box of this split, -1 = past the sequence
+  // token row (in the [num_blocks * BS, row] view of the cache) of every TMA box of this split, -1 = past the sequence
   auto box_row = [&](int i) -> int {
     const int tok0 = tile_lo * TILE + i * rows;
     if (tok0 >= seq_len) return -1;
@@ -158,7 +173,8 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
       const int t = (warp & 3) * 32 + lane;
       for (int g = 0; g < G; ++g) {
         const int64_t pi = ((int64_t)b * p.H + (h0 + g)) * p.num_splits + split;
-        for (int c = 0; c < 4; ++c) p.part_out[pi * DL + c * 128 + t] = 0.f;
+        for (int c = 0; c < NC; ++c)
+          if (c * 128 + t < p.R) p.part_out[pi * p.R + c * 128 + t] = 0.f;
         if (t == 0) p.part_lse[pi] = -INFINITY;
       }
     }
@@ -171,9 +187,10 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
     if (lane == 0) {
       // ===== TMA producer
       mbar_expect_tx(q_full, NKB * min(N, p.H) * 128);   // the full TMA box is always written (OOB heads as zeros)
-      for (int kb = 0; kb < 8; ++kb) tma_load_3d(q_smem + kb * (N * 128), &tmap_qn, kb * 64, h0, b, q_full);
-      tma_load_3d(q_smem + 8 * (N * 128), &tmap_qr, 0, h0, b, q_full);
-      for (int j = 0; j < n_tiles; ++j) {
+      for (int kb = 0; kb < NL; ++kb) tma_load_3d(q_smem + kb * (N * 128), &tmap_qn, kb * 64, h0, b, q_full);
+      if (ROPE) tma_load_3d(q_smem + NL * (N * 128), &tmap_qr, 0, h0, b, q_full);
+      bool ok = true;
+      for (int j = 0; j < n_tiles && ok; ++j) {
         const int st = j % STAGES;
         const uint32_t par = ((j / STAGES) & 1) ^ 1;
         int row[8], n_valid = 0;
@@ -186,14 +203,19 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
         unsigned char* stp = kv_smem + st * STAGE_BYTES;
 #pragma unroll 1
         for (int i = 0; i < NKB; ++i) {
-          const int kb = i == 0 ? NKB - 1 : i - 1;             // rope block first: QK releases it first
+          const int kb = ROPE ? (i == 0 ? NKB - 1 : i - 1) : i;   // rope block first: QK releases it first
           const int slot = st * NKB + kb;
-          mbar_wait(&kv_empty[slot], par);
+          if (!(ok = mbar_wait_lim(&kv_empty[slot], par, give_up))) break;
           mbar_expect_tx(&kv_full[slot], bytes);
           for (int u = 0; u < ppt; ++u)
             if (row[u] >= 0)
-              tma_load_2d_hint(stp + kb * KB_BYTES + u * rows * 128, &tmap_kv, kb * 64, row[u], &kv_full[slot], L2_EVICT_FIRST);
+              tma_load_2d_hint(stp + kb * KB_BYTES + u * rows * 128, &tmap_kv, kb * 64, row[u], &kv_full[slot],
+                               p.H > N ? L2_EVICT_NORMAL : L2_EVICT_FIRST);   // other head groups read the tile again
         }
+      }
+      if (!ok) {                                // let the copies in flight land before the block gives up its memory
+        for (int i = 0; i < STAGES * NKB; ++i)
+          for (int n = 0; n < 4096 && !mbar_try_wait(&kv_full[i], 0) && !mbar_try_wait(&kv_full[i], 1); ++n) {}
       }
     }
   } else if (warp == 1) {
@@ -201,24 +223,24 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
     const bool bf16 = DTypeOf<T>::v == DT_BF16;
     const uint32_t idesc_s = umma_idesc_f16(128, N, bf16);
     const uint32_t idesc_o = idesc_f16_a_mn(128, N, bf16);
-    mbar_wait(q_full, 0);
+    bool ok = mbar_wait_warp(q_full, 0, give_up);
     // descriptors are built once; every MMA adds a compile-time offset (in 16-byte units) to the address field
     const uint64_t d_kv = umma_desc_sw128(kv_smem);
     const uint64_t d_kv_mn = umma_desc_sw128_mn(kv_smem, KB_BYTES);
     const uint64_t d_q = umma_desc_sw128(q_smem);
     const uint64_t d_p = umma_desc_sw128(p_smem);
-    for (int j = 0; j <= n_tiles; ++j) {
+    for (int j = 0; j <= n_tiles && ok; ++j) {
       if (j < n_tiles) {
         // ---- S^T_j = Kc · Q^T, k-block by k-block as they land (M = 128: rows 64..127 are padding, see the header)
         const int st = j % STAGES, sb = j & 1;
         const uint32_t par = (j / STAGES) & 1;
-        mbar_wait(&s_empty[sb], ((j >> 1) & 1) ^ 1);
+        if (!(ok = mbar_wait_warp(&s_empty[sb], ((j >> 1) & 1) ^ 1, give_up))) break;
         tc_fence_after();
 #pragma unroll
         for (int i = 0; i < NKB; ++i) {
-          const int kb = i == 0 ? NKB - 1 : i - 1;
+          const int kb = ROPE ? (i == 0 ? NKB - 1 : i - 1) : i;
           const int slot = st * NKB + kb;
-          mbar_wait(&kv_full[slot], par);
+          if (!(ok = mbar_wait_warp(&kv_full[slot], par, give_up))) break;
           tc_fence_after();
           if (lane == 0) {
             const uint64_t da = d_kv + (uint64_t)((st * STAGE_BYTES + kb * KB_BYTES) >> 4);
@@ -229,28 +251,29 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
           }
           __syncwarp();
         }
+        if (!ok) break;
         if (lane == 0) {
           umma_commit(&s_full[sb]);
-          umma_commit(&kv_empty[st * NKB + NKB - 1]);          // the rope block is only read by QK
+          if (ROPE) umma_commit(&kv_empty[st * NKB + NKB - 1]);   // the rope block is only read by QK
         }
         __syncwarp();
       }
       if (j > 0) {
-        // ---- O^T += V^T · P^T for tile j-1: four 128-dim chunks (k-blocks 2c, 2c+1 read MN-major), K = 64 tokens;
+        // ---- O^T += V^T · P^T for tile j-1: NC 128-dim chunks (k-blocks 2c, 2c+1 read MN-major), K = 64 tokens;
         // each chunk hands its two k-block buffers back to the producer as soon as it retires
         const int jj = j - 1, st = jj % STAGES;
-        mbar_wait(p_full, jj & 1);
+        if (!(ok = mbar_wait_warp(p_full, jj & 1, give_up))) break;
         tc_fence_after();
         if (lane == 0) {
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
+          for (int c = 0; c < NC; ++c) {
 #pragma unroll
             for (int kk = 0; kk < TILE / 16; ++kk) {
               const uint64_t da = d_kv_mn + (uint64_t)((st * STAGE_BYTES + (2 * c) * KB_BYTES + kk * 2048) >> 4);
               umma_f16(tmem_o + c * N, da, d_p + (uint64_t)(kk * 2), idesc_o, (jj | kk) != 0);
             }
             umma_commit(&kv_empty[st * NKB + 2 * c]);
-            umma_commit(&kv_empty[st * NKB + 2 * c + 1]);
+            if (2 * c + 1 < NL) umma_commit(&kv_empty[st * NKB + 2 * c + 1]);
           }
           umma_commit(pv_done);
         }
@@ -267,7 +290,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
     for (int g = 0; g < N; ++g) { m_used[g] = -INFINITY; l_thr[g] = 0.f; }
     for (int j = 0; j < n_tiles; ++j) {
       const int sb = j & 1;
-      mbar_wait(&s_full[sb], (j >> 1) & 1);
+      mbar_wait_lim(&s_full[sb], (j >> 1) & 1, give_up);
       tc_fence_after();
       float s[N];
 #pragma unroll
@@ -300,10 +323,10 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
           m_used[g] = mx;
         }
       }
-      if (j > 0) { mbar_wait(pv_done, (j - 1) & 1); tc_fence_after(); }   // P and O^T are free again
+      if (j > 0) { mbar_wait_lim(pv_done, (j - 1) & 1, give_up); tc_fence_after(); }   // P and O^T are free again
       if (rescale) {       // uniform over the CTA (every thread sees the same column maxima)
 #pragma unroll
-        for (int c4 = 0; c4 < 4; ++c4) {
+        for (int c4 = 0; c4 < NC; ++c4) {
 #pragma unroll
           for (int c = 0; c < N; c += CH) {
             uint32_t ov[CH];
@@ -339,7 +362,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
       if (lane == 0) wred[qd * N + g] = lt;
     }
     bar_sync_softmax();
-    mbar_wait(pv_done, (n_tiles - 1) & 1);
+    mbar_wait_lim(pv_done, (n_tiles - 1) & 1, give_up);
     tc_fence_after();
     float inv[N], lsum[N];
 #pragma unroll
@@ -348,8 +371,9 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
       inv[g] = lsum[g] > 0.f ? 1.f / lsum[g] : 0.f;
     }
 #pragma unroll
-    for (int c4 = 0; c4 < 4; ++c4) {
+    for (int c4 = 0; c4 < NC; ++c4) {
       const int d = c4 * 128 + t;
+      const bool d_ok = d < p.R;
 #pragma unroll
       for (int c = 0; c < N; c += CH) {
         uint32_t ov[CH];
@@ -357,14 +381,14 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
         tmem_ld_wait();
 #pragma unroll
         for (int g = 0; g < CH; ++g) {
-          if (c + g < G) {
+          if (c + g < G && d_ok) {
             const float o = __uint_as_float(ov[g]) * inv[c + g];
             const int hq = h0 + c + g;
             if (p.num_splits == 1) {
-              reinterpret_cast<T*>(p.out)[(int64_t)b * p.out_stride + (int64_t)hq * DL + d] = from_f32<T>(o);
+              reinterpret_cast<T*>(p.out)[(int64_t)b * p.out_stride + (int64_t)hq * p.R + d] = from_f32<T>(o);
             } else {
               const int64_t pi = ((int64_t)b * p.H + hq) * p.num_splits + split;
-              p.part_out[pi * DL + d] = o;
+              p.part_out[pi * p.R + d] = o;
             }
           }
         }
@@ -389,12 +413,13 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
   tc_fence_before();
   __syncthreads();
   if (warp == 1) tmem_dealloc(tmem_base, TMEM_COLS);
+  if (threadIdx.x == 0 && *give_up && p.error) *p.error = 1;
 }
 
 template <typename T>
 __global__ void __launch_bounds__(128) mla_split_reduce(const float* __restrict__ part_out, const float* __restrict__ part_lse,
                                                         T* __restrict__ out, float* __restrict__ lse_out, int H, int S,
-                                                        int64_t out_stride) {
+                                                        int64_t out_stride, int R) {
   const int tok = blockIdx.x, hq = blockIdx.y;
   const int64_t base = ((int64_t)tok * H + hq) * S;
   float m = -INFINITY;
@@ -402,10 +427,10 @@ __global__ void __launch_bounds__(128) mla_split_reduce(const float* __restrict_
   const float m_use = (m == -INFINITY) ? 0.f : m;
   float den = 0.f;
   for (int s = 0; s < S; ++s) den += ex2(part_lse[base + s] - m_use);
-  for (int d = threadIdx.x; d < DL; d += blockDim.x) {
+  for (int d = threadIdx.x; d < R; d += blockDim.x) {
     float o = 0.f;
-    for (int s = 0; s < S; ++s) o += ex2(part_lse[base + s] - m_use) * part_out[(base + s) * DL + d];
-    out[(int64_t)tok * out_stride + (int64_t)hq * DL + d] = from_f32<T>(den > 0.f ? o / den : 0.f);
+    for (int s = 0; s < S; ++s) o += ex2(part_lse[base + s] - m_use) * part_out[(base + s) * R + d];
+    out[(int64_t)tok * out_stride + (int64_t)hq * R + d] = from_f32<T>(den > 0.f ? o / den : 0.f);
   }
   if (lse_out && threadIdx.x == 0) lse_out[(int64_t)tok * H + hq] = den > 0.f ? (m + log2f(den)) * 0.6931471805599453f : -INFINITY;
 }
@@ -424,11 +449,12 @@ static EncodeTiledFn get_encode() {
   return fn;
 }
 
-template <typename T, int N>
+template <typename T, int N, int NL, int ROPE>
 static int launch(const CUtensorMap& tqn, const CUtensorMap& tqr, const CUtensorMap& tkv, const Params& p, dim3 grid,
                   cudaStream_t st) {
-  const int smem = STAGES * STAGE_BYTES + NKB * N * 128 + 8192 + (2 * STAGES * NKB + 8) * 8 + 16 + 4 * N * 4 + MAX_IDS_SMEM * 4 + 1024;
-  auto k = mla_decode_kernel<T, N>;
+  constexpr int NKB = Geo<NL, ROPE>::NKB, STAGES = Geo<NL, ROPE>::STAGES;
+  const int smem = STAGES * Geo<NL, ROPE>::STAGE_BYTES + NKB * N * 128 + 8192 + (2 * STAGES * NKB + 8) * 8 + 16 + 4 * N * 4 + MAX_IDS_SMEM * 4 + 1024;
+  auto k = mla_decode_kernel<T, N, NL, ROPE>;
   static bool a = false;
   if (!a) { cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); a = true; }
   vb_launch(k, grid, dim3(NUM_THREADS), (size_t)smem, st, tqn, tqr, tkv, p);
@@ -437,44 +463,43 @@ static int launch(const CUtensorMap& tqn, const CUtensorMap& tqr, const CUtensor
 
 }  // namespace mla
 
-// q_nope: [B, H, 512] (absorbed W_UK), q_pe: [B, H, 64], cache: [num_blocks, BS, 576]; out: [B, H, 512].
+// q_nope: [B, H, R] (absorbed W_UK), q_pe: [B, H, 64] or null, cache: [num_blocks, BS, R (+ 64)]; out: [B, H, R].
+// bf16 covers every R (a multiple of 8 up to 512) without a rope part and R = 512 with one; fp16 the latter only.
+// `error` (device int, may be null) becomes 1 when a wait inside the kernel ran into its limit.
 EXPORT int vb_mla_decode(const void* q_nope, const void* q_pe, const void* cache, int64_t num_blocks, const int* block_table,
-                         const int* seq_lens, void* out, float* part_out, float* part_lse, float* lse_out, int B, int H,
-                         int BS, int64_t qn_stride_b, int64_t qn_stride_h, int64_t qr_stride_b, int64_t qr_stride_h,
-                         int64_t out_stride, int bt_stride, int num_splits, float scale, int dtype, cudaStream_t st) {
+                         const int* seq_lens, void* out, float* part_out, float* part_lse, float* lse_out, int* error, int B,
+                         int H, int R, int rope, int BS, int64_t qn_stride_b, int64_t qn_stride_h, int64_t qr_stride_b,
+                         int64_t qr_stride_h, int64_t out_stride, int bt_stride, int num_splits, float scale, int dtype,
+                         cudaStream_t st) {
   using namespace mla;
   if (B == 0) return 0;
-  if (dtype == DT_F32) return -1;
+  if (dtype == DT_F32 || R < 8 || R > 512 || R % 8) return -1;
+  if (rope ? (rope != DR || R != 512) : dtype != DT_BF16) return -2;
   if (BS != 16 && BS != 32 && BS != 64 && BS != 128) return -4;
   auto enc = get_encode();
   if (!enc) return -10;
   const bool bf16 = dtype == DT_BF16;
   const CUtensorMapDataType dt = bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
   const int N = H > 16 ? 32 : 16;
+  const int DK = R + rope;
   Params p;
   p.block_table = block_table; p.seq_lens = seq_lens; p.out = out; p.part_out = part_out; p.part_lse = part_lse;
   p.lse_out = lse_out; p.out_stride = out_stride; p.bt_stride = bt_stride; p.H = H; p.BS = BS; p.num_splits = num_splits;
+  p.R = R; p.error = error;
   p.scale_log2 = scale * 1.4426950408889634f;
   CUtensorMap tqn, tqr, tkv;
   const int gbox = H < N ? H : N;
-  {
-    cuuint64_t dims[3] = {(cuuint64_t)DL, (cuuint64_t)H, (cuuint64_t)B};
-    cuuint64_t strides[2] = {(cuuint64_t)qn_stride_h * 2, (cuuint64_t)qn_stride_b * 2};
+  auto enc_q = [&](CUtensorMap* m, const void* ptr, int width, int64_t sb, int64_t sh) {
+    cuuint64_t dims[3] = {(cuuint64_t)width, (cuuint64_t)H, (cuuint64_t)B};
+    cuuint64_t strides[2] = {(cuuint64_t)sh * 2, (cuuint64_t)sb * 2};
     cuuint32_t box[3] = {64, (cuuint32_t)gbox, 1};
     cuuint32_t es[3] = {1, 1, 1};
-    if (enc(&tqn, dt, 3, const_cast<void*>(q_nope), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
-            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
-      return -11;
-  }
-  {
-    cuuint64_t dims[3] = {(cuuint64_t)DR, (cuuint64_t)H, (cuuint64_t)B};
-    cuuint64_t strides[2] = {(cuuint64_t)qr_stride_h * 2, (cuuint64_t)qr_stride_b * 2};
-    cuuint32_t box[3] = {64, (cuuint32_t)gbox, 1};
-    cuuint32_t es[3] = {1, 1, 1};
-    if (enc(&tqr, dt, 3, const_cast<void*>(q_pe), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
-            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
-      return -12;
-  }
+    return enc(m, dt, 3, const_cast<void*>(ptr), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  };
+  if (enc_q(&tqn, q_nope, R, qn_stride_b, qn_stride_h) != CUDA_SUCCESS) return -11;
+  if (rope && enc_q(&tqr, q_pe, DR, qr_stride_b, qr_stride_h) != CUDA_SUCCESS) return -12;
+  if (!rope) tqr = tqn;
   {
     cuuint64_t dims[2] = {(cuuint64_t)DK, (cuuint64_t)num_blocks * BS};
     cuuint64_t strides[1] = {(cuuint64_t)DK * 2};
@@ -486,12 +511,20 @@ EXPORT int vb_mla_decode(const void* q_nope, const void* q_pe, const void* cache
   }
   dim3 grid(num_splits, (H + N - 1) / N, B);
   int rc;
-  if (N == 16) rc = bf16 ? launch<__nv_bfloat16, 16>(tqn, tqr, tkv, p, grid, st) : launch<__half, 16>(tqn, tqr, tkv, p, grid, st);
-  else rc = bf16 ? launch<__nv_bfloat16, 32>(tqn, tqr, tkv, p, grid, st) : launch<__half, 32>(tqn, tqr, tkv, p, grid, st);
+#define GO(TT, NL, RP) rc = N == 16 ? launch<TT, 16, NL, RP>(tqn, tqr, tkv, p, grid, st) : launch<TT, 32, NL, RP>(tqn, tqr, tkv, p, grid, st)
+  const int nl = (R + 63) / 64;
+  if (rope) { if (bf16) GO(__nv_bfloat16, 8, 1); else GO(__half, 8, 1); }
+  else if (nl <= 1) GO(__nv_bfloat16, 1, 0);
+  else if (nl == 2) GO(__nv_bfloat16, 2, 0);
+  else if (nl == 3) GO(__nv_bfloat16, 3, 0);
+  else if (nl == 4) GO(__nv_bfloat16, 4, 0);
+  else if (nl <= 6) GO(__nv_bfloat16, 6, 0);
+  else GO(__nv_bfloat16, 8, 0);
+#undef GO
   if (rc) return rc;
   if (num_splits > 1) {
-    if (bf16) mla_split_reduce<__nv_bfloat16><<<dim3(B, H), 128, 0, st>>>(part_out, part_lse, (__nv_bfloat16*)out, lse_out, H, num_splits, out_stride);
-    else mla_split_reduce<__half><<<dim3(B, H), 128, 0, st>>>(part_out, part_lse, (__half*)out, lse_out, H, num_splits, out_stride);
+    if (bf16) mla_split_reduce<__nv_bfloat16><<<dim3(B, H), 128, 0, st>>>(part_out, part_lse, (__nv_bfloat16*)out, lse_out, H, num_splits, out_stride, R);
+    else mla_split_reduce<__half><<<dim3(B, H), 128, 0, st>>>(part_out, part_lse, (__half*)out, lse_out, H, num_splits, out_stride, R);
   }
   return (int)cudaGetLastError();
 }

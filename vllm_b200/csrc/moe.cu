@@ -62,6 +62,175 @@ __global__ void topk_softmax_kernel(const T* __restrict__ logits, float* __restr
   }
 }
 
+// Router with sigmoid or softmax scores, a selection bias and group-limited choice; one CTA per token, fp32 throughout.
+//   logits: given ([T, E] fp32), or computed here from x [T, H] and w [E, H] (one warp per expert, decode batches)
+//   choice score = score + bias;  a group (n_group equal runs of neighbours) is ranked by the sum of its two best choice
+//   scores (with a bias) or by its best (without);  the k best experts of the `keep` best groups are taken, the lowest
+//   index winning ties;  weight = score WITHOUT the bias (optionally renormalised) * scale
+template <typename TX, typename TW>
+__global__ void __launch_bounds__(256)
+grouped_topk_kernel(const float* __restrict__ logits, const TX* __restrict__ x, const TW* __restrict__ w, int H,
+                    const float* __restrict__ bias, float* __restrict__ out_w, int* __restrict__ out_ids, int E, int k,
+                    int n_group, int keep, int softmax, int renorm, float scale) {
+  extern __shared__ float smf[];
+  float* score = smf;               // [E]
+  float* choice = score + E;        // [E]
+  float* gs = choice + E;           // [n_group]
+  float* xs = gs + n_group;         // [H] when the logits are computed here
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  if (logits) {
+    for (int e = threadIdx.x; e < E; e += blockDim.x) score[e] = logits[(int64_t)t * E + e];
+  } else {
+    const TX* xr = x + (int64_t)t * H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) xs[i] = to_f32(xr[i]);
+    __syncthreads();
+    constexpr int V = Vec16<TW>::N;
+    const bool vec = H % V == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
+    for (int e = warp; e < E; e += n_warps) {
+      const TW* wr = w + (int64_t)e * H;
+      float a = 0.f;
+      if (vec) {
+        for (int i = lane * V; i < H; i += 32 * V) {
+          const Vec16<TW> wv = ld16(wr + i);
+#pragma unroll
+          for (int j = 0; j < V; ++j) a += xs[i + j] * to_f32(wv.e[j]);
+        }
+      } else {
+        for (int i = lane; i < H; i += 32) a += xs[i] * to_f32(wr[i]);
+      }
+      a = warp_sum(a);
+      if (lane == 0) score[e] = a;
+    }
+  }
+  __syncthreads();
+  if (softmax) {
+    float mx = -INFINITY;
+    for (int e = threadIdx.x; e < E; e += blockDim.x) mx = fmaxf(mx, score[e]);
+    mx = warp_max(mx);
+    if (lane == 0) red[warp] = mx;
+    __syncthreads();
+    mx = warp_max(lane < n_warps ? red[lane] : -INFINITY);
+    __syncthreads();
+    float sum = 0.f;
+    for (int e = threadIdx.x; e < E; e += blockDim.x) { score[e] = expf(score[e] - mx); sum += score[e]; }
+    const float inv = 1.f / block_sum(sum, red);
+    for (int e = threadIdx.x; e < E; e += blockDim.x) score[e] *= inv;
+  } else {
+    for (int e = threadIdx.x; e < E; e += blockDim.x) score[e] = 1.f / (1.f + expf(-score[e]));
+  }
+  for (int e = threadIdx.x; e < E; e += blockDim.x) choice[e] = score[e] + (bias ? bias[e] : 0.f);
+  __syncthreads();
+  if (warp) return;                 // the choice is one warp's work
+  auto argmax = [&](const float* v, int n) -> int {
+    float best = -INFINITY;
+    int bi = 0x7fffffff;
+    for (int i = lane; i < n; i += 32)
+      if (v[i] > best) { best = v[i]; bi = i; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+    }
+    return bi;                      // 0x7fffffff: nothing above -inf is left
+  };
+  if (n_group > 1) {
+    const int gsz = E / n_group;
+    for (int g = lane; g < n_group; g += 32) {
+      float a = -INFINITY, b = -INFINITY;
+      for (int i = 0; i < gsz; ++i) {
+        const float c = choice[g * gsz + i];
+        if (c > a) { b = a; a = c; } else if (c > b) { b = c; }
+      }
+      gs[g] = bias && gsz > 1 ? a + b : a;
+    }
+    __syncwarp();
+    // drop the worst groups: what the keep-th best leaves behind.  A taken group is marked by -inf.
+    for (int n = 0; n < keep; ++n) {
+      const int g = argmax(gs, n_group);
+      __syncwarp();
+      if (lane == 0 && g < n_group) gs[g] = -INFINITY;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (gs[e / gsz] != -INFINITY) choice[e] = -INFINITY;
+    __syncwarp();
+  }
+  float wsum = 0.f, mine = 0.f;
+  for (int j = 0; j < k; ++j) {
+    int e = argmax(choice, E);
+    if (e >= E) e = 0;              // fewer than k candidates: cannot happen for a valid configuration
+    const float s = score[e];
+    wsum += s;
+    __syncwarp();
+    if (lane == 0) {
+      choice[e] = -INFINITY;
+      out_ids[(int64_t)t * k + j] = e;
+      if (!renorm) out_w[(int64_t)t * k + j] = s * scale;
+    }
+    if (lane == (j & 31)) mine = s;
+    if (renorm && ((j & 31) == 31 || j == k - 1) && lane <= (j & 31)) out_w[(int64_t)t * k + (j & ~31) + lane] = mine;
+    __syncwarp();
+  }
+  if (renorm)
+    for (int j = lane; j < k; j += 32) out_w[(int64_t)t * k + j] *= scale / (wsum + 1e-20f);
+}
+
+// Grouped GEMM on the CUDA cores for what the tcgen05 kernel (gemm_tc.cu) does not take — fp32, or rows that are not
+// 16-byte multiples:  y[r, n] = act(sum_k x[tok(r), k] * w[e(r), n, k]), rows sorted by expert.  64 x 64 tiles; grid.y
+// enumerates (expert, row tile) pairs, found from `offs` on the device.
+constexpr int GT = 64, GK = 16;
+template <typename T>
+__global__ void __launch_bounds__(256)
+grouped_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict__ y, const int* __restrict__ offs,
+                    const int* __restrict__ row_tok, int N, int K, int E, int act) {
+  __shared__ float as[GK][GT + 4], bs[GK][GT + 4];
+  pdl_trigger();
+  pdl_wait();
+  int tile = blockIdx.y, e = 0, lo = 0, hi = 0;
+  for (; e < E; ++e) {
+    lo = offs[e]; hi = offs[e + 1];
+    const int nt = (hi - lo + GT - 1) / GT;
+    if (tile < nt) break;
+    tile -= nt;
+  }
+  if (e == E) return;
+  const int r0 = lo + tile * GT, n0 = blockIdx.x * GT;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += GK) {
+    for (int i = threadIdx.x; i < GT * GK; i += 256) {
+      const int r = i / GK, kk = i % GK, row = r0 + r, n = n0 + r, kc = k0 + kk;
+      as[kk][r] = (row < hi && kc < K) ? to_f32(x[(int64_t)(row_tok ? row_tok[row] : row) * K + kc]) : 0.f;
+      bs[kk][r] = (n < N && kc < K) ? to_f32(w[((int64_t)e * N + n) * K + kc]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < GK; ++kk) {
+      float a[4], b[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) { a[i] = as[kk][ty * 4 + i]; b[i] = bs[kk][tx * 4 + i]; }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] += a[i] * b[j];
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int row = r0 + ty * 4 + i, n = n0 + tx * 4 + j;
+      float v = acc[i][j];
+      if (act == 2) { v = fmaxf(v, 0.f); v *= v; }
+      if (row < hi && n < N) y[(int64_t)row * N + n] = from_f32<T>(v);
+    }
+}
+
 // counting sort of R = T*k (token, slot) pairs by (mapped) expert id.  One CTA.
 //   ids[i]  : global expert of pair i;  emap (optional): global → local expert or -1 (not on this rank)
 //   sorted_tok[p] : token of the pair placed at sorted position p;  inv[i] : sorted position of pair i (or -1)
@@ -218,10 +387,40 @@ EXPORT int vb_moe_topk_softmax(const void* logits, float* out_w, int* out_ids, i
   return (int)cudaGetLastError();
 }
 
+// x / w null: `logits` are given.  dtypes: x fp32 or the model dtype (x_f32), w the model dtype.
+EXPORT int vb_moe_grouped_topk(const float* logits, const void* x, int x_f32, const void* w, int H, const float* bias,
+                               float* out_w, int* out_ids, int n_tokens, int E, int k, int n_group, int keep, int softmax,
+                               int renorm, float scale, int dtype, cudaStream_t st) {
+  if (n_tokens == 0) return 0;
+  if (E < 1 || E > 4096 || k < 1 || k > E || n_group < 1 || E % n_group || keep < 1 || keep > n_group) return -1;
+  if (!logits && (!x || !w)) return -1;
+  const size_t smem = (size_t)(2 * E + n_group + (logits ? 0 : H)) * sizeof(float);
+  if (smem > 48 * 1024) return -3;
+  const int thr = logits ? (E > 128 ? 256 : 64) : 256;
+#define GO(TX, TW) vb_launch(moe::grouped_topk_kernel<TX, TW>, dim3(n_tokens), dim3(thr), smem, st, logits, (const TX*)x, (const TW*)w, H, bias, out_w, out_ids, E, k, n_group, keep, softmax, renorm, scale)
+  DISPATCH_DTYPE(dtype, T, {
+    if (x_f32) GO(float, T); else GO(T, T);
+  });
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+// x [*, K] read through row_tok (null: x is already in sorted order), w [E, N, K], y [R, N]; act: 0 none, 2 squared ReLU
+EXPORT int vb_moe_grouped_simt(const void* x, const void* w, void* y, const int* offs, const int* row_tok, int R, int N, int K,
+                               int E, int act, int dtype, cudaStream_t st) {
+  if (R == 0) return 0;
+  if (act != 0 && act != 2) return -1;
+  const dim3 grid((N + moe::GT - 1) / moe::GT, R / moe::GT + (E < R ? E : R));
+  DISPATCH_DTYPE(dtype, T, {
+    vb_launch(moe::grouped_simt_kernel<T>, grid, dim3(256), 0, st, (const T*)x, (const T*)w, (T*)y, offs, row_tok, N, K, E, act);
+  });
+  return (int)cudaGetLastError();
+}
+
 EXPORT int vb_moe_align2(const int* ids, const int* emap, int* sorted_tok, int* inv, int* offs, int R, int k, int E,
                          int* sorted_pair, cudaStream_t st) {
   if (E > 4096) return -1;
-  vb_launch(moe::align_kernel, dim3(1), dim3(256), (size_t)(2 * E + 1) * sizeof(int), st, ids, emap, sorted_tok, inv, offs,
+  vb_launch(moe::align_kernel, dim3(1), dim3(R > 4096 ? 1024 : 256), (size_t)(2 * E + 1) * sizeof(int), st, ids, emap, sorted_tok, inv, offs,
             R, k, E, sorted_pair);
   return (int)cudaGetLastError();
 }

@@ -1,0 +1,190 @@
+// fp32 residual stream: embedding entry, and "norm the sublayer's output, then add" (post-norm) steps.
+//
+// Models that keep the residual sum in 32-bit and normalise the OUTPUT of every sublayer run two kernels of this file
+// per layer.  The stream x lives in fp32; beside it every step leaves the 16-bit copy the next GEMM reads (or, in front
+// of the LM head, the model's final norm of it), so the conversion never costs a pass of its own:
+//   embed_stream      x = table[id] * scale (+ pos_table[position]);   out = T(x)
+//   post_norm_add     y = a dense sublayer output row, or the routed sum  sum_j w_j * rows[inv_j]  of an expert layer
+//                     x += rmsnorm(y) * w;   out = T(x)  |  T(rmsnorm(x) * w_next)
+// The combine of the expert layer is the load of post_norm_add: expert outputs are read once, summed in slot order in
+// fp32 (deterministic) and never written back.
+#include "common.cuh"
+
+namespace stream {
+
+template <typename T, int V> struct Pack { T e[V]; };
+template <typename T, int V> VB_DEVICE void load_f32(const T* p, float (&v)[V]) {
+  if constexpr (V == 1) {
+    v[0] = to_f32(p[0]);
+  } else if constexpr (sizeof(T) == 4) {
+#pragma unroll
+    for (int i = 0; i < V; i += 4) {
+      const float4 f = *reinterpret_cast<const float4*>(p + i);
+      v[i] = f.x; v[i + 1] = f.y; v[i + 2] = f.z; v[i + 3] = f.w;
+    }
+  } else {
+    const Vec16<T> x = ld16(p);
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = to_f32(x.e[i]);
+  }
+}
+template <typename T, int V> VB_DEVICE void store_f32(T* p, const float (&v)[V]) {
+  if constexpr (V == 1) {
+    p[0] = from_f32<T>(v[0]);
+  } else if constexpr (sizeof(T) == 4) {
+#pragma unroll
+    for (int i = 0; i < V; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+  } else {
+    Vec16<T> x;
+#pragma unroll
+    for (int i = 0; i < V; ++i) x.e[i] = from_f32<T>(v[i]);
+    st16(p, x);
+  }
+}
+
+// one CTA per token; V consecutive elements per access
+template <typename T, int V>
+__global__ void embed_stream_kernel(const int* __restrict__ ids, const int64_t* __restrict__ positions,
+                                    const T* __restrict__ table, const T* __restrict__ pos_table, float scale,
+                                    float* __restrict__ x, T* __restrict__ out, int H, int vocab, int max_pos) {
+  pdl_trigger();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  const int id = min(max(ids[row], 0), vocab - 1);
+  const T* tr = table + (int64_t)id * H;
+  const T* pr = nullptr;
+  if (pos_table) {
+    int64_t p = positions[row];
+    p = p < 0 ? 0 : (p >= max_pos ? max_pos - 1 : p);
+    pr = pos_table + p * H;
+  }
+  for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+    float v[V];
+    load_f32<T, V>(tr + i, v);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] *= scale;
+    if (pr) {
+      float q[V];
+      load_f32<T, V>(pr + i, q);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[j] += q[j];
+    }
+    store_f32<float, V>(x + row * H + i, v);
+    if (out) store_f32<T, V>(out + row * H + i, v);
+  }
+}
+
+// NV vectors of V elements per thread stay in registers between the reductions (H <= 1024 * NV * V)
+template <typename T, int V, int NV>
+__global__ void __launch_bounds__(1024)
+post_norm_add_kernel(const T* __restrict__ y, int64_t y_stride, const int* __restrict__ inv, const float* __restrict__ pair_w,
+                     int k, const T* __restrict__ w, int w_off, float* __restrict__ x, const T* __restrict__ w_next,
+                     int w_next_off, T* __restrict__ out, int H, float eps) {
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  const int step = blockDim.x * V;
+  float v[NV][V];
+  float ss = 0.f;
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * step;
+    if (i >= H) continue;
+    if (inv) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[n][j] = 0.f;
+      for (int s = 0; s < k; ++s) {
+        const int p = inv[row * k + s];
+        if (p < 0) continue;                            // pair computed by another rank
+        const float ws = pair_w[row * k + s];
+        float r[V];
+        load_f32<T, V>(y + (int64_t)p * y_stride + i, r);
+#pragma unroll
+        for (int j = 0; j < V; ++j) v[n][j] += ws * r[j];
+      }
+    } else {
+      load_f32<T, V>(y + row * y_stride + i, v[n]);
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += v[n][j] * v[n][j];
+  }
+  if (w) {
+    const float r1 = rsqrtf(block_sum(ss, red) / (float)H + eps);
+    ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = threadIdx.x * V + n * step;
+      if (i >= H) continue;
+      float g[V], xv[V];
+      load_f32<T, V>(w + i, g);
+      load_f32<float, V>(x + row * H + i, xv);
+#pragma unroll
+      for (int j = 0; j < V; ++j) {
+        v[n][j] = xv[j] + v[n][j] * r1 * (g[j] + (float)w_off);
+        ss += v[n][j] * v[n][j];
+      }
+      store_f32<float, V>(x + row * H + i, v[n]);
+    }
+  }
+  if (!out) return;
+  float r2 = 1.f;
+  if (w_next) r2 = rsqrtf(block_sum(ss, red) / (float)H + eps);
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * step;
+    if (i >= H) continue;
+    if (w_next) {
+      float g[V];
+      load_f32<T, V>(w_next + i, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[n][j] *= r2 * (g[j] + (float)w_next_off);
+    }
+    store_f32<T, V>(out + row * H + i, v[n]);
+  }
+}
+
+template <typename T> constexpr int vec_of() { return sizeof(T) == 4 ? 4 : 8; }
+static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+}  // namespace stream
+
+// x [T, H] fp32 and (optional) out [T, H] in the model dtype; pos_table may be null (no learned positions)
+EXPORT int vb_embed_stream(const int* ids, const int64_t* positions, const void* table, const void* pos_table, float scale,
+                           float* x, void* out, int T_, int H, int vocab, int max_pos, int dtype, cudaStream_t st) {
+  using namespace stream;
+  if (T_ == 0) return 0;
+  DISPATCH_DTYPE(dtype, T, {
+    constexpr int V = vec_of<T>();
+    const bool vec = H % V == 0 && al16(table) && (!pos_table || al16(pos_table)) && al16(x) && (!out || al16(out));
+    const int items = vec ? H / V : H;
+    const int thr = items >= 256 ? 256 : ((items + 31) / 32) * 32;
+    if (vec) vb_launch(embed_stream_kernel<T, V>, dim3(T_), dim3(thr), 0, st, ids, positions, (const T*)table, (const T*)pos_table, scale, x, (T*)out, H, vocab, max_pos);
+    else vb_launch(embed_stream_kernel<T, 1>, dim3(T_), dim3(thr), 0, st, ids, positions, (const T*)table, (const T*)pos_table, scale, x, (T*)out, H, vocab, max_pos);
+  });
+  return (int)cudaGetLastError();
+}
+
+// inv / pair_w null: y is [T, H].  Else y holds expert output rows and inv [T, k] maps (token, slot) to a row (or -1).
+// w null: no norm, no residual (x unused): out = T(y or the routed sum).  w_off / w_next_off: 1 for weights stored
+// around zero.
+EXPORT int vb_post_norm_add(const void* y, int64_t y_stride, const int* inv, const float* pair_w, int k, const void* w,
+                            int w_off, float* x, const void* w_next, int w_next_off, void* out, int T_, int H, float eps,
+                            int dtype, cudaStream_t st) {
+  using namespace stream;
+  if (T_ == 0) return 0;
+  if (w && !x) return -1;
+#define GO(VV, NVV) vb_launch(post_norm_add_kernel<T, VV, NVV>, dim3(T_), dim3(thr), 0, st, (const T*)y, y_stride, inv, pair_w, k, (const T*)w, w_off, x, (const T*)w_next, w_next_off, (T*)out, H, eps)
+  DISPATCH_DTYPE(dtype, T, {
+    constexpr int V = vec_of<T>();
+    const bool vec = H % V == 0 && y_stride % V == 0 && al16(y) && (!w || al16(w)) && (!x || al16(x)) &&
+                     (!w_next || al16(w_next)) && (!out || al16(out));
+    const int items = vec ? H / V : H;
+    const int thr = items >= 1024 ? 1024 : ((items + 31) / 32) * 32;
+    const int nv = (items + thr - 1) / thr;
+    if (vec) { if (nv <= 1) GO(V, 1); else if (nv <= 4) GO(V, 4); else return -1; }
+    else { if (nv <= 1) GO(1, 1); else if (nv <= 16) GO(1, 16); else return -1; }
+  });
+#undef GO
+  return (int)cudaGetLastError();
+}

@@ -107,6 +107,16 @@ class EngineCore:
     def abort_requests(self, request_ids: list[str]) -> None:
         self.scheduler.finish_requests(request_ids, RequestStatus.FINISHED_ABORTED)
 
+    def run_given(self, entries: list[tuple[str, list[int]]], logits_positions: dict[str, list[int]], sampling_params=None
+                  ) -> dict[str, Any]:
+        """One prescribed step (``Scheduler.schedule_given``): request → logits [places, vocab] fp32."""
+        so = self.scheduler.schedule_given(entries, logits_positions, sampling_params)
+        try:
+            return self.model_executor.execute_model(so).logits or {}
+        except Exception:
+            self._dump_failed_step(so)
+            raise
+
     def step(self) -> tuple[dict[int, EngineCoreOutputs], bool]:
         if not self.scheduler.has_requests():
             return {}, False

@@ -172,8 +172,13 @@ def _cmd_launch(argv: list[str]) -> None:
     render_main(argv)
 
 
+def _cmd_trace(argv: list[str]) -> None:
+    from vllm_b200.engine.replay import main
+    main(argv)
+
+
 COMMANDS = {
-    "launch": _cmd_launch,
+    "launch": _cmd_launch, "trace": _cmd_trace,
     "serve": _cmd_serve, "bench": _cmd_bench, "chat": lambda a: _client(a, True),
     "complete": lambda a: _client(a, False), "run-batch": _cmd_run_batch, "collect-env": _cmd_collect_env,
 }

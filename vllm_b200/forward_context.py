@@ -24,6 +24,10 @@ class AttentionMetadata:
     seq_lens: torch.Tensor         # [B] int32, device
     block_table: torch.Tensor      # [B, max_blocks] int32, device
     slot_mapping: torch.Tensor     # [T] int64, device
+    # host copies of query_start_loc / seq_lens (numpy), where the step was prepared eagerly: layers that choose kernels by
+    # the lengths of a mixed batch read them instead of synchronising
+    host_lens: Any = None
+    latent_plan: Any = None        # layers/latent.py: how a mixed step is split between its attention kernels
     query_start_loc_cpu: Optional[torch.Tensor] = None
     seq_lens_cpu: Optional[torch.Tensor] = None
     decode_only: bool = False      # every request has exactly one new token

@@ -213,7 +213,8 @@ class MLAAttentionCore(nn.Module):
     decode kernel in the reference does."""
 
     def __init__(self, num_heads: int, kv_lora_rank: int, qk_rope_head_dim: int, scale: float,
-                 prefix: str = "") -> None:
+                 prefix: str = "", kv_sharing_target: Optional[str] = None) -> None:
+        """``kv_sharing_target``: name of an earlier layer whose cache this one reads (it owns none and writes nothing)."""
         super().__init__()
         self.num_heads, self.kv_lora_rank, self.qk_rope_head_dim = num_heads, kv_lora_rank, qk_rope_head_dim
         self.scale = scale
@@ -221,7 +222,15 @@ class MLAAttentionCore(nn.Module):
         self.head_size = kv_lora_rank + qk_rope_head_dim
         self.num_kv_heads = 1
         self.sliding_window = None
-        _LAYER_REGISTRY[prefix] = self  # type: ignore[assignment]
+        self.kv_sharing_target = kv_sharing_target
+        self.cache_name = kv_sharing_target or prefix
+        if kv_sharing_target is None:
+            _LAYER_REGISTRY[prefix] = self  # type: ignore[assignment]
+            return
+        owner = _LAYER_REGISTRY.get(kv_sharing_target)
+        if not isinstance(owner, MLAAttentionCore) or owner.head_size != self.head_size:
+            raise ValueError(f"layer {prefix!r} shares the cache of {kv_sharing_target!r}, which is not an earlier latent "
+                             f"cache of width {self.head_size} on this rank")
 
     def get_kv_cache_spec(self, block_size: int, dtype_size: int) -> KVCacheSpec:
         from vllm_b200.parallel.state import get_dcp_group
@@ -275,14 +284,19 @@ class MLAAttentionCore(nn.Module):
         out = (o_c * wc[..., None] + o_new * wn[..., None]) / (wc + wn)[..., None]
         return out.to(q_nope_abs.dtype)
 
-    def forward(self, q_nope_abs: torch.Tensor, q_pe: torch.Tensor, kv_c: torch.Tensor, k_pe: torch.Tensor
-                ) -> torch.Tensor:
+    def bound_cache(self):
+        """(metadata, cache) of this step; (None, None) in a profiling run."""
         ctx = get_forward_context()
-        md = ctx.metadata_for(self.layer_name)
-        kv_cache = ctx.kv_caches.get(self.layer_name)
+        md = ctx.metadata_for(self.cache_name)
+        kv_cache = ctx.kv_caches.get(self.cache_name)
         if md is not None and kv_cache is None:
             raise RuntimeError(f"MLA layer {self.layer_name!r} has no KV cache bound")
-        if md is None or kv_cache is None:
+        return (md, kv_cache) if md is not None else (None, None)
+
+    def forward(self, q_nope_abs: torch.Tensor, q_pe: torch.Tensor, kv_c: torch.Tensor, k_pe: torch.Tensor
+                ) -> torch.Tensor:
+        md, kv_cache = self.bound_cache()
+        if md is None:
             return torch.zeros_like(q_nope_abs)
         from vllm_b200.parallel.state import get_dcp_group
         if get_dcp_group().world_size > 1:

@@ -84,6 +84,21 @@ class ReplicatedLinear(LinearBase):
         param.data.copy_(w)
 
 
+class MergedReplicatedLinear(ReplicatedLinear):
+    """Several replicated matrices over the same input, stacked along the output dim (one GEMM)."""
+
+    def __init__(self, input_size, output_sizes: list[int], bias=False, dtype=None, quant_config=None, prefix="") -> None:
+        self.output_sizes = list(output_sizes)
+        super().__init__(input_size, sum(output_sizes), bias, dtype, quant_config, prefix)
+
+    def weight_loader(self, param: nn.Parameter, w: torch.Tensor, shard_id=None) -> None:
+        if shard_id is None:
+            return super().weight_loader(param, w)
+        dst = param.data.narrow(0, sum(self.output_sizes[:shard_id]), self.output_sizes[shard_id])
+        assert dst.shape == w.shape, (self.prefix, shard_id, dst.shape, w.shape)
+        dst.copy_(w)
+
+
 class ColumnParallelLinear(LinearBase):
     """Y = X W^T with W split along the output dim."""
 

@@ -28,9 +28,13 @@ class FusedMoE(nn.Module):
                  renormalize: bool = True, use_grouped_topk: bool = False, n_group: int = 1, topk_group: int = 1,
                  scoring_func: str = "softmax", routed_scaling_factor: float = 1.0, e_score_bias: bool = False,
                  act: str = "silu", enable_ep: bool = False, reduce_results: bool = True, prefix: str = "",
-                 quant_config=None) -> None:
+                 quant_config=None, gated: bool = True) -> None:
         super().__init__()
         g = get_tp_group()
+        # ``gated`` False: an expert is up → act → down and ``w13_weight`` holds the up projection alone
+        self.gated = gated
+        if not gated and quant_config is not None and getattr(quant_config, "name", "") == "fp8_block":
+            raise NotImplementedError("block-scaled fp8 experts are gated")
         self.tp_rank, self.tp_size = max(g.rank_in_group, 0), g.world_size
         self.num_experts, self.top_k = num_experts, top_k
         self.renormalize = renormalize
@@ -93,7 +97,7 @@ class FusedMoE(nn.Module):
             self.expert_map = None
             self.inter_per_rank = divide(intermediate_size, self.tp_size)
         I = self.inter_per_rank
-        self.w13_weight = nn.Parameter(torch.empty(max(self.local_experts, 1), 2 * I, hidden_size, dtype=dt),
+        self.w13_weight = nn.Parameter(torch.empty(max(self.local_experts, 1), (2 if gated else 1) * I, hidden_size, dtype=dt),
                                        requires_grad=False)
         self.w2_weight = nn.Parameter(torch.empty(max(self.local_experts, 1), hidden_size, I, dtype=dt),
                                       requires_grad=False)
@@ -129,10 +133,11 @@ class FusedMoE(nn.Module):
             w = w * self.routed_scaling_factor
         return w, ids
 
-    def forward(self, x: torch.Tensor, router_logits: torch.Tensor) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, router_logits: Optional[torch.Tensor] = None, routing: Optional[tuple] = None) -> torch.Tensor:
+        """``routing``: (weights [T, k], ids [T, k]) of a router that stands in front of the layer (``GroupedRouter``)."""
         shape = x.shape
         x2 = x.reshape(-1, shape[-1])
-        w, ids = self.select_experts(router_logits.reshape(-1, router_logits.shape[-1]))
+        w, ids = routing if routing is not None else self.select_experts(router_logits.reshape(-1, router_logits.shape[-1]))
         if self.wide_ep:
             out = self.a2a.dispatch_combine(x2, w.to(torch.float32), ids, self._local_experts,
                                             reduce_tp=self.reduce_results)
@@ -147,12 +152,22 @@ class FusedMoE(nn.Module):
             out = get_tp_group().all_reduce(out)
         return out.reshape(shape)
 
+    def forward_post_norm(self, x: torch.Tensor, routing: tuple, stream: torch.Tensor, norm, next_norm=None) -> torch.Tensor:
+        """In place on the fp32 residual stream: stream += norm(moe(x)).  Returns the next GEMM's input (the stream in x's
+        dtype, or ``next_norm`` of it).  On one rank the top-k combine is part of the norm kernel's load."""
+        nw, ng = (None, False) if next_norm is None else (next_norm.weight, next_norm.gemma)
+        if self.tp_size == 1 and not (self.gated or self.ep or self.wide_ep or self.eplb):
+            w, ids = routing
+            return ops.fused_moe_post_norm(stream, x, self.w13_weight, self.w2_weight, w, ids, self.act, self.expert_map,
+                                           norm.weight, norm.eps, norm.gemma, nw, ng)
+        return ops.post_norm_add(stream, self.forward(x, routing=routing), norm.weight, norm.eps, norm.gemma, nw, ng)
+
     def forward_reduce_norm(self, x: torch.Tensor, router_logits: torch.Tensor, residual: torch.Tensor, norm):
         """(normed, residual) = norm(all_reduce(moe(x)) + residual) with the combine, the cross-rank reduction, the
         residual add and the RMSNorm fused around the grouped GEMMs (``ops/moe.py::fused_moe_reduce_norm``): the w2
         epilogue red.adds every weighted row into the accumulator of the rank that owns the token.  None = not covered
         (wide EP, EPLB, fp8 experts, prefill-sized batches, CPU) → the caller uses the unfused sequence."""
-        if (not x.is_cuda or self.wide_ep or self.eplb or self.fp8_block or norm is None
+        if (not x.is_cuda or self.wide_ep or self.eplb or self.fp8_block or norm is None or not self.gated
                 or x.dtype not in (torch.bfloat16, torch.float16) or self.w13_weight.dtype != x.dtype):
             return None
         from vllm_b200 import envs
@@ -233,7 +248,7 @@ class FusedMoE(nn.Module):
         """Contribution of the experts this rank owns (ids are global; the expert map drops the others)."""
         if self.fp8_block and self.w13_weight.dtype == torch.float8_e4m3fn:
             return self._forward_fp8(x2, w, ids)
-        return ops.fused_moe(x2, self.w13_weight, self.w2_weight, w, ids, self.act, self.expert_map)
+        return ops.fused_moe(x2, self.w13_weight, self.w2_weight, w, ids, self.act, self.expert_map, self.gated)
 
     def _dequant(self, wq: torch.Tensor, scale: torch.Tensor) -> torch.Tensor:
         blk = self.fp8_block
@@ -320,6 +335,30 @@ class FusedMoE(nn.Module):
         else:
             off = 0 if shard_id == "w1" else I
             param.data[le, off:off + I].copy_(w[r0:r0 + I])
+
+
+class GroupedRouter(nn.Module):
+    """Expert choice in 32-bit straight from the residual stream: scores (sigmoid or softmax) of x W^T, a selection bias
+    that does not enter the weights, and group-limited top-k.  Decode batches are one kernel (csrc/moe.cu); the logits of
+    larger ones come from one product with fp32 output."""
+
+    def __init__(self, hidden_size: int, num_experts: int, top_k: int, dtype=None, n_group: int = 1, topk_group: int = 1,
+                 scoring_func: str = "sigmoid", renormalize: bool = False, routed_scaling_factor: float = 1.0,
+                 selection_bias: bool = True) -> None:
+        super().__init__()
+        if not 1 <= top_k <= num_experts or num_experts % n_group or not 1 <= topk_group <= n_group:
+            raise ValueError(f"router: top {top_k} of {num_experts} experts, {topk_group} of {n_group} groups")
+        if top_k > topk_group * (num_experts // n_group):
+            raise ValueError(f"router: {topk_group} groups of {num_experts // n_group} hold fewer than {top_k} experts")
+        self.top_k, self.n_group, self.topk_group = top_k, n_group, topk_group
+        self.scoring_func, self.renormalize, self.routed_scaling_factor = scoring_func, renormalize, routed_scaling_factor
+        self.weight = nn.Parameter(torch.empty(num_experts, hidden_size, dtype=dtype or torch.get_default_dtype()),
+                                   requires_grad=False)
+        self.bias = nn.Parameter(torch.zeros(num_experts, dtype=torch.float32), requires_grad=False) if selection_bias else None
+
+    def forward(self, x: torch.Tensor, x_half: Optional[torch.Tensor] = None) -> tuple[torch.Tensor, torch.Tensor]:
+        return ops.router_topk(x, self.weight, self.top_k, self.n_group, self.topk_group, self.renormalize, self.scoring_func,
+                               self.bias, self.routed_scaling_factor, x_half)
 
 
 def make_expert_params_mapping(gate_name: str, down_name: str, up_name: str, num_experts: int,

@@ -111,6 +111,9 @@ def get_model(vllm_config: VllmConfig, device: torch.device,
     mc, lc = vllm_config.model_config, vllm_config.load_config
     cls = resolve_model_cls(mc.architecture, getattr(mc, "model_impl", "auto"))
     t0 = time.perf_counter()
+    if device.type == "cuda" and getattr(cls, "kernel_sources", None):
+        from vllm_b200.ops import cuda_ops
+        cuda_ops().prebuild(cls.kernel_sources)
     old = torch.get_default_dtype()
     torch.set_default_dtype(mc.torch_dtype)
     try:

@@ -14,6 +14,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "LlamaForCausalLM": ("llama", "LlamaForCausalLM"),
     "LLaMAForCausalLM": ("llama", "LlamaForCausalLM"),
     "MistralForCausalLM": ("llama", "MistralForCausalLM"),
+    "PomipelForCausalLM": ("pomipel", "PomipelForCausalLM"),
     "Qwen2ForCausalLM": ("llama", "Qwen2ForCausalLM"),
     "Qwen3ForCausalLM": ("llama", "Qwen3ForCausalLM"),
     "GemmaForCausalLM": ("llama", "GemmaForCausalLM"),

@@ -156,11 +156,60 @@ def paged_attention(q, kv_cache, md, scale, sliding_window=None, logits_soft_cap
 
 
 def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank):
-    if _use_cuda(q_pe):
+    """``q_pe`` None: no rope part."""
+    if _use_cuda(q_nope_abs):
         return cuda_ops().mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank)
     sl = md.seq_lens_cpu if md.seq_lens_cpu is not None else md.seq_lens.cpu()
     qsl = md.query_start_loc_cpu if md.query_start_loc_cpu is not None else md.query_start_loc.cpu()
+    if q_pe is None:
+        q_pe = q_nope_abs[..., :0]
     return ref.mla_decode_attention(q_nope_abs, q_pe, kv_cache, md.block_table, sl, qsl, scale, kv_lora_rank)
+
+
+def mla_attention_rows(q_abs, q_pe, kv_cache, block_table, seq_lens, max_len: int, scale):
+    """Attention over the latent cache for rows with a block table and a number of visible keys each (CUDA)."""
+    cu = cuda_ops()
+    if cu._mla_tc_ok(q_abs, q_pe, kv_cache):
+        return cu.mla_decode_tc(q_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_len)
+    return cu.mla_simt(q_abs, q_pe, kv_cache, block_table, seq_lens, None, scale)
+
+
+def latent_expand_ok(q, v_dim: int, kv_rank: int) -> bool:
+    """Can prompt portions run over expanded keys and values (csrc/mla_prefill.cu)?"""
+    return _use_cuda(q) and cuda_ops().mla_prefill_ok(q, v_dim, kv_rank)
+
+
+def gather_latents(kv_cache, block_table, cu_kv, num_kv: int, max_kv: int):
+    """Cached rows of a batch of sequences, contiguous [num_kv, R] (CUDA)."""
+    out = torch.empty((num_kv, kv_cache.shape[-1]), dtype=kv_cache.dtype, device=kv_cache.device)
+    return cuda_ops().gather_cache(kv_cache, block_table, cu_kv, out, max_kv)
+
+
+def mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0: int, max_q: int, scale) -> None:
+    cuda_ops().mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0, max_q, scale)
+
+
+def latent_norm_cache(lat, q_rank, q_weight, kv_rank, kv_weight, eps, cache=None, slots=None):
+    """RMSNorm of both halves of a latent down-projection; the key / value latents go into their cache rows (and are
+    returned by themselves where no cache is bound)."""
+    if _use_cuda(lat):
+        return cuda_ops().latent_norm_cache(lat, q_rank, q_weight, kv_rank, kv_weight, eps, cache, slots, want_kv=cache is None)
+    return ref.latent_norm_cache(lat, q_rank, q_weight, kv_rank, kv_weight, eps, cache, slots)
+
+
+def embed_stream(ids, positions, table, pos_table=None, scale: float = 1.0):
+    """Entry of an fp32 residual stream: (table[id] * scale + pos_table[position] in fp32, the same in the table's dtype)."""
+    if _use_cuda(table):
+        return cuda_ops().embed_stream(ids, positions, table, pos_table, scale)
+    return ref.embed_stream(ids, positions, table, pos_table, scale)
+
+
+def post_norm_add(x, y, weight, eps, gemma=False, next_weight=None, next_gemma=False):
+    """In place on the fp32 stream: x += rmsnorm(y) * w.  Returns the next GEMM's input in y's dtype: x, or its norm with
+    ``next_weight``."""
+    if _use_cuda(x):
+        return cuda_ops().post_norm_add(x, y, weight, eps, gemma, next_weight, next_gemma)
+    return ref.post_norm_add(x, y, weight, eps, gemma, next_weight, next_gemma)
 
 
 def merge_attn_states(o1, lse1, o2, lse2):
@@ -190,10 +239,32 @@ def grouped_topk(scores, k, n_group, topk_group, renormalize, scoring="sigmoid",
     return ref.grouped_topk(scores, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor)
 
 
-def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None):
+def router_topk(x, gate, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None, routed_scaling_factor=1.0,
+                x_half=None):
+    """Router with 32-bit logits: (weights fp32 [T, k], ids [T, k]) of x [T, H] (fp32 stream or model dtype) with gate [E, H]."""
     if _use_cuda(x):
-        return cuda_ops().fused_moe(x, w13, w2, topk_w, topk_ids, act, expert_map)
-    return ref.fused_moe(x, w13, w2, topk_w, topk_ids, act, expert_map)
+        return cuda_ops().router_topk(x, gate, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor, x_half)
+    return ref.grouped_topk(x.float() @ gate.float().t(), k, n_group, topk_group, renormalize, scoring, bias,
+                            routed_scaling_factor)
+
+
+def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None, gated: bool = True):
+    """``gated`` False: w13 is the plain up projection [E, I, H]."""
+    if _use_cuda(x):
+        return cuda_ops().fused_moe(x, w13, w2, topk_w, topk_ids, act, expert_map, gated)
+    return ref.fused_moe(x, w13, w2, topk_w, topk_ids, act, expert_map, gated)
+
+
+def fused_moe_post_norm(stream, x, w_up, w_down, topk_w, topk_ids, act, expert_map, weight, eps, gemma=False, next_weight=None,
+                        next_gemma=False):
+    """post_norm_add of the routed sum of ungated experts; on CUDA the combine is the load of that kernel."""
+    if _use_cuda(x):
+        from vllm_b200.ops.moe import expert_rows_plain
+        rows, inv = expert_rows_plain(x, w_up, w_down, topk_ids, act, expert_map)
+        return cuda_ops().post_norm_add(stream, rows, weight, eps, gemma, next_weight, next_gemma, inv,
+                                        topk_w.to(torch.float32).contiguous())
+    return ref.post_norm_add(stream, ref.fused_moe(x, w_up, w_down, topk_w, topk_ids, act, expert_map, False), weight, eps, gemma,
+                             next_weight, next_gemma)
 
 
 def block_fp8_linear(x, wq, w_scale, block=128, bias=None):

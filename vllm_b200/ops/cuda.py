@@ -1,8 +1,11 @@
 """ctypes bindings to ``vllm_b200/_C.so`` (built by ``vllm_b200/csrc/build.py``).
 
 Every wrapper passes raw device pointers + the current CUDA stream, so the calls are
-CUDA-graph capturable.  A missing / stale library raises at import: on a GPU box the
-kernels are the only path (no silent PyTorch fallback).
+CUDA-graph capturable.  On a GPU box the kernels are the only path (no silent PyTorch fallback).
+
+A symbol is looked up at its first call.  In a checkout where nothing was built ahead (no ``_C.so``) the source file
+that defines it is compiled then, by itself: a process compiles the kernels its model uses and no others
+(``prebuild`` does a known set in parallel).
 """
 from __future__ import annotations
 
@@ -17,14 +20,53 @@ from vllm_b200 import envs
 _LIB_PATH = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "_C.so")
 
 
-def _load() -> ctypes.CDLL:
+_libs: dict[str, ctypes.CDLL] = {}
+
+
+def _library_for(name: str) -> ctypes.CDLL:
+    """The library that holds symbol ``name``: the full build where there is one, else its source's own."""
+    path = _LIB_PATH
+    if not os.path.exists(path):
+        from vllm_b200.csrc import build as b
+        path = b.build_source(b.source_of(name))
+    if path not in _libs:
+        _libs[path] = ctypes.CDLL(path)
+    return _libs[path]
+
+
+def prebuild(sources) -> None:
+    """Compile these sources (names without suffix) in parallel, unless the full library exists."""
     if not os.path.exists(_LIB_PATH):
-        from vllm_b200.csrc.build import build
-        build()
-    return ctypes.CDLL(_LIB_PATH)
+        from vllm_b200.csrc import build as b
+        b.build_sources(sources)
 
 
-_lib = _load()
+class _Symbol:
+    __slots__ = ("name", "argtypes", "fn")
+
+    def __init__(self, name: str, argtypes: tuple) -> None:
+        self.name, self.argtypes, self.fn = name, argtypes, None
+
+    def resolve(self):
+        fn = getattr(_library_for(self.name), self.name)
+        fn.argtypes = list(self.argtypes)
+        fn.restype = ctypes.c_int
+        self.fn = fn
+        return fn
+
+    def __call__(self, *args):
+        return (self.fn or self.resolve())(*args)
+
+
+_symbols: list[_Symbol] = []
+
+
+def resolve_all() -> None:
+    """Look every declared symbol up (a build check: a missing one raises)."""
+    for sym in _symbols:
+        sym.resolve()
+
+
 _vp, _i, _i64, _f = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_float
 
 _DT = {torch.bfloat16: 0, torch.float16: 1, torch.float32: 2}
@@ -32,11 +74,10 @@ _ACT = {"silu": 0, "gelu": 1, "gelu_tanh": 2, "gelu_pytorch_tanh": 2, "relu": 3,
         "quick_gelu": 6, "relu2": 7}
 
 
-def _sig(name: str, *argtypes):
-    fn = getattr(_lib, name)
-    fn.argtypes = list(argtypes)
-    fn.restype = ctypes.c_int
-    return fn
+def _sig(name: str, *argtypes) -> _Symbol:
+    sym = _Symbol(name, argtypes)
+    _symbols.append(sym)
+    return sym
 
 
 _rms_norm = _sig("vb_rms_norm", _vp, _vp, _vp, _vp, _i, _i, _i64, _f, _i, _i, _vp)
@@ -325,9 +366,34 @@ def merge_attn_states(o1, lse1, o2, lse2):
     return out, lse
 
 
-_mla_decode = _sig("vb_mla_decode", _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i64, _i64, _i64, _i64, _i64,
-                   _i, _i, _f, _i, _vp)
+_mla_decode = _sig("vb_mla_decode", _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i64, _i64,
+                   _i64, _i64, _i64, _i, _i, _f, _i, _vp)
+_mla_prefill = _sig("vb_mla_prefill", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i64, _i, _i, _i, _i, _i, _i64, _i64,
+                    _i64, _i64, _i, _f, _i, _vp)
+_mla_simt = _sig("vb_mla_simt", _vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _i, _i, _i, _i, _i, _i, _i64, _i64, _i64, _i64, _i64,
+                 _i64, _f, _i, _vp)
+_latent_norm = _sig("vb_latent_norm_cache", _vp, _i64, _i, _vp, _vp, _i, _vp, _vp, _vp, _i64, _vp, _i, _f, _i, _vp)
 _mla_ws: dict[int, tuple] = {}
+_kernel_error: dict[int, torch.Tensor] = {}
+
+
+def kernel_error_flag(device: torch.device) -> torch.Tensor:
+    """Device int that a kernel with bounded waits raises when one of them ran into its limit."""
+    key = device.index or 0
+    t = _kernel_error.get(key)
+    if t is None:
+        if torch.cuda.is_current_stream_capturing():
+            raise RuntimeError("the kernel error flag must be allocated before CUDA-graph capture")
+        t = _kernel_error[key] = torch.zeros(1, dtype=torch.int32, device=device)
+    return t
+
+
+def check_kernel_error(device: torch.device) -> None:
+    """Raise if a kernel gave up on a wait since the last check (synchronises)."""
+    t = _kernel_error.get(device.index or 0)
+    if t is not None and int(t.item()):
+        t.zero_()
+        raise RuntimeError("a kernel gave up waiting for a copy or a matrix product; its outputs are not valid")
 
 
 def mla_decode_splits(B: int, H: int, max_seq_len: int) -> int:
@@ -344,9 +410,10 @@ def mla_decode_splits(B: int, H: int, max_seq_len: int) -> int:
 
 def mla_decode_tc(q_nope_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_seq_len: int, num_splits: int = 0,
                   return_lse: bool = False):
-    """tcgen05 MLA decode (csrc/mla_decode.cu): q_nope_abs [B, H, 512], q_pe [B, H, 64], cache [blocks, BS, 576]."""
+    """tcgen05 MLA decode (csrc/mla_decode.cu): q_nope_abs [B, H, R], q_pe [B, H, 64] or None, cache [blocks, BS, R (+64)]."""
     B, H, R = q_nope_abs.shape
-    assert R == 512 and q_pe.shape[-1] == 64 and kv_cache.shape[-1] == 576 and q_nope_abs.stride(-1) == 1 and q_pe.stride(-1) == 1
+    P = 0 if q_pe is None else q_pe.shape[-1]
+    assert kv_cache.shape[-1] == R + P and q_nope_abs.stride(-1) == 1 and (q_pe is None or q_pe.stride(-1) == 1)
     dev = q_nope_abs.device
     splits = num_splits or mla_decode_splits(B, H, max_seq_len)
     out = torch.empty((B, H, R), dtype=q_nope_abs.dtype, device=dev)
@@ -360,108 +427,131 @@ def mla_decode_tc(q_nope_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_
             if torch.cuda.is_current_stream_capturing():
                 raise RuntimeError("MLA split-KV workspace must be allocated before CUDA-graph capture")
             n = max(need, 64 * 128 * 4)
-            ws = _mla_ws[key] = (torch.empty(n * R, dtype=torch.float32, device=dev),
+            ws = _mla_ws[key] = (torch.empty(n * 512, dtype=torch.float32, device=dev),
                                  torch.empty(n, dtype=torch.float32, device=dev))
         po, pl = ws
-    _check(_mla_decode(q_nope_abs.data_ptr(), q_pe.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0],
-                       block_table.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), _p(po), _p(pl), _p(lse), B, H,
-                       kv_cache.shape[1], q_nope_abs.stride(0), q_nope_abs.stride(1), q_pe.stride(0), q_pe.stride(1),
+    err = kernel_error_flag(dev)
+    _check(_mla_decode(q_nope_abs.data_ptr(), _p(q_pe), kv_cache.data_ptr(), kv_cache.shape[0],
+                       block_table.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), _p(po), _p(pl), _p(lse), err.data_ptr(), B,
+                       H, R, P, kv_cache.shape[1], q_nope_abs.stride(0), q_nope_abs.stride(1),
+                       q_pe.stride(0) if P else 0, q_pe.stride(1) if P else 0,
                        out.stride(0), block_table.stride(0), splits, scale, _DT[q_nope_abs.dtype], _st()),
-           f"mla_decode(B={B},H={H})", 2 if splits > 1 else 1)
+           f"mla_decode(B={B},H={H},R={R})", 2 if splits > 1 else 1)
     return (out, lse) if return_lse else out
 
 
 def _mla_tc_ok(q_nope_abs, q_pe, kv_cache) -> bool:
-    return (q_nope_abs.dtype in (torch.bfloat16, torch.float16) and kv_cache.dtype == q_nope_abs.dtype
-            and q_nope_abs.shape[-1] == 512 and q_pe.shape[-1] == 64 and kv_cache.dim() == 3 and kv_cache.shape[-1] == 576
-            and kv_cache.shape[1] in (16, 32, 64, 128) and q_nope_abs.stride(-1) == 1 and q_pe.stride(-1) == 1
+    R = q_nope_abs.shape[-1]
+    if q_pe is None:
+        shape_ok = q_nope_abs.dtype == torch.bfloat16 and R % 8 == 0 and R <= 512 and kv_cache.shape[-1] == R
+    else:
+        shape_ok = (q_nope_abs.dtype in _HALF_DTYPES and R == 512 and q_pe.shape[-1] == 64 and kv_cache.shape[-1] == 576
+                    and q_pe.stride(-1) == 1 and (q_pe.stride(0) * 2) % 16 == 0 and (q_pe.stride(1) * 2) % 16 == 0)
+    return (shape_ok and kv_cache.dtype == q_nope_abs.dtype and kv_cache.dim() == 3
+            and kv_cache.shape[1] in (16, 32, 64, 128) and q_nope_abs.stride(-1) == 1
             and (q_nope_abs.stride(0) * 2) % 16 == 0 and (q_nope_abs.stride(1) * 2) % 16 == 0
-            and (q_pe.stride(0) * 2) % 16 == 0 and (q_pe.stride(1) * 2) % 16 == 0 and envs.VLLM_B200_ATTN != "simt")
+            and q_nope_abs.data_ptr() % 16 == 0 and envs.VLLM_B200_ATTN != "simt")
+
+
+_HALF_DTYPES = (torch.bfloat16, torch.float16)
+
+
+def mla_simt(q_abs, q_pe, kv_cache, block_table, seq_lens, qsl, scale):
+    """Variable-length attention over the latent cache for any width and dtype (csrc/latent.cu); fp32 arithmetic."""
+    T, H, R = q_abs.shape
+    P = 0 if q_pe is None else q_pe.shape[-1]
+    assert kv_cache.shape[-1] == R + P and kv_cache.dtype == q_abs.dtype and kv_cache.is_contiguous()
+    q_abs = q_abs if q_abs.stride(-1) == 1 else q_abs.contiguous()
+    q_pe = q_pe if q_pe is None or q_pe.stride(-1) == 1 else q_pe.contiguous()
+    out = torch.empty((T, H, R), dtype=q_abs.dtype, device=q_abs.device)
+    _check(_mla_simt(q_abs.data_ptr(), _p(q_pe), kv_cache.data_ptr(), out.data_ptr(), block_table.data_ptr(),
+                     block_table.stride(0), seq_lens.data_ptr(), _p(qsl), seq_lens.numel(), T, H, R, P, kv_cache.shape[1],
+                     q_abs.stride(0), q_abs.stride(1), q_pe.stride(0) if P else 0, q_pe.stride(1) if P else 0,
+                     out.stride(0), out.stride(1), scale, _DT[q_abs.dtype], _st()), f"mla_simt(T={T},H={H},R={R})")
+    return out
+
+
+def mla_prefill_ok(q, v_dim: int, kv_lora_rank: int) -> bool:
+    D = q.shape[-1]
+    return (q.dtype in _HALF_DTYPES and D % 8 == 0 and 8 <= D <= 128 and v_dim % 8 == 0 and 8 <= v_dim <= 128
+            and kv_lora_rank % 8 == 0 and envs.VLLM_B200_ATTN != "simt")
+
+
+def mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0: int, max_q: int, scale) -> None:
+    """Causal attention of prompt portions over expanded keys and values (csrc/mla_prefill.cu), written into ``out``.
+    q [T, H, dim], out [T, H, vdim]; k [KV, hl, dim], v [KV, hl, vdim] hold heads h0 .. h0 + hl - 1."""
+    T, H, D = q.shape
+    KV, hl, _ = k.shape
+    VD = v.shape[-1]
+    assert q.stride(2) == 1 and q.stride(1) == D and k.stride(2) == 1 and k.stride(1) == D and v.stride(2) == 1 and v.stride(1) == VD
+    assert out.shape == (T, H, VD) and out.stride(1) == VD and out.stride(2) == 1
+    for t in (q, k, v, out):
+        assert t.data_ptr() % 16 == 0
+    _check(_mla_prefill(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), q_start.data_ptr(), q_len.data_ptr(),
+                        seq_len.data_ptr(), kv_start.data_ptr(), kernel_error_flag(q.device).data_ptr(), q_len.numel(), T, KV, H,
+                        h0, hl, D, VD, q.stride(0), k.stride(0), v.stride(0), out.stride(0), max_q, scale, _DT[q.dtype], _st()),
+           f"mla_prefill(T={T},KV={KV},H={H})")
+
+
+def latent_norm_cache(lat, q_rank: int, q_weight, kv_rank: int, kv_weight, eps: float, cache=None, slots=None, want_kv: bool = True):
+    """(c_q, c_kv): RMSNorm of the two halves of a latent down-projection [T, q_rank + kv_rank]; c_kv also goes into its
+    cache rows (csrc/latent.cu).  kv_rank = 0: queries only."""
+    T = lat.shape[0]
+    cq = torch.empty((T, q_rank), dtype=lat.dtype, device=lat.device)
+    ckv = torch.empty((T, kv_rank), dtype=lat.dtype, device=lat.device) if kv_rank and want_kv else None
+    if cache is not None:
+        assert cache.shape[-1] == kv_rank and cache.dtype == lat.dtype and cache.is_contiguous() and slots.dtype == torch.int64
+    _check(_latent_norm(lat.data_ptr(), lat.stride(0), q_rank, _p(q_weight), cq.data_ptr(), kv_rank, _p(kv_weight), _p(ckv),
+                        _p(cache), kv_rank, _p(slots) if cache is not None else None, T, eps, _DT[lat.dtype], _st()),
+           "latent_norm_cache")
+    return cq, ckv
 
 
 def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank):
-    """MLA as MQA over the latent cache (K = 576-d latent+rope, V = first 512 dims of the same rows).
+    """MLA as MQA over the latent cache (K = latent (+ rope) row, V = the latent part of the same row).
 
     Decode batches run on the tcgen05 MLA kernel (csrc/mla_decode.cu: the latent tile is shared by all heads of the
     CTA and by both matrix products, split-KV for long contexts; no host synchronisation, graph capturable).
-    Shapes it does not cover (other latent widths) use dense batched GEMMs over the gathered pages; mixed / prefill
-    batches use the variable-length reference loop (eager only)."""
-    from vllm_b200.ops import ref
-    if md.decode_only:
-        B, H, R = q_nope_abs.shape
-        if R == kv_lora_rank and _mla_tc_ok(q_nope_abs, q_pe, kv_cache):
-            return mla_decode_tc(q_nope_abs, q_pe, kv_cache, md.block_table, md.seq_lens, scale, md.max_seq_len,
-                                 md.num_splits or 0)
-        bs = kv_cache.shape[1]
-        nbk = max((md.max_seq_len + bs - 1) // bs, 1)
-        lat = kv_cache[md.block_table[:B, :nbk].long()].reshape(B, nbk * bs, -1)        # [B, S, 576]
-        kc, kp = lat[..., :kv_lora_rank], lat[..., kv_lora_rank:]
-        att = (torch.bmm(q_nope_abs, kc.transpose(1, 2)) + torch.bmm(q_pe, kp.transpose(1, 2))).float() * scale
-        pos = torch.arange(nbk * bs, device=att.device)[None, None, :]
-        att = att.masked_fill(pos >= md.seq_lens[:B, None, None], float("-inf"))
-        p = torch.softmax(att, dim=-1).to(q_nope_abs.dtype)
-        return torch.bmm(p, kc)
-    sl = md.seq_lens_cpu if md.seq_lens_cpu is not None else md.seq_lens.cpu()
-    qsl = md.query_start_loc_cpu if md.query_start_loc_cpu is not None else md.query_start_loc.cpu()
-    return ref.mla_decode_attention(q_nope_abs, q_pe, kv_cache, md.block_table, sl, qsl, scale, kv_lora_rank)
+    Everything it does not cover — other widths with a rope part, fp32, variable-length batches — runs on the generic
+    kernel of csrc/latent.cu, which needs no host lengths either."""
+    R = q_nope_abs.shape[-1]
+    if md.decode_only and R == kv_lora_rank and _mla_tc_ok(q_nope_abs, q_pe, kv_cache):
+        return mla_decode_tc(q_nope_abs, q_pe, kv_cache, md.block_table, md.seq_lens, scale, md.max_seq_len,
+                             md.num_splits or 0)
+    B = md.num_reqs
+    return mla_simt(q_nope_abs, q_pe, kv_cache, md.block_table, md.seq_lens[:B],
+                    None if md.decode_only else md.query_start_loc, scale)
 
 
-# ------------------------------------------------------------------ sampling
-def argmax(logits: torch.Tensor) -> torch.Tensor:
-    B, V = logits.shape
-    out = torch.empty(B, dtype=torch.int64, device=logits.device)
-    _check(_argmax(logits.data_ptr(), logits.stride(0), B, V, out.data_ptr(), _DT[logits.dtype], _st()), "argmax")
-    return out
+# ------------------------------------------------------------------ fp32 residual stream (csrc/stream.cu)
+_embed_stream = _sig("vb_embed_stream", _vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _i, _vp)
+_post_norm = _sig("vb_post_norm_add", _vp, _i64, _vp, _vp, _i, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _f, _i, _vp)
 
 
-_step_buf: dict[int, torch.Tensor] = {}
+def embed_stream(ids, positions, table, pos_table, scale: float):
+    """(x fp32, copy of x in the table's dtype — x itself when that is fp32)."""
+    T, H = ids.numel(), table.shape[1]
+    x = torch.empty((T, H), dtype=torch.float32, device=table.device)
+    out = None if table.dtype == torch.float32 else torch.empty((T, H), dtype=table.dtype, device=table.device)
+    assert ids.dtype == torch.int32 and positions.dtype == torch.int64 and table.is_contiguous()
+    _check(_embed_stream(ids.data_ptr(), positions.data_ptr(), table.data_ptr(), _p(pos_table), float(scale), x.data_ptr(),
+                         _p(out), T, H, table.shape[0], 0 if pos_table is None else pos_table.shape[0], _DT[table.dtype], _st()),
+           "embed_stream")
+    return x, (x if out is None else out)
 
 
-def fused_sample(logits, temperature, seeds, step, out: Optional[torch.Tensor] = None):
-    """``step``: per-row int32 [B] noise counters (a python int is broadcast)."""
-    B, V = logits.shape
-    if out is None:
-        out = torch.empty(B, dtype=torch.int64, device=logits.device)
-    if not isinstance(step, torch.Tensor):
-        step = torch.full((B,), int(step) & 0x7FFFFFFF, dtype=torch.int32, device=logits.device)
-    _check(_fused_sample(logits.data_ptr(), logits.stride(0), B, V, temperature.data_ptr(), seeds.data_ptr(),
-                         step.data_ptr(), out.data_ptr(), _DT[logits.dtype], _st()), "fused_sample")
-    return out
-
-
-_fused_sample_cand = _sig("vb_fused_sample_cand", _vp, _i64, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _vp)
-_select_cand = _sig("vb_select_candidate", _vp, _i, _vp, _i, _vp)
-
-
-def fused_sample_candidates(logits_local, temperature, seeds, step, idx_off: int, v_valid: int) -> torch.Tensor:
-    """Per-row best (value, global id) of this rank's vocab shard as a [B, 8] bf16-viewable 16-byte record."""
-    B = logits_local.shape[0]
-    cand = torch.empty((B, 4), dtype=torch.float32, device=logits_local.device)
-    _check(_fused_sample_cand(logits_local.data_ptr(), logits_local.stride(0), B, max(v_valid, 0), temperature.data_ptr(),
-                              seeds.data_ptr(), step.data_ptr(), idx_off, cand.data_ptr(), _DT[logits_local.dtype], _st()),
-           "fused_sample_cand")
-    return cand
-
-
-def select_candidates(cands: torch.Tensor, W: int, out: torch.Tensor) -> torch.Tensor:
-    """cands: [B, W, 4] fp32 records gathered from the W ranks → winning token id per row."""
-    B = out.shape[0]
-    _check(_select_cand(cands.data_ptr(), W, out.data_ptr(), B, _st()), "select_candidate")
-    return out
-
-
-def topk_topp_mask_(logits: torch.Tensor, top_k, top_p, min_p=None) -> torch.Tensor:
-    assert logits.dtype == torch.float32 and logits.is_contiguous()
-    B, V = logits.shape
-    _check(_topk_topp(logits.data_ptr(), B, V, _p(top_k), _p(top_p), _p(min_p), _st()), "topk_topp")
-    return logits
-
-
-def row_lse(logits: torch.Tensor) -> torch.Tensor:
-    B, V = logits.shape
-    out = torch.empty(B, dtype=torch.float32, device=logits.device)
-    _check(_row_lse(logits.data_ptr(), logits.stride(0), B, V, out.data_ptr(), _DT[logits.dtype], _st()), "row_lse")
-    return out
+def post_norm_add(x, y, weight, eps: float, gemma: bool, next_weight=None, next_gemma: bool = False, inv=None, pair_w=None):
+    """In place: x += rmsnorm(y') * w, y' = y [T, H] or (``inv``, ``pair_w`` [T, k]) the weighted sum of expert rows of y.
+    Returns x in y's dtype (x itself when that is fp32), or its norm with ``next_weight``."""
+    T, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.stride(-1) == 1
+    k = 1 if inv is None else inv.numel() // T
+    out = None
+    if next_weight is not None or y.dtype != torch.float32:
+        out = torch.empty((T, H), dtype=y.dtype, device=y.device)
+    _check(_post_norm(y.data_ptr(), y.stride(0), _p(inv), _p(pair_w), k, weight.data_ptr(), int(gemma), x.data_ptr(),
+                      _p(next_weight), int(next_gemma), _p(out), T, H, eps, _DT[y.dtype], _st()), "post_norm_add")
+    return x if out is None else out
 
 
 # ------------------------------------------------------------------ GEMM
@@ -646,7 +736,7 @@ def gemm_ar(c, x, w, residual, norm_w, out, eps, gemma, mode=0, oring_off=0, ori
 
 def gemm_ar_set_trace(t: Optional[torch.Tensor]) -> None:
     """Point the fused kernel's phase stamps ([n_ctas, 8] int64 globaltimer values) at ``t`` (None = off)."""
-    fn = _lib.vb_gemm_ar_set_trace
+    fn = _library_for("vb_gemm_ar_set_trace").vb_gemm_ar_set_trace
     fn.argtypes, fn.restype = [_vp], None
     fn(t.data_ptr() if t is not None else None)
 
@@ -665,7 +755,10 @@ _comm_ar_rows2 = _sig("vb_comm_allreduce_rows2", _vp, _vp, _vp, _vp, _i, _i, _vp
                       _i, _vp)
 _moe_combine = _sig("vb_moe_combine", _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp)
 _moe_gather = _sig("vb_moe_gather", _vp, _vp, _vp, _i, _i, _i, _vp)
-_gemm_grouped = _sig("vb_gemm_tc_grouped", _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp)
+_gemm_grouped = _sig("vb_gemm_tc_grouped2", _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp)
+_grouped_simt = _sig("vb_moe_grouped_simt", _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp)
+_grouped_topk = _sig("vb_moe_grouped_topk", _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp)
+_GROUPED_ACT = {None: 0, "none": 0, "relu2": 2}
 
 
 def topk_softmax(gating, k, renormalize, scale: float = 1.0):
@@ -738,28 +831,79 @@ def moe_combine(y: torch.Tensor, inv: torch.Tensor, w: torch.Tensor, T: int) -> 
     H = y.shape[1]
     k = inv.numel() // T
     out = torch.empty((T, H), dtype=y.dtype, device=y.device)
-    _check(_moe_combine(y.data_ptr(), inv.data_ptr(), w.data_ptr(), out.data_ptr(), T, H, k, _DT[y.dtype], _st()),
-           "moe_combine")
+    if y.dtype in _HALF_DTYPES and H % 8 == 0:
+        _check(_moe_combine(y.data_ptr(), inv.data_ptr(), w.data_ptr(), out.data_ptr(), T, H, k, _DT[y.dtype], _st()),
+               "moe_combine")
+    else:
+        _check(_post_norm(y.data_ptr(), y.stride(0), inv.data_ptr(), w.data_ptr(), k, None, 0, None, None, 0, out.data_ptr(), T, H,
+                          0.0, _DT[y.dtype], _st()), "moe_combine")
     return out
 
 
-def gemm_tc_grouped(xs: torch.Tensor, w: torch.Tensor, offs: torch.Tensor, bn: int) -> torch.Tensor:
-    """Y[r] = xs[r] · w[e(r)]^T, rows sorted by expert (``offs``). w: [E, N, K]."""
+def gemm_tc_grouped(xs: torch.Tensor, w: torch.Tensor, offs: torch.Tensor, bn: int, act: Optional[str] = None,
+                    flat: bool = False) -> torch.Tensor:
+    """Y[r] = act(xs[r] · w[e(r)]^T), rows sorted by expert (``offs``). w: [E, N, K].  ``flat``: the grid follows the row
+    count (large batches) instead of every chunk an expert could have."""
     R, K = xs.shape
     E, N, _ = w.shape
     y = torch.empty((R, N), dtype=xs.dtype, device=xs.device)
-    _check(_gemm_grouped(xs.data_ptr(), w.data_ptr(), y.data_ptr(), offs.data_ptr(), R, N, K, E, bn, _DT[xs.dtype],
-                         _st()), f"gemm_tc_grouped(R={R},N={N},K={K},E={E})")
+    _check(_gemm_grouped(xs.data_ptr(), w.data_ptr(), y.data_ptr(), offs.data_ptr(), R, N, K, E, bn, _GROUPED_ACT[act], int(flat),
+                         _DT[xs.dtype], _st()), f"gemm_tc_grouped(R={R},N={N},K={K},E={E})")
+    return y
+
+
+def grouped_simt(x: torch.Tensor, w: torch.Tensor, offs: torch.Tensor, R: int, row_tok: Optional[torch.Tensor] = None,
+                 act: Optional[str] = None) -> torch.Tensor:
+    """The grouped product on the CUDA cores (any dtype and row width); ``row_tok`` gathers rows of x on the way in."""
+    E, N, K = w.shape
+    assert x.is_contiguous() and w.is_contiguous() and x.dtype == w.dtype
+    y = torch.empty((R, N), dtype=x.dtype, device=x.device)
+    _check(_grouped_simt(x.data_ptr(), w.data_ptr(), y.data_ptr(), offs.data_ptr(), _p(row_tok), R, N, K, E, _GROUPED_ACT[act],
+                         _DT[x.dtype], _st()), f"grouped_simt(R={R},N={N},K={K},E={E})")
     return y
 
 
 def grouped_topk(scores, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None, routed_scaling_factor=1.0):
-    from vllm_b200.ops import ref
-    return ref.grouped_topk(scores, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor)
+    T, E = scores.shape
+    lg = scores.float().contiguous()
+    w = torch.empty((T, k), dtype=torch.float32, device=scores.device)
+    ids = torch.empty((T, k), dtype=torch.int32, device=scores.device)
+    b = None if bias is None else bias.float().contiguous()
+    _check(_grouped_topk(lg.data_ptr(), None, 0, None, 0, _p(b), w.data_ptr(), ids.data_ptr(), T, E, k, n_group,
+                         topk_group if n_group > 1 else 1, int(scoring != "sigmoid"), int(renormalize), float(routed_scaling_factor),
+                         2, _st()), f"grouped_topk(E={E},k={k})")
+    return w, ids
 
 
-def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None):
+ROUTER_FUSED_TOKENS = 256       # above this the logits come from one tensor-core product with fp32 output
+
+
+def router_topk(x, gate, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None, routed_scaling_factor=1.0, x_half=None):
+    """Routing of x [T, H] (fp32 stream or model dtype) with gate [E, H]: 32-bit logits, scores, choice and weights.
+    ``x_half``: the 16-bit copy of x for the large-batch product."""
+    T, H = x.shape
+    E = gate.shape[0]
+    if T > ROUTER_FUSED_TOKENS or H > 8192:
+        xh = x if x.dtype == gate.dtype else x_half
+        if gate.dtype == torch.float32 or xh is None:
+            lg = x.float() @ gate.float().t()
+        else:
+            lg = torch.mm(xh, gate.t(), out_dtype=torch.float32)
+        return grouped_topk(lg, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor)
+    w = torch.empty((T, k), dtype=torch.float32, device=x.device)
+    ids = torch.empty((T, k), dtype=torch.int32, device=x.device)
+    assert x.is_contiguous() and gate.is_contiguous() and (x.dtype == torch.float32 or x.dtype == gate.dtype)
+    assert bias is None or bias.dtype == torch.float32
+    _check(_grouped_topk(None, x.data_ptr(), int(x.dtype == torch.float32), gate.data_ptr(), H, _p(bias), w.data_ptr(),
+                         ids.data_ptr(), T, E, k, n_group, topk_group if n_group > 1 else 1, int(scoring != "sigmoid"),
+                         int(renormalize), float(routed_scaling_factor), _DT[gate.dtype], _st()), f"router_topk(E={E},k={k},H={H})")
+    return w, ids
+
+
+def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None, gated: bool = True):
     from vllm_b200.ops import moe
+    if not gated:
+        return moe.fused_moe_plain(x, w13, w2, topk_w, topk_ids, act, expert_map)
     return moe.fused_moe_cuda(x, w13, w2, topk_w, topk_ids, act, expert_map)
 
 

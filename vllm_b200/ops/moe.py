@@ -47,6 +47,48 @@ def fused_moe_grouped(x, w13, w2, topk_w, topk_ids, act, expert_map):
     return cu.moe_combine(y, inv, topk_w.to(torch.float32).contiguous(), T)
 
 
+def _tile_width(R: int, E: int) -> int:
+    """Token-tile width: average rows per expert rounded up, so that most experts need one chunk."""
+    avg = max(R // max(E, 1), 1)
+    bn = 16
+    while bn < 128 and bn < 2 * avg:
+        bn += 16
+    return bn
+
+
+def expert_rows_plain(x, w_up, w_down, topk_ids, act, expert_map):
+    """Experts without a gate, up → act → down: (rows [R, H] sorted by expert, inv [R]: (token, slot) pair → row).
+
+    Stays on the device at every batch size (no host sync, graph capturable): the flat grouped GEMM sizes its grid by the
+    row count and finds each tile's expert itself, and the activation is applied in the first GEMM's epilogue.  What the
+    tensor-core kernel does not take (fp32, row widths off the 16-byte grid) runs on the CUDA-core grouped kernel."""
+    from vllm_b200.ops import cuda as cu
+    T, k = topk_ids.shape
+    R, E, (N, K) = T * k, w_up.shape[0], w_up.shape[1:]
+    ids = topk_ids if topk_ids.dtype == torch.int32 else topk_ids.to(torch.int32)
+    sorted_tok, inv, offs = cu.moe_align(ids.contiguous(), E, expert_map)
+    x = x.contiguous()
+    fused_act = act == "relu2"
+    if x.dtype in (torch.bfloat16, torch.float16) and w_up.dtype == x.dtype and K % 8 == 0 and N % 8 == 0:
+        xs = cu.moe_gather(x, sorted_tok)
+        bn = _tile_width(R, E)
+        a = cu.gemm_tc_grouped(xs, w_up, offs, bn, act if fused_act else None, flat=True)
+        if not fused_act:
+            a = cu.activation(a, act)
+        return cu.gemm_tc_grouped(a, w_down, offs, bn, flat=True), inv
+    a = cu.grouped_simt(x, w_up, offs, R, sorted_tok, act if fused_act else None)
+    if not fused_act:
+        from vllm_b200.ops import ref
+        a = ref.ACT_FNS[act](a)
+    return cu.grouped_simt(a, w_down, offs, R), inv
+
+
+def fused_moe_plain(x, w_up, w_down, topk_w, topk_ids, act, expert_map):
+    from vllm_b200.ops import cuda as cu
+    rows, inv = expert_rows_plain(x, w_up, w_down, topk_ids, act, expert_map)
+    return cu.moe_combine(rows, inv, topk_w.to(torch.float32).contiguous(), x.shape[0])
+
+
 def fused_moe_fp8_grouped(x, w13q, w13_scale, w2q, w2_scale, topk_w, topk_ids, expert_map):
     """Block-scaled fp8 experts on the device (DeepSeek-V3 checkpoints): align → gather → per-(token,128) fp8 quant →
     grouped tcgen05 f8f6f4 GEMM (w13) → fused SiLU·mul + re-quant → grouped fp8 GEMM (w2) → weighted combine.  Weight

@@ -299,6 +299,35 @@ def partial_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: 
     return torch.einsum("qhk,khd->qhd", p, vf), lse
 
 
+# ------------------------------------------------------------- latent attention / fp32 residual stream
+def latent_norm_cache(lat: torch.Tensor, q_rank: int, q_weight, kv_rank: int, kv_weight, eps: float, cache=None, slots=None):
+    """RMSNorm of both halves of a latent down-projection [T, q_rank + kv_rank]; c_kv also goes into its cache rows."""
+    cq = rms_norm(lat[:, :q_rank], q_weight, eps)
+    if not kv_rank:
+        return cq, None
+    ckv = rms_norm(lat[:, q_rank:q_rank + kv_rank], kv_weight, eps)
+    if cache is not None:
+        concat_and_cache_mla(ckv, ckv[:, :0], cache, slots)
+    return cq, ckv
+
+
+def embed_stream(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, pos_table: Optional[torch.Tensor],
+                 scale: float) -> tuple[torch.Tensor, torch.Tensor]:
+    x = F.embedding(ids, table).float() * scale
+    if pos_table is not None:
+        x = x + pos_table[positions.long()].float()
+    return x, x.to(table.dtype)
+
+
+def post_norm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float, gemma: bool = False,
+                  next_weight: Optional[torch.Tensor] = None, next_gemma: bool = False) -> torch.Tensor:
+    """In place: x (fp32) += rmsnorm(y) * w.  Returns x in y's dtype, or its norm with ``next_weight``."""
+    x += rms_norm(y.float(), weight, eps, gemma)
+    if next_weight is None:
+        return x.to(y.dtype)
+    return rms_norm(x, next_weight, eps, next_gemma).to(y.dtype)
+
+
 # -------------------------------------------------------------- sampling
 def apply_penalties(logits: torch.Tensor, prompt_mask: torch.Tensor, output_counts: torch.Tensor,
                     presence: torch.Tensor, frequency: torch.Tensor, repetition: torch.Tensor) -> torch.Tensor:
@@ -388,7 +417,7 @@ def grouped_topk(scores_in: torch.Tensor, k: int, n_group: int, topk_group: int,
     sel = s + bias.float()[None] if bias is not None else s
     if n_group > 1:
         g = sel.view(T, n_group, E // n_group)
-        gs = g.topk(2, dim=-1).values.sum(-1) if bias is not None else g.max(-1).values
+        gs = g.topk(min(2, E // n_group), dim=-1).values.sum(-1) if bias is not None else g.max(-1).values
         gi = gs.topk(topk_group, dim=-1).indices
         gm = torch.zeros_like(gs).scatter_(1, gi, 1.0)
         mask = gm[:, :, None].expand(T, n_group, E // n_group).reshape(T, E)
@@ -401,9 +430,9 @@ def grouped_topk(scores_in: torch.Tensor, k: int, n_group: int, topk_group: int,
 
 
 def fused_moe(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor,
-              topk_ids: torch.Tensor, act: str = "silu", expert_map: Optional[torch.Tensor] = None
+              topk_ids: torch.Tensor, act: str = "silu", expert_map: Optional[torch.Tensor] = None, gated: bool = True
               ) -> torch.Tensor:
-    """x [T,H]; w13 [E,2I,H] (gate rows then up rows); w2 [E,H,I]. Returns [T,H]."""
+    """x [T,H]; w13 [E,2I,H] (gate rows then up rows) or, not ``gated``, [E,I,H]; w2 [E,H,I]. Returns [T,H]."""
     T, H = x.shape
     E = w13.shape[0]
     out = torch.zeros(T, H, dtype=torch.float32, device=x.device)
@@ -415,6 +444,10 @@ def fused_moe(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torc
         if tok.numel() == 0:
             continue
         h = x[tok].float() @ w13[e].float().t()
+        if not gated:
+            y = ACT_FNS[act](h).to(x.dtype).float() @ w2[e].float().t()
+            out.index_add_(0, tok, y * topk_w[tok, slot].float()[:, None])
+            continue
         I = h.shape[-1] // 2
         a = F.silu(h[:, :I]) if act == "silu" else F.gelu(h[:, :I])
         h = (a * h[:, I:]).to(x.dtype).float()

@@ -250,7 +250,7 @@ class ModelRunner:
         self.dev_tokens: Optional[torch.Tensor] = None
         self.dev_block_rows: list[torch.Tensor] = []
         self._bt_diffs: list[list[tuple[str, int, list[int]]]] = []
-        self._new_rids: list[str] = []
+        self._new_tokens: list[tuple[str, int]] = []     # (request, first token the device table does not have)
         self.prep_host_s = 0.0  # host seconds spent preparing + uploading step inputs (diagnostic)
         self.prep_decode_s, self.prep_decode_n = 0.0, 0
         self.wait_s = 0.0       # host seconds blocked on the device (D2H of sampled ids, staging reuse)
@@ -447,7 +447,7 @@ class ModelRunner:
             self.block_tables_cpu[g][row, :len(ids)] = ids
             self.num_blocks_cpu[g][row] = len(ids)
         if self.gpu_prep:       # admission: the whole row travels once, with this step's uploads (_flush_gpu_state)
-            self._new_rids.append(st.req_id)
+            self._new_tokens.append((st.req_id, 0))
 
     def _add(self, nr) -> None:
         sp = nr.sampling_params
@@ -481,11 +481,13 @@ class ModelRunner:
             row = self.req_index[rid]
             self.num_computed_cpu[row] = c.num_computed_tokens[i]
             toks = c.new_token_ids[i]
-            if toks:  # PP: tokens sampled on another rank
+            if toks:  # tokens this worker does not have: sampled on another rank (PP), or fed in by the caller
                 n0 = c.num_computed_tokens[i]
                 self.token_ids_cpu[row, n0:n0 + len(toks)] = toks
                 self.num_tokens_cpu[row] = max(self.num_tokens_cpu[row], n0 + len(toks))
                 self.num_logical_cpu[row] = max(self.num_logical_cpu[row], self.num_tokens_cpu[row])
+                if self.gpu_prep:
+                    self._new_tokens.append((rid, n0))
             nb = c.new_block_ids[i]
             if nb is not None:
                 for g in range(self.num_kv_groups):
@@ -593,34 +595,35 @@ class ModelRunner:
         scattered into the tables by ``block_table_apply_diffs`` (row, start, count, offset) entries."""
         cu = self._cu
         R = self.max_num_reqs
-        if self._new_rids:
-            rids, self._new_rids = self._new_rids, []
+        if self._new_tokens:
+            fresh, self._new_tokens = self._new_tokens, []
             pin, cap = stg.input_ids, stg.input_ids.numel()
             pv = pin.numpy()
-            d_row, d_cnt, d_off = [], [], []
+            d_row, d_start, d_cnt, d_off = [], [], [], []
             off = 0
-            for rid in rids:
+            for rid, first in fresh:
                 row = self.req_index.get(rid)
                 if row is None:
                     continue
-                n = int(self.num_tokens_cpu[row])
-                for g in range(self.num_kv_groups):      # the whole block list of the row goes through the diff path
-                    k = int(self.num_blocks_cpu[g][row])
+                n = int(self.num_tokens_cpu[row]) - first
+                for g in range(self.num_kv_groups if first == 0 else 0):
+                    k = int(self.num_blocks_cpu[g][row])  # the whole block list of the row goes through the diff path
                     if k:
                         self._bt_diffs[g].append((rid, 0, self.block_tables_cpu[g][row, :k]))
                 if off + n <= cap and len(d_row) < R:
-                    pv[off:off + n] = self.token_ids_cpu[row, :n]
+                    pv[off:off + n] = self.token_ids_cpu[row, first:first + n]
                     d_row.append(row)
+                    d_start.append(first)
                     d_cnt.append(n)
                     d_off.append(off)
                     off += n
                 else:                       # does not fit the packed upload (very long prompts): pageable row copy
-                    self.dev_tokens[row, :n].copy_(torch.from_numpy(self.token_ids_cpu[row, :n].copy()))
+                    self.dev_tokens[row, first:first + n].copy_(torch.from_numpy(self.token_ids_cpu[row, first:first + n].copy()))
                 self.h2d_bytes += n * 4
             n_e = len(d_row)
             if n_e:
                 hv = stg.tok_hdr.numpy()
-                hv[:n_e], hv[n_e:2 * n_e], hv[2 * n_e:3 * n_e], hv[3 * n_e:4 * n_e] = d_row, 0, d_cnt, d_off
+                hv[:n_e], hv[n_e:2 * n_e], hv[2 * n_e:3 * n_e], hv[3 * n_e:4 * n_e] = d_row, d_start, d_cnt, d_off
                 self.tok_hdr_dev[:4 * n_e].copy_(stg.tok_hdr[:4 * n_e], non_blocking=True)
                 # the step's own input_ids buffer doubles as device scratch: prep_step overwrites it afterwards
                 self.input_ids[:off].copy_(pin[:off], non_blocking=True)
@@ -697,7 +700,8 @@ class ModelRunner:
                          self.positions, self.qsl, self.seq_lens, self.slot_mappings[g], self.block_tables[g], nbk,
                          self.block_size, pad_b=pad_b, write_tokens=(g == 0), pad_t=pad_t)
 
-    def _make_metadata(self, nb, T, max_q, max_s, decode_only, cpu_qsl=None, cpu_sl=None) -> dict[int, AttentionMetadata]:
+    def _make_metadata(self, nb, T, max_q, max_s, decode_only, cpu_qsl=None, cpu_sl=None, host_lens=None
+                       ) -> dict[int, AttentionMetadata]:
         nbk = max(cdiv(max_s, self.vblock), 1)
         out = {}
         for g in range(self.num_kv_groups):
@@ -706,7 +710,7 @@ class ModelRunner:
                 query_start_loc=self.qsl[:nb + 1], seq_lens=self.seq_lens[:nb],
                 block_table=self.block_tables[g][:nb] if self.is_cuda else self.block_tables[g][:nb, :nbk],
                 slot_mapping=self.slot_mappings[g][:T], query_start_loc_cpu=cpu_qsl, seq_lens_cpu=cpu_sl,
-                decode_only=decode_only, kv_vt=self.kv_vt[g])
+                decode_only=decode_only, kv_vt=self.kv_vt[g], host_lens=host_lens)
         return out
 
     # ------------------------------------------------------------ forward
@@ -999,7 +1003,7 @@ class ModelRunner:
         decode_only = max_q == 1 and not has_spec
         pad_b = nb
         graph = None
-        simple = not bool(self.complex_cpu[rows].any()) and so.grammar_bitmask is None
+        simple = not bool(self.complex_cpu[rows].any()) and so.grammar_bitmask is None and so.logits_positions is None
         no_filter = not bool(self.filter_cpu[rows].any())
         kv_meta = so.kv_connector_metadata if self.kv_connector is not None else None
         lora_batch = None
@@ -1054,7 +1058,8 @@ class ModelRunner:
         else:
             l0 = self._launches()
             states = [self.states[r] for r in req_ids]
-            md = self._make_metadata(nb, T, max_q, max_s, decode_only, cpu_qsl, cpu_sl)
+            md = self._make_metadata(nb, T, max_q, max_s, decode_only, cpu_qsl, cpu_sl,
+                                     (cu, self.num_computed_cpu[rows] + ns))
             if so.num_common_prefix_blocks and nb >= self.cascade_min_reqs and self.pcp == 1 and self.dcp == 1:
                 self._add_cascade(md, so.num_common_prefix_blocks, rows, ns, nb, T, max_q, max_s)
             if kv_meta:
@@ -1096,6 +1101,8 @@ class ModelRunner:
                 self.kv_connector.save_kv(kv_meta, self.kv_caches)           # freshly computed full blocks
             if isinstance(hidden, dict):  # non-last PP stage
                 return ModelRunnerOutput(kv_connector_output=hidden)
+            if so.logits_positions is not None:
+                return self._wanted_logits(so, hidden, req_ids, rows, ns, cu, stg, t0)
             if any(s.pooling_params is not None for s in states):
                 return self._pool(hidden, states, rows, cu, produces, t0)
             if has_spec:
@@ -1289,6 +1296,21 @@ class ModelRunner:
             ids, vals, ranks = ref.compute_logprobs(logits, tgt, k)
             out[s.req_id] = LogprobsTensors(ids.cpu(), vals.cpu(), ranks.cpu())
         return out
+
+    def _wanted_logits(self, so, hidden, req_ids, rows, ns, cu, stg, t0) -> ModelRunnerOutput:
+        """Logits at the places the step asks for; the tokens are committed, nothing is sampled."""
+        want = [so.logits_positions.get(r) or [] for r in req_ids]
+        idx = [int(cu[j]) + p for j, w in enumerate(want) for p in w]
+        logits = {}
+        if idx:
+            flat = self.model.compute_logits(hidden[torch.tensor(idx, dtype=torch.int64, device=self.device)]).float().cpu()
+            logits = {r: t for r, t, w in zip(req_ids, flat.split([len(w) for w in want]), want) if w}
+        if self.is_cuda:
+            stg.event.record()
+        self.num_computed_cpu[rows] += ns
+        return ModelRunnerOutput(req_ids=req_ids, req_id_to_index={r: i for i, r in enumerate(req_ids)},
+                                 sampled_token_ids=[[] for _ in req_ids], logits=logits,
+                                 forward_ms=(time.perf_counter() - t0) * 1e3)
 
     def _pool(self, hidden, states, rows, cu, produces, t0) -> ModelRunnerOutput:
         from vllm_b200.layers.pooler import pool_hidden
