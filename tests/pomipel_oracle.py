@@ -1,7 +1,7 @@
 """Plain, slow Pomipel in float64, one function per mechanism, from the equations only: the yardstick of the Pomipel tests.
 
-Nothing of the package is used here.  Weights are a dict of checkpoint names; sequences are processed whole, one token and
-one head at a time where that is the clearest way to say it.
+Nothing of the package is used here.  Weights are a dict of checkpoint names; sequences are processed whole, one
+head, one expert and (in the router) one token at a time.
 """
 from __future__ import annotations
 
@@ -40,12 +40,14 @@ def attend(c_q, c, w_uq, w_uk, w_uv, heads, dim, vdim, scale, hide=()):
     """[n, heads * vdim]; query i sees latents 0..i (``hide``: key positions left out, to show that they matter)."""
     n = c.shape[0]
     q, k, v = (c_q @ w_uq.T).view(n, heads, dim), (c @ w_uk.T).view(n, heads, dim), (c @ w_uv.T).view(n, heads, vdim)
-    out = torch.zeros(n, heads, vdim, dtype=c.dtype)
-    for i in range(n):
-        keys = [j for j in range(i + 1) if j not in hide or j == i]
-        s = torch.einsum("hd,khd->hk", q[i], k[keys]) * scale
-        out[i] = torch.einsum("hk,khd->hd", torch.softmax(s, dim=-1), v[keys])
-    return out.reshape(n, heads * vdim)
+    seen = torch.ones(n, n, dtype=torch.bool).tril()
+    for j in hide:
+        seen[j + 1:, j] = False
+    out = []
+    for h in range(heads):
+        s = (q[:, h] @ k[:, h].T * scale).masked_fill(~seen, -math.inf)
+        out.append(torch.softmax(s, dim=-1) @ v[:, h])
+    return torch.cat(out, dim=-1)
 
 
 def route(h, w_router, correction, top, count, keep):
@@ -63,16 +65,22 @@ def route(h, w_router, correction, top, count, keep):
 
 
 def expert(h, up, down):
-    return down @ torch.clamp(up @ h, min=0.0) ** 2
+    return torch.clamp(h @ up.T, min=0.0) ** 2 @ down.T
 
 
 def feed_forward(h, w, p, spec):
     r = spec["router"]
     groups = r.get("groups") or {"count": 1, "keep": 1}
-    out = torch.zeros_like(h)
+    mine = [[] for _ in range(r["experts"])]                   # expert: [(token, weight)]
     for t in range(h.shape[0]):
         for e, weight in route(h[t], w[p + "router"], w[p + "correction"], r["top"], groups["count"], groups["keep"]):
-            out[t] += weight * expert(h[t], w[f"{p}e{e}.up"], w[f"{p}e{e}.down"])
+            mine[e].append((t, weight))
+    out = torch.zeros_like(h)
+    for e, pairs in enumerate(mine):
+        if pairs:
+            at = [t for t, _ in pairs]
+            weight = torch.tensor([x for _, x in pairs], dtype=h.dtype)
+            out[at] += weight[:, None] * expert(h[at], w[f"{p}e{e}.up"], w[f"{p}e{e}.down"])
     return out
 
 
@@ -143,7 +151,8 @@ def wide():
     return config(128, 160, [(mixer(17, 80, 72, 96, 136), moe(64, 8, 2, 2, 1)), (mixer(4, 128, 128, 64, 264), moe(136, 16, 6, 4, 3))])
 
 
-def make_weights(cfg, seed=0, dtype=torch.float32, pos_size=0.3):
+def make_weights(cfg, seed=0, dtype=torch.float32, pos_size=0.3, steady=False):
+    """``steady``: choice scores far apart, so that 16-bit rounding cannot change which experts are chosen."""
     g = torch.Generator().manual_seed(seed)
 
     def mat(*shape, size=1.0):
@@ -167,6 +176,10 @@ def make_weights(cfg, seed=0, dtype=torch.float32, pos_size=0.3):
             w[f"l{i}.norm2"] = vec(H, 0.2)
             r, ff, p = spec["mlp"]["router"], spec["mlp"]["expert"]["ff"], f"l{i}.mlp."
             w[p + "router"], w[p + "correction"] = mat(r["experts"], H), vec(r["experts"], 0.6)
+            if steady:
+                w[p + "router"] = w[p + "router"] * 0.125
+                order = torch.randperm(r["experts"], generator=g).to(dtype)
+                w[p + "correction"] = 0.5 * order - 0.25 * r["experts"] - 1.0 / 16
             for e in range(r["experts"]):
                 w[f"{p}e{e}.up"], w[f"{p}e{e}.down"] = mat(ff, H), mat(H, ff)
     return w

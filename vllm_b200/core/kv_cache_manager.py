@@ -13,7 +13,7 @@ get one block table per group).
 """
 from __future__ import annotations
 
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 from typing import Optional, Sequence
 
 from vllm_b200.core.block_pool import BlockPool, KVCacheBlock, make_block_hasher
@@ -105,6 +105,10 @@ class CrossAttentionSpec(FullAttentionSpec):
 class KVCacheGroupSpec:
     layer_names: list[str]
     spec: KVCacheSpec
+    layer_specs: dict[str, KVCacheSpec] = field(default_factory=dict)     # layers whose rows are narrower than ``spec``'s
+
+    def spec_of(self, layer_name: str) -> KVCacheSpec:
+        return self.layer_specs.get(layer_name, self.spec)
 
 
 @dataclass
@@ -121,11 +125,17 @@ class KVCacheConfig:
 
 
 def group_specs(layer_specs: dict[str, KVCacheSpec]) -> list[KVCacheGroupSpec]:
-    """Layers with identical specs share a group (= one block table)."""
+    """Layers with identical specs share a group (= one block table); so do latent caches of different widths, whose pages
+    hold the same tokens (each layer owns a tensor of its own width)."""
     groups: dict[KVCacheSpec, list[str]] = {}
     for name, spec in layer_specs.items():
-        groups.setdefault(spec, []).append(name)
-    return [KVCacheGroupSpec(names, spec) for spec, names in groups.items()]
+        key = replace(spec, head_size=0) if isinstance(spec, MLAAttentionSpec) else spec
+        groups.setdefault(key, []).append(name)
+    out = []
+    for names in groups.values():
+        widest = max((layer_specs[n] for n in names), key=lambda s: s.page_size_bytes)
+        out.append(KVCacheGroupSpec(names, widest, {n: layer_specs[n] for n in names if layer_specs[n] != widest}))
+    return out
 
 
 def get_kv_cache_config(layer_specs: dict[str, KVCacheSpec], available_bytes: int, max_model_len: int,

@@ -45,8 +45,7 @@ class StepReplay:
         page = cfg.cache_config.block_size
         longest = min(cfg.scheduler_config.max_model_len, cdiv(max_tokens, page) * page)
         cfg.scheduler_config.max_model_len = cfg.model_config.max_model_len = longest
-        self._pool_pages = cdiv(max_tokens, page)
-        cfg.cache_config.num_gpu_blocks_override = self._pool_pages + 1           # + the null page
+        cfg.cache_config.num_gpu_blocks_override = cdiv(max_tokens, page) + 1     # + the null page
         self.core = EngineCore(cfg)
         self.device = self.core.model_executor.worker.device
         self.sampling = SamplingParams(temperature=0.0, max_tokens=1, ignore_eos=True)

@@ -94,6 +94,8 @@ class MergedReplicatedLinear(ReplicatedLinear):
     def weight_loader(self, param: nn.Parameter, w: torch.Tensor, shard_id=None) -> None:
         if shard_id is None:
             return super().weight_loader(param, w)
+        if shard_id >= len(self.output_sizes):
+            raise ValueError(f"{self.prefix} has no part {shard_id}")
         dst = param.data.narrow(0, sum(self.output_sizes[:shard_id]), self.output_sizes[shard_id])
         assert dst.shape == w.shape, (self.prefix, shard_id, dst.shape, w.shape)
         dst.copy_(w)

@@ -331,7 +331,8 @@ class ModelRunner:
                                                        device=self.device)
                     continue
                 if isinstance(s, MLAAttentionSpec):
-                    shape = (cfg.num_blocks, s.phys_block_size, s.head_size)
+                    ls = g.spec_of(name)
+                    shape = (cfg.num_blocks, ls.phys_block_size, ls.head_size)
                 else:
                     shape = (cfg.num_blocks, 2, s.num_kv_heads, getattr(s, "phys_block_size", s.block_size), s.head_size)
                 self.kv_caches[name] = torch.zeros(shape, dtype=kvd, device=self.device)
