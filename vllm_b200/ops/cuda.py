@@ -523,6 +523,64 @@ def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank):
                     None if md.decode_only else md.query_start_loc, scale)
 
 
+# ------------------------------------------------------------------ sampling
+def argmax(logits: torch.Tensor) -> torch.Tensor:
+    B, V = logits.shape
+    out = torch.empty(B, dtype=torch.int64, device=logits.device)
+    _check(_argmax(logits.data_ptr(), logits.stride(0), B, V, out.data_ptr(), _DT[logits.dtype], _st()), "argmax")
+    return out
+
+
+_step_buf: dict[int, torch.Tensor] = {}
+
+
+def fused_sample(logits, temperature, seeds, step, out: Optional[torch.Tensor] = None):
+    """``step``: per-row int32 [B] noise counters (a python int is broadcast)."""
+    B, V = logits.shape
+    if out is None:
+        out = torch.empty(B, dtype=torch.int64, device=logits.device)
+    if not isinstance(step, torch.Tensor):
+        step = torch.full((B,), int(step) & 0x7FFFFFFF, dtype=torch.int32, device=logits.device)
+    _check(_fused_sample(logits.data_ptr(), logits.stride(0), B, V, temperature.data_ptr(), seeds.data_ptr(),
+                         step.data_ptr(), out.data_ptr(), _DT[logits.dtype], _st()), "fused_sample")
+    return out
+
+
+_fused_sample_cand = _sig("vb_fused_sample_cand", _vp, _i64, _i, _i, _vp, _vp, _vp, _i, _vp, _i, _vp)
+_select_cand = _sig("vb_select_candidate", _vp, _i, _vp, _i, _vp)
+
+
+def fused_sample_candidates(logits_local, temperature, seeds, step, idx_off: int, v_valid: int) -> torch.Tensor:
+    """Per-row best (value, global id) of this rank's vocab shard as a [B, 8] bf16-viewable 16-byte record."""
+    B = logits_local.shape[0]
+    cand = torch.empty((B, 4), dtype=torch.float32, device=logits_local.device)
+    _check(_fused_sample_cand(logits_local.data_ptr(), logits_local.stride(0), B, max(v_valid, 0), temperature.data_ptr(),
+                              seeds.data_ptr(), step.data_ptr(), idx_off, cand.data_ptr(), _DT[logits_local.dtype], _st()),
+           "fused_sample_cand")
+    return cand
+
+
+def select_candidates(cands: torch.Tensor, W: int, out: torch.Tensor) -> torch.Tensor:
+    """cands: [B, W, 4] fp32 records gathered from the W ranks → winning token id per row."""
+    B = out.shape[0]
+    _check(_select_cand(cands.data_ptr(), W, out.data_ptr(), B, _st()), "select_candidate")
+    return out
+
+
+def topk_topp_mask_(logits: torch.Tensor, top_k, top_p, min_p=None) -> torch.Tensor:
+    assert logits.dtype == torch.float32 and logits.is_contiguous()
+    B, V = logits.shape
+    _check(_topk_topp(logits.data_ptr(), B, V, _p(top_k), _p(top_p), _p(min_p), _st()), "topk_topp")
+    return logits
+
+
+def row_lse(logits: torch.Tensor) -> torch.Tensor:
+    B, V = logits.shape
+    out = torch.empty(B, dtype=torch.float32, device=logits.device)
+    _check(_row_lse(logits.data_ptr(), logits.stride(0), B, V, out.data_ptr(), _DT[logits.dtype], _st()), "row_lse")
+    return out
+
+
 # ------------------------------------------------------------------ fp32 residual stream (csrc/stream.cu)
 _embed_stream = _sig("vb_embed_stream", _vp, _vp, _vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _i, _vp)
 _post_norm = _sig("vb_post_norm_add", _vp, _i64, _vp, _vp, _i, _vp, _i, _vp, _vp, _i, _vp, _i, _i, _f, _i, _vp)
