@@ -129,21 +129,14 @@ VB_DEVICE void mbar_wait(uint64_t* bar, uint32_t parity) {
   while (!mbar_try_wait(bar, parity)) {}
 }
 
-// Bounded wait: gives up after MBAR_TRIES polls (each poll suspends in hardware, so this is seconds — no valid wait
-// comes near it) or as soon as another thread of the CTA gave up (`give_up` in shared memory).  A kernel that gets
-// `false` drains its own copies, frees its TMEM, raises its error flag and returns.
-constexpr uint32_t MBAR_TRIES = 1u << 20;
-VB_DEVICE bool mbar_wait_lim(uint64_t* bar, uint32_t parity, volatile int* give_up) {
-  for (uint32_t i = 0; i < MBAR_TRIES; ++i) {
-    if (mbar_try_wait(bar, parity)) return true;
-    if (*give_up) return false;
-  }
-  *give_up = 1;
-  return false;
-}
-// the same for a whole warp that goes on in step: every lane gets the same answer
-VB_DEVICE bool mbar_wait_warp(uint64_t* bar, uint32_t parity, volatile int* give_up) {
-  return __all_sync(0xffffffffu, mbar_wait_lim(bar, parity, give_up)) != 0;
+// Bounded waits: a thread has a budget of failed polls for its whole life (each poll suspends in hardware, so this is a
+// good part of a second at least — no valid run comes near it).  Once it is spent every later wait falls through after one
+// poll: the kernel runs to its end with void results and in-bounds accesses, lets its copies in flight land, frees its
+// TMEM and raises its error flag.
+constexpr int MBAR_BUDGET = 1 << 24;
+VB_DEVICE void mbar_wait_lim(uint64_t* bar, uint32_t parity, int& budget) {
+  while (!mbar_try_wait(bar, parity))
+    if (--budget < 0) break;
 }
 
 // ------------------------------------------------- PTX: bulk / tensor copies

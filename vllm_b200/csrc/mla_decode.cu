@@ -87,7 +87,8 @@ VB_HOST_DEVICE uint32_t idesc_f16_a_mn(int M, int N, bool bf16) {
   return umma_idesc_f16(M, N, bf16) | (1u << 15);     // bit 15: A operand is MN-major
 }
 
-template <typename T, int N, int NL, int ROPE>
+// FULL: the latent fills its blocks (R = 64 NL is a compile-time constant)
+template <typename T, int N, int NL, int ROPE, bool FULL>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_constant__ CUtensorMap tmap_qr,
                   const __grid_constant__ CUtensorMap tmap_kv, const Params p) {
@@ -112,10 +113,10 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 1);
   float* wred = reinterpret_cast<float*>(tmem_slot + 2);        // [4][N]
   int* blk_ids = reinterpret_cast<int*>(wred + 4 * N);          // [MAX_IDS_SMEM]
-  __shared__ int give_up_s;
-  volatile int* give_up = &give_up_s;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int budget = MBAR_BUDGET;                  // failed polls left (mbar_wait_lim)
+  const int R = FULL ? NL * 64 : p.R;
   const int split = blockIdx.x, hg = blockIdx.y, b = blockIdx.z;
   const int h0 = hg * N;
   const int G = min(N, p.H - h0);            // real heads of this group
@@ -134,7 +135,6 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
   const int n_tiles = max(tile_hi - tile_lo, 0);
   constexpr uint32_t TMEM_USE = (2 + NC) * N;
   constexpr uint32_t TMEM_COLS = TMEM_USE <= 64 ? 64 : (TMEM_USE <= 128 ? 128 : 256);
-  if (threadIdx.x == 0) give_up_s = 0;
 
   if (warp == 0 && lane == 0) {
     tma_prefetch_desc(&tmap_qn); tma_prefetch_desc(&tmap_qr); tma_prefetch_desc(&tmap_kv);
@@ -174,7 +174,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
       for (int g = 0; g < G; ++g) {
         const int64_t pi = ((int64_t)b * p.H + (h0 + g)) * p.num_splits + split;
         for (int c = 0; c < NC; ++c)
-          if (c * 128 + t < p.R) p.part_out[pi * p.R + c * 128 + t] = 0.f;
+          if (c * 128 + t < R) p.part_out[pi * R + c * 128 + t] = 0.f;
         if (t == 0) p.part_lse[pi] = -INFINITY;
       }
     }
@@ -189,8 +189,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
       mbar_expect_tx(q_full, NKB * min(N, p.H) * 128);   // the full TMA box is always written (OOB heads as zeros)
       for (int kb = 0; kb < NL; ++kb) tma_load_3d(q_smem + kb * (N * 128), &tmap_qn, kb * 64, h0, b, q_full);
       if (ROPE) tma_load_3d(q_smem + NL * (N * 128), &tmap_qr, 0, h0, b, q_full);
-      bool ok = true;
-      for (int j = 0; j < n_tiles && ok; ++j) {
+      for (int j = 0; j < n_tiles && budget >= 0; ++j) {
         const int st = j % STAGES;
         const uint32_t par = ((j / STAGES) & 1) ^ 1;
         int row[8], n_valid = 0;
@@ -205,15 +204,14 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
         for (int i = 0; i < NKB; ++i) {
           const int kb = ROPE ? (i == 0 ? NKB - 1 : i - 1) : i;   // rope block first: QK releases it first
           const int slot = st * NKB + kb;
-          if (!(ok = mbar_wait_lim(&kv_empty[slot], par, give_up))) break;
+          mbar_wait_lim(&kv_empty[slot], par, budget);
           mbar_expect_tx(&kv_full[slot], bytes);
           for (int u = 0; u < ppt; ++u)
             if (row[u] >= 0)
-              tma_load_2d_hint(stp + kb * KB_BYTES + u * rows * 128, &tmap_kv, kb * 64, row[u], &kv_full[slot],
-                               p.H > N ? L2_EVICT_NORMAL : L2_EVICT_FIRST);   // other head groups read the tile again
+              tma_load_2d_hint(stp + kb * KB_BYTES + u * rows * 128, &tmap_kv, kb * 64, row[u], &kv_full[slot], L2_EVICT_FIRST);
         }
       }
-      if (!ok) {                                // let the copies in flight land before the block gives up its memory
+      if (budget < 0) {                         // let the copies in flight land before the block gives up its memory
         for (int i = 0; i < STAGES * NKB; ++i)
           for (int n = 0; n < 4096 && !mbar_try_wait(&kv_full[i], 0) && !mbar_try_wait(&kv_full[i], 1); ++n) {}
       }
@@ -223,24 +221,24 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
     const bool bf16 = DTypeOf<T>::v == DT_BF16;
     const uint32_t idesc_s = umma_idesc_f16(128, N, bf16);
     const uint32_t idesc_o = idesc_f16_a_mn(128, N, bf16);
-    bool ok = mbar_wait_warp(q_full, 0, give_up);
+    mbar_wait_lim(q_full, 0, budget);
     // descriptors are built once; every MMA adds a compile-time offset (in 16-byte units) to the address field
     const uint64_t d_kv = umma_desc_sw128(kv_smem);
     const uint64_t d_kv_mn = umma_desc_sw128_mn(kv_smem, KB_BYTES);
     const uint64_t d_q = umma_desc_sw128(q_smem);
     const uint64_t d_p = umma_desc_sw128(p_smem);
-    for (int j = 0; j <= n_tiles && ok; ++j) {
+    for (int j = 0; j <= n_tiles; ++j) {
       if (j < n_tiles) {
         // ---- S^T_j = Kc · Q^T, k-block by k-block as they land (M = 128: rows 64..127 are padding, see the header)
         const int st = j % STAGES, sb = j & 1;
         const uint32_t par = (j / STAGES) & 1;
-        if (!(ok = mbar_wait_warp(&s_empty[sb], ((j >> 1) & 1) ^ 1, give_up))) break;
+        mbar_wait_lim(&s_empty[sb], ((j >> 1) & 1) ^ 1, budget);
         tc_fence_after();
 #pragma unroll
         for (int i = 0; i < NKB; ++i) {
           const int kb = ROPE ? (i == 0 ? NKB - 1 : i - 1) : i;
           const int slot = st * NKB + kb;
-          if (!(ok = mbar_wait_warp(&kv_full[slot], par, give_up))) break;
+          mbar_wait_lim(&kv_full[slot], par, budget);
           tc_fence_after();
           if (lane == 0) {
             const uint64_t da = d_kv + (uint64_t)((st * STAGE_BYTES + kb * KB_BYTES) >> 4);
@@ -251,7 +249,6 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
           }
           __syncwarp();
         }
-        if (!ok) break;
         if (lane == 0) {
           umma_commit(&s_full[sb]);
           if (ROPE) umma_commit(&kv_empty[st * NKB + NKB - 1]);   // the rope block is only read by QK
@@ -262,7 +259,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
         // ---- O^T += V^T · P^T for tile j-1: NC 128-dim chunks (k-blocks 2c, 2c+1 read MN-major), K = 64 tokens;
         // each chunk hands its two k-block buffers back to the producer as soon as it retires
         const int jj = j - 1, st = jj % STAGES;
-        if (!(ok = mbar_wait_warp(p_full, jj & 1, give_up))) break;
+        mbar_wait_lim(p_full, jj & 1, budget);
         tc_fence_after();
         if (lane == 0) {
 #pragma unroll
@@ -290,7 +287,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
     for (int g = 0; g < N; ++g) { m_used[g] = -INFINITY; l_thr[g] = 0.f; }
     for (int j = 0; j < n_tiles; ++j) {
       const int sb = j & 1;
-      mbar_wait_lim(&s_full[sb], (j >> 1) & 1, give_up);
+      mbar_wait_lim(&s_full[sb], (j >> 1) & 1, budget);
       tc_fence_after();
       float s[N];
 #pragma unroll
@@ -323,7 +320,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
           m_used[g] = mx;
         }
       }
-      if (j > 0) { mbar_wait_lim(pv_done, (j - 1) & 1, give_up); tc_fence_after(); }   // P and O^T are free again
+      if (j > 0) { mbar_wait_lim(pv_done, (j - 1) & 1, budget); tc_fence_after(); }   // P and O^T are free again
       if (rescale) {       // uniform over the CTA (every thread sees the same column maxima)
 #pragma unroll
         for (int c4 = 0; c4 < NC; ++c4) {
@@ -362,7 +359,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
       if (lane == 0) wred[qd * N + g] = lt;
     }
     bar_sync_softmax();
-    mbar_wait_lim(pv_done, (n_tiles - 1) & 1, give_up);
+    mbar_wait_lim(pv_done, (n_tiles - 1) & 1, budget);
     tc_fence_after();
     float inv[N], lsum[N];
 #pragma unroll
@@ -373,7 +370,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
 #pragma unroll
     for (int c4 = 0; c4 < NC; ++c4) {
       const int d = c4 * 128 + t;
-      const bool d_ok = d < p.R;
+      const bool d_ok = d < R;
 #pragma unroll
       for (int c = 0; c < N; c += CH) {
         uint32_t ov[CH];
@@ -385,10 +382,10 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
             const float o = __uint_as_float(ov[g]) * inv[c + g];
             const int hq = h0 + c + g;
             if (p.num_splits == 1) {
-              reinterpret_cast<T*>(p.out)[(int64_t)b * p.out_stride + (int64_t)hq * p.R + d] = from_f32<T>(o);
+              reinterpret_cast<T*>(p.out)[(int64_t)b * p.out_stride + (int64_t)hq * R + d] = from_f32<T>(o);
             } else {
               const int64_t pi = ((int64_t)b * p.H + hq) * p.num_splits + split;
-              p.part_out[pi * p.R + d] = o;
+              p.part_out[pi * R + d] = o;
             }
           }
         }
@@ -413,7 +410,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
   tc_fence_before();
   __syncthreads();
   if (warp == 1) tmem_dealloc(tmem_base, TMEM_COLS);
-  if (threadIdx.x == 0 && *give_up && p.error) *p.error = 1;
+  if (budget < 0 && p.error) *p.error = 1;
 }
 
 template <typename T>
@@ -449,12 +446,12 @@ static EncodeTiledFn get_encode() {
   return fn;
 }
 
-template <typename T, int N, int NL, int ROPE>
+template <typename T, int N, int NL, int ROPE, bool FULL>
 static int launch(const CUtensorMap& tqn, const CUtensorMap& tqr, const CUtensorMap& tkv, const Params& p, dim3 grid,
                   cudaStream_t st) {
   constexpr int NKB = Geo<NL, ROPE>::NKB, STAGES = Geo<NL, ROPE>::STAGES;
   const int smem = STAGES * Geo<NL, ROPE>::STAGE_BYTES + NKB * N * 128 + 8192 + (2 * STAGES * NKB + 8) * 8 + 16 + 4 * N * 4 + MAX_IDS_SMEM * 4 + 1024;
-  auto k = mla_decode_kernel<T, N, NL, ROPE>;
+  auto k = mla_decode_kernel<T, N, NL, ROPE, FULL>;
   static bool a = false;
   if (!a) { cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); a = true; }
   vb_launch(k, grid, dim3(NUM_THREADS), (size_t)smem, st, tqn, tqr, tkv, p);
@@ -511,15 +508,16 @@ EXPORT int vb_mla_decode(const void* q_nope, const void* q_pe, const void* cache
   }
   dim3 grid(num_splits, (H + N - 1) / N, B);
   int rc;
-#define GO(TT, NL, RP) rc = N == 16 ? launch<TT, 16, NL, RP>(tqn, tqr, tkv, p, grid, st) : launch<TT, 32, NL, RP>(tqn, tqr, tkv, p, grid, st)
+#define GO(TT, NL, RP, FL) rc = N == 16 ? launch<TT, 16, NL, RP, FL>(tqn, tqr, tkv, p, grid, st) : launch<TT, 32, NL, RP, FL>(tqn, tqr, tkv, p, grid, st)
   const int nl = (R + 63) / 64;
-  if (rope) { if (bf16) GO(__nv_bfloat16, 8, 1); else GO(__half, 8, 1); }
-  else if (nl <= 1) GO(__nv_bfloat16, 1, 0);
-  else if (nl == 2) GO(__nv_bfloat16, 2, 0);
-  else if (nl == 3) GO(__nv_bfloat16, 3, 0);
-  else if (nl == 4) GO(__nv_bfloat16, 4, 0);
-  else if (nl <= 6) GO(__nv_bfloat16, 6, 0);
-  else GO(__nv_bfloat16, 8, 0);
+  if (rope) { if (bf16) GO(__nv_bfloat16, 8, 1, true); else GO(__half, 8, 1, true); }
+  else if (R == 512) GO(__nv_bfloat16, 8, 0, true);
+  else if (nl <= 1) GO(__nv_bfloat16, 1, 0, false);
+  else if (nl == 2) GO(__nv_bfloat16, 2, 0, false);
+  else if (nl == 3) GO(__nv_bfloat16, 3, 0, false);
+  else if (nl == 4) GO(__nv_bfloat16, 4, 0, false);
+  else if (nl <= 6) GO(__nv_bfloat16, 6, 0, false);
+  else GO(__nv_bfloat16, 8, 0, false);
 #undef GO
   if (rc) return rc;
   if (num_splits > 1) {

@@ -85,9 +85,9 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   uint64_t* p_full = s_empty + 2;
   uint64_t* pv_done = p_full + 1;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 1);
-  volatile int* give_up = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int budget = MBAR_BUDGET;                    // failed polls left (mbar_wait_lim)
   const int b = blockIdx.z, h = blockIdx.y;
   pdl_trigger();
   pdl_wait();
@@ -112,7 +112,6 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     mbar_init(p_full, 128);
     mbar_init(pv_done, 1);
     mbar_fence_init();
-    *give_up = 0;
   }
   if (warp == 1) tmem_alloc(tmem_slot, 512);
   tc_fence_before();
@@ -128,21 +127,22 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       mbar_expect_tx(q_full, NQ * BLK);
 #pragma unroll
       for (int i = 0; i < NQ; ++i) tma_load_3d(q_smem + i * BLK, &tmap_q, i * 64, p.h0 + h, q0, q_full);
-      bool ok = true;
-      for (int j = 0; j < n_tiles && ok; ++j) {
+      for (int j = 0; j < n_tiles; ++j) {
         const int s = j % STAGES;
         const uint32_t par = ((j / STAGES) & 1) ^ 1;
         const int row = kv0 + j * TN;
-        if (!(ok = mbar_wait_lim(&k_empty[s], par, give_up))) break;
+        mbar_wait_lim(&k_empty[s], par, budget);
+        if (budget < 0) break;
         mbar_expect_tx(&k_full[s], NQ * BLK);
 #pragma unroll
         for (int i = 0; i < NQ; ++i) tma_load_3d(k_smem + (s * NQ + i) * BLK, &tmap_k, i * 64, h, row, &k_full[s]);
-        if (!(ok = mbar_wait_lim(&v_empty[s], par, give_up))) break;
+        mbar_wait_lim(&v_empty[s], par, budget);
+        if (budget < 0) break;
         mbar_expect_tx(&v_full[s], NV * BLK);
 #pragma unroll
         for (int i = 0; i < NV; ++i) tma_load_3d(v_smem + (s * NV + i) * BLK, &tmap_v, i * 64, h, row, &v_full[s]);
       }
-      if (!ok) {                                // let the copies in flight land before the block gives up its memory
+      if (budget < 0) {                         // let the copies in flight land before the block gives up its memory
         for (int s = 0; s < STAGES; ++s)
           for (int n = 0; n < 4096 && !(mbar_try_wait(&k_full[s], 0) || mbar_try_wait(&k_full[s], 1)); ++n) {}
         for (int s = 0; s < STAGES; ++s)
@@ -156,12 +156,13 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     const uint32_t idesc_o = umma_idesc_f16(TM, NV * 64, bf16) | (1u << 16);      // bit 16: B operand is MN-major
     const uint64_t d_q = umma_desc_sw128(q_smem), d_k = umma_desc_sw128(k_smem), d_p = umma_desc_sw128(p_smem);
     const uint64_t d_v = desc_mn(v_smem);
-    bool ok = mbar_wait_warp(q_full, 0, give_up);
-    for (int j = 0; j <= n_tiles && ok; ++j) {
+    mbar_wait_lim(q_full, 0, budget);
+    __syncwarp();
+    for (int j = 0; j <= n_tiles; ++j) {
       if (j < n_tiles) {
         const int s = j % STAGES, sb = j & 1;
-        if (!(ok = mbar_wait_warp(&k_full[s], (j / STAGES) & 1, give_up))) break;
-        if (!(ok = mbar_wait_warp(&s_empty[sb], ((j >> 1) & 1) ^ 1, give_up))) break;
+        mbar_wait_lim(&k_full[s], (j / STAGES) & 1, budget);
+        mbar_wait_lim(&s_empty[sb], ((j >> 1) & 1) ^ 1, budget);
         tc_fence_after();
         if (lane == 0) {
 #pragma unroll
@@ -178,8 +179,8 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       }
       if (j > 0) {
         const int jj = j - 1, s = jj % STAGES;
-        if (!(ok = mbar_wait_warp(&v_full[s], (jj / STAGES) & 1, give_up))) break;
-        if (!(ok = mbar_wait_warp(p_full, jj & 1, give_up))) break;
+        mbar_wait_lim(&v_full[s], (jj / STAGES) & 1, budget);
+        mbar_wait_lim(p_full, jj & 1, budget);
         tc_fence_after();
         if (lane == 0) {
 #pragma unroll
@@ -204,7 +205,7 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     for (int j = 0; j < n_tiles; ++j) {
       const int sb = j & 1;
       const uint32_t t_s = tmem_base + sb * 128 + t_lane;
-      mbar_wait_lim(&s_full[sb], (j >> 1) & 1, give_up);
+      mbar_wait_lim(&s_full[sb], (j >> 1) & 1, budget);
       __syncwarp();
       tc_fence_after();
       const int hi = row_valid ? pos0 + r + 1 - j * TN : 0;     // keys [0, hi) of this tile are visible to the row
@@ -234,7 +235,7 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         m_used = mx;
       }
       const float m_ref = m_used == -INFINITY ? 0.f : m_used;
-      if (j > 0) { mbar_wait_lim(pv_done, (j - 1) & 1, give_up); __syncwarp(); tc_fence_after(); }   // P and O are free
+      if (j > 0) { mbar_wait_lim(pv_done, (j - 1) & 1, budget); __syncwarp(); tc_fence_after(); }   // P and O are free
       if (__any_sync(0xffffffffu, rescale)) {
         l_run *= alpha;
 #pragma unroll
@@ -278,7 +279,7 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       mbar_arrive(p_full);
     }
     // ---- epilogue
-    mbar_wait_lim(pv_done, (n_tiles - 1) & 1, give_up);
+    mbar_wait_lim(pv_done, (n_tiles - 1) & 1, budget);
     __syncwarp();
     tc_fence_after();
     const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
@@ -306,7 +307,7 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   tc_fence_before();
   __syncthreads();
   if (warp == 1) tmem_dealloc(tmem_base, 512);
-  if (threadIdx.x == 0 && *give_up && p.error) *p.error = 1;
+  if (budget < 0 && p.error) *p.error = 1;
 }
 
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,

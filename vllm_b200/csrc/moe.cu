@@ -68,7 +68,7 @@ __global__ void topk_softmax_kernel(const T* __restrict__ logits, float* __restr
 //   scores (with a bias) or by its best (without);  the k best experts of the `keep` best groups are taken, the lowest
 //   index winning ties;  weight = score WITHOUT the bias (optionally renormalised) * scale
 template <typename TX, typename TW>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(512)
 grouped_topk_kernel(const float* __restrict__ logits, const TX* __restrict__ x, const TW* __restrict__ w, int H,
                     const float* __restrict__ bias, float* __restrict__ out_w, int* __restrict__ out_ids, int E, int k,
                     int n_group, int keep, int softmax, int renorm, float scale) {
@@ -89,20 +89,31 @@ grouped_topk_kernel(const float* __restrict__ logits, const TX* __restrict__ x, 
     __syncthreads();
     constexpr int V = Vec16<TW>::N;
     const bool vec = H % V == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
-    for (int e = warp; e < E; e += n_warps) {
-      const TW* wr = w + (int64_t)e * H;
-      float a = 0.f;
+    constexpr int EB = 4;                       // experts of a warp in flight together
+    for (int e0 = warp * EB; e0 < E; e0 += n_warps * EB) {
+      float a[EB] = {};
       if (vec) {
         for (int i = lane * V; i < H; i += 32 * V) {
-          const Vec16<TW> wv = ld16(wr + i);
+          Vec16<TW> wv[EB];
 #pragma unroll
-          for (int j = 0; j < V; ++j) a += xs[i + j] * to_f32(wv.e[j]);
+          for (int u = 0; u < EB; ++u) wv[u] = ld16(w + (int64_t)min(e0 + u, E - 1) * H + i);
+#pragma unroll
+          for (int j = 0; j < V; ++j) {
+            const float xv = xs[i + j];
+#pragma unroll
+            for (int u = 0; u < EB; ++u) a[u] += xv * to_f32(wv[u].e[j]);
+          }
         }
       } else {
-        for (int i = lane; i < H; i += 32) a += xs[i] * to_f32(wr[i]);
+        for (int i = lane; i < H; i += 32)
+#pragma unroll
+          for (int u = 0; u < EB; ++u) a[u] += xs[i] * to_f32(w[(int64_t)min(e0 + u, E - 1) * H + i]);
       }
-      a = warp_sum(a);
-      if (lane == 0) score[e] = a;
+#pragma unroll
+      for (int u = 0; u < EB; ++u) {
+        a[u] = warp_sum(a[u]);
+        if (lane == 0 && e0 + u < E) score[e0 + u] = a[u];
+      }
     }
   }
   __syncthreads();
@@ -396,7 +407,7 @@ EXPORT int vb_moe_grouped_topk(const float* logits, const void* x, int x_f32, co
   if (!logits && (!x || !w)) return -1;
   const size_t smem = (size_t)(2 * E + n_group + (logits ? 0 : H)) * sizeof(float);
   if (smem > 48 * 1024) return -3;
-  const int thr = logits ? (E > 128 ? 256 : 64) : 256;
+  const int thr = logits ? (E > 128 ? 256 : 64) : (E > 32 ? 512 : 256);
 #define GO(TX, TW) vb_launch(moe::grouped_topk_kernel<TX, TW>, dim3(n_tokens), dim3(thr), smem, st, logits, (const TX*)x, (const TW*)w, H, bias, out_w, out_ids, E, k, n_group, keep, softmax, renorm, scale)
   DISPATCH_DTYPE(dtype, T, {
     if (x_f32) GO(float, T); else GO(T, T);
