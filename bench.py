@@ -19,7 +19,7 @@ Both arms print the SAME ``metric`` string and measure the SAME thing:
            over R interleaved repetitions after a full warm-up generate; e2e = 64 * K / t_decode.  Every engine
            step inside copies its inputs host -> device from pinned memory and reads the sampled ids back.
 
-``--design pomipel`` measures another workload: a few layers of that design beside the closest model (no contract line).
+``--design pomipel`` measures another workload: a few layers of that design beside the closest model.
 
 ``--impl reference`` runs the UNMODIFIED reference (baseline/_ref if the offline install worked, else the stock
 vLLM wheel of the image — DESIGN.md §0) on its DEFAULT engine: multiprocess engine core, async scheduling,

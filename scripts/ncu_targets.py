@@ -1,6 +1,6 @@
 """Launch each hot kernel a few times so that `ncu --set full -k regex:<name> -s 3 -c 1` can capture it in isolation.
 
-    ncu --set full --clock-control none -k regex:gemm_fp8_kernel -s 3 -c 1 -o gpurun_out/ncu_fp8 \
+    ncu --set full --clock-control none -k regex:gemm_fp8_kernel -s 3 -c 1 -o ncu_fp8 \
         python scripts/ncu_targets.py fp8
 """
 import sys
@@ -55,3 +55,20 @@ if which in ("attn", "mla", "all"):
         qn = (torch.randn(B, 16, 512, device="cuda") * 0.3).to(dt)
         qp = (torch.randn(B, 16, 64, device="cuda") * 0.3).to(dt)
         rep(lambda: cu.mla_decode_tc(qn, qp, cache, bt, sl, 0.07, 4096))
+if which in ("latent", "all"):
+    # latent attention and ungated experts: prompt attention, decode over the latents, grouped products of a prompt step
+    from vllm_b200.benchmarks.latent_layers import _pages, _routing
+    from vllm_b200.ops import moe
+    n, ctx, h, D = 4, 1024, 16, 128
+    i32 = dict(dtype=torch.int32, device="cuda")
+    q, k, v = (torch.randn(n * ctx, h, D, device="cuda", dtype=dt) * 0.3 for _ in range(3))
+    out = torch.empty_like(q)
+    start, lens = torch.arange(0, n * ctx, ctx, **i32), torch.full((n,), ctx, **i32)
+    rep(lambda: cu.mla_prefill(q, k, v, out, start, lens, lens, start, 0, ctx, D ** -0.5))
+    cache, bt, sl = _pages(64, 4096, 512)
+    qa = torch.randn(64, 16, 512, device="cuda", dtype=dt) * 0.3
+    rep(lambda: cu.mla_decode_tc(qa, None, cache, bt, sl, 0.07, 4096))
+    x = torch.randn(4096, 2048, device="cuda", dtype=dt) * 0.1
+    up, down = (torch.randn(*s, device="cuda", dtype=dt) * 0.02 for s in ((32, 1408, 2048), (32, 2048, 1408)))
+    wt, ids = _routing(4096, 32, 6)
+    rep(lambda: moe.expert_rows_plain(x, up, down, ids, "relu2", None))

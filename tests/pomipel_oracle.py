@@ -20,7 +20,7 @@ def unit_rms(x, eps):
 
 
 def centred_norm(x, w, eps):
-    """RMS norm whose weight is stored around zero."""
+    """RMS norm whose gain is one plus the stored weight."""
     return unit_rms(x, eps) * (1.0 + w)
 
 
@@ -179,7 +179,8 @@ def make_weights(cfg, seed=0, dtype=torch.float32, pos_size=0.3, steady=False):
             if steady:
                 w[p + "router"] = w[p + "router"] * 0.125
                 order = torch.randperm(r["experts"], generator=g).to(dtype)
-                w[p + "correction"] = 0.5 * order - 0.25 * r["experts"] - 1.0 / 16
+                # growing steps: sums of two (the rank of a group) do not tie either
+                w[p + "correction"] = (0.5 * order + 0.0625 * order * order - 0.25 * r["experts"] - 1.0 / 16).to(torch.bfloat16).to(dtype)
             for e in range(r["experts"]):
                 w[f"{p}e{e}.up"], w[f"{p}e{e}.down"] = mat(ff, H), mat(H, ff)
     return w

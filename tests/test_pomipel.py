@@ -174,7 +174,7 @@ def test_router_choice_and_weights(E, top, count, keep):
         assert sorted(ids[t].tolist()) == sorted(e for e, _ in want)
         got = dict(zip(ids[t].tolist(), wt[t].tolist()))
         for e, s in want:
-            assert abs(got[e] - s) < 1e-5                      # without the correction, not renormalised
+            assert abs(got[e] - s) < 1e-5                      # the plain score, whatever the correction
 
 
 def test_ungated_experts():

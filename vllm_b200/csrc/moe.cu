@@ -64,7 +64,7 @@ __global__ void topk_softmax_kernel(const T* __restrict__ logits, float* __restr
 
 // Router with sigmoid or softmax scores, a selection bias and group-limited choice; one CTA per token, fp32 throughout.
 //   logits: given ([T, E] fp32), or computed here from x [T, H] and w [E, H] (one warp per expert, decode batches)
-//   choice score = score + bias;  a group (n_group equal runs of neighbours) is ranked by the sum of its two best choice
+//   choice score = score + bias;  a group (one of n_group contiguous runs) is ranked by the sum of its two best choice
 //   scores (with a bias) or by its best (without);  the k best experts of the `keep` best groups are taken, the lowest
 //   index winning ties;  weight = score WITHOUT the bias (optionally renormalised) * scale
 template <typename TX, typename TW>

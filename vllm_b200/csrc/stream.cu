@@ -166,8 +166,8 @@ EXPORT int vb_embed_stream(const int* ids, const int64_t* positions, const void*
 }
 
 // inv / pair_w null: y is [T, H].  Else y holds expert output rows and inv [T, k] maps (token, slot) to a row (or -1).
-// w null: no norm, no residual (x unused): out = T(y or the routed sum).  w_off / w_next_off: 1 for weights stored
-// around zero.
+// w null: no norm, no residual (x unused): out = T(y or the routed sum).  w_off / w_next_off: 1 where
+// the stored weight is the deviation from one.
 EXPORT int vb_post_norm_add(const void* y, int64_t y_stride, const int* inv, const float* pair_w, int k, const void* w,
                             int w_off, float* x, const void* w_next, int w_next_off, void* out, int T_, int H, float eps,
                             int dtype, cudaStream_t st) {

@@ -1,13 +1,13 @@
-"""Pomipel: latent attention (no positions in the scores) + group-limited experts, norms on the sublayers' outputs.
+"""Pomipel: position-free latent attention and group-limited experts in post-norm residual blocks.
 
-    x = embed[token] * embedding.scale + pos[position]                     learned positions, added unscaled
-    x = x + norm1(mixer(x));   x = x + norm2(experts(x))                   sublayers read x itself
-    logits = head norm(x) * logit_scale
+    x_0 = s_e E[t] + P[i]                 token t at index i: scaled embedding plus a learned position
+    x_{n+1} = x_n + N(F_n(x_n))           F_n: attention and experts in turn; the norm N is behind F_n, nothing in front of it
+    logits = s_l W_head N(x_last)
 
 * The stream x stays in fp32 (csrc/stream.cu); each step leaves the 16-bit copy the next GEMM reads.
 * Mixer: ``layers/latent.py``; a layer with ``kv_from`` reads the latent cache of that earlier layer.
 * Feed-forward: ungated squared-ReLU experts (``FusedMoE(gated=False)``) behind a sigmoid router with a selection bias and
-  group-limited choice, in 32-bit (``GroupedRouter``); the weights are the chosen scores, not renormalised.
+  group-limited choice, in 32-bit (``GroupedRouter``); a chosen expert is mixed in with its plain sigmoid score.
 
 Sizes and constants come from the configuration layer by layer: layers may differ in heads, widths and experts, and a
 layer may have no feed-forward.
