@@ -252,10 +252,11 @@ def _ssm_md(q_lens, ctx_lens, rows):
     qsl = torch.tensor([0] + list(torch.tensor(q_lens).cumsum(0)), dtype=torch.int32, device="cuda")
     sl = torch.tensor([c + q for c, q in zip(ctx_lens, q_lens)], dtype=torch.int32, device="cuda")
     bt = torch.tensor(rows, dtype=torch.int32, device="cuda").view(-1, 1).repeat(1, 3).contiguous()
-    return SimpleNamespace(num_reqs=len(q_lens), query_start_loc=qsl, seq_lens=sl, block_table=bt)
+    return SimpleNamespace(num_reqs=len(q_lens), query_start_loc=qsl, seq_lens=sl, block_table=bt, max_query_len=max(q_lens), flat=False,
+                           decode_only=max(q_lens) == 1)
 
 
-@pytest.mark.parametrize("K", [2, 4])
+@pytest.mark.parametrize("K", [1, 2, 3, 4, 6])
 def test_causal_conv1d_with_cached_window(K):
     torch.manual_seed(10)
     C, q_lens, ctx = 384, [5, 1, 17, 1], [0, 9, 3, 0]
@@ -275,7 +276,7 @@ def test_causal_conv1d_with_cached_window(K):
         xin = torch.cat([win.t(), x[s:s + n].float()], 0)                   # [K-1+n, C]
         conv = (xin.unfold(0, K, 1) * w.float()[None]).sum(-1) + b.float()
         close(out[s:s + n], torch.nn.functional.silu(conv), atol=2e-3, rtol=2e-3)
-        close(pool[rows[i], :C * (K - 1)].view(C, K - 1), xin[-(K - 1):].t(), atol=1e-6, rtol=0)
+        close(pool[rows[i], :C * (K - 1)].view(C, K - 1), xin[n:].t(), atol=1e-6, rtol=0)
         assert torch.equal(pool[rows[i], C * (K - 1):], pool0[rows[i], C * (K - 1):])      # rest of the row untouched
         s += n
 
@@ -305,28 +306,34 @@ def test_selective_scan_mamba1():
 
 @pytest.mark.parametrize("N,G", [(128, 1), (64, 2), (32, 4)])
 def test_ssd_scan_mamba2_matches_chunked_reference(N, G):
+    from vllm_b200 import ops
     torch.manual_seed(12)
     nh, hd, q_lens, ctx, rows = 8, 16, [70, 1, 9], [0, 11, 5], [1, 4, 2]
-    T = sum(q_lens)
     d_inner = nh * hd
-    xbc = torch.randn(T, d_inner + 2 * G * N, device="cuda") * 0.5
-    dt_raw = torch.randn(T, nh, device="cuda")
+    seqs = [torch.randn(c + n, d_inner + 2 * G * N, device="cuda") * 0.5 for c, n in zip(ctx, q_lens)]
+    dts = [torch.randn(c + n, nh, device="cuda") for c, n in zip(ctx, q_lens)]
     dt_bias, A_log, D = torch.randn(nh, device="cuda") * 0.3, torch.randn(nh, device="cuda") * 0.3, torch.randn(nh, device="cuda")
     off = 24
-    pool = torch.randn(6, off + nh * hd * N, device="cuda") * 0.3
+    pool = torch.randn(6, off + nh * ops.scan_state_elems(N, hd), device="cuda") * 0.3
     pool0 = pool.clone()
-    y = cu().ssd_scan(xbc, dt_raw, dt_bias, A_log, D, pool, off, _ssm_md(q_lens, ctx, rows), nh, hd, G, N)
-    s = 0
+
+    def step(parts, at):            # at: tokens before this step, per request
+        live = [i for i, p in enumerate(parts) if p]
+        md = _ssm_md([parts[i] for i in live], [at[i] for i in live], [rows[i] for i in live])
+        y = cu().ssd_scan(torch.cat([seqs[i][at[i]:at[i] + parts[i]] for i in live]),
+                          torch.cat([dts[i][at[i]:at[i] + parts[i]] for i in live]), dt_bias, A_log, D, pool, off, md, nh, hd, G, N)
+        return dict(zip(live, y.split([parts[i] for i in live])))
+    step(ctx, [0, 0, 0])
+    got = step(q_lens, ctx)
     for i, n in enumerate(q_lens):
-        h0 = pool0[rows[i], off:].view(nh, hd, N).clone() if ctx[i] > 0 else None
-        seg = xbc[s:s + n]
-        xs, Bs, Cs = seg.split([d_inner, G * N, G * N], -1)
-        dt = torch.nn.functional.softplus(dt_raw[s:s + n] + dt_bias)
-        ye, hf = ref.ssd_chunk_scan(xs.view(n, nh, hd), dt, -torch.exp(A_log), Bs.view(n, G, N), Cs.view(n, G, N), 16, h0)
-        ye = ye + D[None, :, None] * xs.view(n, nh, hd)
-        close(y[s:s + n], ye.reshape(n, d_inner), atol=5e-3, rtol=5e-3)
-        close(pool[rows[i], off:].view(nh, hd, N), hf, atol=5e-3, rtol=5e-3)
-        s += n
+        xs, Bs, Cs = seqs[i].split([d_inner, G * N, G * N], -1)
+        t = ctx[i] + n
+        dt = torch.nn.functional.softplus(dts[i] + dt_bias)
+        ye, _ = ref.ssd_chunk_scan(xs.view(t, nh, hd), dt, -torch.exp(A_log), Bs.view(t, G, N), Cs.view(t, G, N), 16, None)
+        ye = ye + D[None, :, None] * xs.view(t, nh, hd)
+        close(got[i], ye.reshape(t, d_inner)[ctx[i]:], atol=5e-3, rtol=5e-3)
+    untouched = [r for r in range(6) if r not in rows]
+    assert torch.equal(pool[untouched], pool0[untouched]) and torch.equal(pool[:, :off], pool0[:, :off])
 
 
 def test_gdn_scan_matches_recurrence():

@@ -7,9 +7,11 @@ vllm/v1/core/kv_cache_manager.py:232-570 (``get_computed_blocks``,
 block reclamation for sliding-window layers), kv_cache_coordinator.py
 (hybrid groups sharing one pool).
 
-All groups share one ``BlockPool``; every group uses the same page size in
-bytes so a physical block id is valid in every layer's tensor (hybrid models
-get one block table per group).
+Attention groups share one ``BlockPool``: a block id is valid in every attention
+layer's tensor (hybrid models get one block table per group).  Recurrent layers
+form one group of their own whose "blocks" are state slots, one per live request,
+from a second, much smaller pool: the state of a layer is allocated once per
+slot, not once per page of tokens.
 """
 from __future__ import annotations
 
@@ -122,14 +124,21 @@ class KVCacheConfig:
     num_blocks: int
     kv_cache_tensors: list[KVCacheTensor] = field(default_factory=list)
     kv_cache_groups: list[KVCacheGroupSpec] = field(default_factory=list)
+    num_state_slots: int = 0      # rows of the recurrent layers' state tensors (row 0 takes the padding of graph buckets)
 
 
 def group_specs(layer_specs: dict[str, KVCacheSpec]) -> list[KVCacheGroupSpec]:
-    """Layers with identical specs share a group (= one block table); so do latent caches of different widths, whose pages
-    hold the same tokens (each layer owns a tensor of its own width)."""
+    """Layers whose pages hold the same tokens share a group (= one block table), whatever their widths and head counts: each
+    layer owns a tensor of its own shape.  Recurrent layers all share one group (= one state slot per request)."""
     groups: dict[KVCacheSpec, list[str]] = {}
     for name, spec in layer_specs.items():
-        key = replace(spec, head_size=0) if isinstance(spec, MLAAttentionSpec) else spec
+        key = spec
+        if isinstance(spec, MLAAttentionSpec):
+            key = replace(spec, head_size=0)
+        elif isinstance(spec, FullAttentionSpec):
+            key = replace(spec, num_kv_heads=0, head_size=0)
+        elif isinstance(spec, MambaSpec):
+            key = replace(spec, state_bytes=0)
         groups.setdefault(key, []).append(name)
     out = []
     for names in groups.values():
@@ -138,22 +147,37 @@ def group_specs(layer_specs: dict[str, KVCacheSpec]) -> list[KVCacheGroupSpec]:
     return out
 
 
+# part of the cache memory that state slots may take where token pages compete for it
+STATE_SHARE = 0.4
+
+
 def get_kv_cache_config(layer_specs: dict[str, KVCacheSpec], available_bytes: int, max_model_len: int,
                         num_gpu_blocks_override: Optional[int] = None,
-                        auto_fit_max_model_len: bool = False) -> tuple[KVCacheConfig, int]:
-    """Size the pool. Returns (config, possibly reduced max_model_len)."""
+                        auto_fit_max_model_len: bool = False, max_num_seqs: int = 256) -> tuple[KVCacheConfig, int]:
+    """Size the pools. Returns (config, possibly reduced max_model_len)."""
     if not layer_specs:
         return KVCacheConfig(num_blocks=2), max_model_len
     groups = group_specs(layer_specs)
-    # every layer owns its own tensor of ``num_blocks`` pages (pages of different groups — attention K/V pages,
-    # sliding-window pages, recurrent-state pages — may differ in size); block ids are shared across groups, so the
-    # pool size is what fits when every layer gets one page per block
-    per_block = sum(s.page_size_bytes for s in layer_specs.values())
-    page = max(g.spec.page_size_bytes for g in groups)
-    num_blocks = int(available_bytes // max(per_block, 1))
+    state = [s for s in layer_specs.values() if isinstance(s, MambaSpec)]
+    pages = [s for s in layer_specs.values() if not isinstance(s, MambaSpec)]
+    num_slots = 0
+    if state:
+        # one slot per request that may run, fewer where they would crowd out the token pages (requests then wait for one)
+        per_slot = sum(s.page_size_bytes for s in state)
+        budget = int(available_bytes * (STATE_SHARE if pages and num_gpu_blocks_override is None else 1.0))
+        num_slots = max(min(max_num_seqs + 1, budget // max(per_slot, 1)), 2)
+        available_bytes -= num_slots * per_slot
+        if available_bytes < 0:
+            raise ValueError(f"no room for the recurrent state of one request ({per_slot} bytes per request)")
+    # every attention layer owns its own tensor of ``num_blocks`` pages (pages of different groups — attention K/V pages,
+    # sliding-window pages — may differ in size); block ids are shared across groups, so the pool size is what fits when
+    # every layer gets one page per block
+    per_block = sum(s.page_size_bytes for s in pages)
+    num_blocks = int(available_bytes // per_block) if pages else 2
     if num_gpu_blocks_override is not None:
         num_blocks = num_gpu_blocks_override
-    need_blocks = sum(cdiv(g.spec.max_memory_usage_bytes(max_model_len), g.spec.page_size_bytes) for g in groups) + 1
+    need_blocks = sum(cdiv(g.spec.max_memory_usage_bytes(max_model_len), g.spec.page_size_bytes) for g in groups
+                      if not isinstance(g.spec, MambaSpec)) + 1
     if num_blocks < need_blocks:
         if auto_fit_max_model_len and num_blocks > 2:
             bs = groups[0].spec.block_size
@@ -163,8 +187,9 @@ def get_kv_cache_config(layer_specs: dict[str, KVCacheSpec], available_bytes: in
                 f"KV cache too small: {num_blocks} blocks available but one request of max_model_len="
                 f"{max_model_len} needs {need_blocks}; lower max_model_len or raise "
                 f"gpu_memory_utilization")
-    tensors = [KVCacheTensor(size=sp.page_size_bytes * num_blocks, shared_by=[name]) for name, sp in layer_specs.items()]
-    return KVCacheConfig(num_blocks=num_blocks, kv_cache_tensors=tensors, kv_cache_groups=groups), max_model_len
+    tensors = [KVCacheTensor(size=sp.page_size_bytes * (num_slots if isinstance(sp, MambaSpec) else num_blocks), shared_by=[name])
+               for name, sp in layer_specs.items()]
+    return KVCacheConfig(num_blocks=num_blocks, num_state_slots=num_slots, kv_cache_tensors=tensors, kv_cache_groups=groups), max_model_len
 
 
 # ---------------------------------------------------------------------------
@@ -290,7 +315,7 @@ class SlidingWindowManager(SingleTypeManager):
 
 
 class MambaManager(SingleTypeManager):
-    """One state block per request regardless of length."""
+    """One state slot per request regardless of length (``pool`` holds slots, not token pages)."""
 
     def blocks_needed(self, request_id, num_tokens, new_computed) -> int:
         return 0 if self.req_to_blocks.get(request_id) else 1
@@ -308,6 +333,9 @@ class MambaManager(SingleTypeManager):
 
     def find_longest_hit(self, hashes, max_blocks):
         return []
+
+    def num_common_prefix_blocks(self, request_id: str, num_running: int) -> int:
+        return 0
 
 
 def _manager_for(spec: KVCacheSpec, pool: BlockPool, gid: int) -> SingleTypeManager:
@@ -360,7 +388,11 @@ class KVCacheManager:
         self.block_size = groups[0].spec.block_size if groups else 16
         self.pool = BlockPool(kv_cache_config.num_blocks, enable_caching, enable_kv_cache_events,
                               self.block_size)
-        self.managers = [_manager_for(g.spec, self.pool, i) for i, g in enumerate(groups)]
+        # state slots of the recurrent layers: a pool of their own, never prefix-cached
+        self.state_pool = BlockPool(kv_cache_config.num_state_slots, False, False, self.block_size) \
+            if any(isinstance(g.spec, MambaSpec) for g in groups) else None
+        self.managers = [_manager_for(g.spec, self.state_pool if isinstance(g.spec, MambaSpec) else self.pool, i)
+                         for i, g in enumerate(groups)]
         self.num_groups = len(self.managers)
         self.block_hasher = make_block_hasher(self.block_size, hash_algo) if enable_caching else None
         self.prefix_cache_stats = PrefixCacheStats()
@@ -449,8 +481,13 @@ class KVCacheManager:
             m.remove_skipped_blocks(rid, request.num_computed_tokens)
         num_computed = request.num_computed_tokens + num_new_computed_tokens
         total = min(num_computed + num_new_tokens + num_lookahead_tokens, self.max_model_len)
-        needed = sum(m.blocks_needed(rid, total, nc) for m, nc in zip(self.managers, new_computed))
-        if needed > self.pool.get_num_free_blocks():
+        needed = slots = 0
+        for m, nc in zip(self.managers, new_computed):
+            if m.pool is self.state_pool:
+                slots += m.blocks_needed(rid, total, nc)
+            else:
+                needed += m.blocks_needed(rid, total, nc)
+        if needed > self.pool.get_num_free_blocks() or (slots and slots > self.state_pool.get_num_free_blocks()):
             return None
         if self.enable_caching:
             for nc in new_computed:

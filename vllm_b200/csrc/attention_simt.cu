@@ -77,6 +77,7 @@ __global__ void __launch_bounds__(THREADS) paged_attn_kernel(const AttnParams p)
   int kv_end = p.causal ? pos_last + 1 : seq_len;
   int kv_begin = 0;
   if (p.window > 0) kv_begin = max(0, pos0 - p.window + 1);
+  if (p.chunk > 0) kv_begin = max(kv_begin, pos0 / p.chunk * p.chunk);
   int page_lo = kv_begin / BS, page_hi = (kv_end + BS - 1) / BS;
   const int n_pages_total = page_hi - page_lo;
   const int per_split = (n_pages_total + p.num_splits - 1) / p.num_splits;

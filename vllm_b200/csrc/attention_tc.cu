@@ -45,6 +45,9 @@ struct Params {
   float scale_log2;
   int flat_B;              // > 0: grid.x enumerates the (request, query tile) pairs of `flat_B` requests (device-side
                            //      schedule from qsl: the launch geometry depends only on the bucket, not on the lengths)
+  int chunk;               // > 0: a query sees the keys of its own chunk of positions only
+  const float* sinks;      // optional [Hq] logits in the softmax denominator that have no key
+  float out_scale;         // factor of the output
 };
 
 VB_DEVICE void tma_load_3d(void* dst, const void* tmap, int c0, int c1, int c2, uint64_t* bar) {
@@ -130,7 +133,8 @@ fmha_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ 
   const int pos0 = seq_len - q_len + tok0;
   const int pos_last = pos0 + n_tok - 1;
   const int kv_end = p.causal ? pos_last + 1 : seq_len;
-  const int kv_begin = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  int kv_begin = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  if (p.chunk > 0) kv_begin = max(kv_begin, pos0 / p.chunk * p.chunk);
   int tile_lo = kv_begin / TILE_N, tile_hi = (kv_end + TILE_N - 1) / TILE_N;
   {
     const int total = tile_hi - tile_lo;
@@ -277,6 +281,7 @@ fmha_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ 
     const int tq = r / p.G, g = r % p.G;
     const bool row_valid = tq < n_tok && r < p.G * p.TQ;
     const int qpos = row_valid ? pos0 + tq : -1;
+    const int row_lo = max(p.window > 0 ? qpos - p.window + 1 : 0, p.chunk > 0 ? max(qpos, 0) / p.chunk * p.chunk : 0);
     float m_used = -INFINITY, l_run = 0.f;
     for (int j = 0; j < n_tiles; ++j) {
       const int sb = j & 1;
@@ -286,7 +291,7 @@ fmha_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ 
       tc_fence_after();
       // valid column range for this row: [lo, hi)
       int hi = min(kv_end, p.causal ? qpos + 1 : kv_end) - tile_pos;
-      int lo = max(kv_begin, p.window > 0 ? qpos - p.window + 1 : 0) - tile_pos;
+      int lo = max(kv_begin, row_lo) - tile_pos;
       if (!row_valid) hi = -1;
       // ---- pass 1: row max
       float mx = -INFINITY;
@@ -359,10 +364,18 @@ fmha_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ 
     // ---- epilogue
     mbar_wait(pv_done, (n_tiles - 1) & 1);
     tc_fence_after();
-    const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
     const int64_t tok = q0 + tok0 + tq;
     const int hq = h * p.G + g;
+    float inv = l_run > 0.f ? 1.f / l_run : 0.f;
     if (p.num_splits == 1) {
+      if (p.sinks && row_valid) {                    // the sink joins the denominator once, behind the last key
+        const float sink = p.sinks[hq] * 1.4426950408889634f;
+        const float top = fmaxf(m_used, sink), f = ex2(m_used - top);
+        l_run = l_run * f + ex2(sink - top);
+        m_used = top;
+        inv = f / l_run;
+      }
+      inv *= p.out_scale;
       T* orow = reinterpret_cast<T*>(p.out) + tok * p.out_stride + (int64_t)hq * D;
 #pragma unroll
       for (int c = 0; c < D; c += 32) {
@@ -411,19 +424,20 @@ fmha_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ 
 template <typename T, int DD>
 __global__ void __launch_bounds__(DD) split_reduce(const float* __restrict__ part_out, const float* __restrict__ part_lse,
                                                    T* __restrict__ out, float* __restrict__ lse_out, int Hq, int S,
-                                                   int64_t out_stride) {
+                                                   int64_t out_stride, const float* __restrict__ sinks, float out_scale) {
   const int tok = blockIdx.x, hq = blockIdx.y, d = threadIdx.x;
   const int64_t base = ((int64_t)tok * Hq + hq) * S;
-  float m = -INFINITY;
+  const float sink = sinks ? sinks[hq] * 1.4426950408889634f : -INFINITY;
+  float m = sink;
   for (int s = 0; s < S; ++s) m = fmaxf(m, part_lse[base + s]);
   const float m_use = (m == -INFINITY) ? 0.f : m;
-  float den = 0.f, o = 0.f;
+  float den = sinks ? ex2(sink - m_use) : 0.f, o = 0.f;
   for (int s = 0; s < S; ++s) {
     const float wgt = ex2(part_lse[base + s] - m_use);
     den += wgt;
     o += wgt * part_out[(base + s) * DD + d];
   }
-  out[(int64_t)tok * out_stride + (int64_t)hq * DD + d] = from_f32<T>(den > 0.f ? o / den : 0.f);
+  out[(int64_t)tok * out_stride + (int64_t)hq * DD + d] = from_f32<T>(den > 0.f ? o / den * out_scale : 0.f);
   if (lse_out && d == 0) lse_out[(int64_t)tok * Hq + hq] = den > 0.f ? (m + log2f(den)) * 0.6931471805599453f : -INFINITY;
 }
 
@@ -444,26 +458,13 @@ static EncodeTiledFn get_encode() {
 }  // namespace fmha
 
 // kv_cache: [nb, 2, Hkv, BS*D] with K pages [BS, D] and V pages stored transposed [D, BS].
-EXPORT int vb_fmha_tc2(const void* q, const void* kv_cache, int64_t num_blocks, const int* block_table,
-                       const int* seq_lens, const int* qsl, void* out, float* part_out, float* part_lse,
-                       float* lse_out, int B, int T_total, int max_q_len, int Hq, int Hkv, int64_t q_stride,
-                       int64_t out_stride, int bt_stride, int num_splits, int window, float scale, int causal,
-                       int flat, int dtype, cudaStream_t st);
-EXPORT int vb_fmha_tc(const void* q, const void* kv_cache, int64_t num_blocks, const int* block_table,
-                      const int* seq_lens, const int* qsl, void* out, float* part_out, float* part_lse,
-                      float* lse_out, int B, int T_total, int max_q_len, int Hq, int Hkv, int64_t q_stride,
-                      int64_t out_stride, int bt_stride, int num_splits, int window, float scale, int causal,
-                      int dtype, cudaStream_t st) {
-  return vb_fmha_tc2(q, kv_cache, num_blocks, block_table, seq_lens, qsl, out, part_out, part_lse, lse_out, B, T_total,
-                     max_q_len, Hq, Hkv, q_stride, out_stride, bt_stride, num_splits, window, scale, causal, 0, dtype, st);
-}
 // flat != 0 (varlen only): the grid is sized from (T_total, B) alone — T_total / TQ + B tiles bound every split of
 // T_total tokens over B requests — so one captured launch serves any mixed batch of that bucket.
 EXPORT int vb_fmha_tc2(const void* q, const void* kv_cache, int64_t num_blocks, const int* block_table,
                        const int* seq_lens, const int* qsl, void* out, float* part_out, float* part_lse,
                        float* lse_out, int B, int T_total, int max_q_len, int Hq, int Hkv, int64_t q_stride,
                        int64_t out_stride, int bt_stride, int num_splits, int window, float scale, int causal,
-                       int flat, int dtype, cudaStream_t st) {
+                       int flat, int chunk, const float* sinks, float out_scale, int dtype, cudaStream_t st) {
   using namespace fmha;
   if (B == 0) return 0;
   if (dtype == DT_F32) return -1;
@@ -479,6 +480,7 @@ EXPORT int vb_fmha_tc2(const void* q, const void* kv_cache, int64_t num_blocks, 
   p.Hkv = Hkv; p.G = G; p.TQ = qsl ? TILE_M / G : 1; p.num_splits = qsl ? 1 : num_splits; p.window = window;
   p.causal = causal; p.scale_log2 = scale * 1.4426950408889634f;
   p.flat_B = (flat && qsl) ? B : 0;
+  p.chunk = chunk; p.sinks = sinks; p.out_scale = out_scale;
   CUtensorMap tq, tk, tv;
   {  // q: [T, Hq, D] with token stride q_stride; box {64, G, TQ}
     cuuint64_t dims[3] = {(cuuint64_t)D, (cuuint64_t)Hq, (cuuint64_t)T_total};
@@ -524,8 +526,8 @@ EXPORT int vb_fmha_tc2(const void* q, const void* kv_cache, int64_t num_blocks, 
   int rc = (int)cudaGetLastError();
   if (rc) return rc;
   if (!qsl && p.num_splits > 1) {
-    if (bf16) split_reduce<__nv_bfloat16, D><<<dim3(B, Hq), D, 0, st>>>(part_out, part_lse, (__nv_bfloat16*)out, lse_out, Hq, p.num_splits, out_stride);
-    else split_reduce<__half, D><<<dim3(B, Hq), D, 0, st>>>(part_out, part_lse, (__half*)out, lse_out, Hq, p.num_splits, out_stride);
+    if (bf16) split_reduce<__nv_bfloat16, D><<<dim3(B, Hq), D, 0, st>>>(part_out, part_lse, (__nv_bfloat16*)out, lse_out, Hq, p.num_splits, out_stride, sinks, out_scale);
+    else split_reduce<__half, D><<<dim3(B, Hq), D, 0, st>>>(part_out, part_lse, (__half*)out, lse_out, Hq, p.num_splits, out_stride, sinks, out_scale);
   }
   return (int)cudaGetLastError();
 }

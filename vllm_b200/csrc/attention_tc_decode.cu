@@ -36,6 +36,9 @@ struct Params {
   int bt_stride;
   int Hq, Hkv, G, num_splits, window, B;
   float scale_log2;
+  int chunk;               // > 0: the query sees the keys of its own chunk of positions only
+  const float* sinks;      // optional [Hq] logits in the softmax denominator that have no key
+  float out_scale;         // factor of the output
 };
 
 VB_DEVICE void tma_load_3d(void* dst, const void* tmap, int c0, int c1, int c2, uint64_t* bar) {
@@ -119,6 +122,7 @@ fmha_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
     const int seq_len = p.seq_lens[b];
     kv_end = seq_len;
     kv_begin = p.window > 0 ? max(0, seq_len - p.window) : 0;
+    if (p.chunk > 0) kv_begin = max(kv_begin, (seq_len - 1) / p.chunk * p.chunk);
     tile_lo = kv_begin / TILE;
     int tile_hi = (kv_end + TILE - 1) / TILE;
     const int per = (tile_hi - tile_lo + p.num_splits - 1) / p.num_splits;
@@ -341,9 +345,17 @@ fmha_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         const float o = __uint_as_float(ov[g]) * inv;
         const int hq = h * G + g;
         if (p.num_splits == 1) {
-          reinterpret_cast<T*>(p.out)[(int64_t)b * p.out_stride + (int64_t)hq * D + d] = from_f32<T>(o);
+          float top = m_used[g], f = 1.f, den = l;       // the sink joins the denominator once, behind the last key
+          if (p.sinks) {
+            const float sink = p.sinks[hq] * 1.4426950408889634f;
+            top = fmaxf(top, sink);
+            f = ex2(m_used[g] - top);
+            den = l * f + ex2(sink - top);
+          }
+          const float r = p.sinks ? __uint_as_float(ov[g]) * (f / den) : o;
+          reinterpret_cast<T*>(p.out)[(int64_t)b * p.out_stride + (int64_t)hq * D + d] = from_f32<T>(r * p.out_scale);
           if (p.lse_out && d == 0)
-            p.lse_out[(int64_t)b * p.Hq + hq] = l > 0.f ? (m_used[g] + log2f(l)) * 0.6931471805599453f : -INFINITY;
+            p.lse_out[(int64_t)b * p.Hq + hq] = den > 0.f ? (top + log2f(den)) * 0.6931471805599453f : -INFINITY;
         } else {
           const int64_t pi = ((int64_t)b * p.Hq + hq) * p.num_splits + split;
           p.part_out[pi * D + d] = o;
@@ -361,20 +373,21 @@ fmha_decode_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
 
 template <typename T>
 __global__ void __launch_bounds__(128) split_reduce(const float* __restrict__ part_out, const float* __restrict__ part_lse,
-                                                    T* __restrict__ out, float* __restrict__ lse_out, int Hq, int S,
-                                                    int64_t out_stride) {
+                                                   T* __restrict__ out, float* __restrict__ lse_out, int Hq, int S,
+                                                   int64_t out_stride, const float* __restrict__ sinks, float out_scale) {
   const int tok = blockIdx.x, hq = blockIdx.y, d = threadIdx.x;
   const int64_t base = ((int64_t)tok * Hq + hq) * S;
-  float m = -INFINITY;
+  const float sink = sinks ? sinks[hq] * 1.4426950408889634f : -INFINITY;
+  float m = sink;
   for (int s = 0; s < S; ++s) m = fmaxf(m, part_lse[base + s]);
   const float m_use = (m == -INFINITY) ? 0.f : m;
-  float den = 0.f, o = 0.f;
+  float den = sinks ? ex2(sink - m_use) : 0.f, o = 0.f;
   for (int s = 0; s < S; ++s) {
     const float wgt = ex2(part_lse[base + s] - m_use);
     den += wgt;
     o += wgt * part_out[(base + s) * D + d];
   }
-  out[(int64_t)tok * out_stride + (int64_t)hq * D + d] = from_f32<T>(den > 0.f ? o / den : 0.f);
+  out[(int64_t)tok * out_stride + (int64_t)hq * D + d] = from_f32<T>(den > 0.f ? o / den * out_scale : 0.f);
   if (lse_out && d == 0) lse_out[(int64_t)tok * Hq + hq] = den > 0.f ? (m + log2f(den)) * 0.6931471805599453f : -INFINITY;
 }
 
@@ -409,7 +422,8 @@ static int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMa
 EXPORT int vb_fmha_tc_decode(const void* q, const void* kv_cache, int64_t num_blocks, const int* block_table,
                              const int* seq_lens, void* out, float* part_out, float* part_lse, float* lse_out, int B,
                              int Hq, int Hkv, int64_t q_stride, int64_t out_stride, int bt_stride, int num_splits,
-                             int window, float scale, int dtype, cudaStream_t st) {
+                             int window, float scale, int chunk, const float* sinks, float out_scale, int dtype,
+                             cudaStream_t st) {
   using namespace fmha_dec;
   if (B == 0) return 0;
   if (dtype == DT_F32) return -1;
@@ -423,6 +437,7 @@ EXPORT int vb_fmha_tc_decode(const void* q, const void* kv_cache, int64_t num_bl
   p.block_table = block_table; p.seq_lens = seq_lens; p.out = out; p.part_out = part_out; p.part_lse = part_lse;
   p.lse_out = lse_out; p.out_stride = out_stride; p.bt_stride = bt_stride; p.Hq = Hq; p.Hkv = Hkv; p.G = G;
   p.num_splits = num_splits; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.B = B;
+  p.chunk = chunk; p.sinks = sinks; p.out_scale = out_scale;
   CUtensorMap tq, tk, tv;
   {
     cuuint64_t dims[3] = {(cuuint64_t)D, (cuuint64_t)Hq, (cuuint64_t)B};
@@ -468,8 +483,8 @@ EXPORT int vb_fmha_tc_decode(const void* q, const void* kv_cache, int64_t num_bl
 #undef VB_GO
   if (rc) return rc;
   if (num_splits > 1) {
-    if (bf16) split_reduce<__nv_bfloat16><<<dim3(B, Hq), 128, 0, st>>>(part_out, part_lse, (__nv_bfloat16*)out, lse_out, Hq, num_splits, out_stride);
-    else split_reduce<__half><<<dim3(B, Hq), 128, 0, st>>>(part_out, part_lse, (__half*)out, lse_out, Hq, num_splits, out_stride);
+    if (bf16) split_reduce<__nv_bfloat16><<<dim3(B, Hq), 128, 0, st>>>(part_out, part_lse, (__nv_bfloat16*)out, lse_out, Hq, num_splits, out_stride, sinks, out_scale);
+    else split_reduce<__half><<<dim3(B, Hq), 128, 0, st>>>(part_out, part_lse, (__half*)out, lse_out, Hq, num_splits, out_stride, sinks, out_scale);
   }
   return (int)cudaGetLastError();
 }

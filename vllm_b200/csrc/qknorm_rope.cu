@@ -51,6 +51,7 @@ struct Params {
   int64_t q_stride, k_stride, v_stride;
   int T, Hq, Hkv, D, rot, BS;
   int neox, gemma, kv_fp8, vt;
+  int keep32;                              // the normalised head stays in 32 bits on its way to the rotation
   float eps, k_inv_scale, v_inv_scale;
 };
 
@@ -113,7 +114,8 @@ __global__ void __launch_bounds__(256) qknorm_rope_cache_kernel(const Params p) 
     for (int j = 0; j < E; ++j) {
       float g = to_f32(wv.e[j]);
       if (p.gemma) g += 1.f;
-      f[j] = to_f32(from_f32<T>(f[j] * inv * g));     // round through T like the unfused norm does
+      f[j] *= inv * g;
+      if (!p.keep32) f[j] = to_f32(from_f32<T>(f[j]));     // round through T like the unfused norm does
     }
   }
   if (p.rot > 0) {
@@ -161,10 +163,68 @@ __global__ void __launch_bounds__(256) qknorm_rope_cache_kernel(const Params p) 
   }
 }
 
+// The same for every head size, rotated width, value width and dtype: one warp per (token, head), the head in shared memory,
+// 32-bit between norm and rotation.  DV: value width; DC: width of a cache row.
+constexpr int ANY_MAX_D = 512, ANY_WARPS = 4;
+template <typename T>
+__global__ void __launch_bounds__(ANY_WARPS * 32) qknorm_rope_any_kernel(const Params p, int DV, int DC) {
+  __shared__ float buf[ANY_WARPS][ANY_MAX_D];
+  pdl_trigger();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  float* f = buf[threadIdx.x >> 5];
+  const int items = p.Hq + 2 * p.Hkv;
+  const int64_t wg = (int64_t)blockIdx.x * ANY_WARPS + (threadIdx.x >> 5);
+  if (wg >= (int64_t)p.T * items) return;
+  const int t = (int)(wg / items), it = (int)(wg % items), D = p.D;
+  const int64_t slot = p.slot_mapping ? p.slot_mapping[t] : -1;
+  const bool do_cache = p.kv_cache != nullptr && slot >= 0;
+  const int64_t blk = do_cache ? slot / p.BS : 0;
+  const int off = do_cache ? (int)(slot % p.BS) : 0;
+  T* cache = reinterpret_cast<T*>(p.kv_cache);
+  if (it >= p.Hq + p.Hkv) {
+    if (!do_cache || p.v == nullptr) return;
+    const int h = it - p.Hq - p.Hkv;
+    const T* v = reinterpret_cast<const T*>(p.v) + t * p.v_stride + (int64_t)h * DV;
+    T* dst = cache + ((blk * 2 + 1) * p.Hkv + h) * p.BS * (int64_t)DC + (p.vt ? off : off * DC);
+    for (int d = lane; d < DV; d += 32) dst[p.vt ? (int64_t)d * p.BS : d] = v[d];
+    return;
+  }
+  const bool is_k = it >= p.Hq;
+  const int h = is_k ? it - p.Hq : it;
+  T* base = is_k ? reinterpret_cast<T*>(p.k) + t * p.k_stride + (int64_t)h * D
+                 : reinterpret_cast<T*>(p.q) + t * p.q_stride + (int64_t)h * D;
+  const T* w = reinterpret_cast<const T*>(is_k ? p.k_w : p.q_w);
+  float ss = 0.f;
+  for (int d = lane; d < D; d += 32) { const float x = to_f32(base[d]); f[d] = x; ss += x * x; }
+  if (w != nullptr) {
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)D + p.eps);
+    for (int d = lane; d < D; d += 32) f[d] *= inv * (to_f32(w[d]) + (p.gemma ? 1.f : 0.f));
+  }
+  __syncwarp();
+  T* dst = is_k && do_cache ? cache + ((blk * 2 * p.Hkv + h) * p.BS + off) * (int64_t)DC : nullptr;
+  const int half = p.rot / 2;
+  const float* cs = p.rot > 0 ? p.cos_sin + p.positions[t] * p.rot : nullptr;
+  for (int d = lane; d < D; d += 32) {
+    float x = f[d];
+    if (d < p.rot) {
+      const int i = p.neox ? d % half : d >> 1;
+      const bool first = p.neox ? d < half : (d & 1) == 0;
+      const float o = f[p.neox ? (first ? d + half : d - half) : d ^ 1];
+      const float co = cs[i], si = cs[half + i];
+      x = first ? x * co - o * si : x * co + o * si;
+    }
+    const T y = from_f32<T>(x);
+    base[d] = y;
+    if (dst) dst[d] = y;
+  }
+}
+
 }  // namespace
 
 // q, k: [T, H*D] views of the fused qkv buffer (rotated / normalised in place); v may be null (no cache write of V);
-// kv_cache may be null (norm + rope only).  flags: bit0 fp8 cache, bit1 transposed V pages.
+// kv_cache may be null (norm + rope only).  flags: bit0 fp8 cache, bit1 transposed V pages, bit2 no rounding to T between the
+// norm and the rotation.
 EXPORT int vb_qknorm_rope_cache(const int64_t* positions, void* q, void* k, const void* v, const void* q_w, const void* k_w,
                                 const float* cos_sin, int rot, int T, int Hq, int Hkv, int D, int64_t q_stride,
                                 int64_t k_stride, int64_t v_stride, void* kv_cache, const int64_t* slot_mapping, int BS,
@@ -187,7 +247,7 @@ EXPORT int vb_qknorm_rope_cache(const int64_t* positions, void* q, void* k, cons
   p.positions = positions; p.q = q; p.k = k; p.v = v; p.q_w = q_w; p.k_w = k_w; p.cos_sin = cos_sin;
   p.kv_cache = kv_cache; p.slot_mapping = slot_mapping; p.q_stride = q_stride; p.k_stride = k_stride; p.v_stride = v_stride;
   p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.rot = rot; p.BS = BS; p.neox = neox; p.gemma = gemma;
-  p.kv_fp8 = flags & 1; p.vt = (flags >> 1) & 1; p.eps = eps; p.k_inv_scale = 1.f / k_scale; p.v_inv_scale = 1.f / v_scale;
+  p.kv_fp8 = flags & 1; p.vt = (flags >> 1) & 1; p.keep32 = (flags >> 2) & 1; p.eps = eps; p.k_inv_scale = 1.f / k_scale; p.v_inv_scale = 1.f / v_scale;
   const int64_t warps = (int64_t)T * (Hq + 2 * Hkv);
   const int wpb = 8;
   const unsigned blocks = (unsigned)((warps + wpb - 1) / wpb);
@@ -199,5 +259,22 @@ EXPORT int vb_qknorm_rope_cache(const int64_t* positions, void* q, void* k, cons
       default: vb_launch(qknorm_rope_cache_kernel<TT, 16>, dim3(blocks), dim3(wpb * 32), 0, st, p); break;
     }
   });
+  return (int)cudaGetLastError();
+}
+
+// Every other shape and dtype.  The cache holds the model dtype.
+EXPORT int vb_qknorm_rope_any(const int64_t* positions, void* q, void* k, const void* v, const void* q_w, const void* k_w,
+                              const float* cos_sin, int rot, int T, int Hq, int Hkv, int D, int DV, int DC, int64_t q_stride,
+                              int64_t k_stride, int64_t v_stride, void* kv_cache, const int64_t* slot_mapping, int BS, int neox,
+                              int gemma, int vt, float eps, int dtype, cudaStream_t st) {
+  if (T == 0) return 0;
+  if (D > ANY_MAX_D || rot > D || rot % 2 || DC < D || DC < DV) return -1;
+  Params p = {};
+  p.positions = positions; p.q = q; p.k = k; p.v = v; p.q_w = q_w; p.k_w = k_w; p.cos_sin = cos_sin;
+  p.kv_cache = kv_cache; p.slot_mapping = slot_mapping; p.q_stride = q_stride; p.k_stride = k_stride; p.v_stride = v_stride;
+  p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.rot = rot; p.BS = BS; p.neox = neox; p.gemma = gemma; p.vt = vt; p.eps = eps;
+  const int64_t warps = (int64_t)T * (Hq + 2 * Hkv);
+  dim3 grid((unsigned)((warps + ANY_WARPS - 1) / ANY_WARPS));
+  DISPATCH_DTYPE(dtype, TT, vb_launch(qknorm_rope_any_kernel<TT>, grid, dim3(ANY_WARPS * 32), 0, st, p, DV, DC));
   return (int)cudaGetLastError();
 }

@@ -1,12 +1,10 @@
 // State-space / linear-attention kernels over the paged recurrent-state cache (sm_100a):
 //   causal depthwise conv1d with cached window     (Mamba-1/2, gated delta net; prefill, chunked prefill, decode)
 //   Mamba-1 selective scan                          (per-channel A, state N <= 32)
-//   Mamba-2 SSD scan / selective_state_update       (scalar decay per head, state [hd, N] per head)
 //   gated delta rule scan                           (Qwen3-Next GDN: rank-1 corrected state [dk, dv] per head)
 //
 // Reference ops: csrc/libtorch_stable/mamba/selective_scan_fwd.cu, vllm/model_executor/layers/mamba/ops/
-// causal_conv1d.py, mamba_ssm.py (selective_state_update), ssd_combined.py (+ ssd_chunk_scan / state passing),
-// fla ops/fused_recurrent (GDN decode).  One design replaces that family here: every op is a varlen kernel driven
+// causal_conv1d.py, fla ops/fused_recurrent (GDN decode).  One design replaces that family here: every op is a varlen kernel driven
 // by device-resident `query_start_loc` / `seq_lens` / cache-row ids, reads and writes the request's state row in
 // the cache pool in place, and walks the request's tokens in order with the state held in registers — decode is
 // the q = 1 case of the same kernel, so there is one code path, no host loop, no `.tolist()`, and every batch shape
@@ -19,44 +17,85 @@
 namespace {
 
 VB_DEVICE float silu_f(float x) { return x / (1.f + __expf(-x)); }
-VB_DEVICE float softplus_f(float x) { return x > 20.f ? x : log1pf(__expf(x)); }
 
 // ------------------------------------------------------------------ causal conv1d (+ SiLU), window cached per request
-// grid (num_reqs, ceil(C / 256)); thread = one channel, walks the request's tokens with the k-1 window in registers.
-template <typename T, int K>
-__global__ void __launch_bounds__(256) causal_conv1d_kernel(const T* __restrict__ x, int64_t x_stride, float* __restrict__ out,
+// Thread = one channel x TT consecutive tokens of the batch: the grid depends on the token count alone, and a long prompt is
+// spread over all SMs.  A token's request is found from query_start_loc.  The cached window of a request (the last K - 1
+// inputs) is read and rewritten by one thread only, the one that has the request's first token; it also takes the tokens
+// behind its tile that still look into the old window.  KT: compile-time tap count, 0: any up to MAX_TAPS.
+constexpr int CONV_TT = 16, MAX_TAPS = 16;
+template <typename T, int KT>
+__global__ void __launch_bounds__(128) causal_conv1d_kernel(const T* __restrict__ x, int64_t x_stride, float* __restrict__ out,
                                                              int64_t out_stride, const T* __restrict__ w,
                                                              const T* __restrict__ bias, float* __restrict__ state,
                                                              int64_t state_stride, const int* __restrict__ qsl,
                                                              const int* __restrict__ seq_lens,
-                                                             const int* __restrict__ rows, int64_t rows_stride, int C,
-                                                             int act) {
+                                                             const int* __restrict__ rows, int64_t rows_stride, int num_reqs,
+                                                             int n_tok, int C, int taps, int act) {
+  constexpr int KM = KT ? KT : MAX_TAPS;
   pdl_trigger();
   pdl_wait();
-  const int r = blockIdx.x;
+  const int K = KT ? KT : taps;
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
-  const int t0 = qsl[r], t1 = qsl[r + 1];
-  if (c >= C || t1 <= t0) return;
-  const bool has_init = seq_lens[r] - (t1 - t0) > 0;
-  float* st = state + (int64_t)rows[r * rows_stride] * state_stride + (int64_t)c * (K - 1);
-  float win[K];
-#pragma unroll
-  for (int j = 0; j < K - 1; ++j) win[j] = has_init ? st[j] : 0.f;
-  float wr[K];
-#pragma unroll
-  for (int j = 0; j < K; ++j) wr[j] = to_f32(w[(int64_t)c * K + j]);
-  const float b = bias ? to_f32(bias[c]) : 0.f;
-  for (int t = t0; t < t1; ++t) {
-    win[K - 1] = to_f32(x[t * x_stride + c]);
-    float acc = b;
-#pragma unroll
-    for (int j = 0; j < K; ++j) acc += wr[j] * win[j];
-    out[t * out_stride + c] = act ? silu_f(acc) : acc;
-#pragma unroll
-    for (int j = 0; j < K - 1; ++j) win[j] = win[j + 1];
+  if (c >= C) return;
+  const int tile0 = blockIdx.x * CONV_TT, tile1 = min(tile0 + CONV_TT, n_tok);
+  const int total = qsl[num_reqs];
+  // last request that starts at or before the tile and is not empty there
+  int r = 0;
+  for (int lo = 0, hi = num_reqs - 1; lo <= hi;) {
+    const int mid = (lo + hi) >> 1;
+    if (qsl[mid] <= tile0) { r = mid; lo = mid + 1; } else hi = mid - 1;
   }
+  float wr[KM];
 #pragma unroll
-  for (int j = 0; j < K - 1; ++j) st[j] = win[j];
+  for (int j = 0; j < KM; ++j) wr[j] = j < K ? to_f32(w[(int64_t)c * K + j]) : 0.f;
+  const float b = bias ? to_f32(bias[c]) : 0.f;
+  int t = tile0;
+  while (t < tile1) {
+    if (t >= total) {                                   // padding of a graph bucket
+      out[t * out_stride + c] = 0.f;
+      ++t;
+      continue;
+    }
+    while (t >= qsl[r + 1]) ++r;
+    const int t0 = qsl[r], t1 = qsl[r + 1];
+    const bool first = t == t0;
+    if (!first && t < t0 + K - 1) { t = min(t0 + K - 1, t1); continue; }      // an earlier thread's tokens
+    const int end = first ? min(t1, max(tile1, t0 + K - 1)) : min(t1, tile1);
+    float win[KM];                                      // inputs t - K + 1 .. t - 1, then t
+    if (first) {
+      float* st = state + (int64_t)rows[r * rows_stride] * state_stride + (int64_t)c * (K - 1);
+      const bool has_init = seq_lens[r] - (t1 - t0) > 0;
+#pragma unroll
+      for (int j = 0; j < KM; ++j) win[j] = j < K - 1 && has_init ? st[j] : 0.f;
+      const int q = t1 - t0;
+#pragma unroll
+      for (int j = 0; j < KM; ++j) {
+        if (j >= K - 1) continue;
+        const int p = q - (K - 1) + j;                  // token of this step, or p + K - 1 = j + q of the old window
+        float v = 0.f;
+        if (p >= 0) v = to_f32(x[(int64_t)(t0 + p) * x_stride + c]);
+        else {
+#pragma unroll
+          for (int i = 0; i < KM; ++i) if (i == j + q) v = win[i];
+        }
+        st[j] = v;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < KM; ++j) win[j] = j < K - 1 ? to_f32(x[(int64_t)(t - (K - 1) + j) * x_stride + c]) : 0.f;
+    }
+#pragma unroll 4
+    for (; t < end; ++t) {
+      const float in = to_f32(x[(int64_t)t * x_stride + c]);
+      float acc = b;
+#pragma unroll
+      for (int j = 0; j < KM; ++j) acc += wr[j] * (j == K - 1 ? in : win[j]);
+      out[(int64_t)t * out_stride + c] = act ? silu_f(acc) : acc;
+#pragma unroll
+      for (int j = 0; j < KM - 1; ++j) win[j] = j == K - 2 ? in : win[j + 1];
+    }
+  }
 }
 
 // ------------------------------------------------------------------ Mamba-1 selective scan
@@ -95,58 +134,6 @@ __global__ void __launch_bounds__(128) selective_scan_kernel(const float* __rest
   }
 #pragma unroll
   for (int n = 0; n < N; ++n) st[n] = h[n];
-}
-
-// ------------------------------------------------------------------ Mamba-2 SSD scan (decode == q = 1)
-// warp = (request, head, p); lane holds NPL = N / 32 state elements of row p.
-//   h[p, n] = exp(dt·A_h) h[p, n] + dt x[p] B[g, n];   y[p] = Σ_n h[p, n] C[g, n] + D_h x[p]
-// xbc: [T, conv_dim] fp32 = x (nh*hd) | B (G*N) | C (G*N) (the conv1d output); dt_raw: [T, nh] (+dt_bias, softplus,
-// clamp in-kernel).
-template <int NPL>
-__global__ void __launch_bounds__(256) ssd_scan_kernel(const float* __restrict__ xbc, int64_t xbc_stride,
-                                                        const float* __restrict__ dt_raw, int64_t dt_stride,
-                                                        const float* __restrict__ dt_bias, const float* __restrict__ A_log,
-                                                        const float* __restrict__ D, float* __restrict__ y,
-                                                        float* __restrict__ state, int64_t state_stride, int64_t state_off,
-                                                        const int* __restrict__ qsl, const int* __restrict__ seq_lens,
-                                                        const int* __restrict__ rows, int64_t rows_stride, int nh, int hd,
-                                                        int G, float dt_min, float dt_max) {
-  pdl_trigger();
-  pdl_wait();
-  constexpr int N = NPL * 32;
-  const int lane = threadIdx.x & 31;
-  const int r = blockIdx.y;
-  const int wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);      // (head, p)
-  const int t0 = qsl[r], t1 = qsl[r + 1];
-  if (wid >= nh * hd || t1 <= t0) return;
-  const int hh = wid / hd, p = wid % hd;
-  const int g = hh / (nh / G);
-  const bool has_init = seq_lens[r] - (t1 - t0) > 0;
-  float* st = state + (int64_t)rows[r * rows_stride] * state_stride + state_off + ((int64_t)hh * hd + p) * N + lane * NPL;
-  float h[NPL];
-#pragma unroll
-  for (int i = 0; i < NPL; ++i) h[i] = has_init ? st[i] : 0.f;
-  const float a = -__expf(A_log[hh]), dd = D[hh], db = dt_bias[hh];
-  const int d_inner = nh * hd;
-  for (int t = t0; t < t1; ++t) {
-    const float* row = xbc + (int64_t)t * xbc_stride;
-    float dtv = softplus_f(dt_raw[(int64_t)t * dt_stride + hh] + db);
-    dtv = fminf(fmaxf(dtv, dt_min), dt_max);
-    const float xv = row[hh * hd + p];
-    const float dA = __expf(dtv * a), dx = dtv * xv;
-    const float* Bp = row + d_inner + g * N + lane * NPL;
-    const float* Cp = row + d_inner + G * N + g * N + lane * NPL;
-    float acc = 0.f;
-#pragma unroll
-    for (int i = 0; i < NPL; ++i) {
-      h[i] = dA * h[i] + dx * Bp[i];
-      acc += h[i] * Cp[i];
-    }
-    acc = warp_sum(acc);
-    if (lane == 0) y[(int64_t)t * d_inner + hh * hd + p] = acc + dd * xv;
-  }
-#pragma unroll
-  for (int i = 0; i < NPL; ++i) st[i] = h[i];
 }
 
 // ------------------------------------------------------------------ gated delta rule scan (GDN)
@@ -203,19 +190,19 @@ __global__ void __launch_bounds__(256) gdn_scan_kernel(const float* __restrict__
 
 }  // namespace
 
-// x: [T, C] (T-typed), out: [T, C] fp32; state rows hold the (k-1)-window at offset 0 ([C, k-1] fp32).
+// x: [T, C], out: [T, C] fp32 (rows behind the last request are zeroed); state rows hold the (k-1)-window at offset 0 ([C, k-1] fp32).
 // rows: cache-row id of each request (block_table[:, 0], int32, stride rows_stride).
 EXPORT int vb_causal_conv1d(const void* x, int64_t x_stride, float* out, int64_t out_stride, const void* w, const void* bias,
                             float* state, int64_t state_stride, const int* qsl, const int* seq_lens, const int* rows,
-                            int64_t rows_stride, int num_reqs, int C, int K, int act, int dtype, cudaStream_t st) {
-  if (num_reqs == 0) return 0;
-  if (dtype == DT_F32 || K < 2 || K > 4) return -1;
-  dim3 grid(num_reqs, (C + 255) / 256);
-#define GO(KK) vb_launch(causal_conv1d_kernel<TT, KK>, grid, dim3(256), 0, st, reinterpret_cast<const TT*>(x), x_stride, out, \
+                            int64_t rows_stride, int num_reqs, int n_tok, int C, int K, int act, int dtype, cudaStream_t st) {
+  if (num_reqs == 0 || n_tok == 0) return 0;
+  if (K < 1 || K > MAX_TAPS) return -1;
+  dim3 grid((n_tok + CONV_TT - 1) / CONV_TT, (C + 127) / 128);
+#define GO(KK) vb_launch(causal_conv1d_kernel<TT, KK>, grid, dim3(128), 0, st, reinterpret_cast<const TT*>(x), x_stride, out, \
                          out_stride, reinterpret_cast<const TT*>(w), reinterpret_cast<const TT*>(bias), state, state_stride,   \
-                         qsl, seq_lens, rows, rows_stride, C, act)
-  DISPATCH_HALF(dtype, TT, {
-    if (K == 2) GO(2); else if (K == 3) GO(3); else GO(4);
+                         qsl, seq_lens, rows, rows_stride, num_reqs, n_tok, C, K, act)
+  DISPATCH_DTYPE(dtype, TT, {
+    if (K == 2) GO(2); else if (K == 3) GO(3); else if (K == 4) GO(4); else GO(0);
   });
 #undef GO
   return (int)cudaGetLastError();
@@ -230,27 +217,6 @@ EXPORT int vb_selective_scan(const float* x, const float* dt, const float* B, co
 #define GO(NN) vb_launch(selective_scan_kernel<NN>, grid, dim3(128), 0, st, x, dt, B, C, A, D, y, state, state_stride, \
                          state_off, qsl, seq_lens, rows, rows_stride, di)
   if (N == 16) GO(16); else if (N == 8) GO(8); else if (N == 32) GO(32); else return -1;
-#undef GO
-  return (int)cudaGetLastError();
-}
-
-EXPORT int vb_ssd_scan(const float* xbc, int64_t xbc_stride, const float* dt_raw, int64_t dt_stride, const float* dt_bias,
-                       const float* A_log, const float* D, float* y, float* state, int64_t state_stride, int64_t state_off,
-                       const int* qsl, const int* seq_lens, const int* rows, int64_t rows_stride, int num_reqs, int nh, int hd,
-                       int G, int N, float dt_min, float dt_max, cudaStream_t st) {
-  if (num_reqs == 0) return 0;
-  if (N % 32 || N > 256 || nh % G) return -1;
-  const int wpb = 8;
-  dim3 grid((nh * hd + wpb - 1) / wpb, num_reqs);
-#define GO(P) vb_launch(ssd_scan_kernel<P>, grid, dim3(wpb * 32), 0, st, xbc, xbc_stride, dt_raw, dt_stride, dt_bias, A_log, D, \
-                        y, state, state_stride, state_off, qsl, seq_lens, rows, rows_stride, nh, hd, G, dt_min, dt_max)
-  switch (N / 32) {
-    case 1: GO(1); break;
-    case 2: GO(2); break;
-    case 4: GO(4); break;
-    case 8: GO(8); break;
-    default: return -1;
-  }
 #undef GO
   return (int)cudaGetLastError();
 }

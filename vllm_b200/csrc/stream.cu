@@ -6,6 +6,8 @@
 //   embed_stream      x = table[id] * scale (+ pos_table[position]);   out = T(x)
 //   post_norm_add     y = a dense sublayer output row, or the routed sum  sum_j w_j * rows[inv_j]  of an expert layer
 //                     x += rmsnorm(y) * w;   out = T(x)  |  T(rmsnorm(x) * w_next)
+//   norm_add          the same step for blocks with a norm on either side of a sublayer, layer norms or RMS norms:
+//                     x += m norm(y + bias);   out = T(norm_next(x))       (or x = table[id] at the model's entry)
 // The combine of the expert layer is the load of post_norm_add: expert outputs are read once, summed in slot order in
 // fp32 (deterministic) and never written back.
 #include "common.cuh"
@@ -144,6 +146,90 @@ post_norm_add_kernel(const T* __restrict__ y, int64_t y_stride, const int* __res
   }
 }
 
+// mean and variance (or the mean square) over the row held in v, then (v - mean) * rstd * w + b in place
+template <typename T, int V, int NV, bool LN>
+VB_DEVICE void normalise(float (&v)[NV][V], const T* w, const T* b, int w_off, int H, float eps, float* red) {
+  const int step = blockDim.x * V;
+  float mean = 0.f;
+  if constexpr (LN) {
+    float s = 0.f;
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+      if (threadIdx.x * V + n * step < H)
+#pragma unroll
+        for (int j = 0; j < V; ++j) s += v[n][j];
+    mean = block_sum(s, red) / (float)H;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int n = 0; n < NV; ++n)
+    if (threadIdx.x * V + n * step < H)
+#pragma unroll
+      for (int j = 0; j < V; ++j) { v[n][j] -= mean; ss += v[n][j] * v[n][j]; }
+  const float r = 1.f / sqrtf(block_sum(ss, red) / (float)H + eps);
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * step;
+    if (i >= H) continue;
+    float g[V], o[V];
+    load_f32<T, V>(w + i, g);
+    if (b) load_f32<T, V>(b + i, o);
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[n][j] = v[n][j] * r * (g[j] + (float)w_off) + (b ? o[j] : 0.f);
+  }
+}
+
+// entry (ids): x = table[id];  else x += mult * norm1(y + y_bias).  out = norm2(x), or x where w2 is null
+template <typename T, int V, int NV, bool LN>
+__global__ void __launch_bounds__(1024)
+norm_add_kernel(const int* __restrict__ ids, int vocab, const T* __restrict__ y, int64_t y_stride, const float* __restrict__ y_bias,
+                const T* __restrict__ w1, const T* __restrict__ b1, float mult, float* __restrict__ x, const T* __restrict__ w2,
+                const T* __restrict__ b2, int w_off, T* __restrict__ out, int H, float eps) {
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  const int step = blockDim.x * V;
+  const T* src = y + (ids ? (int64_t)min(max(ids[row], 0), vocab - 1) * H : row * y_stride);
+  float v[NV][V];
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * step;
+    if (i >= H) continue;
+    load_f32<T, V>(src + i, v[n]);
+    if (y_bias) {
+      float b[V];
+      load_f32<float, V>(y_bias + i, b);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[n][j] += b[j];
+    }
+  }
+  if (!ids) {
+    normalise<T, V, NV, LN>(v, w1, b1, w_off, H, eps, red);
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = threadIdx.x * V + n * step;
+      if (i >= H) continue;
+      float xv[V];
+      load_f32<float, V>(x + row * H + i, xv);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[n][j] = xv[j] + mult * v[n][j];
+    }
+  }
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * step;
+    if (i < H) store_f32<float, V>(x + row * H + i, v[n]);
+  }
+  if (!out) return;
+  if (w2) normalise<T, V, NV, LN>(v, w2, b2, w_off, H, eps, red);
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * step;
+    if (i < H) store_f32<T, V>(out + row * H + i, v[n]);
+  }
+}
+
 template <typename T> constexpr int vec_of() { return sizeof(T) == 4 ? 4 : 8; }
 static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
@@ -179,6 +265,34 @@ EXPORT int vb_post_norm_add(const void* y, int64_t y_stride, const int* inv, con
     constexpr int V = vec_of<T>();
     const bool vec = H % V == 0 && y_stride % V == 0 && al16(y) && (!w || al16(w)) && (!x || al16(x)) &&
                      (!w_next || al16(w_next)) && (!out || al16(out));
+    const int items = vec ? H / V : H;
+    const int thr = items >= 1024 ? 1024 : ((items + 31) / 32) * 32;
+    const int nv = (items + thr - 1) / thr;
+    if (vec) { if (nv <= 1) GO(V, 1); else if (nv <= 4) GO(V, 4); else return -1; }
+    else { if (nv <= 1) GO(1, 1); else if (nv <= 16) GO(1, 16); else return -1; }
+  });
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+// One step of an fp32 stream between sublayers: x += mult * norm1(y + y_bias), out = norm2(x) in the model dtype.  At the
+// model's entry ``ids`` pick rows of y = the embedding table [vocab, H] instead and x is written.  ln: layer norms (with b1,
+// b2), else RMS norms with weights w + w_off.  w2 null: out = T(x).
+EXPORT int vb_norm_add(const int* ids, int vocab, const void* y, int64_t y_stride, const float* y_bias, const void* w1,
+                       const void* b1, float mult, float* x, const void* w2, const void* b2, int w_off, int ln, void* out,
+                       int T_, int H, float eps, int dtype, cudaStream_t st) {
+  using namespace stream;
+  if (T_ == 0) return 0;
+  if (!ids && !w1) return -1;
+#define GO(VV, NVV)                                                                                                          \
+  do {                                                                                                                       \
+    if (ln) vb_launch(norm_add_kernel<T, VV, NVV, true>, dim3(T_), dim3(thr), 0, st, ids, vocab, (const T*)y, y_stride, y_bias, (const T*)w1, (const T*)b1, mult, x, (const T*)w2, (const T*)b2, w_off, (T*)out, H, eps); \
+    else vb_launch(norm_add_kernel<T, VV, NVV, false>, dim3(T_), dim3(thr), 0, st, ids, vocab, (const T*)y, y_stride, y_bias, (const T*)w1, (const T*)b1, mult, x, (const T*)w2, (const T*)b2, w_off, (T*)out, H, eps); \
+  } while (0)
+  DISPATCH_DTYPE(dtype, T, {
+    constexpr int V = vec_of<T>();
+    auto ok = [](const void* p) { return !p || al16(p); };
+    const bool vec = H % V == 0 && y_stride % V == 0 && ok(y) && ok(y_bias) && ok(w1) && ok(b1) && ok(x) && ok(w2) && ok(b2) && ok(out);
     const int items = vec ? H / V : H;
     const int thr = items >= 1024 ? 1024 : ((items + 31) / 32) * 32;
     const int nv = (items + thr - 1) / thr;

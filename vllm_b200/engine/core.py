@@ -71,11 +71,14 @@ class EngineCore:
         max_len = self.vllm_config.scheduler_config.max_model_len
         # one config per worker (pipeline stages own different layers); every worker must end up with the same
         # number of blocks because block ids are global to the scheduler
-        cfgs = [get_kv_cache_config(sp, mm, max_len, cc.num_gpu_blocks_override, auto_fit_max_model_len=False)[0]
-                for sp in specs]
+        seqs = self.vllm_config.scheduler_config.max_num_seqs
+        cfgs = [get_kv_cache_config(sp, mm, max_len, cc.num_gpu_blocks_override, False, seqs)[0] for sp in specs]
         nblk = min(c.num_blocks for c in cfgs)
         if any(c.num_blocks != nblk for c in cfgs):
-            cfgs = [get_kv_cache_config(sp, mm, max_len, nblk, auto_fit_max_model_len=False)[0] for sp in specs]
+            cfgs = [get_kv_cache_config(sp, mm, max_len, nblk, False, seqs)[0] for sp in specs]
+        slots = [c.num_state_slots for c in cfgs if c.num_state_slots]
+        for c in cfgs:           # slot ids are global to the scheduler as well
+            c.num_state_slots = min(slots) if c.num_state_slots else 0
         cfg = cfgs[0]
         cc.num_gpu_blocks = cfg.num_blocks
         ex.initialize_from_config(cfgs if len(cfgs) > 1 else cfg)

@@ -38,7 +38,7 @@ class StepReplay:
     def __init__(self, model: str, dtype: str = "bfloat16", max_tokens: int = 2048, max_requests: int = MAX_LIVE_REQUESTS,
                  **engine_args: Any) -> None:
         kw = dict(dtype=dtype, skip_tokenizer_init=True, enforce_eager=True, enable_prefix_caching=False, max_num_seqs=max_requests,
-                  max_num_batched_tokens=max_tokens, gpu_memory_utilization=0.5, kv_cache_memory_bytes=1 << 30,
+                  max_num_batched_tokens=max_tokens, gpu_memory_utilization=0.5, kv_cache_memory_bytes=16 << 30,
                   distributed_executor_backend="uni")
         args = EngineArgs(model=model, **{**kw, **engine_args})
         cfg = args.create_engine_config()

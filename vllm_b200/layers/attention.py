@@ -35,8 +35,15 @@ class Attention(nn.Module):
                  sliding_window: Optional[int] = None, logits_soft_cap: float = 0.0, prefix: str = "",
                  causal: bool = True, rope: Optional[nn.Module] = None,
                  alibi_slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
-                 chunk_size: int = 0) -> None:
+                 chunk_size: int = 0, v_head_size: Optional[int] = None, fused_prologue: bool = False,
+                 out_scale: float = 1.0) -> None:
+        """``v_head_size``: value width where it is not ``head_size`` (cache rows are as wide as the wider one).
+        ``fused_prologue``: q/k norms, rotation and cache write are one kernel for whatever shape and dtype, 32-bit between norm
+        and rotation.  ``out_scale``: factor of the output, applied in 32-bit."""
         super().__init__()
+        self.v_head_size = v_head_size or head_size
+        self.cache_head_size = max(head_size, self.v_head_size)
+        self.fused_prologue, self.out_scale = fused_prologue, float(out_scale)
         self.chunk_size = int(chunk_size or 0)        # chunked-local attention (Llama-4 rope layers)
         # ALiBi slopes / attention-sink logits of THIS rank's heads (buffers follow the module's device)
         self.register_buffer("alibi_slopes", None if alibi_slopes is None else alibi_slopes.float(), persistent=False)
@@ -58,10 +65,10 @@ class Attention(nn.Module):
             if self.sliding_window or self.alibi_slopes is not None or self.sinks is not None or self.chunk_size:
                 raise NotImplementedError("decode context parallelism covers full causal attention (no sliding window / "
                                           "ALiBi / sinks / chunked-local layers)")
-            return FullAttentionSpec(block_size=block_size * d, num_kv_heads=self.num_kv_heads, head_size=self.head_size,
+            return FullAttentionSpec(block_size=block_size * d, num_kv_heads=self.num_kv_heads, head_size=self.cache_head_size,
                                      dtype_size=dtype_size, dcp=d)
         cls = SlidingWindowSpec if self.sliding_window else FullAttentionSpec
-        return cls(block_size=block_size, num_kv_heads=self.num_kv_heads, head_size=self.head_size,
+        return cls(block_size=block_size, num_kv_heads=self.num_kv_heads, head_size=self.cache_head_size,
                    dtype_size=dtype_size, sliding_window=self.sliding_window)
 
     def _forward_dcp(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions, md, kv_cache) -> torch.Tensor:
@@ -118,8 +125,9 @@ class Attention(nn.Module):
         return out.to(q.dtype).reshape(T, h * D)
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
-                positions: Optional[torch.Tensor] = None, qk_norm: Optional[tuple] = None) -> torch.Tensor:
-        """q: [T, Hq*D], k/v: [T, Hkv*D] → [T, Hq*D]. If the layer has a ``rope``,
+                positions: Optional[torch.Tensor] = None, qk_norm: Optional[tuple] = None,
+                out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """q: [T, Hq*D], k: [T, Hkv*D], v: [T, Hkv*DV] → [T, Hq*DV] (``out``: a buffer for it, any token stride). If the layer has a ``rope``,
         rotation and the KV write happen in one fused kernel.  ``qk_norm`` = (q_norm, k_norm) per-head RMSNorm modules
         (Qwen3 / Gemma-3 / OLMo-2 style): on CUDA they are fused with the rotation and the cache insert into ONE launch
         (csrc/qknorm_rope.cu), otherwise applied here before the rotation."""
@@ -133,6 +141,8 @@ class Attention(nn.Module):
                                "cover this worker's layers)")
         if md is None or kv_cache is None:
             # memory-profiling run: no cache; keep the data flow (and the GEMM shapes) intact
+            if self.v_head_size != D or out is not None:
+                return (q.new_empty(T, self.num_heads * self.v_head_size) if out is None else out).zero_()
             if self.rope is not None and positions is not None:
                 q, k = self.rope(positions, q, k)
             return q.clone() if q.shape[-1] == self.num_heads * D else q
@@ -148,15 +158,16 @@ class Attention(nn.Module):
         if qk_norm is not None:
             qn, kn = qk_norm
             fused = (md is not None and kv_cache is not None and q.is_cuda and pcp is None and mpos is None
-                     and self.rope is not None and positions is not None and q.dtype in (torch.bfloat16, torch.float16)
+                     and self.rope is not None and positions is not None
                      and kv_cache.dtype == q.dtype and getattr(qn, "gemma", False) == getattr(kn, "gemma", False)
                      and qn.eps == kn.eps and not envs.VLLM_B200_FORCE_REF_OPS
-                     and ops.cuda_ops().qknorm_rope_ok(D, self.rope.cos_sin_cache.shape[-1], self.rope.is_neox_style))
+                     and (self.fused_prologue or (q.dtype in (torch.bfloat16, torch.float16) and ops.cuda_ops().qknorm_rope_ok(
+                         D, self.rope.cos_sin_cache.shape[-1], self.rope.is_neox_style))))
             if fused:
                 ops.cuda_ops().fused_qk_norm_rope(positions, q, k, qn.weight, kn.weight, self.rope.cos_sin_cache, D, qn.eps,
                                                   self.rope.is_neox_style, v=v, kv_cache=kv_cache,
                                                   slot_mapping=md.slot_mapping, gemma=getattr(qn, "gemma", False),
-                                                  vt=md.kv_vt)
+                                                  vt=md.kv_vt, v_head_dim=self.v_head_size, keep32=self.fused_prologue)
                 positions = None            # rotation and cache insert are done: skip them below
                 skip_cache_write = True
             else:
@@ -167,6 +178,14 @@ class Attention(nn.Module):
             skip_cache_write = False
         if skip_cache_write:
             pass
+        elif self.v_head_size != D:
+            if pcp is not None or mpos is not None:
+                raise NotImplementedError("unequal key and value widths with prefill context parallelism or M-RoPE")
+            if self.rope is not None and positions is not None:
+                q, k = self.rope(positions, q, k)
+            wide = [torch.nn.functional.pad(x.reshape(T, self.num_kv_heads, -1), (0, self.cache_head_size - w))
+                    for x, w in ((k, D), (v, self.v_head_size))]
+            ops.reshape_and_cache(*wide, kv_cache, md.slot_mapping, vt=md.kv_vt)
         elif mpos is not None:
             # multimodal rotary ids differ per channel section for image tokens: rotate un-fused, then the ordinary
             # cache write (text-only steps take the fused path below with 1-D positions = index + per-request delta)
@@ -190,7 +209,7 @@ class Attention(nn.Module):
             ops.reshape_and_cache(k.view(T, self.num_kv_heads, D), v.view(T, self.num_kv_heads, D),
                                   kv_cache, md.slot_mapping, vt=md.kv_vt)
         if (md.cascade is not None and self.causal and not self.sliding_window and self.alibi_slopes is None
-                and self.sinks is None and not self.chunk_size):
+                and self.sinks is None and not self.chunk_size and self.v_head_size == D and out is None):
             # shared prefix: its K/V are read once for the whole batch (all queries sit after it → no causal mask),
             # the per-request remainders are attended separately, the two partial softmaxes are merged by their LSE
             md_p, md_s = md.cascade
@@ -200,10 +219,12 @@ class Attention(nn.Module):
             out, _ = ops.merge_attn_states(o1, l1, o2, l2)
             Attention.cascade_calls += 1
             return out.view(T, self.num_heads * D)
-        out = ops.paged_attention(q.view(T, self.num_heads, D), kv_cache, md, self.scale,
-                                  self.sliding_window, self.logits_soft_cap, self.causal,
-                                  alibi_slopes=self.alibi_slopes, sinks=self.sinks, chunk_size=self.chunk_size)
-        return out.view(T, self.num_heads * D)
+        buf = None if out is None else out.view(T, self.num_heads, self.v_head_size)
+        o = ops.paged_attention(q.view(T, self.num_heads, D), kv_cache, md, self.scale,
+                                self.sliding_window, self.logits_soft_cap, self.causal, out=buf,
+                                alibi_slopes=self.alibi_slopes, sinks=self.sinks, chunk_size=self.chunk_size,
+                                v_head_size=self.v_head_size, out_scale=self.out_scale)
+        return o.view(T, self.num_heads * self.v_head_size) if out is None else out
 
 
 class MLAAttentionCore(nn.Module):

@@ -85,18 +85,55 @@ class ReplicatedLinear(LinearBase):
 
 
 class MergedReplicatedLinear(ReplicatedLinear):
-    """Several replicated matrices over the same input, stacked along the output dim (one GEMM)."""
+    """Several replicated matrices over the same input, stacked along the output dim (one GEMM).  ``align``: every part starts
+    at a multiple of this many outputs (zero rows between), so that its columns of the result can be read in vectors."""
 
-    def __init__(self, input_size, output_sizes: list[int], bias=False, dtype=None, quant_config=None, prefix="") -> None:
+    def __init__(self, input_size, output_sizes: list[int], bias=False, dtype=None, quant_config=None, prefix="",
+                 align: int = 1) -> None:
         self.output_sizes = list(output_sizes)
-        super().__init__(input_size, sum(output_sizes), bias, dtype, quant_config, prefix)
+        self.offsets, total = [], 0
+        for n in self.output_sizes:
+            self.offsets.append(total)
+            total += -(-n // align) * align
+        super().__init__(input_size, total, bias, dtype, quant_config, prefix)
+        if total != sum(self.output_sizes):
+            self.weight.data.zero_()
+
+    def parts(self, y: torch.Tensor) -> list[torch.Tensor]:
+        return [y.narrow(-1, o, n) for o, n in zip(self.offsets, self.output_sizes)]
 
     def weight_loader(self, param: nn.Parameter, w: torch.Tensor, shard_id=None) -> None:
         if shard_id is None:
             return super().weight_loader(param, w)
         if shard_id >= len(self.output_sizes):
             raise ValueError(f"{self.prefix} has no part {shard_id}")
-        dst = param.data.narrow(0, sum(self.output_sizes[:shard_id]), self.output_sizes[shard_id])
+        dst = param.data.narrow(0, self.offsets[shard_id], self.output_sizes[shard_id])
+        assert dst.shape == w.shape, (self.prefix, shard_id, dst.shape, w.shape)
+        dst.copy_(w)
+
+
+class SummedReplicatedLinear(ReplicatedLinear):
+    """sum_i W_i x_i over inputs of their own as one GEMM: the inputs lie side by side in ``buffer``, part i at a multiple of
+    ``align`` elements."""
+
+    def __init__(self, input_sizes: list[int], output_size, dtype=None, prefix="", align: int = 8) -> None:
+        self.input_sizes = list(input_sizes)
+        self.offsets, total = [], 0
+        for n in self.input_sizes:
+            self.offsets.append(total)
+            total += -(-n // align) * align
+        super().__init__(total, output_size, False, dtype, None, prefix)
+        self.padded = total != sum(self.input_sizes)
+        if self.padded:
+            self.weight.data.zero_()
+
+    def buffer(self, like: torch.Tensor) -> tuple[torch.Tensor, list[torch.Tensor]]:
+        """(a row of inputs per row of ``like``, its parts)."""
+        x = (like.new_zeros if self.padded else like.new_empty)((like.shape[0], self.input_size))
+        return x, [x.narrow(1, o, n) for o, n in zip(self.offsets, self.input_sizes)]
+
+    def weight_loader(self, param: nn.Parameter, w: torch.Tensor, shard_id=None) -> None:
+        dst = param.data.narrow(1, self.offsets[shard_id], self.input_sizes[shard_id])
         assert dst.shape == w.shape, (self.prefix, shard_id, dst.shape, w.shape)
         dst.copy_(w)
 

@@ -3,8 +3,8 @@
 Behavioural reference: vllm/model_executor/layers/mamba/mamba_mixer.py (conv state + SSM state kept per request
 in the KV-cache pool through ``MambaSpec``; causal-conv1d + selective-scan ops).
 
-State layout: one pool block per request holds ``[conv_state (d_inner x (k-1)) | ssm_state (d_inner x d_state)]``
-in fp32.  Decode batches (one token per request) are fully vectorised over the batch — gather states by block id,
+State layout: one state slot per request holds ``[conv_state (d_inner x (k-1)) | ssm_state (d_inner x d_state)]``
+in fp32.  Decode batches (one token per request) are fully vectorised over the batch — gather states by slot id,
 one fused update, scatter back — with no host synchronisation, so they replay inside CUDA graphs.  Prefill /
 mixed batches walk each request's segment (chunked prefill resumes from the cached state).
 """
@@ -17,6 +17,7 @@ import torch
 import torch.nn as nn
 import torch.nn.functional as F
 
+from vllm_b200 import ops
 from vllm_b200.core.kv_cache_manager import KVCacheSpec, MambaSpec
 from vllm_b200.forward_context import get_forward_context
 from vllm_b200.layers import attention as _attn
@@ -155,14 +156,16 @@ class Mamba2Mixer(nn.Module):
     projection.  Reference: vllm/model_executor/layers/mamba/mamba_mixer2.py (+ ops/ssd_*.py, causal_conv1d.py,
     mamba_ssm.py ``selective_state_update``).
 
-    Cache block per request (fp32): ``[conv_state (conv_dim x (k-1)) | ssm_state (heads x head_dim x d_state)]``.
-    Decode batches are one vectorised state update (graph-capturable); prefill / mixed batches run the chunked SSD
-    scan per request and resume from the cached state (chunked prefill, prefix resume)."""
+    State slot per request (fp32): ``[conv_state (conv_dim x (k-1)) | ssm_state]``.  On CUDA three varlen kernels (convolution,
+    scan, gated norm) serve prompts, portions and decode steps of every size; the plain path keeps the state as
+    [heads, head_dim, d_state] and runs the chunked SSD scan per request.
+
+    ``own_projections`` False: a block that merges this mixer's projections with others' calls ``mix`` between them."""
 
     def __init__(self, hidden: int, num_heads: int, head_dim: int, d_state: int, d_conv: int, n_groups: int,
                  use_bias: bool, use_conv_bias: bool, chunk_size: int, eps: float, dtype, prefix: str,
                  time_step_limit: tuple[float, float] = (0.0, float("inf")), norm_before_gate: bool = False,
-                 norm_groups: int = 1) -> None:
+                 norm_groups: int = 1, own_projections: bool = True) -> None:
         super().__init__()
         self.nh, self.hd, self.N, self.k, self.G = num_heads, head_dim, d_state, d_conv, n_groups
         self.norm_groups = norm_groups        # gated RMSNorm statistics per group of channels (Nemotron-H, Zamba-2, Falcon-H1)
@@ -172,8 +175,10 @@ class Mamba2Mixer(nn.Module):
         self.conv_dim = self.d_inner + 2 * n_groups * d_state
         self.chunk = chunk_size
         self.dt_min, self.dt_max = time_step_limit
-        self.in_proj = ReplicatedLinear(hidden, 2 * self.d_inner + 2 * n_groups * d_state + num_heads, use_bias, dtype,
-                                        None, f"{prefix}.in_proj")
+        if own_projections:
+            self.in_proj = ReplicatedLinear(hidden, 2 * self.d_inner + 2 * n_groups * d_state + num_heads, use_bias, dtype,
+                                            None, f"{prefix}.in_proj")
+            self.out_proj = ReplicatedLinear(self.d_inner, hidden, use_bias, dtype, None, f"{prefix}.out_proj")
         self.conv_weight = nn.Parameter(torch.empty(self.conv_dim, d_conv, dtype=dtype), requires_grad=False)
         self.conv_bias = nn.Parameter(torch.zeros(self.conv_dim, dtype=dtype), requires_grad=False) if use_conv_bias else None
         self.dt_bias = nn.Parameter(torch.ones(num_heads, dtype=torch.float32), requires_grad=False)
@@ -181,9 +186,10 @@ class Mamba2Mixer(nn.Module):
         self.D = nn.Parameter(torch.ones(num_heads, dtype=torch.float32), requires_grad=False)
         self.norm_weight = nn.Parameter(torch.ones(self.d_inner, dtype=dtype), requires_grad=False)
         self.norm_eps = eps
-        self.out_proj = ReplicatedLinear(self.d_inner, hidden, use_bias, dtype, None, f"{prefix}.out_proj")
         self.layer_name = prefix
-        self.state_elems = self.conv_dim * (d_conv - 1) + num_heads * head_dim * d_state
+        self.conv_elems = -(-self.conv_dim * (d_conv - 1) // 4) * 4           # the state behind it starts at 16 bytes
+        self.ssm_elems = num_heads * head_dim * d_state
+        self.state_elems = self.conv_elems + max(num_heads * ops.scan_state_elems(d_state, head_dim), self.ssm_elems)
         self.num_kv_heads, self.head_size, self.sliding_window = 1, 0, None
         assert prefix not in _attn._LAYER_REGISTRY, f"duplicate layer name {prefix}"
         _attn._LAYER_REGISTRY[prefix] = self
@@ -192,25 +198,25 @@ class Mamba2Mixer(nn.Module):
         return MambaSpec(block_size=block_size, state_bytes=self.state_elems * 4)
 
     def _split_state(self, st: torch.Tensor):
-        nconv = self.conv_dim * (self.k - 1)
+        nconv, o = self.conv_dim * (self.k - 1), self.conv_elems
         return (st[..., :nconv].reshape(*st.shape[:-1], self.conv_dim, self.k - 1),
-                st[..., nconv:].reshape(*st.shape[:-1], self.nh, self.hd, self.N))
+                st[..., o:o + self.ssm_elems].reshape(*st.shape[:-1], self.nh, self.hd, self.N))
+
+    def _store_state(self, cache: torch.Tensor, slots, conv_state: torch.Tensor, h: torch.Tensor) -> None:
+        nconv, o = self.conv_dim * (self.k - 1), self.conv_elems
+        cache[slots, :nconv] = conv_state.reshape(*conv_state.shape[:-2], nconv)
+        cache[slots, o:o + self.ssm_elems] = h.reshape(*h.shape[:-3], self.ssm_elems)
 
     def _dt(self, dt: torch.Tensor) -> torch.Tensor:
         dt = F.softplus(dt.float() + self.dt_bias)
         return dt.clamp(self.dt_min, self.dt_max) if (self.dt_min > 0 or self.dt_max != float("inf")) else dt
 
-    def _gated_norm(self, y: torch.Tensor, z: torch.Tensor) -> torch.Tensor:
+    def _gated_norm(self, y: torch.Tensor, z: torch.Tensor, out=None, scale: float = 1.0) -> torch.Tensor:
+        """y fp32 → z's dtype."""
         if self.norm_before_gate is None:
-            return y.float() * F.silu(z.float())
-        y = y.float() if self.norm_before_gate else y.float() * F.silu(z.float())
-        if self.norm_groups > 1:
-            g = y.view(*y.shape[:-1], self.norm_groups, -1)
-            y = (g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + self.norm_eps)).view(y.shape)
-        else:
-            y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + self.norm_eps)
-        y = self.norm_weight.float() * y
-        return y * F.silu(z.float()) if self.norm_before_gate else y
+            y = (y * F.silu(z.float()) * scale)
+            return y.to(z.dtype) if out is None else out.copy_(y)
+        return ops.gated_norm(y, z, self.norm_weight, self.norm_groups, self.norm_eps, not self.norm_before_gate, out, scale)
 
     def _segment(self, xbc: torch.Tensor, dt: torch.Tensor, conv_state: torch.Tensor, h: torch.Tensor):
         """ONE request: xbc [q, conv_dim], dt [q, nh] raw → (y [q, d_inner] fp32, conv_state, h)."""
@@ -225,32 +231,39 @@ class Mamba2Mixer(nn.Module):
         y, h = ref.ssd_chunk_scan(x.view(q, self.nh, self.hd), self._dt(dt), -torch.exp(self.A_log),
                                   B.view(q, self.G, self.N), C.view(q, self.G, self.N), self.chunk, h)
         y = y + self.D[None, :, None] * x.view(q, self.nh, self.hd)
-        return y.reshape(q, self.d_inner), xin[-(self.k - 1):].t().float(), h
+        return y.reshape(q, self.d_inner), xin[q:].t().float(), h
 
     def forward(self, hidden: torch.Tensor) -> torch.Tensor:
+        z, xbc, dt = self.in_proj(hidden).split([self.d_inner, self.conv_dim, self.nh], dim=-1)
+        return self.out_proj(self.mix(z, xbc, dt))
+
+    def mix(self, z: torch.Tensor, xbc: torch.Tensor, dt: torch.Tensor, out: Optional[torch.Tensor] = None, scale: float = 1.0
+            ) -> torch.Tensor:
+        """Everything between the projections: z [T, d_inner], xbc [T, conv_dim], dt [T, heads] (row strides free) → [T, d_inner]
+        times ``scale`` in the model dtype (into ``out`` where given)."""
         ctx = get_forward_context()
         md = ctx.metadata_for(self.layer_name)
         cache = ctx.kv_caches.get(self.layer_name)
-        z, xbc, dt = self.in_proj(hidden).split([self.d_inner, self.conv_dim, self.nh], dim=-1)
-        T = hidden.shape[0]
-        dev = hidden.device
-        if md is None or cache is None:                      # profiling run: one stateless sequence
-            y, _, _ = self._segment(xbc, dt, torch.zeros(self.conv_dim, self.k - 1, device=dev),
-                                    torch.zeros(self.nh, self.hd, self.N, device=dev))
-            return self.out_proj(self._gated_norm(y, z).to(hidden.dtype))
-        if _cuda_ssm(xbc) and self.N % 32 == 0 and self.N <= 256 and 2 <= self.k <= 4:
-            from vllm_b200.ops import cuda_ops
-            cu = cuda_ops()
+        T, dev = xbc.shape[0], xbc.device
+        if md is None or cache is None:                      # profiling run: no state
+            y = torch.zeros(T, self.d_inner, device=dev) if xbc.is_cuda else self._segment(
+                xbc, dt, torch.zeros(self.conv_dim, self.k - 1, device=dev), torch.zeros(self.nh, self.hd, self.N, device=dev))[0]
+            return self._gated_norm(y, z, out, scale)
+        if ops._use_cuda(xbc):
+            cu = ops.cuda_ops()
             xa = cu.causal_conv1d(xbc, self.conv_weight, self.conv_bias, cache, md)
-            y = cu.ssd_scan(xa, dt.float(), self.dt_bias, self.A_log, self.D, cache, self.conv_dim * (self.k - 1), md,
+            y = cu.ssd_scan(xa, dt, self.dt_bias, self.A_log, self.D, cache, self.conv_elems, md,
                             self.nh, self.hd, self.G, self.N, self.dt_min, self.dt_max)
-            return self.out_proj(self._gated_norm(y, z).to(hidden.dtype))
+            return self._gated_norm(y, z, out, scale)
         cache = cache.view(cache.shape[0], -1).view(torch.float32) if cache.dtype != torch.float32 else cache
-        out = torch.zeros(T, self.d_inner, dtype=torch.float32, device=dev)
+        y = torch.zeros(T, self.d_inner, dtype=torch.float32, device=dev)
         if md.decode_only:
             Bn = md.num_reqs
             slots = md.block_table[:Bn, 0].long()
             conv_state, h = self._split_state(cache[slots])
+            fresh = (md.seq_lens[:Bn] <= 1).to(dev)            # a one-token prompt starts from nothing
+            conv_state = conv_state.masked_fill(fresh[:, None, None], 0.0)
+            h = h.masked_fill(fresh[:, None, None, None], 0.0)
             xin = torch.cat([conv_state, xbc[:Bn].float()[:, :, None]], dim=-1)            # [B, conv_dim, k]
             conv = (xin * self.conv_weight.float()[None]).sum(-1)
             if self.conv_bias is not None:
@@ -264,9 +277,9 @@ class Mamba2Mixer(nn.Module):
             dtv = self._dt(dt[:Bn])                                                         # [B, nh]
             dA = torch.exp(dtv * (-torch.exp(self.A_log))[None])
             h = h * dA[:, :, None, None] + (dtv[:, :, None] * x)[..., None] * Bm[:, :, None, :]
-            y = (h * Cm[:, :, None, :]).sum(-1) + self.D[None, :, None] * x
-            cache[slots] = torch.cat([xin[:, :, 1:].reshape(Bn, -1), h.reshape(Bn, -1)], dim=-1)
-            out[:Bn] = y.reshape(Bn, self.d_inner)
+            o = (h * Cm[:, :, None, :]).sum(-1) + self.D[None, :, None] * x
+            self._store_state(cache, slots, xin[:, :, 1:], h)
+            y[:Bn] = o.reshape(Bn, self.d_inner)
         else:
             qsl = (md.query_start_loc_cpu if md.query_start_loc_cpu is not None else md.query_start_loc.cpu()).tolist()
             sls = (md.seq_lens_cpu if md.seq_lens_cpu is not None else md.seq_lens.cpu()).tolist()
@@ -281,7 +294,6 @@ class Mamba2Mixer(nn.Module):
                 else:
                     conv_state = torch.zeros(self.conv_dim, self.k - 1, dtype=torch.float32, device=dev)
                     h = torch.zeros(self.nh, self.hd, self.N, dtype=torch.float32, device=dev)
-                y, conv_state, h = self._segment(xbc[s:e], dt[s:e], conv_state, h)
-                cache[slots[i]] = torch.cat([conv_state.reshape(-1), h.reshape(-1)])
-                out[s:e] = y
-        return self.out_proj(self._gated_norm(out, z).to(hidden.dtype))
+                y[s:e], conv_state, h = self._segment(xbc[s:e], dt[s:e], conv_state, h)
+                self._store_state(cache, slots[i], conv_state, h)
+        return self._gated_norm(y, z, out, scale)

@@ -147,7 +147,7 @@ _CACHE: dict[tuple, RotaryEmbedding] = {}
 def get_rope(head_size: int, rotary_dim: int, max_position: int, base: float, is_neox_style: bool = True,
              rope_scaling: Optional[dict[str, Any]] = None) -> RotaryEmbedding:
     key = (head_size, rotary_dim, max_position, base, is_neox_style,
-           repr(sorted(rope_scaling.items())) if rope_scaling else None)
+           repr(sorted(rope_scaling.items())) if rope_scaling else None, str(torch.get_default_device()))
     if key not in _CACHE:
         _CACHE[key] = RotaryEmbedding(head_size, rotary_dim, max_position, base, is_neox_style, rope_scaling)
     return _CACHE[key]

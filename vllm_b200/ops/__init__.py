@@ -95,7 +95,6 @@ def activation(x: torch.Tensor, name: str) -> torch.Tensor:
 
 
 _HALF = (torch.bfloat16, torch.float16)
-_SIMT_ATTN_SHAPES = {(128, 64), (64, 64), (32, 64), (128, 32), (128, 16), (64, 32), (64, 16), (256, 32), (32, 32), (32, 16)}
 
 
 def _rope_ok(q, cos_sin_cache, head_dim) -> bool:
@@ -104,8 +103,15 @@ def _rope_ok(q, cos_sin_cache, head_dim) -> bool:
     return q.dtype in _HALF and head_dim % 8 == 0 and (rot // 2) % 8 == 0 and (head_dim - rot) % 8 == 0
 
 
-def cuda_attention_supported(D: int, BS: int, dtype, vt: bool) -> bool:
-    return dtype in _HALF and (vt or (D, BS) in _SIMT_ATTN_SHAPES)
+def cuda_attention_supported(D: int, DV: int, BS: int, G: int, dtype, kv_dtype, vt: bool = False) -> bool:
+    """Every head shape has a kernel where the cache holds the model dtype (csrc/attention_any.cu takes what the others do
+    not); fp8 caches need a shape of csrc/attention_simt.cu."""
+    return vt or (kv_dtype == dtype and max(D, DV) <= 512) or cuda_ops()._simt_attention_ok(D, DV, BS, G, dtype)
+
+
+def cuda_cache_write_supported(D: int, dtype) -> bool:
+    """Layers without a fused prologue write their keys and values with the vectorised kernel (no host synchronisation)."""
+    return dtype in _HALF and D % 8 == 0
 
 
 def rotary_embedding(positions, q, k, cos_sin_cache, head_dim, is_neox=True):
@@ -142,17 +148,31 @@ def concat_and_cache_mla(kv_c, k_pe, kv_cache, slot_mapping) -> None:
 
 def paged_attention(q, kv_cache, md, scale, sliding_window=None, logits_soft_cap=0.0, causal=True,
                     out: Optional[torch.Tensor] = None, alibi_slopes: Optional[torch.Tensor] = None,
-                    sinks: Optional[torch.Tensor] = None, chunk_size: int = 0, return_lse: bool = False):
-    """``md``: AttentionMetadata (see vllm_b200.forward_context)."""
-    if _use_cuda(q) and cuda_attention_supported(q.shape[-1], kv_cache.shape[3], q.dtype, md.kv_vt):
+                    sinks: Optional[torch.Tensor] = None, chunk_size: int = 0, return_lse: bool = False,
+                    v_head_size: Optional[int] = None, out_scale: float = 1.0):
+    """``md``: AttentionMetadata (see vllm_b200.forward_context).  ``v_head_size``: value width where it is not the keys'.
+    ``out``: [T, Hq, value width] to write into; ``out_scale``: its factor."""
+    if _use_cuda(q) and cuda_attention_supported(q.shape[2], v_head_size or q.shape[2], kv_cache.shape[3],
+                                                 q.shape[1] // kv_cache.shape[2], q.dtype, kv_cache.dtype, md.kv_vt):
         return cuda_ops().paged_attention(q, kv_cache, md, scale, sliding_window, logits_soft_cap, causal, out,
                                           return_lse=return_lse, alibi_slopes=alibi_slopes, sinks=sinks,
-                                          chunk_size=chunk_size)
+                                          chunk_size=chunk_size, v_head_size=v_head_size, out_scale=out_scale)
     sl = md.seq_lens_cpu if md.seq_lens_cpu is not None else md.seq_lens.cpu()
     qsl = md.query_start_loc_cpu if md.query_start_loc_cpu is not None else md.query_start_loc.cpu()
-    return ref.paged_attention(q, kv_cache, md.block_table, sl, qsl, scale,
-                               causal=causal, sliding_window=sliding_window, logits_soft_cap=logits_soft_cap,
-                               alibi_slopes=alibi_slopes, sinks=sinks, chunk_size=chunk_size, return_lse=return_lse)
+    pad = kv_cache.shape[-1] - q.shape[-1]
+    if pad:                                   # cache rows as wide as the wider of key and value
+        q = torch.nn.functional.pad(q, (0, pad))
+    got = ref.paged_attention(q, kv_cache, md.block_table, sl, qsl, scale,
+                              causal=causal, sliding_window=sliding_window, logits_soft_cap=logits_soft_cap,
+                              alibi_slopes=alibi_slopes, sinks=sinks, chunk_size=chunk_size, return_lse=return_lse)
+    o, lse = got if return_lse else (got, None)
+    if v_head_size is not None:
+        o = o[..., :v_head_size]
+    if out_scale != 1.0:
+        o = o * out_scale
+    if out is not None:
+        o = out.copy_(o)
+    return (o, lse) if return_lse else o
 
 
 def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank):
@@ -210,6 +230,39 @@ def post_norm_add(x, y, weight, eps, gemma=False, next_weight=None, next_gemma=F
     if _use_cuda(x):
         return cuda_ops().post_norm_add(x, y, weight, eps, gemma, next_weight, next_gemma)
     return ref.post_norm_add(x, y, weight, eps, gemma, next_weight, next_gemma)
+
+
+def norm_add(x, y, y_bias, norm, mult: float, next_norm, eps: float):
+    """In place on the fp32 stream: x += mult * norm(y + y_bias), layer norms (weight, bias); ``y_bias`` fp32 or None.  Returns the
+    next GEMM's input in y's dtype: next_norm(x), or x where that is None."""
+    if _use_cuda(x):
+        return cuda_ops().norm_add(x, y, y_bias, norm, mult, next_norm, eps)
+    return ref.norm_add(x, y, y_bias, norm, mult, next_norm, eps)
+
+
+def embed_norm(ids, table, next_norm, eps: float):
+    """Entry of an fp32 stream in front of a normed sublayer: (table[ids] fp32, next_norm of it in the table's dtype)."""
+    if _use_cuda(table):
+        x = torch.empty((ids.numel(), table.shape[1]), dtype=torch.float32, device=table.device)
+        return x, cuda_ops().norm_add(x, table, None, None, 1.0, next_norm, eps, ids=ids)
+    x = torch.nn.functional.embedding(ids, table).float()
+    return x, ref.layer_norm(x, *next_norm, eps).to(table.dtype)
+
+
+def scan_state_elems(R: int, C: int) -> int:
+    """Floats that a head's [R, C] state takes in a slot: the lane layout of csrc/linear_attn.cu."""
+    if not 1 <= R <= 512:
+        raise ValueError(f"state of {R} rows: the scan kernels hold up to 512")
+    rows = max(16, 1 << (R - 1).bit_length())
+    return -(-C // 4) * 4 * rows
+
+
+def gated_norm(y, z, weight, groups: int, eps: float, gate_first: bool, out=None, scale: float = 1.0):
+    """RMS norm of y (fp32) over equal parts with the gate silu(z) before or behind it; in z's dtype."""
+    if _use_cuda(y):
+        return cuda_ops().gated_norm(y, z, weight, groups, eps, gate_first, out, scale)
+    o = ref.gated_norm(y, z, weight, groups, eps, gate_first) * scale
+    return o.to(z.dtype) if out is None else out.copy_(o)
 
 
 def merge_attn_states(o1, lse1, o2, lse2):

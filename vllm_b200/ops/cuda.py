@@ -92,9 +92,11 @@ _paged_attention = _sig("vb_paged_attention", _vp, _vp, _vp, _vp, _vp, _vp, _vp,
 _paged_attention_ex = _sig("vb_paged_attention_ex", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
                            _i64, _i64, _i, _i, _i, _f, _f, _f, _i, _i, _i, _vp, _vp, _i, _vp)
 _fmha_tc = _sig("vb_fmha_tc2", _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i64, _i64, _i,
-                _i, _i, _f, _i, _i, _i, _vp)
+                _i, _i, _f, _i, _i, _i, _vp, _f, _i, _vp)
 _fmha_tc_decode = _sig("vb_fmha_tc_decode", _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i64, _i64, _i,
-                       _i, _i, _f, _i, _vp)
+                       _i, _i, _f, _i, _vp, _f, _i, _vp)
+_any_attention = _sig("vb_any_attention", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i64, _i64, _i, _i, _i,
+                      _i, _f, _f, _f, _vp, _vp, _i, _vp)
 _merge_states = _sig("vb_merge_attn_states", _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i, _i, _vp)
 _argmax = _sig("vb_argmax", _vp, _i64, _i, _i, _vp, _i, _vp)
 _fused_sample = _sig("vb_fused_sample", _vp, _i64, _i, _i, _vp, _vp, _vp, _vp, _i, _vp)
@@ -299,44 +301,76 @@ def decode_splits(B: int, Hkv: int, max_seq_len: int, block_size: int) -> int:
     return max(1, min(s, pages))
 
 
+_SIMT_SHAPES = {(128, 64), (64, 64), (32, 64), (128, 32), (128, 16), (64, 32), (64, 16), (256, 32), (32, 32), (32, 16)}
+
+
+def tc_attention_ok(D: int, DV: int, G: int) -> bool:
+    """Head shapes of the tensor-core attention kernels (csrc/attention_tc*.cu)."""
+    return D == 128 and DV == 128 and G <= 128 and 128 % G == 0
+
+
+def _simt_attention_ok(D: int, DV: int, BS: int, G: int, dtype) -> bool:
+    return (dtype in _HALF_DTYPES and D == DV and (D, BS) in _SIMT_SHAPES and G <= 8 and G & (G - 1) == 0)
+
+
 def paged_attention(q, kv_cache, md, scale, sliding_window=None, logits_soft_cap=0.0, causal=True, out=None,
-                    kv_scale: float = 1.0, return_lse: bool = False, alibi_slopes=None, sinks=None, chunk_size: int = 0):
+                    kv_scale: float = 1.0, return_lse: bool = False, alibi_slopes=None, sinks=None, chunk_size: int = 0,
+                    v_head_size: Optional[int] = None, out_scale: float = 1.0):
+    """``out``: [T, Hq, DV] (any token stride) to write into."""
     T, Hq, D = q.shape
     Hkv, BS = kv_cache.shape[2], kv_cache.shape[3]
+    DV = v_head_size or D
+    G = Hq // Hkv
     if out is None:
         # (bucket padding rows are written by no CTA: keep them finite for the row-wise layers that follow)
-        out = (torch.zeros if md.flat else torch.empty)((T, Hq, D), dtype=q.dtype, device=q.device)
+        out = (torch.zeros if md.flat else torch.empty)((T, Hq, DV), dtype=q.dtype, device=q.device)
+    elif md.flat:
+        out.zero_()
+    assert out.stride(-1) == 1 and out.stride(1) == DV and q.stride(-1) == 1 and q.stride(1) == D
     lse = torch.empty((T, Hq), dtype=torch.float32, device=q.device) if return_lse else None
     bt = md.block_table
+    if alibi_slopes is not None:
+        alibi_slopes = alibi_slopes.to(device=q.device, dtype=torch.float32).contiguous()
+    if sinks is not None:
+        sinks = sinks.to(device=q.device, dtype=torch.float32).contiguous()
+    chunk_size = int(chunk_size or 0)
     if md.kv_vt:
         # tcgen05 kernel over the tensor-core cache layout
-        assert D == 128 and BS == 64 and not logits_soft_cap and alibi_slopes is None and sinks is None and not chunk_size, \
-            "tensor-core attention: D=128, 64-token pages, no soft-cap / ALiBi / sinks / chunked-local mask"
+        assert tc_attention_ok(D, DV, G) and BS == 64 and not logits_soft_cap and alibi_slopes is None, \
+            "tensor-core attention: D=128, 64-token pages, no soft-cap / ALiBi"
         # batch-invariant mode: a decode row takes the varlen kernel it would take inside a mixed batch
         decode = md.decode_only and not (batch_invariant() and md.query_start_loc is not None)
         splits = (md.num_splits or decode_splits(md.num_reqs, Hkv, md.max_seq_len, 128)) if decode else 1
+        if chunk_size and chunk_size <= 4096:
+            splits = 1                                   # a chunk is all that a query reads
         ws = _get_attn_ws(md.num_reqs, Hq, D, splits, q.device) if splits > 1 else None
-        G = Hq // Hkv
         if decode and G <= 16 and (G & (G - 1)) == 0 and causal:
             # swap-AB decode kernel: KV tokens on the MMA M axis
             rc = _fmha_tc_decode(q.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0], bt.data_ptr(),
                                  md.seq_lens.data_ptr(), out.data_ptr(), _p(ws.part_out) if ws else None,
                                  _p(ws.part_lse) if ws else None, _p(lse), md.num_reqs, Hq, Hkv, q.stride(0),
-                                 out.stride(0), bt.stride(0), splits, sliding_window or 0, scale, _DT[q.dtype],
-                                 _st())
+                                 out.stride(0), bt.stride(0), splits, sliding_window or 0, scale, chunk_size, _p(sinks),
+                                 out_scale, _DT[q.dtype], _st())
             _check(rc, f"fmha_tc_decode(G={G})", 2 if splits > 1 else 1)
             return (out, lse) if return_lse else out
         rc = _fmha_tc(q.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0], bt.data_ptr(), md.seq_lens.data_ptr(),
                       None if decode else md.query_start_loc.data_ptr(), out.data_ptr(),
                       _p(ws.part_out) if ws else None, _p(ws.part_lse) if ws else None, _p(lse), md.num_reqs, T,
                       md.max_query_len, Hq, Hkv, q.stride(0), out.stride(0), bt.stride(0), splits,
-                      sliding_window or 0, scale, int(causal), int(md.flat and not decode), _DT[q.dtype], _st())
+                      sliding_window or 0, scale, int(causal), int(md.flat and not decode), chunk_size, _p(sinks), out_scale,
+                      _DT[q.dtype], _st())
         _check(rc, f"fmha_tc(G={Hq // Hkv})", 2 if splits > 1 else 1)
         return (out, lse) if return_lse else out
-    if alibi_slopes is not None:
-        alibi_slopes = alibi_slopes.to(device=q.device, dtype=torch.float32).contiguous()
-    if sinks is not None:
-        sinks = sinks.to(device=q.device, dtype=torch.float32).contiguous()
+    if not _simt_attention_ok(D, DV, BS, G, q.dtype) or out_scale != 1.0:
+        assert kv_cache.dtype == q.dtype, "the generic attention kernel reads caches of the model dtype"
+        # one token per request needs no offsets (and the same arithmetic serves prompts and decode steps)
+        rc = _any_attention(q.data_ptr(), kv_cache.data_ptr(), bt.data_ptr(), md.seq_lens.data_ptr(),
+                            None if md.decode_only else md.query_start_loc.data_ptr(), out.data_ptr(), _p(lse), md.num_reqs,
+                            1 if md.decode_only else md.max_query_len, Hq, Hkv, D, DV, kv_cache.shape[4], BS, q.stride(0),
+                            out.stride(0), bt.stride(0), sliding_window or 0, chunk_size, int(causal), scale, logits_soft_cap,
+                            out_scale, _p(alibi_slopes), _p(sinks), _DT[q.dtype], _st())
+        _check(rc, f"any_attention(D={D}, DV={DV}, G={G})")
+        return (out, lse) if return_lse else out
     n_launch = 1
     if md.decode_only and not (batch_invariant() and md.query_start_loc is not None):
         splits = md.num_splits or decode_splits(md.num_reqs, Hkv, md.max_seq_len, BS)
@@ -346,13 +380,13 @@ def paged_attention(q, kv_cache, md, scale, sliding_window=None, logits_soft_cap
                                  out.data_ptr(), _p(ws.part_out) if ws else None, _p(ws.part_lse) if ws else None,
                                  _p(lse), md.num_reqs, 1, Hq, Hkv, D, BS, q.stride(0), out.stride(0), bt.stride(0),
                                  splits, sliding_window or 0, scale, logits_soft_cap, kv_scale, int(causal),
-                                 _kv_fp8(kv_cache), _DT[q.dtype], _p(alibi_slopes), _p(sinks), int(chunk_size or 0), _st())
+                                 _kv_fp8(kv_cache), _DT[q.dtype], _p(alibi_slopes), _p(sinks), chunk_size, _st())
     else:
         rc = _paged_attention_ex(q.data_ptr(), kv_cache.data_ptr(), bt.data_ptr(), md.seq_lens.data_ptr(),
                                  md.query_start_loc.data_ptr(), out.data_ptr(), None, None, _p(lse), md.num_reqs,
                                  md.max_query_len, Hq, Hkv, D, BS, q.stride(0), out.stride(0), bt.stride(0), 1,
                                  sliding_window or 0, scale, logits_soft_cap, kv_scale, int(causal),
-                                 _kv_fp8(kv_cache), _DT[q.dtype], _p(alibi_slopes), _p(sinks), int(chunk_size or 0), _st())
+                                 _kv_fp8(kv_cache), _DT[q.dtype], _p(alibi_slopes), _p(sinks), chunk_size, _st())
     _check(rc, f"paged_attention(D={D}, BS={BS}, G={Hq // Hkv})", n_launch)
     return (out, lse) if return_lse else out
 
@@ -609,6 +643,22 @@ def post_norm_add(x, y, weight, eps: float, gemma: bool, next_weight=None, next_
         out = torch.empty((T, H), dtype=y.dtype, device=y.device)
     _check(_post_norm(y.data_ptr(), y.stride(0), _p(inv), _p(pair_w), k, weight.data_ptr(), int(gemma), x.data_ptr(),
                       _p(next_weight), int(next_gemma), _p(out), T, H, eps, _DT[y.dtype], _st()), "post_norm_add")
+    return x if out is None else out
+
+
+_norm_add = _sig("vb_norm_add", _vp, _i, _vp, _i64, _vp, _vp, _vp, _f, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _f, _i, _vp)
+
+
+def norm_add(x, y, y_bias, norm, mult: float, next_norm, eps: float, ids=None):
+    """In place on the fp32 stream: x += mult * norm(y + y_bias), or (``ids``) x = y[ids] with y the embedding table.  ``norm``,
+    ``next_norm``: (weight, bias) of layer norms.  Returns next_norm(x) — or x — in y's dtype."""
+    T, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and y.stride(-1) == 1 and (ids is None or ids.dtype == torch.int32)
+    w1, b1 = norm if norm is not None else (None, None)
+    w2, b2 = next_norm if next_norm is not None else (None, None)
+    out = torch.empty((T, H), dtype=y.dtype, device=y.device) if w2 is not None or y.dtype != torch.float32 else None
+    _check(_norm_add(_p(ids), y.shape[0], y.data_ptr(), y.stride(0), _p(y_bias), _p(w1), _p(b1), mult, x.data_ptr(), _p(w2), _p(b2),
+                     0, 1, _p(out), T, H, eps, _DT[y.dtype], _st()), "norm_add")
     return x if out is None else out
 
 
@@ -1213,19 +1263,35 @@ def qknorm_rope_ok(head_dim: int, rot: int, is_neox: bool) -> bool:
     return True
 
 
+_qknorm_rope_any = _sig("vb_qknorm_rope_any", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i64, _i64, _i64, _vp,
+                        _vp, _i, _i, _i, _i, _f, _i, _vp)
+
+
 def fused_qk_norm_rope(positions, q, k, q_weight, k_weight, cos_sin_cache, head_dim, eps, is_neox=True, *, v=None,
                        kv_cache=None, slot_mapping=None, gemma: bool = False, k_scale: float = 1.0, v_scale: float = 1.0,
-                       vt: bool = False):
-    """In place: per-head RMSNorm(q), RMSNorm(k) → RoPE → (optionally) K/V insert into the paged cache; one launch."""
+                       vt: bool = False, v_head_dim: Optional[int] = None, keep32: bool = False):
+    """In place: per-head RMSNorm(q), RMSNorm(k) → RoPE → (optionally) K/V insert into the paged cache; one launch.
+    ``keep32``: no rounding to the model dtype between the norm and the rotation."""
     T = q.shape[0]
     Hq, Hkv = q.shape[-1] // head_dim, k.shape[-1] // head_dim
     rot = cos_sin_cache.shape[-1] if cos_sin_cache is not None else 0
     assert q.stride(-1) == 1 and k.stride(-1) == 1
-    flags = 0
+    flags = 4 if keep32 else 0
     BS = 1
+    dv = v_head_dim or head_dim
+    dc = max(head_dim, dv)
     if kv_cache is not None:
-        flags = _kv_fp8(kv_cache) | (2 if vt else 0)
-        BS = kv_cache.shape[3]
+        flags |= _kv_fp8(kv_cache) | (2 if vt else 0)
+        BS, dc = kv_cache.shape[3], kv_cache.shape[4]
+    step = min(head_dim // 32, 16 // q.element_size())          # elements of one vector access of the register kernel
+    vec = all(t is None or (t.stride(0) % step == 0 and t.data_ptr() % (step * t.element_size()) == 0) for t in (q, k, v)) if step else False
+    if not (q.dtype in _HALF_DTYPES and dv == dc == head_dim and vec and qknorm_rope_ok(head_dim, rot, is_neox)):
+        assert not flags & 1, "this head shape needs a cache of the model dtype"
+        _check(_qknorm_rope_any(_p(positions), q.data_ptr(), k.data_ptr(), _p(v), _p(q_weight), _p(k_weight), _p(cos_sin_cache),
+                                rot, T, Hq, Hkv, head_dim, dv, dc, q.stride(0), k.stride(0), v.stride(0) if v is not None else 0,
+                                _p(kv_cache), _p(slot_mapping), BS, int(is_neox), int(gemma), int(vt), eps, _DT[q.dtype], _st()),
+               "qknorm_rope_any")
+        return q, k
     _check(_qknorm_rope(_p(positions), q.data_ptr(), k.data_ptr(), _p(v), _p(q_weight), _p(k_weight), _p(cos_sin_cache),
                         rot, T, Hq, Hkv, head_dim, q.stride(0), k.stride(0), v.stride(0) if v is not None else 0,
                         _p(kv_cache), _p(slot_mapping), BS, int(is_neox), int(gemma), flags, eps, k_scale, v_scale,
@@ -1288,12 +1354,16 @@ def convert_fp8(x: torch.Tensor, scale: float = 1.0, to_fp8: bool = True, out_dt
     return out
 
 
-# ------------------------------------------------------------------ SSM / linear attention (csrc/ssm.cu)
-_conv1d = _sig("vb_causal_conv1d", _vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _i64, _i, _i, _i, _i, _i, _vp)
+# ------------------------------------------------------------------ SSM / linear attention (csrc/ssm.cu, linear_attn.cu)
+_conv1d = _sig("vb_causal_conv1d", _vp, _i64, _vp, _i64, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _i64, _i, _i, _i, _i, _i, _i, _vp)
 _sel_scan = _sig("vb_selective_scan", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _vp, _vp, _vp, _i64, _i, _i, _i,
                  _vp)
-_ssd_scan = _sig("vb_ssd_scan", _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _vp, _vp, _vp, _i64, _i, _i, _i,
-                 _i, _i, _f, _f, _vp)
+_ssd_scan = _sig("vb_ssd_scan", _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _vp, _vp, _vp, _i64, _i, _i, _i, _i,
+                 _i, _i, _f, _f, _i, _vp)
+_gla_scan = _sig("vb_gla_scan", _vp, _vp, _vp, _i64, _i64, _i64, _f, _vp, _vp, _i64, _vp, _vp, _i, _f, _vp, _vp, _i64, _i64, _vp, _vp,
+                 _vp, _i64, _i, _i, _i, _i, _i, _i, _vp)
+_gla_decay = _sig("vb_gla_decay", _vp, _i64, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp)
+_gated_norm = _sig("vb_gated_norm", _vp, _vp, _i64, _vp, _i, _vp, _i64, _i, _i, _i, _i, _f, _f, _i, _vp)
 _gdn_scan = _sig("vb_gdn_scan", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _vp, _vp, _vp, _i64, _i, _i, _i, _i, _vp)
 
 
@@ -1305,14 +1375,15 @@ def _state_view(cache: torch.Tensor) -> torch.Tensor:
 
 def causal_conv1d(x, weight, bias, cache, md, act: bool = True) -> torch.Tensor:
     """Depthwise causal conv over each request's tokens with the (k-1)-window kept at the head of its state row.
-    x [T, C] (bf16/fp16, any row stride) → fp32 [T, C]; the window in the cache is advanced in place."""
+    x [T, C] (any dtype and row stride) → fp32 [T, C]; the window in the cache is advanced in place."""
     T, C = x.shape
     st = _state_view(cache)
-    out = torch.zeros((T, C), dtype=torch.float32, device=x.device)
+    out = torch.empty((T, C), dtype=torch.float32, device=x.device)
     bt = md.block_table
+    assert x.stride(1) == 1 and weight.is_contiguous() and weight.dtype == x.dtype
     _check(_conv1d(x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), weight.data_ptr(), _p(bias), st.data_ptr(),
                    st.stride(0), md.query_start_loc.data_ptr(), md.seq_lens.data_ptr(), bt.data_ptr(), bt.stride(0),
-                   md.num_reqs, C, weight.shape[-1], int(act), _DT[x.dtype], _st()), "causal_conv1d")
+                   md.num_reqs, T, C, weight.shape[-1], int(act), _DT[x.dtype], _st()), "causal_conv1d")
     return out
 
 
@@ -1330,19 +1401,61 @@ def selective_scan(x, dt, B, C, A, D, cache, state_off: int, md) -> torch.Tensor
     return y
 
 
+def _scan_out(T: int, n: int, md, device) -> torch.Tensor:
+    """Output rows of a scan; rows of no request (bucket padding) must be finite."""
+    return (torch.zeros if md.flat else torch.empty)((T, n), dtype=torch.float32, device=device)
+
+
 def ssd_scan(xbc, dt_raw, dt_bias, A_log, D, cache, state_off: int, md, nh: int, hd: int, G: int, N: int,
              dt_min: float = 0.0, dt_max: float = float("inf")) -> torch.Tensor:
-    """Mamba-2: conv output xbc fp32 [T, nh*hd + 2*G*N], raw dt [T, nh] fp32 → y [T, nh*hd] (D skip included)."""
+    """Mamba-2: conv output xbc fp32 [T, nh*hd + 2*G*N], raw dt [T, nh] (any dtype and row stride) → y [T, nh*hd] fp32 (D skip
+    included); the states at ``state_off`` of the request's slot (``ops.scan_state_elems``) advance in place."""
     T = xbc.shape[0]
     st = _state_view(cache)
-    y = torch.zeros((T, nh * hd), dtype=torch.float32, device=xbc.device)
+    y = _scan_out(T, nh * hd, md, xbc.device)
     bt = md.block_table
     dt_max = min(dt_max, 3.0e38)
+    assert xbc.dtype == torch.float32 and xbc.stride(1) == 1 and dt_raw.stride(1) == 1
     _check(_ssd_scan(xbc.data_ptr(), xbc.stride(0), dt_raw.data_ptr(), dt_raw.stride(0), dt_bias.data_ptr(),
                      A_log.data_ptr(), D.data_ptr(), y.data_ptr(), st.data_ptr(), st.stride(0), state_off,
-                     md.query_start_loc.data_ptr(), md.seq_lens.data_ptr(), bt.data_ptr(), bt.stride(0), md.num_reqs, nh, hd,
-                     G, N, dt_min, dt_max, _st()), "ssd_scan")
+                     md.query_start_loc.data_ptr(), md.seq_lens.data_ptr(), bt.data_ptr(), bt.stride(0), md.num_reqs,
+                     md.max_query_len, nh, hd, G, N, dt_min, dt_max, _DT[dt_raw.dtype], _st()), "ssd_scan")
     return y
+
+
+def gla_scan(q, k, v, a1, a2, a2_bias, tau: float, q_scale: float, cache, md, H: int, R: int, C: int, state_off: int = 0):
+    """Gated linear attention: q, k [T, H*R], v [T, H*C] (row strides free), decay sigmoid(a1 @ a2.T + a2_bias)^(1/tau) per key
+    channel → o [T, H*C] fp32; the slot's states advance in place."""
+    T = q.shape[0]
+    st = _state_view(cache)
+    o = _scan_out(T, H * C, md, q.device)
+    bt = md.block_table
+    rank = a1.shape[1]
+    assert all(t.stride(1) == 1 and t.dtype == q.dtype for t in (q, k, v, a1)) and a2.is_contiguous() and a2.dtype == q.dtype
+    alpha = None
+    if not md.decode_only:          # whole prompts: once per token and channel; decode steps evaluate it in the scan
+        alpha = torch.empty((T, H * R), dtype=torch.float32, device=q.device)
+        _check(_gla_decay(a1.data_ptr(), a1.stride(0), a2.data_ptr(), a2_bias.data_ptr(), alpha.data_ptr(), T, H * R, rank,
+                          1.0 / tau, _DT[q.dtype], _st()), "gla_decay")
+    _check(_gla_scan(q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), k.stride(0), v.stride(0), q_scale, _p(alpha),
+                     a1.data_ptr(), a1.stride(0), a2.data_ptr(), a2_bias.data_ptr(), rank, 1.0 / tau, o.data_ptr(), st.data_ptr(),
+                     st.stride(0), state_off, md.query_start_loc.data_ptr(), md.seq_lens.data_ptr(), bt.data_ptr(), bt.stride(0),
+                     md.num_reqs, md.max_query_len, H, R, C, _DT[q.dtype], _st()), "gla_scan")
+    return o
+
+
+def gated_norm(y, z, weight, groups: int, eps: float, gate_first: bool, out=None, scale: float = 1.0):
+    """y fp32 [T, n]: RMS norm over ``groups`` equal parts, silu(z) before (``gate_first``) or behind it, times the weight
+    (repeated along the parts where it is shorter) and ``scale``; in z's dtype."""
+    T, n = y.shape
+    if out is None:
+        out = torch.empty((T, n), dtype=z.dtype, device=z.device)
+    W = n // groups
+    wl = weight.numel()
+    assert y.is_contiguous() and z.stride(1) == 1 and out.stride(1) == 1 and weight.dtype == z.dtype and n % groups == 0 and n % wl == 0
+    _check(_gated_norm(y.data_ptr(), z.data_ptr(), z.stride(0), weight.data_ptr(), wl, out.data_ptr(), out.stride(0), T, groups, W,
+                       int(gate_first), eps, scale, _DT[z.dtype], _st()), "gated_norm")
+    return out
 
 
 def gdn_scan(q, k, v, g, beta, cache, state_off: int, md) -> torch.Tensor:

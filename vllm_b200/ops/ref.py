@@ -328,6 +328,35 @@ def post_norm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: f
     return rms_norm(x, next_weight, eps, next_gemma).to(y.dtype)
 
 
+def norm_add(x: torch.Tensor, y: torch.Tensor, y_bias: Optional[torch.Tensor], norm, mult: float, next_norm, eps: float
+             ) -> torch.Tensor:
+    """In place: x (fp32) += mult * layer_norm(y + y_bias).  Returns x in y's dtype, or its layer norm with ``next_norm``."""
+    yf = y.float() if y_bias is None else y.float() + y_bias
+    x += mult * layer_norm(yf, *norm, eps)
+    return (x if next_norm is None else layer_norm(x, *next_norm, eps)).to(y.dtype)
+
+
+def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, gate_first: bool) -> torch.Tensor:
+    """fp32: rms norm of y over ``groups`` equal parts, times the weight (repeated along the parts), silu(z) first or last."""
+    gate = F.silu(z.float())
+    y = y.float() * gate if gate_first else y.float()
+    g = y.reshape(y.shape[0], groups, -1)
+    y = (g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)).reshape(y.shape)
+    y = y * weight.float().repeat(y.shape[1] // weight.numel())
+    return y if gate_first else y * gate
+
+
+def gated_linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, alpha: torch.Tensor, state: torch.Tensor
+                      ) -> tuple[torch.Tensor, torch.Tensor]:
+    """One sequence.  q, k, alpha [T, H, R], v [T, H, C], state [H, R, C] fp32 → (o [T, H, C], final state):
+    S = diag(alpha) S + k v^T, o = S^T q."""
+    o = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        state = alpha[t][..., None] * state + k[t][..., None] * v[t][:, None]
+        o[t] = (state * q[t][..., None]).sum(1)
+    return o, state
+
+
 # -------------------------------------------------------------- sampling
 def apply_penalties(logits: torch.Tensor, prompt_mask: torch.Tensor, output_counts: torch.Tensor,
                     presence: torch.Tensor, frequency: torch.Tensor, repetition: torch.Tensor) -> torch.Tensor:

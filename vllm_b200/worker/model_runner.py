@@ -319,22 +319,19 @@ class ModelRunner:
                 and not isinstance(s, MLAAttentionSpec) and getattr(s, "head_size", 0) == 128
                 and s.block_size == 64 and getattr(s, "dcp", 1) == 1 and kvd in (torch.bfloat16, torch.float16)
                 and self.dtype in (torch.bfloat16, torch.float16)
-                # features only the generic kernel implements keep the whole group on the standard layout
-                and all(not getattr(attention_layers().get(n), "logits_soft_cap", 0.0)
-                        and getattr(attention_layers().get(n), "alibi_slopes", None) is None
-                        and getattr(attention_layers().get(n), "sinks", None) is None
-                        and not getattr(attention_layers().get(n), "chunk_size", 0) for n in g.layer_names)))
+                # head shapes and features only the generic kernels implement keep the whole group on the standard layout
+                and all(self._tensor_core_layer(attention_layers().get(n)) for n in g.layer_names)))
             for name in g.layer_names:
                 self.layer_to_group[name] = gid
+                ls = g.spec_of(name)
                 if isinstance(s, MambaSpec):
-                    self.kv_caches[name] = torch.zeros((cfg.num_blocks, s.state_bytes // 4), dtype=torch.float32,
+                    self.kv_caches[name] = torch.zeros((cfg.num_state_slots, ls.state_bytes // 4), dtype=torch.float32,
                                                        device=self.device)
                     continue
                 if isinstance(s, MLAAttentionSpec):
-                    ls = g.spec_of(name)
                     shape = (cfg.num_blocks, ls.phys_block_size, ls.head_size)
                 else:
-                    shape = (cfg.num_blocks, 2, s.num_kv_heads, getattr(s, "phys_block_size", s.block_size), s.head_size)
+                    shape = (cfg.num_blocks, 2, ls.num_kv_heads, getattr(ls, "phys_block_size", ls.block_size), ls.head_size)
                 self.kv_caches[name] = torch.zeros(shape, dtype=kvd, device=self.device)
         if self.kv_connector is not None and hasattr(self.kv_connector, "register_kv_caches"):
             self.kv_connector.register_kv_caches(self.kv_caches)
@@ -347,6 +344,15 @@ class ModelRunner:
         n_sets = 3 if self.is_cuda else 1
         self.staging = [_Staging(self.max_num_tokens, R, MB, G, self.is_cuda) for _ in range(n_sets)]
         self._init_gpu_prep()
+
+    @staticmethod
+    def _tensor_core_layer(layer) -> bool:
+        from vllm_b200.ops import cuda_ops
+        if layer is None:
+            return True
+        d, hq, hkv = layer.head_size, getattr(layer, "num_heads", 1), layer.num_kv_heads
+        return (not getattr(layer, "logits_soft_cap", 0.0) and getattr(layer, "alibi_slopes", None) is None
+                and cuda_ops().tc_attention_ok(d, getattr(layer, "v_head_size", d), max(hq // max(hkv, 1), 1)))
 
     def _init_gpu_prep(self) -> None:
         """Persistent device mirrors of the per-request token ids and block tables (reference:
@@ -1416,12 +1422,18 @@ class ModelRunner:
     # -------------------------------------------------------- CUDA graphs
     def _attention_kernels_cover_model(self) -> bool:
         """False when some attention layer would fall back to the plain-PyTorch op (which syncs with the host)."""
-        from vllm_b200.ops import cuda_attention_supported
+        from vllm_b200.ops import cuda_attention_supported, cuda_cache_write_supported
         for name, cache in self.kv_caches.items():
             layer = attention_layers().get(name)
             if layer is None or cache.dim() != 5:
                 continue
-            if not cuda_attention_supported(cache.shape[4], cache.shape[3], self.dtype, self.kv_vt[self.layer_to_group[name]]):
+            vt = self.kv_vt[self.layer_to_group[name]]
+            d = layer.head_size
+            if not cuda_attention_supported(d, getattr(layer, "v_head_size", d), cache.shape[3],
+                                            layer.num_heads // cache.shape[2], self.dtype, cache.dtype, vt):
+                return False
+            # a fused prologue writes any shape; else the vectorised cache write has to cover the layer
+            if not (vt or getattr(layer, "fused_prologue", False) or cuda_cache_write_supported(d, self.dtype)):
                 return False
         return True
 
