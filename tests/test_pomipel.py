@@ -11,13 +11,7 @@ import pytest
 import torch
 
 from tests import pomipel_oracle as po
-
-# largest row error over the spread of the logits
-TOL = {"float32": 2e-4, "bfloat16": 0.12}
-PLACES = [pytest.param(("cpu", "float32"), id="cpu-float32"),
-          pytest.param(("cuda", "bfloat16"), id="cuda-bfloat16", marks=pytest.mark.gpu),
-          pytest.param(("cuda", "float32"), id="cuda-float32", marks=pytest.mark.gpu)]
-
+from tests.replay_utils import PLACES, TOL, Engine, check_greedy, generate, make_llm, portions
 
 @pytest.fixture(autouse=True)
 def _few_threads():
@@ -33,48 +27,11 @@ def place(request):
     return request.param
 
 
-class Engine:
-    """A replay of one model; ``feed`` runs steps and collects logits per request and position."""
-
-    def __init__(self, path, place, max_tokens=1024, **kw):
-        from vllm_b200.engine.replay import StepReplay
-        self.replay = StepReplay(path, place[1], max_tokens, device=place[0], **kw)
-        self.at, self.rows = {}, {}
-
-    def feed(self, *steps):
-        """A step is a list of (request, tokens, finished?)."""
-        for step in steps:
-            got = self.replay.step([dict(id=r, tokens=t, want=list(range(len(t)))) for r, t, *_ in step],
-                                   [r for r, _, *e in step if e and e[0]])
-            n = 0
-            for r, t, *_ in step:
-                self.rows.setdefault(r, []).append(torch.from_numpy(got[n:n + len(t)]))
-                n += len(t)
-        return self
-
-    def logits(self, r):
-        return torch.cat(self.rows.pop(r))
-
-    def __enter__(self):
-        return self
-
-    def __exit__(self, *_):
-        self.replay.shutdown()
-
-
 def _model(tmp_path, cfg, seed=0, place=("cpu", "float32"), plant=None, **kw):
     w = po.make_weights(cfg, seed, steady=place[1] == "bfloat16", **kw)
     if plant:
         po.plant_key(cfg, w, *plant)
     return po.save_model(cfg, w, tmp_path / "model"), w
-
-
-def _portions(toks, sizes):
-    out, i, k = [], 0, 0
-    while i < len(toks):
-        out.append(toks[i:i + sizes[k % len(sizes)]])
-        i, k = i + sizes[k % len(sizes)], k + 1
-    return out
 
 
 # ------------------------------------------------------------------------------------------------ configuration and checkpoint
@@ -221,7 +178,7 @@ def test_prompt_token_by_token_and_portions_agree_with_the_equations(tmp_path, p
         e.feed(*[[("single", [t], i == 149)] for i, t in enumerate(toks)])
         assert po.row_error(e.logits("single"), want) < tol
         for k, sizes in enumerate([(2,), (3, 2, 5), (63, 2, 64, 2), (17, 1, 1, 40), (16, 17, 65), (100, 2, 1)]):
-            parts = _portions(toks, sizes)
+            parts = portions(toks, sizes)
             e.feed(*[[(f"p{k}", p, i == len(parts) - 1)] for i, p in enumerate(parts)])
             assert po.row_error(e.logits(f"p{k}"), want) < tol, sizes
 
@@ -245,7 +202,7 @@ def test_unequal_requests_in_one_batch(tmp_path, place):
     path, w = _model(tmp_path, cfg, 5, place)
     reqs = {"a": po.tokens(cfg, 140, 1), "b": po.tokens(cfg, 9, 2), "c": po.tokens(cfg, 75, 3), "d": po.tokens(cfg, 33, 4)}
     sizes = {"a": (70, 1, 2, 67), "b": (1,), "c": (2, 40, 1), "d": (33,)}
-    parts = {r: _portions(t, sizes[r]) for r, t in reqs.items()}
+    parts = {r: portions(t, sizes[r]) for r, t in reqs.items()}
     starts = {"a": 0, "b": 0, "c": 1, "d": 3}
     steps = []
     for n in range(40):
@@ -336,27 +293,8 @@ def test_long_decoding(tmp_path, place):
 
 
 # ------------------------------------------------------------------------------------------------ generation
-def _llm(path, place, **kw):
-    from vllm_b200 import LLM
-    d = dict(device=place[0], dtype=place[1], max_model_len=320, max_num_seqs=8, max_num_batched_tokens=64, skip_tokenizer_init=True,
-             kv_cache_memory_bytes=16 << 20)
-    return LLM(path, **{**d, **kw})
-
-
-def _generate(llm, prompts, n):
-    from vllm_b200 import SamplingParams
-    outs = llm.generate([{"prompt_token_ids": p} for p in prompts],
-                        SamplingParams(max_tokens=n, temperature=0.0, ignore_eos=True, detokenize=False))
-    return [list(o.outputs[0].token_ids) for o in outs]
-
-
 def _check_greedy(cfg, w, prompts, got, slack):
-    """Every generated token is the best by the equations, within ``slack`` of the logits' spread."""
-    for p, out in zip(prompts, got):
-        lg = po.forward(cfg, w, p + out[:-1])[len(p) - 1:]
-        spread = lg.std()
-        for row, t in zip(lg, out):
-            assert float(row.max() - row[t]) <= slack * float(spread)
+    check_greedy(lambda toks: po.forward(cfg, w, toks), prompts, got, slack)
 
 
 def test_greedy_generation(tmp_path, place):
@@ -364,8 +302,8 @@ def test_greedy_generation(tmp_path, place):
     cfg = po.small()
     path, w = _model(tmp_path, cfg, 10, place)
     prompts = [po.tokens(cfg, n, n) for n in (1, 3, 40, 100, 130, 17)]
-    llm = _llm(path, place)
-    got = _generate(llm, prompts, 12)
+    llm = make_llm(path, place)
+    got = generate(llm, prompts, 12)
     assert all(len(g) == 12 for g in got)
     _check_greedy(cfg, w, prompts, got, 1e-3 if place[1] == "float32" else 0.25)
     if place[1] == "float32":
@@ -373,7 +311,7 @@ def test_greedy_generation(tmp_path, place):
     if place == ("cuda", "bfloat16"):
         runner = llm.llm_engine.engine_core.engine_core.model_executor.worker.runner
         assert runner.graphs and any(getattr(g, "replays", 0) for g in runner.graphs.values())    # decode steps replay graphs
-    assert _generate(llm, prompts[3:5], 4) == [g[:4] for g in got[3:5]]                           # and the prefix cache serves them
+    assert generate(llm, prompts[3:5], 4) == [g[:4] for g in got[3:5]]                           # and the prefix cache serves them
     llm.shutdown()
 
 
@@ -382,12 +320,12 @@ def test_generation_with_preemption(tmp_path):
     cfg = po.small()
     path, w = _model(tmp_path, cfg, 11)
     prompts = [po.tokens(cfg, n, n) for n in (60, 62, 50, 61)]
-    llm = _llm(path, ("cpu", "float32"), num_gpu_blocks_override=7, enable_prefix_caching=False)
+    llm = make_llm(path, ("cpu", "float32"), num_gpu_blocks_override=7, enable_prefix_caching=False)
     sched = llm.llm_engine.engine_core.engine_core.scheduler
     seen = []
     orig = sched._preempt
     sched._preempt = lambda r: (seen.append(r.request_id), orig(r))[1]
-    got = _generate(llm, prompts, 20)
+    got = generate(llm, prompts, 20)
     assert seen
     _check_greedy(cfg, w, prompts, got, 1e-3)
     llm.shutdown()
@@ -400,8 +338,8 @@ def test_parallel_ranks_generate_the_same(tmp_path, kw):
                              (po.mixer(2, 16, 8, 16, 24), po.moe(16, 4, 2, 1, 1)), (po.mixer(2, 32, 16, 8, 24, kv_from=2), po.moe(8, 4, 3, 2, 2))])
     path, w = _model(tmp_path, cfg, 12)
     prompts = [po.tokens(cfg, n, n) for n in (5, 70, 33)]
-    llm = _llm(path, ("cpu", "float32"), distributed_executor_backend="mp", **kw)
-    got = _generate(llm, prompts, 6)
+    llm = make_llm(path, ("cpu", "float32"), distributed_executor_backend="mp", **kw)
+    got = generate(llm, prompts, 6)
     llm.shutdown()
     _check_greedy(cfg, w, prompts, got, 1e-3)
 

@@ -7,6 +7,7 @@ Reference: vllm/config/model.py (``ModelConfig``), transformers_utils/config.py.
 from __future__ import annotations
 
 import copy
+import glob
 import json
 import math
 import os
@@ -793,6 +794,31 @@ def get_preset_hf_config(name: str) -> Optional[dict[str, Any]]:
     return copy.deepcopy(cfg) if cfg is not None else None
 
 
+# positions of a Legelix model where max_model_len is not given (the design itself sets no limit)
+LEGELIX_MAX_LEN = 131072
+# rank of a gated-linear layer's decay where no checkpoint gives it (random weights)
+LEGELIX_DECAY_RANK = 16
+
+
+def safetensors_shapes(path: str) -> dict[str, list[int]]:
+    """Tensor name → shape of every safetensors file in a folder, from the headers alone."""
+    out = {}
+    for fn in sorted(glob.glob(os.path.join(path, "*.safetensors"))):
+        with open(fn, "rb") as f:
+            head = json.loads(f.read(int.from_bytes(f.read(8), "little")))
+        out.update({k: v["shape"] for k, v in head.items() if k != "__metadata__"})
+    return out
+
+
+def _fill_decay_ranks(c: dict, path: str) -> None:
+    """The rank of a gated-linear layer's decay is given by its tensors only."""
+    shapes = safetensors_shapes(path)
+    for i, l in enumerate(c["layers"]):
+        a1 = shapes.get(f"l{i}.mix.a1")
+        if l["type"] == "gla" and a1 is not None:
+            l["mixer"]["rank"] = a1[0]
+
+
 def _flatten_nested_config(c: dict) -> None:
     """Families whose config.json nests or renames the fields the engine sizes the KV cache from."""
     if c.get("architecture") == "Pomipel":
@@ -816,6 +842,28 @@ def _flatten_nested_config(c: dict) -> None:
             j = m.get("kv_from")
             if j is not None and not (0 <= j < i and mixers[j].get("kv_from") is None and mixers[j]["kv_rank"] == m["kv_rank"]):
                 raise ValueError(f"layer {i}: kv_from {j} must name an earlier layer with a latent of its own and the same kv_rank")
+    if c.get("architecture") == "Legelix":
+        layers = c["layers"]
+        left = [l["mixer"]["left"] for l in layers if l["type"] == "parallel"]
+        for i, l in enumerate(layers):
+            m = l["mixer"]
+            if l["type"] == "gla":
+                m.setdefault("rank", LEGELIX_DECAY_RANK)
+            if l["type"] == "parallel":
+                a, r = m["left"], m["right"]
+                if a["heads"] % a["kv_heads"] or r["heads"] % r["groups"] or (r["heads"] * r["vdim"]) % r["norm_groups"]:
+                    raise ValueError(f"layer {i}: heads must divide into kv_heads, groups and norm_groups")
+                if a["rot"]["dims"] % 2 or a["rot"]["dims"] > a["dim"] or a["mask"]["size"] < 1:
+                    raise ValueError(f"layer {i}: rotated dimensions must be even and within the head, and a chunk hold a position")
+        c.setdefault("architectures", ["LegelixForCausalLM"])
+        c.setdefault("model_type", "legelix")
+        c.setdefault("vocab_size", c["vocab"])
+        c.setdefault("hidden_size", c["width"])
+        c.setdefault("num_hidden_layers", len(layers))
+        c.setdefault("max_position_embeddings", LEGELIX_MAX_LEN)
+        c.setdefault("num_attention_heads", max((a["heads"] for a in left), default=1))
+        c.setdefault("num_key_value_heads", max((a["kv_heads"] for a in left), default=1))
+        c.setdefault("head_dim", max((max(a["dim"], a["vdim"]) for a in left), default=128))
     if c.get("model_type") == "dbrx":
         a, f = c.get("attn_config") or {}, c.get("ffn_config") or {}
         c.setdefault("hidden_size", c.get("d_model"))
@@ -895,7 +943,10 @@ class ModelConfig:
         path = os.path.join(self.model, "config.json") if os.path.isdir(self.model) else None
         if path and os.path.exists(path):
             with open(path) as f:
-                return json.load(f)
+                c = json.load(f)
+            if c.get("architecture") == "Legelix":
+                _fill_decay_ranks(c, self.model)
+            return c
         cfg = get_preset_hf_config(self.model)
         if cfg is None:
             raise ValueError(

@@ -113,7 +113,8 @@ def get_model(vllm_config: VllmConfig, device: torch.device,
     t0 = time.perf_counter()
     if device.type == "cuda" and getattr(cls, "kernel_sources", None):
         from vllm_b200.ops import cuda_ops
-        cuda_ops().prebuild(cls.kernel_sources)
+        src = cls.kernel_sources
+        cuda_ops().prebuild(src(mc.hf_config, mc.torch_dtype) if callable(src) else src)
     old = torch.get_default_dtype()
     torch.set_default_dtype(mc.torch_dtype)
     try:

@@ -15,6 +15,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "LLaMAForCausalLM": ("llama", "LlamaForCausalLM"),
     "MistralForCausalLM": ("llama", "MistralForCausalLM"),
     "PomipelForCausalLM": ("pomipel", "PomipelForCausalLM"),
+    "LegelixForCausalLM": ("legelix", "LegelixForCausalLM"),
     "Qwen2ForCausalLM": ("llama", "Qwen2ForCausalLM"),
     "Qwen3ForCausalLM": ("llama", "Qwen3ForCausalLM"),
     "GemmaForCausalLM": ("llama", "GemmaForCausalLM"),
