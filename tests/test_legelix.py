@@ -383,7 +383,7 @@ def test_states_remember_the_first_tokens(tmp_path, place):
     cfg = lo.config(64, 96, [lo.gated(2, 16, 24, 16.0, 40), lo.parallel(lo.left(2, 1, 16, 16, 20), lo.right(2, 16, 12, conv=3), 32)])
     path, w = _model(tmp_path, cfg, 9, lasting=True)
     a = tokens(cfg, 130, 1)
-    b = tokens(cfg, 40, 2) + a[40:]
+    b = [5] * 40 + a[40:]
     wa, wb = lo.forward(cfg, w, a), lo.forward(cfg, w, b)
     assert row_error(wa[-1:], wb[-1:]) > 3 * TOL["bfloat16"]
     with Engine(path, place) as e:
