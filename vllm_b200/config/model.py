@@ -766,7 +766,25 @@ def pomipel_config(*, vocab: int, width: int, layers: int, heads: int, dim: int,
                      embedding=dict(scale=width ** 0.5), norm=dict(eps=1e-6), logit_scale=1.0), **kw)
 
 
+def legelix_config(*, vocab: int, width: int, layers: list[str], heads: int, kv_heads: int, dim: int, chunk: int, ssm_heads: int,
+                   ssm_dim: int, state: int, groups: int, conv: int, gla_heads: int, gla_dim: int, gla_vdim: int, ff: int, **kw) -> dict[str, Any]:
+    """A Legelix config.json whose layers of a kind ("parallel", "gla") are alike."""
+    left = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, mask=dict(size=chunk), scale=dim ** -0.5,
+                rot=dict(base=10000.0, dims=dim, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192)))
+    right = dict(heads=ssm_heads, vdim=ssm_dim, state=state, groups=groups, conv=conv, norm_groups=groups)
+    mixers = dict(parallel=dict(left=left, right=right, left_scale=0.7, right_scale=0.7),
+                  gla=dict(heads=gla_heads, dim=gla_dim, vdim=gla_vdim, tau=16.0))
+    out = [dict(type=t, mixer=copy.deepcopy(mixers[t]), mlp=dict(kind="dense", ff=ff)) for t in layers]
+    return dict(dict(architecture="Legelix", vocab=vocab, width=width, layers=out, norm=dict(eps=1e-6), residual_mult=1.0), **kw)
+
+
 PRESETS.update({
+    "legelix-tiny": legelix_config(vocab=320, width=80, layers=["gla", "parallel", "gla"], heads=4, kv_heads=2, dim=24, chunk=100, ssm_heads=4,
+                                   ssm_dim=16, state=24, groups=2, conv=4, gla_heads=2, gla_dim=20, gla_vdim=28, ff=120,
+                                   max_position_embeddings=1024, torch_dtype="float32"),
+    "legelix-small": legelix_config(vocab=4096, width=1024, layers=["parallel", "gla", "gla", "parallel"], heads=8, kv_heads=2, dim=128,
+                                    chunk=2048, ssm_heads=16, ssm_dim=64, state=64, groups=1, conv=4, gla_heads=4, gla_dim=128, gla_vdim=256,
+                                    ff=2048, max_position_embeddings=8192, torch_dtype="bfloat16"),
     "pomipel-tiny": pomipel_config(vocab=320, width=80, layers=3, heads=2, dim=24, vdim=40, q_rank=56, kv_rank=48, ff=56, experts=6,
                                    top=2, groups=3, keep=2, max_positions=512, share_every=2, torch_dtype="float32"),
     # the layer sizes of "deepseek-small", for side-by-side measurements

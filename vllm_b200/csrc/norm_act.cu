@@ -137,6 +137,19 @@ __global__ void act_and_mul_kernel(T* __restrict__ out, const T* __restrict__ x,
   }
 }
 
+// widths that are no multiple of a vector; IL: gate_i and up_i are neighbours
+template <typename T, int ACT, bool IL>
+__global__ void act_and_mul_scalar_kernel(T* __restrict__ out, const T* __restrict__ x, int d, int64_t total) {
+  pdl_trigger();
+  pdl_wait();
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = i / d;
+    const int c = (int)(i - t * d);
+    const T* row = x + t * 2 * d;
+    out[i] = from_f32<T>(act_fn<ACT>(to_f32(row[IL ? 2 * c : c])) * to_f32(row[IL ? 2 * c + 1 : d + c]));
+  }
+}
+
 // interleaved variant: x[t, 2i] = gate_i, x[t, 2i+1] = up_i (the weight layout of the fused gate_up GEMM epilogue)
 template <typename T>
 __global__ void silu_mul_interleaved_kernel(T* __restrict__ out, const T* __restrict__ x, int d, int64_t total_vec) {
@@ -227,7 +240,16 @@ EXPORT int vb_act_and_mul(void* out, const void* x, int64_t T, int d, int act, i
   if (T == 0) return 0;
   DISPATCH_DTYPE(dtype, TT, {
     constexpr int N = Vec16<TT>::N;
-    if (d % N != 0) return -1;
+    if (d % N != 0) {
+      const int64_t n = T * d;
+      const int nb = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+      switch (act) {
+        case ACT_SILU: vb_launch(act_and_mul_scalar_kernel<TT, ACT_SILU, false>, nb, 256, 0, st, (TT*)out, (const TT*)x, d, n); break;
+        case ACT_GELU: vb_launch(act_and_mul_scalar_kernel<TT, ACT_GELU, false>, nb, 256, 0, st, (TT*)out, (const TT*)x, d, n); break;
+        default: vb_launch(act_and_mul_scalar_kernel<TT, ACT_GELU_TANH, false>, nb, 256, 0, st, (TT*)out, (const TT*)x, d, n); break;
+      }
+      return (int)cudaGetLastError();
+    }
     const int64_t total = T * (d / N);
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     switch (act) {
@@ -241,7 +263,14 @@ EXPORT int vb_act_and_mul(void* out, const void* x, int64_t T, int d, int act, i
 
 EXPORT int vb_silu_mul_interleaved(void* out, const void* x, int64_t T, int d, int dtype, cudaStream_t st) {
   if (T == 0) return 0;
-  if (dtype == DT_F32 || d % 8 != 0) return -1;
+  if (dtype == DT_F32 || d % 8 != 0) {
+    const int64_t n = T * d;
+    const int nb = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+    DISPATCH_DTYPE(dtype, TT, {
+      vb_launch(act_and_mul_scalar_kernel<TT, ACT_SILU, true>, nb, 256, 0, st, (TT*)out, (const TT*)x, d, n);
+    });
+    return (int)cudaGetLastError();
+  }
   const int64_t total = T * (d / 8);
   const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
   DISPATCH_HALF(dtype, TT, {

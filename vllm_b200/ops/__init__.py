@@ -64,7 +64,7 @@ def silu_and_mul(x: torch.Tensor) -> torch.Tensor:
 
 def silu_and_mul_interleaved(x: torch.Tensor) -> torch.Tensor:
     """silu(x[..., 0::2]) * x[..., 1::2]: the activation for gate_up weights stored as interleaved (gate_i, up_i) rows."""
-    if _use_cuda(x) and x.dtype in (torch.bfloat16, torch.float16) and (x.shape[-1] // 2) % 8 == 0:
+    if _use_cuda(x):
         return cuda_ops().silu_and_mul_interleaved(x)
     return (torch.nn.functional.silu(x[..., 0::2].float()) * x[..., 1::2].float()).to(x.dtype)
 

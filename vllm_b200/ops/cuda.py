@@ -137,11 +137,23 @@ def num_sms() -> int:
 
 
 # ------------------------------------------------------------------ norms / act
+def _rows(x: torch.Tensor) -> torch.Tensor:
+    """Contiguous and at a 16-byte address, as the vectorised row kernels read it.  (``contiguous`` alone keeps a column slice
+    of a single row where it is.)"""
+    x = x.contiguous()
+    return x if x.data_ptr() % 16 == 0 else x.clone()
+
+
+def _heads(x: torch.Tensor) -> torch.Tensor:
+    """Rows of heads, any row stride, for kernels that read heads in 16-byte vectors."""
+    return x if x.data_ptr() % 16 == 0 and (x.stride(0) * x.element_size()) % 16 == 0 else x.clone(memory_format=torch.contiguous_format)
+
+
 def rms_norm(x, weight, eps, gemma=False):
     H = x.shape[-1]
     x2 = x.reshape(-1, H)
-    if x2.stride(-1) != 1:
-        x2 = x2.contiguous()
+    if x2.stride(-1) != 1 or x2.data_ptr() % 16 or (x2.stride(0) * x2.element_size()) % 16:
+        x2 = x2.clone(memory_format=torch.contiguous_format)
     out = torch.empty((x2.shape[0], H), dtype=x.dtype, device=x.device)
     _check(_rms_norm(out.data_ptr(), x2.data_ptr(), None, weight.data_ptr(), x2.shape[0], H, x2.stride(0), eps,
                      int(gemma), _DT[x.dtype], _st()), "rms_norm")
@@ -160,7 +172,7 @@ def fused_add_rms_norm(x, residual, weight, eps, gemma=False):
 
 def layer_norm(x, weight, bias, eps):
     H = x.shape[-1]
-    xc = x.contiguous()
+    xc = _rows(x)
     out = torch.empty_like(xc)
     _check(_layer_norm(out.data_ptr(), xc.data_ptr(), weight.data_ptr(), _p(bias), xc.numel() // H, H, eps,
                        _DT[x.dtype], _st()), "layer_norm")
@@ -169,7 +181,7 @@ def layer_norm(x, weight, bias, eps):
 
 def act_and_mul(x, act: str):
     d = x.shape[-1] // 2
-    xc = x.contiguous()
+    xc = _rows(x)
     out = torch.empty(x.shape[:-1] + (d,), dtype=x.dtype, device=x.device)
     _check(_act_and_mul(out.data_ptr(), xc.data_ptr(), xc.numel() // (2 * d), d, _ACT[act], _DT[x.dtype], _st()),
            "act_and_mul")
@@ -182,14 +194,14 @@ _silu_mul_il = _sig("vb_silu_mul_interleaved", _vp, _vp, _i64, _i, _i, _vp)
 def silu_and_mul_interleaved(x):
     """x[..., 2i] = gate_i, x[..., 2i+1] = up_i → silu(gate) * up."""
     d = x.shape[-1] // 2
-    xc = x.contiguous()
+    xc = _rows(x)
     out = torch.empty(x.shape[:-1] + (d,), dtype=x.dtype, device=x.device)
     _check(_silu_mul_il(out.data_ptr(), xc.data_ptr(), xc.numel() // (2 * d), d, _DT[x.dtype], _st()), "silu_mul_interleaved")
     return out
 
 
 def activation(x, name: str):
-    xc = x.contiguous()
+    xc = _rows(x)
     out = torch.empty_like(xc)
     _check(_activation(out.data_ptr(), xc.data_ptr(), xc.numel(), _ACT[name], _DT[x.dtype], _st()), "activation")
     return out
@@ -205,6 +217,7 @@ def rope_and_cache(positions, q, k, v, cos_sin_cache, head_dim, is_neox, kv_cach
     T = q.shape[0]
     Hq, Hkv = q.shape[-1] // head_dim, k.shape[-1] // head_dim
     assert q.stride(-1) == 1 and k.stride(-1) == 1 and v.stride(-1) == 1
+    q, k, v = _heads(q), _heads(k), _heads(v)
     rot = cos_sin_cache.shape[-1]
     flags = _kv_fp8(kv_cache) | (2 if vt else 0)
     _check(_rope_and_cache(positions.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), cos_sin_cache.data_ptr(),
@@ -220,6 +233,7 @@ def rotary_embedding(positions, q, k, cos_sin_cache, head_dim, is_neox=True):
     Hkv = k.shape[-1] // head_dim if k is not None else 0
     if q.stride(-1) != 1:
         q = q.contiguous()
+    q, k = _heads(q), None if k is None else _heads(k)
     rot = cos_sin_cache.shape[-1]
     _check(_rope_and_cache(positions.data_ptr(), q.data_ptr(), _p(k), None, cos_sin_cache.data_ptr(), rot, T, Hq,
                            Hkv, head_dim, q.stride(0), k.stride(0) if k is not None else 0, 0, None, None, 1,
@@ -230,6 +244,7 @@ def rotary_embedding(positions, q, k, cos_sin_cache, head_dim, is_neox=True):
 def reshape_and_cache(key, value, kv_cache, slot_mapping, k_scale: float = 1.0, v_scale: float = 1.0,
                       vt: bool = False):
     T, Hkv, D = key.shape
+    key, value = _heads(key), _heads(value)
     _check(_rope_and_cache(None, None, key.data_ptr(), value.data_ptr(), None, 0, T, 0, Hkv, D, 0, key.stride(0),
                            value.stride(0), kv_cache.data_ptr(), slot_mapping.data_ptr(), kv_cache.shape[3], 1,
                            _kv_fp8(kv_cache) | (2 if vt else 0), k_scale, v_scale, _DT[key.dtype], _st()),
