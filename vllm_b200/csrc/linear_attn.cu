@@ -11,15 +11,16 @@
 //
 // state_scan: a CTA owns a column tile of one head of one request.  Producer warps stage a block of tokens (decays, keys,
 // queries, values, in fp32) into one half of shared memory while consumer warps run the recurrence over the other; one
-// barrier per block of TB tokens.  A consumer lane holds 2 NP rows x 4 columns of S in registers as packed pairs of rows, so
-// that the three products per element are fma.rn.f32x2; the sum over the rows ends in a few shuffles.  In memory a head's
+// barrier per block of TB tokens, and the loads of the block after next are in flight meanwhile.  A consumer lane holds 2 NP
+// rows x 4 Q columns of S in registers as packed pairs of rows, so that the three products per element are fma.rn.f32x2; the
+// sum over the rows ends in a few shuffles.  In memory a head's
 // state is stored in the order the lanes hold it ([column quad][row in lane][lane][4]): every access is a full 16-byte
 // vector per lane and consecutive across the warp.
 #include "common.cuh"
 
 namespace lattn {
 
-VB_DEVICE float silu_f(float x) { return x / (1.f + __expf(-x)); }
+VB_DEVICE float silu_f(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 VB_DEVICE float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 // sigmoid(z)^(1/tau), through the logarithm so that z of either sign keeps its digits
 VB_DEVICE float decay_of(float z, float inv_tau) {
@@ -37,6 +38,16 @@ VB_DEVICE float4 ld_any4(const void* p, int64_t i, int dt) {      // i and p ali
   if (dt == DT_BF16) { a = unpack2<__nv_bfloat16>(u.x); b = unpack2<__nv_bfloat16>(u.y); }
   else { a = unpack2<__half>(u.x); b = unpack2<__half>(u.y); }
   return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// up to four elements, zeros behind the n-th; not inlined: the path of odd sizes and addresses
+__device__ __noinline__ float4 ld_some(const void* p, int64_t i, int dt, int n) {
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (n > 0) v.x = ld_any(p, i, dt);
+  if (n > 1) v.y = ld_any(p, i + 1, dt);
+  if (n > 2) v.z = ld_any(p, i + 2, dt);
+  if (n > 3) v.w = ld_any(p, i + 3, dt);
+  return v;
 }
 
 using pair_t = unsigned long long;      // two fp32
@@ -71,18 +82,43 @@ struct ScanParams {
   float* out;                                // [T, H * C]
   float* state; int64_t state_stride, state_off, head_elems;
   const int* qsl; const int* seq_lens; const int* rows; int64_t rows_stride;
-  int H, groups, R, C, TB, vec;
+  int H, groups, R, C;
+  int vec, vec_v, vec_o, vec_a;              // accesses in units of four elements
 };
 
-// NP row pairs per lane, L lanes share the rows: capacity 2 NP L rows; a warp covers 32 / L quads of columns
-template <int NP, int L, int MODE>
-__global__ void __launch_bounds__(384) state_scan_kernel(const ScanParams p) {
+// N sums per lane over the lanes lr, lr ^ D, ...: each step hands half of the columns to the other lane; ``at``: first column left
+template <int N, int D>
+VB_DEVICE void reduce_columns(float* s, int lr, int& at) {
+  if constexpr (D > 0) {
+    const bool up = (lr & D) != 0;
+    if constexpr (N > 1) {
+#pragma unroll
+      for (int i = 0; i < N / 2; ++i) {
+        const float keep = up ? s[i + N / 2] : s[i], send = up ? s[i] : s[i + N / 2];
+        s[i] = keep + __shfl_xor_sync(0xffffffffu, send, D);
+      }
+      at += up ? N / 2 : 0;
+      reduce_columns<N / 2, D / 2>(s, lr, at);
+    } else {
+      s[0] += __shfl_xor_sync(0xffffffffu, s[0], D);
+      reduce_columns<1, D / 2>(s, lr, at);
+    }
+  }
+}
+
+// NP row pairs per lane, L lanes share the rows (capacity 2 NP L rows); a lane holds Q quads of columns, a warp 32 / L times as
+// many.  Wide lanes (Q = 4) read the staged rows from shared memory for more columns at a time, narrow ones make more warps.
+template <int NP, int L, int MODE, int Q, int TB>
+__global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_kernel(const ScanParams p) {
   constexpr int RL = 2 * NP;                 // rows per lane
   constexpr int RP = RL * L;                 // padded rows
-  constexpr int CW = 32 / L * 4;             // columns per warp
+  constexpr int LG = 32 / L;
+  constexpr int CW = LG * 4 * Q;             // columns per warp
+  constexpr int NT = PRODUCERS * 32;
   extern __shared__ __align__(16) float sm[];
   const int warps = (blockDim.x >> 5) - PRODUCERS;        // consumers
-  const int CT = warps * CW, TB = p.TB;
+  const int CT = warps * CW;
+  // a staged token: keys RP | queries RP | values 2 CT (each twice) | decay, decay, dt, - | decays RP (per channel)
   const int per_tok = (MODE == DECAY_HEAD ? 2 : 3) * RP + 2 * CT + 4;
   float* bufs = sm;                                       // 2 x TB x per_tok
   float* obuf = sm + 2 * TB * per_tok;                    // 2 x TB x CT
@@ -92,94 +128,135 @@ __global__ void __launch_bounds__(384) state_scan_kernel(const ScanParams p) {
   const int t0 = p.qsl[req], t1 = p.qsl[req + 1], n = t1 - t0;
   if (n <= 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const bool has_init = p.seq_lens[req] > n;
   const int R = p.R, C = p.C;
-  const int g = h / (p.H / p.groups);
   const int nblk = (n + TB - 1) / TB;
 
   if (warp >= warps) {
-    // ================= producers
+    // ================= producers: the loads of a block are in flight while the block before it is computed
     const int tid = threadIdx.x - warps * 32;
-    constexpr int NT = PRODUCERS * 32;
-    auto stage = [&](int blk) {
+    const int g = h / (p.H / p.groups);
+    constexpr int NI = (TB * (RP / 4) + NT - 1) / NT;     // row vectors per thread and operand
+    constexpr int NVI = (TB * 32 + NT - 1) / NT;          // value vectors per thread held ahead (of wider tiles the rest is late)
+    float4 rk[NI], rq[NI], ra[NI], rv[NVI];
+    float rdt = 0.f;
+    const int cv = CT / 4;
+    auto value4 = [&](int64_t tok, int c) {
+      const int64_t i = tok * p.v_stride + (int64_t)h * C + c;
+      return p.vec_v ? ld_any4(p.v, i, p.v_dt) : ld_some(p.v, i, p.v_dt, C - c);
+    };
+    auto fetch = [&](int blk) {
+      const int tb = min(TB, n - blk * TB);
+      const int64_t tok0 = t0 + (int64_t)blk * TB;
+      const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int it = tid + i * NT, t = it / (RP / 4), r = (it % (RP / 4)) * 4;
+        rk[i] = rq[i] = ra[i] = zero;
+        if (t >= tb || r >= R) continue;
+        const int64_t ki = (tok0 + t) * p.k_stride + (int64_t)g * R + r, qi = (tok0 + t) * p.q_stride + (int64_t)g * R + r;
+        rk[i] = p.vec ? ld_any4(p.k, ki, p.k_dt) : ld_some(p.k, ki, p.k_dt, R - r);
+        rq[i] = p.vec ? ld_any4(p.q, qi, p.q_dt) : ld_some(p.q, qi, p.q_dt, R - r);
+        if constexpr (MODE == DECAY_GIVEN) {
+          const int64_t ai = ((tok0 + t) * p.H + h) * (int64_t)R + r;
+          ra[i] = p.vec ? *reinterpret_cast<const float4*>(p.alpha + ai) : ld_some(p.alpha, ai, DT_F32, R - r);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < NVI; ++i) {
+        const int it = tid + i * NT, t = it / cv, c = c0 + (it - t * cv) * 4;
+        rv[i] = zero;
+        if (t < tb && c < C) rv[i] = value4(tok0 + t, c);
+      }
+      if constexpr (MODE == DECAY_HEAD)
+        if (tid < tb) rdt = ld_any(p.dt, (tok0 + tid) * p.dt_stride + h, p.dt_dt);
+    };
+    auto store = [&](int blk) {
       float* b = bufs + (blk & 1) * TB * per_tok;
       const int tb = min(TB, n - blk * TB);
       const int64_t tok0 = t0 + (int64_t)blk * TB;
       if constexpr (MODE == DECAY_HEAD) {
-        // [k | q] rows, then values, then (decay, dt); the decay goes first: keys are scaled by dt
-        const float A = -expf(p.A_log[h]), db = p.dt_bias[h];
-        for (int i = tid; i < tb; i += NT) {
-          const float dt = fminf(fmaxf(softplus_f(ld_any(p.dt, (tok0 + i) * p.dt_stride + h, p.dt_dt) + db), p.dt_min), p.dt_max);
-          float* s = b + i * per_tok + 2 * RP + 2 * CT;
-          s[0] = s[1] = expf(A * dt);
-          s[2] = dt;
+        if (tid < tb) {
+          const float dt = fminf(fmaxf(softplus_f(rdt + p.dt_bias[h]), p.dt_min), p.dt_max);
+          float* d = b + tid * per_tok + 2 * RP + 2 * CT;
+          d[0] = d[1] = expf(-expf(p.A_log[h]) * dt);
+          d[2] = dt;
         }
         asm volatile("bar.sync 1, %0;" ::"n"(NT) : "memory");
       }
-      if (p.vec) {
-        const int rq = RP / 4;
-        for (int i = tid; i < tb * rq; i += NT) {
-          const int t = i / rq, r = (i - t * rq) * 4;
-          float* row = b + t * per_tok;
-          float4 kk = make_float4(0.f, 0.f, 0.f, 0.f), qq = kk;
-          if (r < R) {
-            kk = ld_any4(p.k, (tok0 + t) * p.k_stride + (int64_t)g * R + r, p.k_dt);
-            qq = ld_any4(p.q, (tok0 + t) * p.q_stride + (int64_t)g * R + r, p.q_dt);
-          }
-          const float ks = MODE == DECAY_HEAD ? row[2 * RP + 2 * CT + 2] : 1.f;
-          *reinterpret_cast<float4*>(row + r) = make_float4(kk.x * ks, kk.y * ks, kk.z * ks, kk.w * ks);
-          *reinterpret_cast<float4*>(row + RP + r) = make_float4(qq.x * p.q_scale, qq.y * p.q_scale, qq.z * p.q_scale, qq.w * p.q_scale);
-          if constexpr (MODE == DECAY_GIVEN) {
-            float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (r < R) a = *reinterpret_cast<const float4*>(p.alpha + ((tok0 + t) * p.H + h) * (int64_t)R + r);
-            *reinterpret_cast<float4*>(row + 2 * RP + 2 * CT + 4 + r) = a;
-          }
-        }
-      } else {
-        for (int i = tid; i < tb * RP; i += NT) {
-          const int t = i / RP, r = i - t * RP;
-          float* row = b + t * per_tok;
-          float kk = 0.f, qq = 0.f;
-          if (r < R) {
-            kk = ld_any(p.k, (tok0 + t) * p.k_stride + (int64_t)g * R + r, p.k_dt);
-            qq = ld_any(p.q, (tok0 + t) * p.q_stride + (int64_t)g * R + r, p.q_dt);
-          }
-          row[r] = MODE == DECAY_HEAD ? kk * row[2 * RP + 2 * CT + 2] : kk;
-          row[RP + r] = qq * p.q_scale;
-          if constexpr (MODE == DECAY_GIVEN)
-            row[2 * RP + 2 * CT + 4 + r] = r < R ? p.alpha[((tok0 + t) * p.H + h) * (int64_t)R + r] : 0.f;
-        }
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int it = tid + i * NT, t = it / (RP / 4), r = (it % (RP / 4)) * 4;
+        if (t >= tb) continue;
+        float* row = b + t * per_tok;
+        const float ks = MODE == DECAY_HEAD ? row[2 * RP + 2 * CT + 2] : 1.f;
+        *reinterpret_cast<float4*>(row + r) = make_float4(rk[i].x * ks, rk[i].y * ks, rk[i].z * ks, rk[i].w * ks);
+        *reinterpret_cast<float4*>(row + RP + r) =
+            make_float4(rq[i].x * p.q_scale, rq[i].y * p.q_scale, rq[i].z * p.q_scale, rq[i].w * p.q_scale);
+        if constexpr (MODE == DECAY_GIVEN) *reinterpret_cast<float4*>(row + 2 * RP + 2 * CT + 4 + r) = ra[i];
       }
       if constexpr (MODE == DECAY_LOWRANK) {
         for (int r = tid; r < RP; r += NT) {
-          if (r >= R) { for (int t = 0; t < tb; ++t) b[t * per_tok + 2 * RP + 2 * CT + 4 + r] = 0.f; continue; }
           const int64_t w0 = ((int64_t)h * R + r) * p.rank;
-          const float bias = ld_any(p.a2_b, (int64_t)h * R + r, p.a_dt);
+          const float bias = r < R ? ld_any(p.a2_b, (int64_t)h * R + r, p.a_dt) : 0.f;
           for (int t = 0; t < tb; ++t) {
             float z = bias;
-            for (int j = 0; j < p.rank; ++j) z += ld_any(p.a2, w0 + j, p.a_dt) * ld_any(p.a1, (tok0 + t) * p.a1_stride + j, p.a_dt);
-            b[t * per_tok + 2 * RP + 2 * CT + 4 + r] = decay_of(z, p.inv_tau);
+            const int64_t y0 = (tok0 + t) * p.a1_stride;
+            if (r < R) {
+              if (p.vec_a) {
+#pragma unroll 4
+                for (int j = 0; j < p.rank; j += 4) {
+                  const float4 w = ld_any4(p.a2, w0 + j, p.a_dt), y = ld_any4(p.a1, y0 + j, p.a_dt);
+                  z += w.x * y.x; z += w.y * y.y; z += w.z * y.z; z += w.w * y.w;
+                }
+              } else {
+                for (int j = 0; j < p.rank; ++j) z += ld_any(p.a2, w0 + j, p.a_dt) * ld_any(p.a1, y0 + j, p.a_dt);
+              }
+            }
+            b[t * per_tok + 2 * RP + 2 * CT + 4 + r] = r < R ? decay_of(z, p.inv_tau) : 0.f;
           }
         }
       }
-      for (int i = tid; i < tb * CT; i += NT) {
-        const int t = i / CT, c = i - t * CT;
-        const float v = c0 + c < C ? ld_any(p.v, (tok0 + t) * p.v_stride + (int64_t)h * C + c0 + c, p.v_dt) : 0.f;
-        *reinterpret_cast<float2*>(b + t * per_tok + 2 * RP + 2 * c) = make_float2(v, v);
+      auto put = [&](int t, int c, float4 v) {
+        float4* d = reinterpret_cast<float4*>(b + t * per_tok + 2 * RP + 2 * c);
+        d[0] = make_float4(v.x, v.x, v.y, v.y);
+        d[1] = make_float4(v.z, v.z, v.w, v.w);
+      };
+#pragma unroll
+      for (int i = 0; i < NVI; ++i) {
+        const int it = tid + i * NT, t = it / cv, c = (it - t * cv) * 4;
+        if (t < tb) put(t, c, rv[i]);
+      }
+      for (int it = tid + NVI * NT; it < tb * cv; it += NT) {
+        const int t = it / cv, c = (it - t * cv) * 4;
+        put(t, c, c0 + c < C ? value4(tok0 + t, c0 + c) : make_float4(0.f, 0.f, 0.f, 0.f));
       }
     };
     auto flush = [&](int blk) {
       const float* o = obuf + (blk & 1) * TB * CT;
       const int tb = min(TB, n - blk * TB);
+      if (p.vec_o) {
+        for (int i = tid; i < tb * cv; i += NT) {
+          const int t = i / cv, c = (i - t * cv) * 4;
+          if (c0 + c < C)
+            *reinterpret_cast<float4*>(p.out + (t0 + (int64_t)blk * TB + t) * p.H * C + (int64_t)h * C + c0 + c) =
+                *reinterpret_cast<const float4*>(o + t * CT + c);
+        }
+        return;
+      }
       for (int i = tid; i < tb * CT; i += NT) {
         const int t = i / CT, c = i - t * CT;
         if (c0 + c < C) p.out[(t0 + (int64_t)blk * TB + t) * p.H * C + (int64_t)h * C + c0 + c] = o[i];
       }
     };
-    stage(0);
+    fetch(0);
+    store(0);
+    if (nblk > 1) fetch(1);
     bar_all();
     for (int blk = 0; blk < nblk; ++blk) {
-      if (blk + 1 < nblk) stage(blk + 1);
+      if (blk + 1 < nblk) {
+        store(blk + 1);
+        if (blk + 2 < nblk) fetch(blk + 2);
+      }
       if (blk > 0) flush(blk - 1);
       bar_all();
     }
@@ -188,20 +265,23 @@ __global__ void __launch_bounds__(384) state_scan_kernel(const ScanParams p) {
   }
 
   // ================= consumers
-  const int lr = lane % L, quad = warp * (32 / L) + lane / L;         // quad of columns inside the tile
-  const int cq = c0 / 4 + quad;                                       // ... of the head
-  const bool live = cq * 4 < C;
-  float* st = p.state + (int64_t)p.rows[req * p.rows_stride] * p.state_stride + p.state_off + (int64_t)h * p.head_elems +
-              (int64_t)cq * RP * 4 + lr * 4;
-  pair_t S[4][NP];
+  const int lr = lane % L, lg = lane / L;
+  auto quad_of = [&](int j) { return (warp * Q + j) * LG + lg; };     // quad of columns inside the tile
+  const bool has_init = p.seq_lens[req] > n;
+  float* st = p.state + (int64_t)p.rows[req * p.rows_stride] * p.state_stride + p.state_off + (int64_t)h * p.head_elems + lr * 4;
+  pair_t S[Q][4][NP];
 #pragma unroll
-  for (int i = 0; i < NP; ++i) {
-    float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
-    if (has_init && live) {
-      x = *reinterpret_cast<const float4*>(st + (2 * i) * L * 4);
-      y = *reinterpret_cast<const float4*>(st + (2 * i + 1) * L * 4);
+  for (int j = 0; j < Q; ++j) {
+    const int64_t cq = c0 / 4 + quad_of(j);
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
+      if (has_init && cq * 4 < C) {
+        x = *reinterpret_cast<const float4*>(st + (cq * RP + (2 * i) * L) * 4);
+        y = *reinterpret_cast<const float4*>(st + (cq * RP + (2 * i + 1) * L) * 4);
+      }
+      S[j][0][i] = pack(x.x, y.x); S[j][1][i] = pack(x.y, y.y); S[j][2][i] = pack(x.z, y.z); S[j][3][i] = pack(x.w, y.w);
     }
-    S[0][i] = pack(x.x, y.x); S[1][i] = pack(x.y, y.y); S[2][i] = pack(x.z, y.z); S[3][i] = pack(x.w, y.w);
   }
   const float dskip = MODE == DECAY_HEAD ? p.D[h] : 0.f;
   bar_all();
@@ -209,10 +289,10 @@ __global__ void __launch_bounds__(384) state_scan_kernel(const ScanParams p) {
     const float* b = bufs + (blk & 1) * TB * per_tok;
     float* o = obuf + (blk & 1) * TB * CT;
     const int tb = min(TB, n - blk * TB);
-#pragma unroll 2
+#pragma unroll(Q == 1 ? 2 : 1)
     for (int t = 0; t < tb; ++t) {
       const float* row = b + t * per_tok;
-      pair_t kk[NP], qq[NP], aa[NP], vv[4];
+      pair_t kk[NP], qq[NP], aa[NP];
       auto ld_rows = [&](const float* src, pair_t (&dst)[NP]) {
         if constexpr (NP == 1) dst[0] = *reinterpret_cast<const pair_t*>(src + lr * RL);
         else {
@@ -232,44 +312,47 @@ __global__ void __launch_bounds__(384) state_scan_kernel(const ScanParams p) {
       } else {
         ld_rows(row + 2 * RP + 2 * CT + 4, aa);
       }
-      const ulonglong2 v01 = *reinterpret_cast<const ulonglong2*>(row + 2 * RP + quad * 8);
-      const ulonglong2 v23 = *reinterpret_cast<const ulonglong2*>(row + 2 * RP + quad * 8 + 4);
-      vv[0] = v01.x; vv[1] = v01.y; vv[2] = v23.x; vv[3] = v23.y;
-      float s[4];
+      float s[4 * Q];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        pair_t acc;
+      for (int j = 0; j < Q; ++j) {
+        const float* vp = row + 2 * RP + quad_of(j) * 8;
+        const ulonglong2 v01 = *reinterpret_cast<const ulonglong2*>(vp), v23 = *reinterpret_cast<const ulonglong2*>(vp + 4);
+        const pair_t vv[4] = {v01.x, v01.y, v23.x, v23.y};
 #pragma unroll
-        for (int i = 0; i < NP; ++i) {
-          S[c][i] = fma2(aa[i], S[c][i], mul2(kk[i], vv[c]));
-          acc = i == 0 ? mul2(S[c][i], qq[i]) : fma2(S[c][i], qq[i], acc);
+        for (int c = 0; c < 4; ++c) {
+          pair_t acc;
+#pragma unroll
+          for (int i = 0; i < NP; ++i) {
+            S[j][c][i] = fma2(aa[i], S[j][c][i], mul2(kk[i], vv[c]));
+            acc = i == 0 ? mul2(S[j][c][i], qq[i]) : fma2(S[j][c][i], qq[i], acc);
+          }
+          const float2 f = unpack(acc);
+          s[j * 4 + c] = f.x + f.y;
         }
-        const float2 f = unpack(acc);
-        s[c] = f.x + f.y;
       }
-      // four sums over L lanes: halve the columns twice, then add the rest up
-      constexpr int H1 = L / 2, H2 = L / 4;
-      const bool up1 = (lr & H1) != 0, up2 = (lr & H2) != 0;
-      float x0 = up1 ? s[2] : s[0], x1 = up1 ? s[3] : s[1];
-      x0 += __shfl_xor_sync(0xffffffffu, up1 ? s[0] : s[2], H1);
-      x1 += __shfl_xor_sync(0xffffffffu, up1 ? s[1] : s[3], H1);
-      float x = up2 ? x1 : x0;
-      x += __shfl_xor_sync(0xffffffffu, up2 ? x0 : x1, H2);
+      // 4 Q sums over L lanes: halve the columns while there are two or more, then add the rest up
+      int at = 0;
+      reduce_columns<4 * Q, L / 2>(s, lr, at);
+      constexpr int LEFT = 4 * Q > L ? 4 * Q / L : 1, SAME = L > 4 * Q ? L / (4 * Q) : 1;   // sums per lane, lanes with the same
+      if ((lr & (SAME - 1)) == 0) {
 #pragma unroll
-      for (int d = H2 / 2; d > 0; d >>= 1) x += __shfl_xor_sync(0xffffffffu, x, d);
-      if ((lr & (H2 - 1)) == 0) {
-        const int c = quad * 4 + (up1 ? 2 : 0) + (up2 ? 1 : 0);
-        o[t * CT + c] = MODE == DECAY_HEAD ? x + dskip * row[2 * RP + 2 * c] : x;
+        for (int i = 0; i < LEFT; ++i) {
+          const int c = quad_of((at + i) >> 2) * 4 + ((at + i) & 3);
+          o[t * CT + c] = MODE == DECAY_HEAD ? s[i] + dskip * row[2 * RP + 2 * c] : s[i];
+        }
       }
     }
     bar_all();
   }
-  if (live) {
+#pragma unroll
+  for (int j = 0; j < Q; ++j) {
+    const int64_t cq = c0 / 4 + quad_of(j);
+    if (cq * 4 >= C) continue;
 #pragma unroll
     for (int i = 0; i < NP; ++i) {
-      const float2 a = unpack(S[0][i]), b = unpack(S[1][i]), c = unpack(S[2][i]), d = unpack(S[3][i]);
-      *reinterpret_cast<float4*>(st + (2 * i) * L * 4) = make_float4(a.x, b.x, c.x, d.x);
-      *reinterpret_cast<float4*>(st + (2 * i + 1) * L * 4) = make_float4(a.y, b.y, c.y, d.y);
+      const float2 a = unpack(S[j][0][i]), bb = unpack(S[j][1][i]), c = unpack(S[j][2][i]), d = unpack(S[j][3][i]);
+      *reinterpret_cast<float4*>(st + (cq * RP + (2 * i) * L) * 4) = make_float4(a.x, bb.x, c.x, d.x);
+      *reinterpret_cast<float4*>(st + (cq * RP + (2 * i + 1) * L) * 4) = make_float4(a.y, bb.y, c.y, d.y);
     }
   }
 }
@@ -303,42 +386,50 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ a1
     if (t < nt) out[(int64_t)(t0 + t) * CH + c] = decay_of(z[t], inv_tau);
 }
 
-// (token, group of W channels) per group of WPG warps: rms over the group of y (gate first: of y silu(z)), times w, (gate
-// last: times silu(z)), times a constant; w repeats after w_len channels
+// (token, group of W channels) per group of wpg warps: rms over the group of y (gate first: of y silu(z)), times w, (gate
+// last: times silu(z)), times a constant; w repeats after w_len channels.  NV vectors of V elements per lane stay in registers.
+constexpr int GN_NV = 4;
 template <typename T, int V>
-__global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, int64_t z_stride,
-                                                          const T* __restrict__ w, int w_len, T* __restrict__ out,
-                                                          int64_t out_stride, int64_t n_rows, int groups, int W, int gate_first,
-                                                          float eps, float scale, int wpg) {
-  __shared__ float red[8];
+__global__ void __launch_bounds__(1024) gated_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, int64_t z_stride,
+                                                           const T* __restrict__ w, int w_len, T* __restrict__ out,
+                                                           int64_t out_stride, int64_t n_rows, int groups, int W, int gate_first,
+                                                           float eps, float scale, int wpg) {
+  __shared__ float red[32];
   pdl_trigger();
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int per_cta = 8 / wpg, sub = warp / wpg;
+  const int per_cta = (blockDim.x >> 5) / wpg, sub = warp / wpg;
   const int64_t row = (int64_t)blockIdx.x * per_cta + sub;
   const bool ok = row < n_rows;
   const int64_t tok = ok ? row / groups : 0;
-  const int g = ok ? (int)(row % groups) : 0;
+  const int g = ok ? (int)(row - tok * groups) : 0;
   const float* yr = y + (tok * groups + g) * (int64_t)W;
   const T* zr = z + tok * z_stride + (int64_t)g * W;
   const int i0 = ((warp % wpg) * 32 + lane) * V, step = wpg * 32 * V;
   constexpr int dt = DTypeOf<T>::v;
-  float ss = 0.f;
-  if (ok)
-    for (int i = i0; i < W; i += step) {
-      if constexpr (V == 4) {
-        float4 a = *reinterpret_cast<const float4*>(yr + i);
-        if (gate_first) {
-          const float4 b = ld_any4(zr, i, dt);
-          a.x *= silu_f(b.x); a.y *= silu_f(b.y); a.z *= silu_f(b.z); a.w *= silu_f(b.w);
-        }
-        ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
-      } else {
-        float a = yr[i];
-        if (gate_first) a *= silu_f(to_f32(zr[i]));
-        ss += a * a;
-      }
+  auto load = [&](int i, float (&a)[V], float (&b)[V]) {
+    if constexpr (V == 4) {
+      const float4 x = *reinterpret_cast<const float4*>(yr + i), u = ld_any4(zr, i, dt);
+      a[0] = x.x; a[1] = x.y; a[2] = x.z; a[3] = x.w;
+      b[0] = silu_f(u.x); b[1] = silu_f(u.y); b[2] = silu_f(u.z); b[3] = silu_f(u.w);
+    } else {
+      a[0] = yr[i];
+      b[0] = silu_f(to_f32(zr[i]));
     }
+  };
+  float a[GN_NV][V], b[GN_NV][V], ss = 0.f;
+  auto square = [&](const float (&u)[V], const float (&v)[V]) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) { const float x = gate_first ? u[j] * v[j] : u[j]; ss += x * x; }
+  };
+#pragma unroll
+  for (int k = 0; k < GN_NV; ++k)
+    if (ok && i0 + k * step < W) { load(i0 + k * step, a[k], b[k]); square(a[k], b[k]); }
+  for (int i = i0 + GN_NV * step; ok && i < W; i += step) {            // rows too long for the registers
+    float u[V], v[V];
+    load(i, u, v);
+    square(u, v);
+  }
   ss = warp_sum(ss);
   if (wpg > 1) {
     if (lane == 0) red[warp] = ss;
@@ -349,45 +440,76 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
   if (!ok) return;
   const float r = scale / sqrtf(ss / (float)W + eps);
   T* orow = out + tok * out_stride + (int64_t)g * W;
-  for (int i = i0; i < W; i += step) {
-    const int wi = (int)(((int64_t)g * W + i) % w_len);
+  const int w0 = w_len > W ? g * W : 0;                                // (w_len is W, a multiple or a divisor of it)
+  auto emit = [&](int i, const float (&u)[V], const float (&v)[V]) {
+    const int wi = w_len < W ? i % w_len : w0 + i;
     if constexpr (V == 4) {
-      const float4 a = *reinterpret_cast<const float4*>(yr + i), b = ld_any4(zr, i, dt), ww = ld_any4(w, wi, dt);
-      const float o0 = a.x * silu_f(b.x) * ww.x * r, o1 = a.y * silu_f(b.y) * ww.y * r;
-      const float o2 = a.z * silu_f(b.z) * ww.z * r, o3 = a.w * silu_f(b.w) * ww.w * r;
+      const float4 ww = ld_any4(w, wi, dt);
+      const float o0 = u[0] * v[0] * ww.x * r, o1 = u[1] * v[1] * ww.y * r, o2 = u[2] * v[2] * ww.z * r, o3 = u[3] * v[3] * ww.w * r;
       if constexpr (dt == DT_F32) *reinterpret_cast<float4*>(orow + i) = make_float4(o0, o1, o2, o3);
       else *reinterpret_cast<uint2*>(orow + i) = make_uint2(pack2<T>(o0, o1), pack2<T>(o2, o3));
     } else {
-      orow[i] = from_f32<T>(yr[i] * silu_f(to_f32(zr[i])) * to_f32(w[wi]) * r);
+      orow[i] = from_f32<T>(u[0] * v[0] * to_f32(w[wi]) * r);
     }
+  };
+#pragma unroll
+  for (int k = 0; k < GN_NV; ++k)
+    if (i0 + k * step < W) emit(i0 + k * step, a[k], b[k]);
+  for (int i = i0 + GN_NV * step; i < W; i += step) {
+    float u[V], v[V];
+    load(i, u, v);
+    emit(i, u, v);
   }
 }
 
-template <int NP, int L>
-int scan_shape(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t st) {
-  constexpr int RP = 2 * NP * L, CW = 32 / L * 4;
-  // narrow tiles while they are needed to fill the SMs, wide ones (fewer copies of the staged rows) otherwise
-  int warps = 8;
-  while (warps > 1 && ((warps / 2) * CW >= p.C || (int64_t)num_reqs * p.H * ((p.C + warps * CW - 1) / (warps * CW)) < 148)) warps /= 2;
-  const int CT = warps * CW;
-  const int per_tok = (mode == DECAY_HEAD ? 2 : 3) * RP + 2 * CT + 4;
-  int TB = 16;
-  while (TB > 1 && (TB / 2 >= max_len || (size_t)(2 * TB * (per_tok + CT)) * 4 > 100 * 1024)) TB /= 2;
-  p.TB = TB;
+template <int NP, int L, int Q, int TB>
+int scan_launch(ScanParams& p, int mode, int num_reqs, int warps, cudaStream_t st) {
+  constexpr int RP = 2 * NP * L, CW = 32 / L * 4 * Q;
+  const int CT = warps * CW, per_tok = (mode == DECAY_HEAD ? 2 : 3) * RP + 2 * CT + 4;
   const size_t smem = (size_t)(2 * TB * (per_tok + CT)) * 4;
   dim3 grid((p.C + CT - 1) / CT, p.H, num_reqs), block(32 * (warps + PRODUCERS));
 #define GO(M)                                                                                             \
   do {                                                                                                    \
-    auto kern = state_scan_kernel<NP, L, M>;                                                              \
+    auto kern = state_scan_kernel<NP, L, M, Q, TB>;                                                       \
     static bool set = false;                                                                              \
-    if (!set) { cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 101 * 1024); set = true; } \
+    if (!set) { cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); set = true; } \
     vb_launch(kern, grid, block, smem, st, p);                                                            \
   } while (0)
-  if (mode == DECAY_GIVEN) GO(DECAY_GIVEN);
-  else if (mode == DECAY_LOWRANK) GO(DECAY_LOWRANK);
-  else GO(DECAY_HEAD);
+  if (smem > 200 * 1024) return -4;
+  if (mode == DECAY_HEAD) GO(DECAY_HEAD);
+  else if (mode == DECAY_GIVEN) GO(DECAY_GIVEN);
+  else if constexpr (TB == 1) GO(DECAY_LOWRANK);
+  else return -5;                                  // prompts bring their decays
 #undef GO
   return (int)cudaGetLastError();
+}
+
+constexpr int SMS = 148;
+template <int NP, int L>
+int scan_shape(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t st) {
+  constexpr int LG = 32 / L, QMAX = NP <= 2 ? 4 : NP == 4 ? 2 : 1;      // state registers per lane: 8 NP Q
+  const int64_t quads = (int64_t)num_reqs * p.H * ((p.C + 3) / 4);      // of the whole launch
+  const int head_quads = (p.C + 3) / 4;
+  auto tile_warps = [&](int q) {                                        // warps that a CTA needs for one head's columns, at most 8
+    int w = 1;
+    while (w < 8 && w * q * LG < head_quads) w *= 2;
+    return w;
+  };
+  if (max_len == 1) {
+    // decode: the state's bytes count; two quads per lane keep enough of them in flight where there are many states
+    if (QMAX >= 2 && quads / (2 * LG) >= 8 * SMS * 3) return scan_launch<NP, L, QMAX >= 2 ? 2 : 1, 1>(p, mode, num_reqs, tile_warps(2), st);
+    int w = tile_warps(1);
+    while (w > 1 && quads / (w * LG) < SMS) w /= 2;
+    return scan_launch<NP, L, 1, 1>(p, mode, num_reqs, w, st);
+  }
+  // prompts: the widest lanes that still give every scheduler of the GPU a warp, then CTAs small enough to fill the SMs
+  int q = QMAX;
+  if (quads / (q * LG) < SMS * 4) q = 1;
+  int w = tile_warps(q);
+  while (w > 1 && quads / (w * q * LG) < SMS * 3 / 4) w /= 2;
+  constexpr int TB = NP <= 4 ? 16 : 8;
+  if (QMAX > 1 && q == QMAX) return scan_launch<NP, L, QMAX, TB>(p, mode, num_reqs, w, st);
+  return scan_launch<NP, L, 1, TB>(p, mode, num_reqs, w, st);
 }
 
 inline bool al(const void* p, int64_t n) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) % (size_t)n) == 0; }
@@ -399,6 +521,9 @@ int scan(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t st) {
   if (p.state_stride % 4 || p.state_off % 4 || !al(p.state, 16)) return -2;
   p.vec = p.R % 4 == 0 && p.q_stride % 4 == 0 && p.k_stride % 4 == 0 && al(p.q, 4 * esz(p.q_dt)) && al(p.k, 4 * esz(p.k_dt)) &&
           al(p.alpha, 16);
+  p.vec_v = p.C % 4 == 0 && p.v_stride % 4 == 0 && al(p.v, 4 * esz(p.v_dt));
+  p.vec_o = p.C % 4 == 0 && al(p.out, 16);
+  p.vec_a = p.rank % 4 == 0 && p.a1_stride % 4 == 0 && al(p.a1, 4 * esz(p.a_dt)) && al(p.a2, 4 * esz(p.a_dt));
   const int rp = p.R <= 16 ? 16 : p.R <= 32 ? 32 : p.R <= 64 ? 64 : p.R <= 128 ? 128 : p.R <= 256 ? 256 : 512;
   if (p.R > 512) return -3;
   p.head_elems = (int64_t)((p.C + 3) / 4) * 4 * rp;
@@ -477,11 +602,14 @@ EXPORT int vb_gated_norm(const float* y, const void* z, int64_t z_stride, const 
   const int e = esz(dtype);
   const bool vec = W % 4 == 0 && w_len % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0 && al(y, 16) && al(z, 4 * e) &&
                    al(w, 4 * e) && al(out, 4 * e);
-  const int wpg = W <= 512 ? 1 : W <= 1024 ? 2 : W <= 2048 ? 4 : 8;
-  dim3 grid((unsigned)((rows + 8 / wpg - 1) / (8 / wpg)));
+  const int per_warp = vec ? 32 * 4 * GN_NV : 32 * GN_NV;
+  int wpg = 1;
+  while (wpg < 32 && wpg * per_warp < W) wpg *= 2;
+  const int warps = wpg > 8 ? wpg : 8, per_cta = warps / wpg;
+  dim3 grid((unsigned)((rows + per_cta - 1) / per_cta)), block(warps * 32);
   DISPATCH_DTYPE(dtype, T, {
-    if (vec) vb_launch(gated_norm_kernel<T, 4>, grid, dim3(256), 0, st, y, (const T*)z, z_stride, (const T*)w, w_len, (T*)out, out_stride, rows, groups, W, gate_first, eps, scale, wpg);
-    else vb_launch(gated_norm_kernel<T, 1>, grid, dim3(256), 0, st, y, (const T*)z, z_stride, (const T*)w, w_len, (T*)out, out_stride, rows, groups, W, gate_first, eps, scale, wpg);
+    if (vec) vb_launch(gated_norm_kernel<T, 4>, grid, block, 0, st, y, (const T*)z, z_stride, (const T*)w, w_len, (T*)out, out_stride, rows, groups, W, gate_first, eps, scale, wpg);
+    else vb_launch(gated_norm_kernel<T, 1>, grid, block, 0, st, y, (const T*)z, z_stride, (const T*)w, w_len, (T*)out, out_stride, rows, groups, W, gate_first, eps, scale, wpg);
   });
   return (int)cudaGetLastError();
 }

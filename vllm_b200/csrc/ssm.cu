@@ -19,41 +19,54 @@ namespace {
 VB_DEVICE float silu_f(float x) { return x / (1.f + __expf(-x)); }
 
 // ------------------------------------------------------------------ causal conv1d (+ SiLU), window cached per request
-// Thread = one channel x TT consecutive tokens of the batch: the grid depends on the token count alone, and a long prompt is
+// Thread = V channels x TT consecutive tokens of the batch: the grid depends on the token count alone, and a long prompt is
 // spread over all SMs.  A token's request is found from query_start_loc.  The cached window of a request (the last K - 1
 // inputs) is read and rewritten by one thread only, the one that has the request's first token; it also takes the tokens
 // behind its tile that still look into the old window.  KT: compile-time tap count, 0: any up to MAX_TAPS.
-constexpr int CONV_TT = 16, MAX_TAPS = 16;
-template <typename T, int KT>
+constexpr int MAX_TAPS = 16;
+template <typename T, int V> VB_DEVICE void ld_ch(const T* p, float (&v)[V]) {
+  if constexpr (V == 2 && sizeof(T) == 2) {
+    const float2 f = unpack2<T>(*reinterpret_cast<const uint32_t*>(p));
+    v[0] = f.x; v[1] = f.y;
+  } else {
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = to_f32(p[i]);
+  }
+}
+template <typename T, int KT, int V>
 __global__ void __launch_bounds__(128) causal_conv1d_kernel(const T* __restrict__ x, int64_t x_stride, float* __restrict__ out,
                                                              int64_t out_stride, const T* __restrict__ w,
                                                              const T* __restrict__ bias, float* __restrict__ state,
                                                              int64_t state_stride, const int* __restrict__ qsl,
                                                              const int* __restrict__ seq_lens,
                                                              const int* __restrict__ rows, int64_t rows_stride, int num_reqs,
-                                                             int n_tok, int C, int taps, int act) {
+                                                             int n_tok, int C, int taps, int act, int TT) {
   constexpr int KM = KT ? KT : MAX_TAPS;
   pdl_trigger();
   pdl_wait();
   const int K = KT ? KT : taps;
-  const int c = blockIdx.y * blockDim.x + threadIdx.x;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (c >= C) return;
-  const int tile0 = blockIdx.x * CONV_TT, tile1 = min(tile0 + CONV_TT, n_tok);
+  const int tile0 = blockIdx.x * TT, tile1 = min(tile0 + TT, n_tok);
   const int total = qsl[num_reqs];
-  // last request that starts at or before the tile and is not empty there
+  // last request that starts at or before the tile
   int r = 0;
   for (int lo = 0, hi = num_reqs - 1; lo <= hi;) {
     const int mid = (lo + hi) >> 1;
     if (qsl[mid] <= tile0) { r = mid; lo = mid + 1; } else hi = mid - 1;
   }
-  float wr[KM];
+  float wr[KM][V], b[V];
 #pragma unroll
-  for (int j = 0; j < KM; ++j) wr[j] = j < K ? to_f32(w[(int64_t)c * K + j]) : 0.f;
-  const float b = bias ? to_f32(bias[c]) : 0.f;
+  for (int j = 0; j < KM; ++j)
+#pragma unroll
+    for (int v = 0; v < V; ++v) wr[j][v] = j < K ? to_f32(w[(int64_t)(c + v) * K + j]) : 0.f;
+#pragma unroll
+  for (int v = 0; v < V; ++v) b[v] = bias ? to_f32(bias[c + v]) : 0.f;
   int t = tile0;
   while (t < tile1) {
     if (t >= total) {                                   // padding of a graph bucket
-      out[t * out_stride + c] = 0.f;
+#pragma unroll
+      for (int v = 0; v < V; ++v) out[t * out_stride + c + v] = 0.f;
       ++t;
       continue;
     }
@@ -62,38 +75,54 @@ __global__ void __launch_bounds__(128) causal_conv1d_kernel(const T* __restrict_
     const bool first = t == t0;
     if (!first && t < t0 + K - 1) { t = min(t0 + K - 1, t1); continue; }      // an earlier thread's tokens
     const int end = first ? min(t1, max(tile1, t0 + K - 1)) : min(t1, tile1);
-    float win[KM];                                      // inputs t - K + 1 .. t - 1, then t
+    float win[KM][V];                                   // inputs t - K + 1 .. t - 1
     if (first) {
-      float* st = state + (int64_t)rows[r * rows_stride] * state_stride + (int64_t)c * (K - 1);
       const bool has_init = seq_lens[r] - (t1 - t0) > 0;
-#pragma unroll
-      for (int j = 0; j < KM; ++j) win[j] = j < K - 1 && has_init ? st[j] : 0.f;
       const int q = t1 - t0;
 #pragma unroll
-      for (int j = 0; j < KM; ++j) {
-        if (j >= K - 1) continue;
-        const int p = q - (K - 1) + j;                  // token of this step, or p + K - 1 = j + q of the old window
-        float v = 0.f;
-        if (p >= 0) v = to_f32(x[(int64_t)(t0 + p) * x_stride + c]);
-        else {
+      for (int v = 0; v < V; ++v) {
+        float* st = state + (int64_t)rows[r * rows_stride] * state_stride + (int64_t)(c + v) * (K - 1);
 #pragma unroll
-          for (int i = 0; i < KM; ++i) if (i == j + q) v = win[i];
+        for (int j = 0; j < KM; ++j) win[j][v] = j < K - 1 && has_init ? st[j] : 0.f;
+#pragma unroll
+        for (int j = 0; j < KM; ++j) {
+          if (j >= K - 1) continue;
+          const int p = q - (K - 1) + j;                // token of this step, or place j + q of the old window
+          float nv = 0.f;
+          if (p >= 0) nv = to_f32(x[(int64_t)(t0 + p) * x_stride + c + v]);
+          else {
+#pragma unroll
+            for (int i = 0; i < KM; ++i) if (i == j + q) nv = win[i][v];
+          }
+          st[j] = nv;
         }
-        st[j] = v;
       }
     } else {
 #pragma unroll
-      for (int j = 0; j < KM; ++j) win[j] = j < K - 1 ? to_f32(x[(int64_t)(t - (K - 1) + j) * x_stride + c]) : 0.f;
+      for (int j = 0; j < KM; ++j) {
+        if (j < K - 1) ld_ch<T, V>(x + (int64_t)(t - (K - 1) + j) * x_stride + c, win[j]);
+        else {
+#pragma unroll
+          for (int v = 0; v < V; ++v) win[j][v] = 0.f;
+        }
+      }
     }
 #pragma unroll 4
     for (; t < end; ++t) {
-      const float in = to_f32(x[(int64_t)t * x_stride + c]);
-      float acc = b;
+      float in[V], acc[V];
+      ld_ch<T, V>(x + (int64_t)t * x_stride + c, in);
 #pragma unroll
-      for (int j = 0; j < KM; ++j) acc += wr[j] * (j == K - 1 ? in : win[j]);
-      out[(int64_t)t * out_stride + c] = act ? silu_f(acc) : acc;
+      for (int v = 0; v < V; ++v) {
+        acc[v] = b[v];
 #pragma unroll
-      for (int j = 0; j < KM - 1; ++j) win[j] = j == K - 2 ? in : win[j + 1];
+        for (int j = 0; j < KM; ++j) acc[v] += wr[j][v] * (j == K - 1 ? in[v] : win[j][v]);
+        if (act) acc[v] = silu_f(acc[v]);
+#pragma unroll
+        for (int j = 0; j < KM - 1; ++j) win[j][v] = j == K - 2 ? in[v] : win[j + 1][v];
+      }
+      float* o = out + (int64_t)t * out_stride + c;
+      if constexpr (V == 2) *reinterpret_cast<float2*>(o) = make_float2(acc[0], acc[1]);
+      else o[0] = acc[0];
     }
   }
 }
@@ -197,14 +226,23 @@ EXPORT int vb_causal_conv1d(const void* x, int64_t x_stride, float* out, int64_t
                             int64_t rows_stride, int num_reqs, int n_tok, int C, int K, int act, int dtype, cudaStream_t st) {
   if (num_reqs == 0 || n_tok == 0) return 0;
   if (K < 1 || K > MAX_TAPS) return -1;
-  dim3 grid((n_tok + CONV_TT - 1) / CONV_TT, (C + 127) / 128);
-#define GO(KK) vb_launch(causal_conv1d_kernel<TT, KK>, grid, dim3(128), 0, st, reinterpret_cast<const TT*>(x), x_stride, out, \
+  // tokens per thread: one where most requests bring one (each is a walk through the state of its own), more in prompts
+  const int tile = n_tok <= 2 * num_reqs ? 1 : n_tok <= 16 * num_reqs ? 4 : 16;
+  const bool two = dtype != DT_F32 && C % 2 == 0 && x_stride % 2 == 0 && out_stride % 2 == 0 &&
+                   (reinterpret_cast<uintptr_t>(x) & 3) == 0 && (reinterpret_cast<uintptr_t>(out) & 7) == 0;
+  dim3 grid((n_tok + tile - 1) / tile, (C + (two ? 255 : 127)) / (two ? 256 : 128));
+#define GO(KK)                                                                                                                  \
+  do {                                                                                                                          \
+    if (two) GO2(KK, 2); else GO2(KK, 1);                                                                                       \
+  } while (0)
+#define GO2(KK, VV) vb_launch(causal_conv1d_kernel<TT, KK, VV>, grid, dim3(128), 0, st, reinterpret_cast<const TT*>(x), x_stride, out, \
                          out_stride, reinterpret_cast<const TT*>(w), reinterpret_cast<const TT*>(bias), state, state_stride,   \
-                         qsl, seq_lens, rows, rows_stride, num_reqs, n_tok, C, K, act)
+                         qsl, seq_lens, rows, rows_stride, num_reqs, n_tok, C, K, act, tile)
   DISPATCH_DTYPE(dtype, TT, {
     if (K == 2) GO(2); else if (K == 3) GO(3); else if (K == 4) GO(4); else GO(0);
   });
 #undef GO
+#undef GO2
   return (int)cudaGetLastError();
 }
 
