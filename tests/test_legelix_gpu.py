@@ -175,6 +175,37 @@ def test_gla_scan_over_steps(H, d, dv, rank, dtype):
         assert pool[[0, 2, 5]].isnan().all()
 
 
+@pytest.mark.parametrize("R", [12, 32, 60, 128, 200])
+@pytest.mark.parametrize("ssd", [True, False])
+def test_scan_forms_agree(R, ssd):
+    """Lanes hold few or many rows depending on how much runs at once: sequences alone, all together and token by token."""
+    from vllm_b200 import ops
+    C, dtype, B, n = 40, BF, 48, 21
+    for H in (1, 24):
+        width = H * C + 2 * R if ssd else 2 * H * R + H * C + 4
+        x = _rand(B * n, width, seed=1).to(F32 if ssd else dtype).cuda()
+        dt, A, D, tb = _rand(B * n, H, seed=2).cuda(), _rand(H, seed=3).cuda(), _rand(H, seed=4).cuda(), _rand(H, seed=5).cuda()
+        a2, a2b = _rand(H * R, 4, seed=6).to(dtype).cuda(), (_rand(H * R, seed=7) + 2).to(dtype).cuda()
+
+        def run(pool, rows, q_len, at, pick):
+            md = _md([q_len] * len(rows), [at] * len(rows), _slots([r + 1 for r in rows]))
+            if ssd:
+                return _cu().ssd_scan(x[pick], dt[pick], tb, A, D, pool, 0, md, H, C, 1, R)
+            q, k, v, a1 = x[pick].split([H * R, H * R, H * C, 4], -1)
+            return _cu().gla_scan(q, k, v, a1, a2, a2b, 8.0, 0.3, pool, md, H, R, C)
+
+        def pool():
+            return torch.full((B + 1, H * ops.scan_state_elems(R, C)), float("nan"), device="cuda")
+        everything = torch.arange(B * n).view(B, n)
+        many = run(pool(), range(B), n, 0, everything.flatten()).view(B, n, H * C)
+        one = run(pool(), [7], n, 0, everything[7])
+        _close(one, many[7], 3e-6)
+        p = pool()
+        first = run(p, range(B), n - 3, 0, everything[:, :n - 3].flatten()).view(B, n - 3, H * C)      # and decode from there
+        rest = [run(p, range(B), 1, n - 3 + j, everything[:, n - 3 + j]) for j in range(3)]
+        _close(torch.cat([first, torch.stack(rest, 1)], 1), many, 3e-6)
+
+
 # ------------------------------------------------------------------------------------------------ attention
 def _paged(k, v, lens, page, vt):
     """Scatter per-request keys [n, G, D] and values [n, G, DV] over shuffled pages: (cache, block table)."""

@@ -14,8 +14,8 @@
 // barrier per block of TB tokens, and the loads of the block after next are in flight meanwhile.  A consumer lane holds 2 NP
 // rows x 4 Q columns of S in registers as packed pairs of rows, so that the three products per element are fma.rn.f32x2; the
 // sum over the rows ends in a few shuffles.  In memory a head's
-// state is stored in the order the lanes hold it ([column quad][row in lane][lane][4]): every access is a full 16-byte
-// vector per lane and consecutive across the warp.
+// state is stored in the order the lanes of decode steps hold it: every access of theirs is a full 16-byte vector per lane and
+// consecutive across the warp.
 #include "common.cuh"
 
 namespace lattn {
@@ -38,6 +38,17 @@ VB_DEVICE float4 ld_any4(const void* p, int64_t i, int dt) {      // i and p ali
   if (dt == DT_BF16) { a = unpack2<__nv_bfloat16>(u.x); b = unpack2<__nv_bfloat16>(u.y); }
   else { a = unpack2<__half>(u.x); b = unpack2<__half>(u.y); }
   return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// values of four elements as they lie in memory
+VB_DEVICE float4 values4(uint4 u, int dt) {
+  if (dt == DT_F32) return make_float4(__uint_as_float(u.x), __uint_as_float(u.y), __uint_as_float(u.z), __uint_as_float(u.w));
+  const float2 a = dt == DT_BF16 ? unpack2<__nv_bfloat16>(u.x) : unpack2<__half>(u.x);
+  const float2 b = dt == DT_BF16 ? unpack2<__nv_bfloat16>(u.y) : unpack2<__half>(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+VB_DEVICE uint4 bits4(float4 v) {
+  return make_uint4(__float_as_uint(v.x), __float_as_uint(v.y), __float_as_uint(v.z), __float_as_uint(v.w));
 }
 
 // up to four elements, zeros behind the n-th; not inlined: the path of odd sizes and addresses
@@ -68,7 +79,6 @@ VB_DEVICE float2 unpack(pair_t a) {
 VB_DEVICE void bar_all() { asm volatile("bar.sync 0;" ::: "memory"); }
 
 enum : int { DECAY_GIVEN = 0, DECAY_LOWRANK = 1, DECAY_HEAD = 2 };
-constexpr int PRODUCERS = 4;            // warps
 
 struct ScanParams {
   const void* q; const void* k; const void* v;
@@ -106,14 +116,22 @@ VB_DEVICE void reduce_columns(float* s, int lr, int& at) {
   }
 }
 
-// NP row pairs per lane, L lanes share the rows (capacity 2 NP L rows); a lane holds Q quads of columns, a warp 32 / L times as
-// many.  Wide lanes (Q = 4) read the staged rows from shared memory for more columns at a time, narrow ones make more warps.
-template <int NP, int L, int MODE, int Q, int TB>
+// Place of row r in a column quad's [RP][4] block: the order in which the lanes of the decode form (SL lanes, SNP pairs) hold them.
+template <int SNP, int SL> VB_DEVICE int row_place(int r) {
+  if constexpr (SNP == 1) return (r & 1) * SL + (r >> 1);
+  else return ((r >> 2) / SL * 4 + (r & 3)) * SL + (r >> 2) % SL;
+}
+
+// NP row pairs per lane, L lanes share the rows (capacity 2 NP L rows); a lane holds Q quads of columns.  Decode steps want many
+// warps and whole vectors of state (SNP, SL: the form whose order the state has in memory).  Prompts want many rows per lane:
+// a staged row is then read by few lanes for many columns, and the sum over the lanes is short.
+template <int NP, int L, int SNP, int SL, int MODE, int Q, int TB, int PRODUCERS>
 __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_kernel(const ScanParams p) {
   constexpr int RL = 2 * NP;                 // rows per lane
   constexpr int RP = RL * L;                 // padded rows
   constexpr int LG = 32 / L;
   constexpr int CW = LG * 4 * Q;             // columns per warp
+  constexpr int U = TB >= 4 ? 4 : TB;        // tokens whose sums are reduced together
   constexpr int NT = PRODUCERS * 32;
   extern __shared__ __align__(16) float sm[];
   const int warps = (blockDim.x >> 5) - PRODUCERS;        // consumers
@@ -137,38 +155,61 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
     const int g = h / (p.H / p.groups);
     constexpr int NI = (TB * (RP / 4) + NT - 1) / NT;     // row vectors per thread and operand
     constexpr int NVI = (TB * 32 + NT - 1) / NT;          // value vectors per thread held ahead (of wider tiles the rest is late)
-    float4 rk[NI], rq[NI], ra[NI], rv[NVI];
-    float rdt = 0.f;
+    uint4 rk[NI], rq[NI], rv[NVI];
+    float4 ra[NI];
+    uint32_t rdt = 0;
+    // what the registers hold: operands as they lie in memory (one branch per block, no conversion and no predicate between
+    // the loads, or each of them would be waited for), or fp32 bits where sizes or addresses are odd
+    const bool fast16 = p.vec && p.vec_v && p.k_dt != DT_F32, fast32 = p.vec && p.vec_v && p.k_dt == DT_F32;
+    const int dt = fast16 ? p.k_dt : DT_F32;
     const int cv = CT / 4;
-    auto value4 = [&](int64_t tok, int c) {
-      const int64_t i = tok * p.v_stride + (int64_t)h * C + c;
-      return p.vec_v ? ld_any4(p.v, i, p.v_dt) : ld_some(p.v, i, p.v_dt, C - c);
-    };
+    int vt[NVI], vc[NVI];                                 // token and column of the value vectors
+#pragma unroll
+    for (int i = 0; i < NVI; ++i) { vt[i] = (tid + i * NT) / cv; vc[i] = (tid + i * NT - vt[i] * cv) * 4; }
+    const float neg_a = MODE == DECAY_HEAD ? -expf(p.A_log[h]) : 0.f, db = MODE == DECAY_HEAD ? p.dt_bias[h] : 0.f;
+    auto slow_value = [&](int64_t tok, int c) { return bits4(ld_some(p.v, tok * p.v_stride + (int64_t)h * C + c, p.v_dt, C - c)); };
     auto fetch = [&](int blk) {
       const int tb = min(TB, n - blk * TB);
       const int64_t tok0 = t0 + (int64_t)blk * TB;
-      const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+      auto token = [&](int t) { return tok0 + min(t, tb - 1); };       // the rest reads the last token again
+      if constexpr (MODE == DECAY_HEAD) {
+        const int64_t i = token(tid) * p.dt_stride + h;
+        if (p.dt_dt == DT_F32) rdt = reinterpret_cast<const uint32_t*>(p.dt)[i];
+        else rdt = reinterpret_cast<const uint16_t*>(p.dt)[i];
+      }
+      auto load = [&](auto vec_type) {
+        using V = decltype(vec_type);
+        constexpr int ES = sizeof(V) / 4;
+        auto get = [&](uint4& d, const void* base, int64_t i) {
+          const V u = *reinterpret_cast<const V*>(reinterpret_cast<const char*>(base) + i * ES);
+          d.x = u.x; d.y = u.y;
+          if constexpr (ES == 4) { d.z = u.z; d.w = u.w; }
+        };
 #pragma unroll
-      for (int i = 0; i < NI; ++i) {
-        const int it = tid + i * NT, t = it / (RP / 4), r = (it % (RP / 4)) * 4;
-        rk[i] = rq[i] = ra[i] = zero;
-        if (t >= tb || r >= R) continue;
-        const int64_t ki = (tok0 + t) * p.k_stride + (int64_t)g * R + r, qi = (tok0 + t) * p.q_stride + (int64_t)g * R + r;
-        rk[i] = p.vec ? ld_any4(p.k, ki, p.k_dt) : ld_some(p.k, ki, p.k_dt, R - r);
-        rq[i] = p.vec ? ld_any4(p.q, qi, p.q_dt) : ld_some(p.q, qi, p.q_dt, R - r);
-        if constexpr (MODE == DECAY_GIVEN) {
-          const int64_t ai = ((tok0 + t) * p.H + h) * (int64_t)R + r;
-          ra[i] = p.vec ? *reinterpret_cast<const float4*>(p.alpha + ai) : ld_some(p.alpha, ai, DT_F32, R - r);
+        for (int i = 0; i < NI; ++i) {
+          const int it = tid + i * NT, r = min((it % (RP / 4)) * 4, R - 4);
+          const int64_t tok = token(it / (RP / 4));
+          get(rk[i], p.k, tok * p.k_stride + (int64_t)g * R + r);
+          get(rq[i], p.q, tok * p.q_stride + (int64_t)g * R + r);
+          if constexpr (MODE == DECAY_GIVEN) ra[i] = *reinterpret_cast<const float4*>(p.alpha + (tok * p.H + h) * (int64_t)R + r);
         }
-      }
 #pragma unroll
-      for (int i = 0; i < NVI; ++i) {
-        const int it = tid + i * NT, t = it / cv, c = c0 + (it - t * cv) * 4;
-        rv[i] = zero;
-        if (t < tb && c < C) rv[i] = value4(tok0 + t, c);
+        for (int i = 0; i < NVI; ++i) get(rv[i], p.v, token(vt[i]) * p.v_stride + (int64_t)h * C + min(c0 + vc[i], C - 4));
+      };
+      if (fast16) load(uint2{});
+      else if (fast32) load(uint4{});
+      else {
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          const int it = tid + i * NT, r = (it % (RP / 4)) * 4;
+          const int64_t tok = token(it / (RP / 4));
+          rk[i] = bits4(ld_some(p.k, tok * p.k_stride + (int64_t)g * R + r, p.k_dt, R - r));
+          rq[i] = bits4(ld_some(p.q, tok * p.q_stride + (int64_t)g * R + r, p.q_dt, R - r));
+          if constexpr (MODE == DECAY_GIVEN) ra[i] = ld_some(p.alpha, (tok * p.H + h) * (int64_t)R + r, DT_F32, R - r);
+        }
+#pragma unroll
+        for (int i = 0; i < NVI; ++i) rv[i] = slow_value(token(vt[i]), c0 + vc[i]);
       }
-      if constexpr (MODE == DECAY_HEAD)
-        if (tid < tb) rdt = ld_any(p.dt, (tok0 + tid) * p.dt_stride + h, p.dt_dt);
     };
     auto store = [&](int blk) {
       float* b = bufs + (blk & 1) * TB * per_tok;
@@ -176,10 +217,11 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
       const int64_t tok0 = t0 + (int64_t)blk * TB;
       if constexpr (MODE == DECAY_HEAD) {
         if (tid < tb) {
-          const float dt = fminf(fmaxf(softplus_f(rdt + p.dt_bias[h]), p.dt_min), p.dt_max);
+          const float raw = p.dt_dt == DT_F32 ? __uint_as_float(rdt) : p.dt_dt == DT_BF16 ? unpack2<__nv_bfloat16>(rdt).x : unpack2<__half>(rdt).x;
+          const float step = fminf(fmaxf(softplus_f(raw + db), p.dt_min), p.dt_max);
           float* d = b + tid * per_tok + 2 * RP + 2 * CT;
-          d[0] = d[1] = expf(-expf(p.A_log[h]) * dt);
-          d[2] = dt;
+          d[0] = d[1] = expf(neg_a * step);
+          d[2] = step;
         }
         asm volatile("bar.sync 1, %0;" ::"n"(NT) : "memory");
       }
@@ -189,10 +231,11 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
         if (t >= tb) continue;
         float* row = b + t * per_tok;
         const float ks = MODE == DECAY_HEAD ? row[2 * RP + 2 * CT + 2] : 1.f;
-        *reinterpret_cast<float4*>(row + r) = make_float4(rk[i].x * ks, rk[i].y * ks, rk[i].z * ks, rk[i].w * ks);
-        *reinterpret_cast<float4*>(row + RP + r) =
-            make_float4(rq[i].x * p.q_scale, rq[i].y * p.q_scale, rq[i].z * p.q_scale, rq[i].w * p.q_scale);
-        if constexpr (MODE == DECAY_GIVEN) *reinterpret_cast<float4*>(row + 2 * RP + 2 * CT + 4 + r) = ra[i];
+        const bool in = r < R;
+        const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), kv = in ? values4(rk[i], dt) : zero, qv = in ? values4(rq[i], dt) : zero;
+        *reinterpret_cast<float4*>(row + r) = make_float4(kv.x * ks, kv.y * ks, kv.z * ks, kv.w * ks);
+        *reinterpret_cast<float4*>(row + RP + r) = make_float4(qv.x * p.q_scale, qv.y * p.q_scale, qv.z * p.q_scale, qv.w * p.q_scale);
+        if constexpr (MODE == DECAY_GIVEN) *reinterpret_cast<float4*>(row + 2 * RP + 2 * CT + 4 + r) = in ? ra[i] : zero;
       }
       if constexpr (MODE == DECAY_LOWRANK) {
         for (int r = tid; r < RP; r += NT) {
@@ -223,12 +266,11 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
       };
 #pragma unroll
       for (int i = 0; i < NVI; ++i) {
-        const int it = tid + i * NT, t = it / cv, c = (it - t * cv) * 4;
-        if (t < tb) put(t, c, rv[i]);
+        if (vt[i] < tb) put(vt[i], vc[i], values4(rv[i], dt));
       }
       for (int it = tid + NVI * NT; it < tb * cv; it += NT) {
         const int t = it / cv, c = (it - t * cv) * 4;
-        put(t, c, c0 + c < C ? value4(tok0 + t, c0 + c) : make_float4(0.f, 0.f, 0.f, 0.f));
+        put(t, c, values4(slow_value(tok0 + t, c0 + c), DT_F32));
       }
     };
     auto flush = [&](int blk) {
@@ -267,8 +309,10 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
   // ================= consumers
   const int lr = lane % L, lg = lane / L;
   auto quad_of = [&](int j) { return (warp * Q + j) * LG + lg; };     // quad of columns inside the tile
+  auto row_of = [&](int i) { return NP == 1 ? lr * 2 : ((i >> 1) * L + lr) * 4 + (i & 1) * 2; };      // first row of pair i
   const bool has_init = p.seq_lens[req] > n;
-  float* st = p.state + (int64_t)p.rows[req * p.rows_stride] * p.state_stride + p.state_off + (int64_t)h * p.head_elems + lr * 4;
+  float* st = p.state + (int64_t)p.rows[req * p.rows_stride] * p.state_stride + p.state_off + (int64_t)h * p.head_elems;
+  auto at_row = [&](int64_t cq, int r) { return st + (cq * RP + row_place<SNP, SL>(r)) * 4; };
   pair_t S[Q][4][NP];
 #pragma unroll
   for (int j = 0; j < Q; ++j) {
@@ -277,8 +321,8 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
     for (int i = 0; i < NP; ++i) {
       float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
       if (has_init && cq * 4 < C) {
-        x = *reinterpret_cast<const float4*>(st + (cq * RP + (2 * i) * L) * 4);
-        y = *reinterpret_cast<const float4*>(st + (cq * RP + (2 * i + 1) * L) * 4);
+        x = *reinterpret_cast<const float4*>(at_row(cq, row_of(i)));
+        y = *reinterpret_cast<const float4*>(at_row(cq, row_of(i) + 1));
       }
       S[j][0][i] = pack(x.x, y.x); S[j][1][i] = pack(x.y, y.y); S[j][2][i] = pack(x.z, y.z); S[j][3][i] = pack(x.w, y.w);
     }
@@ -289,56 +333,75 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
     const float* b = bufs + (blk & 1) * TB * per_tok;
     float* o = obuf + (blk & 1) * TB * CT;
     const int tb = min(TB, n - blk * TB);
-#pragma unroll(Q == 1 ? 2 : 1)
-    for (int t = 0; t < tb; ++t) {
-      const float* row = b + t * per_tok;
-      pair_t kk[NP], qq[NP], aa[NP];
-      auto ld_rows = [&](const float* src, pair_t (&dst)[NP]) {
-        if constexpr (NP == 1) dst[0] = *reinterpret_cast<const pair_t*>(src + lr * RL);
-        else {
+    // U tokens at a time: their sums are reduced together (fewer shuffles, and none of them waits for the one before)
+    for (int tg = 0; tg < tb; tg += U) {
+      float s[U * 4 * Q];
 #pragma unroll
-          for (int i = 0; i < NP; i += 2) {
-            const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(src + lr * RL + 2 * i);
-            dst[i] = u.x; dst[i + 1] = u.y;
-          }
+      for (int u = 0; u < U; ++u) {
+        if (tg + u >= tb) {                      // behind the last token: nothing may touch the state
+#pragma unroll
+          for (int i = 0; i < 4 * Q; ++i) s[u * 4 * Q + i] = 0.f;
+          continue;
         }
-      };
-      ld_rows(row, kk);
-      ld_rows(row + RP, qq);
-      if constexpr (MODE == DECAY_HEAD) {
-        const pair_t a = *reinterpret_cast<const pair_t*>(row + 2 * RP + 2 * CT);
-#pragma unroll
-        for (int i = 0; i < NP; ++i) aa[i] = a;
-      } else {
-        ld_rows(row + 2 * RP + 2 * CT + 4, aa);
-      }
-      float s[4 * Q];
-#pragma unroll
-      for (int j = 0; j < Q; ++j) {
-        const float* vp = row + 2 * RP + quad_of(j) * 8;
-        const ulonglong2 v01 = *reinterpret_cast<const ulonglong2*>(vp), v23 = *reinterpret_cast<const ulonglong2*>(vp + 4);
-        const pair_t vv[4] = {v01.x, v01.y, v23.x, v23.y};
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          pair_t acc;
-#pragma unroll
-          for (int i = 0; i < NP; ++i) {
-            S[j][c][i] = fma2(aa[i], S[j][c][i], mul2(kk[i], vv[c]));
-            acc = i == 0 ? mul2(S[j][c][i], qq[i]) : fma2(S[j][c][i], qq[i], acc);
+        const float* row = b + (tg + u) * per_tok;
+        constexpr int M = NP == 1 ? 1 : NP / 2, P = NP == 1 ? 1 : 2;      // vectors of rows, pairs in one
+        auto ld_rows = [&](const float* src, pair_t (&dst)[P]) {
+          if constexpr (NP == 1) dst[0] = *reinterpret_cast<const pair_t*>(src);
+          else {
+            const ulonglong2 w = *reinterpret_cast<const ulonglong2*>(src);
+            dst[0] = w.x; dst[P - 1] = w.y;
           }
-          const float2 f = unpack(acc);
-          s[j * 4 + c] = f.x + f.y;
+        };
+        pair_t vv[Q][4], acc[Q][4];
+#pragma unroll
+        for (int j = 0; j < Q; ++j) {
+          const float* vp = row + 2 * RP + quad_of(j) * 8;
+          const ulonglong2 v01 = *reinterpret_cast<const ulonglong2*>(vp), v23 = *reinterpret_cast<const ulonglong2*>(vp + 4);
+          vv[j][0] = v01.x; vv[j][1] = v01.y; vv[j][2] = v23.x; vv[j][3] = v23.y;
         }
+        pair_t ah = 0;
+        if constexpr (MODE == DECAY_HEAD) ah = *reinterpret_cast<const pair_t*>(row + 2 * RP + 2 * CT);
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          pair_t kk[P], qq[P], aa[P];
+          const int r = row_of(2 * m);
+          ld_rows(row + r, kk);
+          ld_rows(row + RP + r, qq);
+          if constexpr (MODE == DECAY_HEAD) {
+#pragma unroll
+            for (int i = 0; i < P; ++i) aa[i] = ah;
+          } else {
+            ld_rows(row + 2 * RP + 2 * CT + 4 + r, aa);
+          }
+#pragma unroll
+          for (int j = 0; j < Q; ++j)
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+#pragma unroll
+              for (int i = 0; i < P; ++i) {
+                pair_t& S1 = S[j][c][P * m + i];
+                S1 = fma2(aa[i], S1, mul2(kk[i], vv[j][c]));
+                acc[j][c] = m + i == 0 ? mul2(S1, qq[i]) : fma2(S1, qq[i], acc[j][c]);
+              }
+        }
+#pragma unroll
+        for (int j = 0; j < Q; ++j)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            const float2 f = unpack(acc[j][c]);
+            s[(u * Q + j) * 4 + c] = f.x + f.y;
+          }
       }
-      // 4 Q sums over L lanes: halve the columns while there are two or more, then add the rest up
+      // the sums over L lanes: halve their number while there are two or more, then add the rest up
+      constexpr int N = 4 * Q * U;
       int at = 0;
-      reduce_columns<4 * Q, L / 2>(s, lr, at);
-      constexpr int LEFT = 4 * Q > L ? 4 * Q / L : 1, SAME = L > 4 * Q ? L / (4 * Q) : 1;   // sums per lane, lanes with the same
+      reduce_columns<N, L / 2>(s, lr, at);
+      constexpr int LEFT = N > L ? N / L : 1, SAME = L > N ? L / N : 1;      // sums per lane, lanes with the same
       if ((lr & (SAME - 1)) == 0) {
 #pragma unroll
         for (int i = 0; i < LEFT; ++i) {
-          const int c = quad_of((at + i) >> 2) * 4 + ((at + i) & 3);
-          o[t * CT + c] = MODE == DECAY_HEAD ? s[i] + dskip * row[2 * RP + 2 * c] : s[i];
+          const int x = at + i, t = tg + x / (4 * Q), c = quad_of(x / 4 % Q) * 4 + (x & 3);
+          if (t < tb) o[t * CT + c] = MODE == DECAY_HEAD ? s[i] + dskip * b[t * per_tok + 2 * RP + 2 * c] : s[i];
         }
       }
     }
@@ -351,8 +414,8 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
 #pragma unroll
     for (int i = 0; i < NP; ++i) {
       const float2 a = unpack(S[j][0][i]), bb = unpack(S[j][1][i]), c = unpack(S[j][2][i]), d = unpack(S[j][3][i]);
-      *reinterpret_cast<float4*>(st + (cq * RP + (2 * i) * L) * 4) = make_float4(a.x, bb.x, c.x, d.x);
-      *reinterpret_cast<float4*>(st + (cq * RP + (2 * i + 1) * L) * 4) = make_float4(a.y, bb.y, c.y, d.y);
+      *reinterpret_cast<float4*>(at_row(cq, row_of(i))) = make_float4(a.x, bb.x, c.x, d.x);
+      *reinterpret_cast<float4*>(at_row(cq, row_of(i) + 1)) = make_float4(a.y, bb.y, c.y, d.y);
     }
   }
 }
@@ -462,54 +525,61 @@ __global__ void __launch_bounds__(1024) gated_norm_kernel(const float* __restric
   }
 }
 
-template <int NP, int L, int Q, int TB>
-int scan_launch(ScanParams& p, int mode, int num_reqs, int warps, cudaStream_t st) {
+template <int NP, int L, int SNP, int SL, int MODE, int Q, int TB, int PRODUCERS>
+int scan_launch(ScanParams& p, int num_reqs, int warps, cudaStream_t st) {
+  static_assert(NP * L == SNP * SL, "one state layout");
   constexpr int RP = 2 * NP * L, CW = 32 / L * 4 * Q;
-  const int CT = warps * CW, per_tok = (mode == DECAY_HEAD ? 2 : 3) * RP + 2 * CT + 4;
+  const int CT = warps * CW, per_tok = (MODE == DECAY_HEAD ? 2 : 3) * RP + 2 * CT + 4;
   const size_t smem = (size_t)(2 * TB * (per_tok + CT)) * 4;
-  dim3 grid((p.C + CT - 1) / CT, p.H, num_reqs), block(32 * (warps + PRODUCERS));
-#define GO(M)                                                                                             \
-  do {                                                                                                    \
-    auto kern = state_scan_kernel<NP, L, M, Q, TB>;                                                       \
-    static bool set = false;                                                                              \
-    if (!set) { cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); set = true; } \
-    vb_launch(kern, grid, block, smem, st, p);                                                            \
-  } while (0)
   if (smem > 200 * 1024) return -4;
-  if (mode == DECAY_HEAD) GO(DECAY_HEAD);
-  else if (mode == DECAY_GIVEN) GO(DECAY_GIVEN);
-  else if constexpr (TB == 1) GO(DECAY_LOWRANK);
-  else return -5;                                  // prompts bring their decays
-#undef GO
+  auto kern = state_scan_kernel<NP, L, SNP, SL, MODE, Q, TB, PRODUCERS>;
+  static bool set = false;
+  if (!set) { cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); set = true; }
+  vb_launch(kern, dim3((p.C + CT - 1) / CT, p.H, num_reqs), dim3(32 * (warps + PRODUCERS)), smem, st, p);
   return (int)cudaGetLastError();
 }
 
 constexpr int SMS = 148;
-template <int NP, int L>
+// SNP, SL: decode form; NP1, L1 and NP2, L2: prompt forms, few and many rows per lane
+template <int SNP, int SL, int NP1, int L1, int NP2, int L2>
 int scan_shape(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t st) {
-  constexpr int LG = 32 / L, QMAX = NP <= 2 ? 4 : NP == 4 ? 2 : 1;      // state registers per lane: 8 NP Q
-  const int64_t quads = (int64_t)num_reqs * p.H * ((p.C + 3) / 4);      // of the whole launch
   const int head_quads = (p.C + 3) / 4;
-  auto tile_warps = [&](int q) {                                        // warps that a CTA needs for one head's columns, at most 8
+  const int64_t quads = (int64_t)num_reqs * p.H * head_quads;           // of the whole launch
+  // warps per CTA: at most 8, no more than one head's columns need (``per``: quads of a warp), fewer while SMs would stay empty
+  auto cta_warps = [&](int per, int64_t ctas) {
     int w = 1;
-    while (w < 8 && w * q * LG < head_quads) w *= 2;
+    while (w < 8 && w * per < head_quads) w *= 2;
+    while (w > 1 && quads / (w * per) < ctas) w /= 2;
     return w;
   };
   if (max_len == 1) {
-    // decode: the state's bytes count; two quads per lane keep enough of them in flight where there are many states
-    if (QMAX >= 2 && quads / (2 * LG) >= 8 * SMS * 3) return scan_launch<NP, L, QMAX >= 2 ? 2 : 1, 1>(p, mode, num_reqs, tile_warps(2), st);
-    int w = tile_warps(1);
-    while (w > 1 && quads / (w * LG) < SMS) w /= 2;
-    return scan_launch<NP, L, 1, 1>(p, mode, num_reqs, w, st);
+    // the state's bytes count; two quads per lane keep more of them in flight where there are many states
+    constexpr int Q2 = SNP <= 4 ? 2 : 1;
+    const bool many = quads / (2 * (32 / SL)) >= 8 * SMS * 3;
+    const int w = many ? cta_warps(Q2 * (32 / SL), 1) : cta_warps(32 / SL, SMS);
+#define DECODE(M) (many ? scan_launch<SNP, SL, SNP, SL, M, Q2, 1, 4>(p, num_reqs, w, st) : scan_launch<SNP, SL, SNP, SL, M, 1, 1, 4>(p, num_reqs, w, st))
+    if (mode == DECAY_HEAD) return DECODE(DECAY_HEAD);
+    if (mode == DECAY_GIVEN) return DECODE(DECAY_GIVEN);
+    return DECODE(DECAY_LOWRANK);
+#undef DECODE
   }
-  // prompts: the widest lanes that still give every scheduler of the GPU a warp, then CTAs small enough to fill the SMs
-  int q = QMAX;
-  if (quads / (q * LG) < SMS * 4) q = 1;
-  int w = tile_warps(q);
-  while (w > 1 && quads / (w * q * LG) < SMS * 3 / 4) w /= 2;
-  constexpr int TB = NP <= 4 ? 16 : 8;
-  if (QMAX > 1 && q == QMAX) return scan_launch<NP, L, QMAX, TB>(p, mode, num_reqs, w, st);
-  return scan_launch<NP, L, 1, TB>(p, mode, num_reqs, w, st);
+  if (mode == DECAY_LOWRANK) return -5;                                 // prompts bring their decays
+  constexpr int TB = 8;
+  constexpr int64_t CTAS = SMS * 3 / 4, WARPS = SMS * 3;                // measured: where the next form begins to win
+  const bool head = mode == DECAY_HEAD;
+  if (quads / (32 / L2) >= WARPS) {
+    const int w = cta_warps(32 / L2, CTAS);
+    return head ? scan_launch<NP2, L2, SNP, SL, DECAY_HEAD, 1, TB, 2>(p, num_reqs, w, st)      // two CTAs fit on an SM
+                : scan_launch<NP2, L2, SNP, SL, DECAY_GIVEN, 1, TB, 4>(p, num_reqs, w, st);
+  }
+  if (quads / (32 / L1) >= WARPS) {
+    const int w = cta_warps(32 / L1, CTAS);
+    return head ? scan_launch<NP1, L1, SNP, SL, DECAY_HEAD, 1, TB, 4>(p, num_reqs, w, st)
+                : scan_launch<NP1, L1, SNP, SL, DECAY_GIVEN, 1, TB, 4>(p, num_reqs, w, st);
+  }
+  const int w = cta_warps(32 / SL, CTAS);
+  return head ? scan_launch<SNP, SL, SNP, SL, DECAY_HEAD, 1, TB, 4>(p, num_reqs, w, st)
+              : scan_launch<SNP, SL, SNP, SL, DECAY_GIVEN, 1, TB, 4>(p, num_reqs, w, st);
 }
 
 inline bool al(const void* p, int64_t n) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) % (size_t)n) == 0; }
@@ -528,12 +598,12 @@ int scan(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t st) {
   if (p.R > 512) return -3;
   p.head_elems = (int64_t)((p.C + 3) / 4) * 4 * rp;
   switch (rp) {
-    case 16: return scan_shape<1, 8>(p, mode, num_reqs, max_len, st);
-    case 32: return scan_shape<1, 16>(p, mode, num_reqs, max_len, st);
-    case 64: return scan_shape<2, 16>(p, mode, num_reqs, max_len, st);
-    case 128: return scan_shape<2, 32>(p, mode, num_reqs, max_len, st);
-    case 256: return scan_shape<4, 32>(p, mode, num_reqs, max_len, st);
-    default: return scan_shape<8, 32>(p, mode, num_reqs, max_len, st);
+    case 16: return scan_shape<1, 8, 2, 4, 4, 2>(p, mode, num_reqs, max_len, st);
+    case 32: return scan_shape<1, 16, 2, 8, 4, 4>(p, mode, num_reqs, max_len, st);
+    case 64: return scan_shape<2, 16, 4, 8, 8, 4>(p, mode, num_reqs, max_len, st);
+    case 128: return scan_shape<2, 32, 4, 16, 8, 8>(p, mode, num_reqs, max_len, st);
+    case 256: return scan_shape<4, 32, 8, 16, 8, 16>(p, mode, num_reqs, max_len, st);
+    default: return scan_shape<8, 32, 8, 32, 8, 32>(p, mode, num_reqs, max_len, st);
   }
 }
 
