@@ -72,3 +72,22 @@ if which in ("latent", "all"):
     up, down = (torch.randn(*s, device="cuda", dtype=dt) * 0.02 for s in ((32, 1408, 2048), (32, 2048, 1408)))
     wt, ids = _routing(4096, 32, 6)
     rep(lambda: moe.expert_rows_plain(x, up, down, ids, "relu2", None))
+if which in ("scan", "all"):
+    # Legelix: scans of prompts (1024 tokens each) and of a decode batch, at the sizes of a 2048-wide model
+    from vllm_b200.forward_context import AttentionMetadata
+    from vllm_b200.ops import scan_state_elems
+    MH, GH, i32 = 64, 8, dict(dtype=torch.int32, device="cuda")
+    for n, q in ((4, 1024), (64, 1)):
+        T = n * q
+        md = AttentionMetadata(num_reqs=n, num_actual_tokens=T, max_query_len=q, max_seq_len=q, query_start_loc=torch.arange(0, T + 1, q, **i32),
+                               seq_lens=torch.full((n,), q + (q == 1), **i32), block_table=(torch.arange(n, **i32) + 1).view(-1, 1),
+                               slot_mapping=None, decode_only=q == 1)
+        xa, dts = torch.randn(T, MH * 64 + 256, device="cuda") * 0.3, torch.randn(T, MH, device="cuda").to(dt)
+        A, D, b = [torch.randn(MH, device="cuda") * 0.3 for _ in range(3)]
+        pool = torch.zeros(n + 1, MH * scan_state_elems(128, 64), device="cuda")
+        rep(lambda: cu.ssd_scan(xa, dts, b, A, D, pool, 0, md, MH, 64, 1, 128))
+        x = (torch.randn(T, GH * (128 + 128 + 256) + 16, device="cuda") * 0.3).to(dt)
+        qq, kk, vv, a1 = x.split([GH * 128, GH * 128, GH * 256, 16], -1)
+        a2, a2b = torch.randn(GH * 128, 16, device="cuda").to(dt), torch.randn(GH * 128, device="cuda").to(dt)
+        pool2 = torch.zeros(n + 1, GH * scan_state_elems(128, 256), device="cuda")
+        rep(lambda: cu.gla_scan(qq, kk, vv, a1, a2, a2b, 16.0, 0.09, pool2, md, GH, 128, 256))

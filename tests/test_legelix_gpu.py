@@ -229,17 +229,18 @@ def _paged(k, v, lens, page, vt):
     return cache.cuda(), table.cuda()
 
 
-SHAPES = [(6, 2, 48, 48), (4, 4, 16, 40), (5, 1, 40, 16), (3, 3, 7, 9), (8, 2, 128, 128), (12, 4, 80, 80), (2, 1, 192, 160), (6, 2, 128, 128)]
+SHAPES = [(6, 2, 48, 48), (4, 4, 16, 40), (5, 1, 40, 16), (3, 3, 7, 9), (8, 2, 128, 128), (12, 4, 80, 80), (2, 1, 192, 160), (6, 2, 128, 128), (8, 2, 64, 64), (4, 4, 32, 32),
+          (6, 2, 64, 64)]
 
 
 @pytest.mark.parametrize("H,G,D,DV", SHAPES)
 @pytest.mark.parametrize("dtype", [BF, F32])
-@pytest.mark.parametrize("sinks", [True, False])
-def test_chunk_local_attention(H, G, D, DV, dtype, sinks):
+@pytest.mark.parametrize("sinks,factor", [(True, 0.6), (False, 0.6), (True, 1.0)])
+def test_chunk_local_attention(H, G, D, DV, dtype, sinks, factor):
     """Portions that start anywhere, chunks of several sizes, one-token steps, pages in any order."""
     from vllm_b200 import ops
     vt = dtype == BF and _cu().tc_attention_ok(D, DV, H // G)
-    scale, factor = 1.3 * D ** -0.5, 0.6
+    scale = 1.3 * D ** -0.5
     for size, q_lens, ctx in ((50, [9, 70, 1, 2], [41, 0, 49, 50]), (64, [1, 1, 1, 1], [63, 64, 0, 200]), (1000, [200, 3], [3, 130]),
                               (1, [4, 1], [0, 9]), (130, [1, 1], [259, 260]), (200, [150], [120])):
         lens = [c + q for c, q in zip(ctx, q_lens)]

@@ -156,8 +156,13 @@ class LegelixForCausalLM(LlamaForCausalLM):
                 continue
             a = spec["mixer"]["left"]
             out |= {"ssm", "qknorm_rope"}
-            tc = half and ops.cuda_ops().tc_attention_ok(a["dim"], a["vdim"], a["heads"] // a["kv_heads"])
-            out |= {"attention_tc", "attention_tc_decode"} if tc else {"attention_any"}
+            cu, d, dv, group = ops.cuda_ops(), a["dim"], a["vdim"], a["heads"] // a["kv_heads"]
+            if half and cu.tc_attention_ok(d, dv, group):
+                out |= {"attention_tc", "attention_tc_decode"}
+            elif spec["mixer"]["left_scale"] == 1.0 and cu._simt_attention_ok(d, dv, 64, group, dtype):
+                out.add("attention_simt")
+            else:
+                out.add("attention_any")
         return sorted(out)
 
     # checkpoint tensor (behind "l<i>.") → (parameter, shard)
