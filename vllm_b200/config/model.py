@@ -778,7 +778,35 @@ def legelix_config(*, vocab: int, width: int, layers: list[str], heads: int, kv_
     return dict(dict(architecture="Legelix", vocab=vocab, width=width, layers=out, norm=dict(eps=1e-6), residual_mult=1.0), **kw)
 
 
+def kopadra_config(*, vocab: int, width: int, layers: list[str], heads: int, kv_heads: int, dim: int, mem_heads: int, mem_dim: int,
+                   mem_vdim: int, ff: int, expert_ff: int, experts: int, identity: int, top: int, groups: int, keep: int, shared_ff: int,
+                   **kw) -> dict[str, Any]:
+    """A Kopadra config.json.  A layer is "mixer+feed-forward": "attention", "reuse" (attention over the keys of the "attention" before it)
+    or "mlstm", then "dense" or "moe"; layers of a kind are alike."""
+    rot = dict(base=500000.0, dims=dim, scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0))
+    attn = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, rot=rot)
+    mlps = dict(dense=dict(kind="dense", ff=ff),
+                moe=dict(kind="moe", expert=dict(ff=expert_ff), shared=dict(ff=shared_ff),
+                         router=dict(experts=experts, identity=identity, top=top, scale=1.0, groups=dict(count=groups, keep=keep))))
+    out, owner = [], None
+    for i, kind in enumerate(layers):
+        mixer, mlp = kind.split("+")
+        if mixer == "mlstm":
+            m = dict(heads=mem_heads, dim=mem_dim, vdim=mem_vdim, gate_cap=15.0)
+        else:
+            m = dict(attn, **(dict(kv_from=owner) if mixer == "reuse" else {}))
+            owner = i if mixer == "attention" else owner
+        out.append(dict(type="mlstm" if mixer == "mlstm" else "attention", mixer=copy.deepcopy(m), mlp=copy.deepcopy(mlps[mlp])))
+    return dict(dict(architecture="Kopadra", vocab=vocab, width=width, layers=out, norm=dict(eps=1e-6), logit_softcap=30.0), **kw)
+
+
 PRESETS.update({
+    "kopadra-tiny": kopadra_config(vocab=320, width=80, layers=["attention+dense", "mlstm+moe", "reuse+moe"], heads=4, kv_heads=2, dim=24,
+                                   mem_heads=2, mem_dim=20, mem_vdim=28, ff=120, expert_ff=40, experts=6, identity=3, top=2, groups=3, keep=2,
+                                   shared_ff=56, max_position_embeddings=1024, torch_dtype="float32"),
+    "kopadra-small": kopadra_config(vocab=4096, width=1024, layers=["attention+dense", "mlstm+moe", "attention+moe", "reuse+dense"], heads=8,
+                                    kv_heads=2, dim=128, mem_heads=4, mem_dim=128, mem_vdim=256, ff=2816, expert_ff=512, experts=16,
+                                    identity=8, top=4, groups=4, keep=2, shared_ff=512, max_position_embeddings=8192, torch_dtype="bfloat16"),
     "legelix-tiny": legelix_config(vocab=320, width=80, layers=["gla", "parallel", "gla"], heads=4, kv_heads=2, dim=24, chunk=100, ssm_heads=4,
                                    ssm_dim=16, state=24, groups=2, conv=4, gla_heads=2, gla_dim=20, gla_vdim=28, ff=120,
                                    max_position_embeddings=1024, torch_dtype="float32"),
@@ -812,8 +840,8 @@ def get_preset_hf_config(name: str) -> Optional[dict[str, Any]]:
     return copy.deepcopy(cfg) if cfg is not None else None
 
 
-# positions of a Legelix model where max_model_len is not given (the design itself sets no limit)
-LEGELIX_MAX_LEN = 131072
+# positions of a model whose design sets no limit, where max_model_len is not given
+OPEN_MAX_LEN = 131072
 # rank of a gated-linear layer's decay where no checkpoint gives it (random weights)
 LEGELIX_DECAY_RANK = 16
 
@@ -878,10 +906,39 @@ def _flatten_nested_config(c: dict) -> None:
         c.setdefault("vocab_size", c["vocab"])
         c.setdefault("hidden_size", c["width"])
         c.setdefault("num_hidden_layers", len(layers))
-        c.setdefault("max_position_embeddings", LEGELIX_MAX_LEN)
+        c.setdefault("max_position_embeddings", OPEN_MAX_LEN)
         c.setdefault("num_attention_heads", max((a["heads"] for a in left), default=1))
         c.setdefault("num_key_value_heads", max((a["kv_heads"] for a in left), default=1))
         c.setdefault("head_dim", max((max(a["dim"], a["vdim"]) for a in left), default=128))
+    if c.get("architecture") == "Kopadra":
+        layers = c["layers"]
+        attn = [l["mixer"] for l in layers if l["type"] == "attention"]
+        moes = [l["mlp"]["router"] for l in layers if l.get("mlp") and l["mlp"].get("kind") == "moe"]
+        for i, l in enumerate(layers):
+            m = l["mixer"]
+            if l["type"] != "attention":
+                continue
+            rot, j = m.get("rot"), m.get("kv_from")
+            if m["heads"] % m["kv_heads"]:
+                raise ValueError(f"layer {i}: heads must divide into kv_heads")
+            if rot and (rot["dims"] % 2 or rot["dims"] > m["dim"]):
+                raise ValueError(f"layer {i}: rotated dimensions must be even and within the head")
+            if j is not None and not (0 <= j < i and layers[j]["type"] == "attention" and layers[j]["mixer"].get("kv_from") is None
+                                      and all(layers[j]["mixer"][k] == m[k] for k in ("heads", "kv_heads", "dim", "vdim"))):
+                raise ValueError(f"layer {i}: kv_from {j} must name an earlier attention layer with keys of its own and the same head shapes")
+        c.setdefault("architectures", ["KopadraForCausalLM"])
+        c.setdefault("model_type", "kopadra")
+        c.setdefault("vocab_size", c["vocab"])
+        c.setdefault("hidden_size", c["width"])
+        c.setdefault("num_hidden_layers", len(layers))
+        c.setdefault("max_position_embeddings", OPEN_MAX_LEN)
+        c.setdefault("num_attention_heads", max((a["heads"] for a in attn), default=1))
+        c.setdefault("num_key_value_heads", max((a["kv_heads"] for a in attn), default=1))
+        c.setdefault("head_dim", max((max(a["dim"], a["vdim"]) for a in attn), default=128))
+        c.setdefault("final_logit_softcapping", c.get("logit_softcap"))
+        if moes:
+            c.setdefault("num_experts", max(r["experts"] for r in moes))
+            c.setdefault("num_experts_per_tok", max(r["top"] for r in moes))
     if c.get("model_type") == "dbrx":
         a, f = c.get("attn_config") or {}, c.get("ffn_config") or {}
         c.setdefault("hidden_size", c.get("d_model"))

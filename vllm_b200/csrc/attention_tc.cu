@@ -288,6 +288,7 @@ fmha_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ 
       const uint32_t t_s = tmem_s0 + sb * 128 + t_lane;
       const int tile_pos = (tile_lo + j) * TILE_N;
       mbar_wait(&s_full[sb], (j >> 1) & 1);
+      __syncwarp();
       tc_fence_after();
       // valid column range for this row: [lo, hi)
       int hi = min(kv_end, p.causal ? qpos + 1 : kv_end) - tile_pos;
@@ -311,14 +312,14 @@ fmha_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ 
       float alpha = 1.f;
       bool rescale = false;
       if (mx > m_used + 8.f || (m_used == -INFINITY && mx > -INFINITY)) {
-        alpha = (m_used == -INFINITY) ? 0.f : ex2(m_used - mx);
-        rescale = (m_used != -INFINITY);
+        rescale = m_used != -INFINITY;
+        if (rescale) alpha = ex2(m_used - mx);
         m_used = mx;
       }
       const float m_ref = (m_used == -INFINITY) ? 0.f : m_used;
       // P (single smem buffer) and O may only be touched once PV_{j-1} has retired
-      if (j > 0) { mbar_wait(pv_done, (j - 1) & 1); tc_fence_after(); }
-      if (rescale) {
+      if (j > 0) { mbar_wait(pv_done, (j - 1) & 1); __syncwarp(); tc_fence_after(); }
+      if (__any_sync(0xffffffffu, rescale)) {          // TMEM accesses are the whole warp's: rows that keep their maximum have alpha 1
         l_run *= alpha;
 #pragma unroll
         for (int c = 0; c < D; c += 32) {
@@ -363,6 +364,7 @@ fmha_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ 
     }
     // ---- epilogue
     mbar_wait(pv_done, (n_tiles - 1) & 1);
+    __syncwarp();
     tc_fence_after();
     const int64_t tok = q0 + tok0 + tq;
     const int hq = h * p.G + g;

@@ -2,12 +2,16 @@
 //
 //   S_t = diag(a_t) S_{t-1} + k_t v_t^T,    o_t = S_t^T q_t        S [R, C] fp32 per (request, head)
 //
-// covers gated linear attention (a decay per key channel: R = key width, C = value width) and the Mamba-2 state-space scan
-// (one decay exp(-exp(A_log) dt) per head; k = dt B, q = C, v = x: R = state size, C = head width, plus the D x skip).
+// covers gated linear attention (a decay per key channel: R = key width, C = value width), the Mamba-2 state-space scan
+// (one decay exp(-exp(A_log) dt) per head; k = dt B, q = C, v = x: R = state size, C = head width, plus the D x skip) and the
+// matrix memory of xLSTM (a decay and an input factor per head, exp(f + m' - m) and exp(i - m) with a running maximum m; one more
+// column of S, whose value is always 1, is the normaliser n).
 //
 //   state_scan    variable-length: a request's tokens in order, decode is the one-token case of the same kernel
 //   gla_decay     a = sigmoid(W2 y + b)^(1/tau) for whole prompts (decode steps evaluate it inside state_scan)
-//   gated_norm    RMS norm over equal groups of channels with the silu gate before or behind it
+//   memory_gates  log gates -> (decay, input factor, exp(-m)) per token and head; m is carried in the slot
+//   gated_norm    RMS norm over equal groups of channels with a silu or sigmoid gate before or behind it; of a matrix memory, the
+//                 division by max(|n . q|, exp(-m)) in front of it
 //
 // state_scan: a CTA owns a column tile of one head of one request.  Producer warps stage a block of tokens (decays, keys,
 // queries, values, in fp32) into one half of shared memory while consumer warps run the recurrence over the other; one
@@ -78,7 +82,8 @@ VB_DEVICE float2 unpack(pair_t a) {
 // barrier over the whole CTA, reached from the producers' and the consumers' code
 VB_DEVICE void bar_all() { asm volatile("bar.sync 0;" ::: "memory"); }
 
-enum : int { DECAY_GIVEN = 0, DECAY_LOWRANK = 1, DECAY_HEAD = 2 };
+enum : int { DECAY_GIVEN = 0, DECAY_LOWRANK = 1, DECAY_HEAD = 2, DECAY_GATES = 3 };
+constexpr bool head_decay(int mode) { return mode == DECAY_HEAD || mode == DECAY_GATES; }      // one decay and key factor per head
 
 struct ScanParams {
   const void* q; const void* k; const void* v;
@@ -89,10 +94,12 @@ struct ScanParams {
   const void* a1; int64_t a1_stride; int a_dt; const void* a2; const void* a2_b; int rank; float inv_tau;   // DECAY_LOWRANK
   const void* dt; int64_t dt_stride; int dt_dt;                                                            // DECAY_HEAD
   const float* dt_bias; const float* A_log; const float* D; float dt_min, dt_max;
-  float* out;                                // [T, H * C]
+  const float4* gates;                       // DECAY_GATES: [T, H] (decay, key factor, ...)
+  float* out;                                // [T, H * CO]
   float* state; int64_t state_stride, state_off, head_elems;
   const int* qsl; const int* seq_lens; const int* rows; int64_t rows_stride;
   int H, groups, R, C;
+  int CV, CO;                                // columns that v has and columns of an output row; C but for DECAY_GATES
   int vec, vec_v, vec_o, vec_a;              // accesses in units of four elements
 };
 
@@ -136,8 +143,8 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
   extern __shared__ __align__(16) float sm[];
   const int warps = (blockDim.x >> 5) - PRODUCERS;        // consumers
   const int CT = warps * CW;
-  // a staged token: keys RP | queries RP | values 2 CT (each twice) | decay, decay, dt, - | decays RP (per channel)
-  const int per_tok = (MODE == DECAY_HEAD ? 2 : 3) * RP + 2 * CT + 4;
+  // a staged token: keys RP | queries RP | values 2 CT (each twice) | decay, decay, key factor, - | decays RP (per channel)
+  const int per_tok = (head_decay(MODE) ? 2 : 3) * RP + 2 * CT + 4;
   float* bufs = sm;                                       // 2 x TB x per_tok
   float* obuf = sm + 2 * TB * per_tok;                    // 2 x TB x CT
   pdl_trigger();
@@ -158,6 +165,7 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
     uint4 rk[NI], rq[NI], rv[NVI];
     float4 ra[NI];
     uint32_t rdt = 0;
+    float2 rgate = make_float2(0.f, 0.f);
     // what the registers hold: operands as they lie in memory (one branch per block, no conversion and no predicate between
     // the loads, or each of them would be waited for), or fp32 bits where sizes or addresses are odd
     const bool fast16 = p.vec && p.vec_v && p.k_dt != DT_F32, fast32 = p.vec && p.vec_v && p.k_dt == DT_F32;
@@ -167,7 +175,7 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
 #pragma unroll
     for (int i = 0; i < NVI; ++i) { vt[i] = (tid + i * NT) / cv; vc[i] = (tid + i * NT - vt[i] * cv) * 4; }
     const float neg_a = MODE == DECAY_HEAD ? -expf(p.A_log[h]) : 0.f, db = MODE == DECAY_HEAD ? p.dt_bias[h] : 0.f;
-    auto slow_value = [&](int64_t tok, int c) { return bits4(ld_some(p.v, tok * p.v_stride + (int64_t)h * C + c, p.v_dt, C - c)); };
+    auto slow_value = [&](int64_t tok, int c) { return bits4(ld_some(p.v, tok * p.v_stride + (int64_t)h * p.CV + c, p.v_dt, p.CV - c)); };
     auto fetch = [&](int blk) {
       const int tb = min(TB, n - blk * TB);
       const int64_t tok0 = t0 + (int64_t)blk * TB;
@@ -177,6 +185,7 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
         if (p.dt_dt == DT_F32) rdt = reinterpret_cast<const uint32_t*>(p.dt)[i];
         else rdt = reinterpret_cast<const uint16_t*>(p.dt)[i];
       }
+      if constexpr (MODE == DECAY_GATES) rgate = *reinterpret_cast<const float2*>(p.gates + token(tid) * p.H + h);
       auto load = [&](auto vec_type) {
         using V = decltype(vec_type);
         constexpr int ES = sizeof(V) / 4;
@@ -194,7 +203,7 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
           if constexpr (MODE == DECAY_GIVEN) ra[i] = *reinterpret_cast<const float4*>(p.alpha + (tok * p.H + h) * (int64_t)R + r);
         }
 #pragma unroll
-        for (int i = 0; i < NVI; ++i) get(rv[i], p.v, token(vt[i]) * p.v_stride + (int64_t)h * C + min(c0 + vc[i], C - 4));
+        for (int i = 0; i < NVI; ++i) get(rv[i], p.v, token(vt[i]) * p.v_stride + (int64_t)h * p.CV + min(c0 + vc[i], p.CV - 4));
       };
       if (fast16) load(uint2{});
       else if (fast32) load(uint4{});
@@ -225,12 +234,20 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
         }
         asm volatile("bar.sync 1, %0;" ::"n"(NT) : "memory");
       }
+      if constexpr (MODE == DECAY_GATES) {
+        if (tid < tb) {
+          float* d = b + tid * per_tok + 2 * RP + 2 * CT;
+          d[0] = d[1] = rgate.x;
+          d[2] = rgate.y;
+        }
+        asm volatile("bar.sync 1, %0;" ::"n"(NT) : "memory");
+      }
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
         const int it = tid + i * NT, t = it / (RP / 4), r = (it % (RP / 4)) * 4;
         if (t >= tb) continue;
         float* row = b + t * per_tok;
-        const float ks = MODE == DECAY_HEAD ? row[2 * RP + 2 * CT + 2] : 1.f;
+        const float ks = head_decay(MODE) ? row[2 * RP + 2 * CT + 2] : 1.f;
         const bool in = r < R;
         const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), kv = in ? values4(rk[i], dt) : zero, qv = in ? values4(rq[i], dt) : zero;
         *reinterpret_cast<float4*>(row + r) = make_float4(kv.x * ks, kv.y * ks, kv.z * ks, kv.w * ks);
@@ -260,6 +277,16 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
         }
       }
       auto put = [&](int t, int c, float4 v) {
+        if constexpr (MODE == DECAY_GATES) {                 // behind the values: zeros up to a quad's end, the one, zeros
+          const int past = c0 + c - p.CV;
+          if (past > -4) {
+            const int one = p.CO - 4 - p.CV;
+            if (past >= 0) v.x = past == one ? 1.f : 0.f;
+            if (past >= -1) v.y = past + 1 == one ? 1.f : 0.f;
+            if (past >= -2) v.z = past + 2 == one ? 1.f : 0.f;
+            v.w = past + 3 == one ? 1.f : 0.f;
+          }
+        }
         float4* d = reinterpret_cast<float4*>(b + t * per_tok + 2 * RP + 2 * c);
         d[0] = make_float4(v.x, v.x, v.y, v.y);
         d[1] = make_float4(v.z, v.z, v.w, v.w);
@@ -279,15 +306,15 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
       if (p.vec_o) {
         for (int i = tid; i < tb * cv; i += NT) {
           const int t = i / cv, c = (i - t * cv) * 4;
-          if (c0 + c < C)
-            *reinterpret_cast<float4*>(p.out + (t0 + (int64_t)blk * TB + t) * p.H * C + (int64_t)h * C + c0 + c) =
+          if (c0 + c < p.CO)
+            *reinterpret_cast<float4*>(p.out + (t0 + (int64_t)blk * TB + t) * p.H * p.CO + (int64_t)h * p.CO + c0 + c) =
                 *reinterpret_cast<const float4*>(o + t * CT + c);
         }
         return;
       }
       for (int i = tid; i < tb * CT; i += NT) {
         const int t = i / CT, c = i - t * CT;
-        if (c0 + c < C) p.out[(t0 + (int64_t)blk * TB + t) * p.H * C + (int64_t)h * C + c0 + c] = o[i];
+        if (c0 + c < p.CO) p.out[(t0 + (int64_t)blk * TB + t) * p.H * p.CO + (int64_t)h * p.CO + c0 + c] = o[i];
       }
     };
     fetch(0);
@@ -360,14 +387,14 @@ __global__ void __launch_bounds__(384, TB == 1 && NP <= 2 ? 2 : 1) state_scan_ke
           vv[j][0] = v01.x; vv[j][1] = v01.y; vv[j][2] = v23.x; vv[j][3] = v23.y;
         }
         pair_t ah = 0;
-        if constexpr (MODE == DECAY_HEAD) ah = *reinterpret_cast<const pair_t*>(row + 2 * RP + 2 * CT);
+        if constexpr (head_decay(MODE)) ah = *reinterpret_cast<const pair_t*>(row + 2 * RP + 2 * CT);
 #pragma unroll
         for (int m = 0; m < M; ++m) {
           pair_t kk[P], qq[P], aa[P];
           const int r = row_of(2 * m);
           ld_rows(row + r, kk);
           ld_rows(row + RP + r, qq);
-          if constexpr (MODE == DECAY_HEAD) {
+          if constexpr (head_decay(MODE)) {
 #pragma unroll
             for (int i = 0; i < P; ++i) aa[i] = ah;
           } else {
@@ -449,14 +476,103 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ a1
     if (t < nt) out[(int64_t)(t0 + t) * CH + c] = decay_of(z[t], inv_tau);
 }
 
-// (token, group of W channels) per group of wpg warps: rms over the group of y (gate first: of y silu(z)), times w, (gate
-// last: times silu(z)), times a constant; w repeats after w_len channels.  NV vectors of V elements per lane stay in registers.
-constexpr int GN_NV = 4;
+// Gates of a matrix memory, one CTA per request and head.  z = W h + b, capped: z' = cap tanh(z / cap); log input gate i = z'_i, log
+// forget gate f = log sigmoid(z'_f);  m_t = max(m_{t-1} + f_t, i_t), m before the first token 0;  out = (exp(f + m_{t-1} - m_t),
+// exp(i - m_t), exp(-m_t), 0).  A token maps m to max(m + F, M) with (F, M) = (f, i), and so does a run of tokens: blocks of GATE_T
+// tokens are scanned in parallel.  logits null: one token per request, and the two products are computed here.
+constexpr int GATE_T = 256;
+struct GateParams {
+  const void* h; int64_t h_stride; const void* w; int W;
+  const float* logits;                       // [T, 2 H], before the bias
+  const float* bias; float cap;              // [2 H]: input gates, forget gates
+  float4* out;
+  float* state; int64_t state_stride, m_off;
+  const int* qsl; const int* seq_lens; const int* rows; int64_t rows_stride;
+  int H;
+};
+VB_DEVICE float2 compose(float2 a, float2 b) { return make_float2(a.x + b.x, fmaxf(a.y + b.x, b.y)); }      // a, then b
+
 template <typename T, int V>
-__global__ void __launch_bounds__(1024) gated_norm_kernel(const float* __restrict__ y, const T* __restrict__ z, int64_t z_stride,
-                                                           const T* __restrict__ w, int w_len, T* __restrict__ out,
+__global__ void __launch_bounds__(GATE_T) memory_gates_kernel(const GateParams p) {
+  __shared__ float red[32];
+  __shared__ float2 runs[GATE_T / 32];
+  __shared__ float ms[GATE_T];
+  pdl_trigger();
+  pdl_wait();
+  const int req = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int t0 = p.qsl[req], n = p.qsl[req + 1] - t0;
+  if (n <= 0) return;
+  float* slot = p.state + (int64_t)p.rows[req * p.rows_stride] * p.state_stride + p.m_off + hd;
+  float m = p.seq_lens[req] > n ? *slot : 0.f;
+  const float bi = p.bias[hd], bf = p.bias[p.H + hd];
+  auto capped = [&](float z) { return p.cap * tanhf(z / p.cap); };
+  auto log_sigmoid = [](float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); };
+  auto gates = [&](float f, float i, float before, float after) {
+    return make_float4(expf(f + before - after), expf(i - after), expf(-after), 0.f);
+  };
+  if (p.logits == nullptr) {
+    const T* h = reinterpret_cast<const T*>(p.h) + (int64_t)t0 * p.h_stride;
+    const T* wi = reinterpret_cast<const T*>(p.w) + (int64_t)hd * p.W;
+    const T* wf = wi + (int64_t)p.H * p.W;
+    float zi = 0.f, zf = 0.f;
+    for (int c = tid * V; c < p.W; c += GATE_T * V) {
+      if constexpr (V == 4) {
+        constexpr int dt = DTypeOf<T>::v;
+        const float4 x = ld_any4(h, c, dt), a = ld_any4(wi, c, dt), b = ld_any4(wf, c, dt);
+        zi += x.x * a.x; zi += x.y * a.y; zi += x.z * a.z; zi += x.w * a.w;
+        zf += x.x * b.x; zf += x.y * b.y; zf += x.z * b.z; zf += x.w * b.w;
+      } else {
+        const float x = to_f32(h[c]);
+        zi += x * to_f32(wi[c]); zf += x * to_f32(wf[c]);
+      }
+    }
+    zi = block_sum(zi, red);
+    zf = block_sum(zf, red);
+    if (tid == 0) {
+      const float i = capped(zi + bi), f = log_sigmoid(capped(zf + bf)), after = fmaxf(f + m, i);
+      p.out[(int64_t)t0 * p.H + hd] = gates(f, i, m, after);
+      *slot = after;
+    }
+    return;
+  }
+  for (int b0 = 0; b0 < n; b0 += GATE_T) {
+    const int t = b0 + tid;
+    float i = -INFINITY, f = 0.f;                               // behind the last token: m stays
+    if (t < n) {
+      const float* z = p.logits + (int64_t)(t0 + t) * 2 * p.H + hd;
+      i = capped(z[0] + bi);
+      f = log_sigmoid(capped(z[p.H] + bf));
+    }
+    float2 run = make_float2(f, i);
+#pragma unroll
+    for (int d = 1; d < 32; d *= 2) {
+      const float2 o = make_float2(__shfl_up_sync(0xffffffffu, run.x, d), __shfl_up_sync(0xffffffffu, run.y, d));
+      if (lane >= d) run = compose(o, run);
+    }
+    if (lane == 31) runs[warp] = run;
+    __syncthreads();
+    float before = m;                                           // m in front of this warp's tokens
+    for (int w = 0; w < warp; ++w) before = fmaxf(before + runs[w].x, runs[w].y);
+    const float after = fmaxf(before + run.x, run.y);
+    ms[tid] = after;
+    __syncthreads();
+    if (t < n) p.out[(int64_t)(t0 + t) * p.H + hd] = gates(f, i, tid ? ms[tid - 1] : m, after);
+    m = ms[GATE_T - 1];
+    __syncthreads();
+  }
+  if (tid == 0) *slot = m;
+}
+
+// (token, group of W channels) per group of wpg warps: rms over the group of y (gate first: of y g(z)), times w, (gate last:
+// times g(z)), times a constant; w repeats after w_len channels.  NV vectors of V elements per lane stay in registers.
+// gates not null (a matrix memory's rows of y, y_row wide): y is first divided by max(|y[n_col]|, gates.z) + 1e-6.
+constexpr int GN_NV = 4;
+struct RowDivisor { const float4* gates; int n_col; };
+template <typename T, int V>
+__global__ void __launch_bounds__(1024) gated_norm_kernel(const float* __restrict__ y, int y_row, const T* __restrict__ z,
+                                                           int64_t z_stride, const T* __restrict__ w, int w_len, T* __restrict__ out,
                                                            int64_t out_stride, int64_t n_rows, int groups, int W, int gate_first,
-                                                           float eps, float scale, int wpg) {
+                                                           int sigmoid_gate, RowDivisor by, float eps, float scale, int wpg) {
   __shared__ float red[32];
   pdl_trigger();
   pdl_wait();
@@ -466,18 +582,20 @@ __global__ void __launch_bounds__(1024) gated_norm_kernel(const float* __restric
   const bool ok = row < n_rows;
   const int64_t tok = ok ? row / groups : 0;
   const int g = ok ? (int)(row - tok * groups) : 0;
-  const float* yr = y + (tok * groups + g) * (int64_t)W;
+  const float* yr = y + (tok * groups + g) * (int64_t)y_row;
   const T* zr = z + tok * z_stride + (int64_t)g * W;
   const int i0 = ((warp % wpg) * 32 + lane) * V, step = wpg * 32 * V;
   constexpr int dt = DTypeOf<T>::v;
+  const float f = by.gates && ok ? 1.f / (fmaxf(fabsf(yr[by.n_col]), by.gates[row].z) + 1e-6f) : 1.f;
+  auto gate = [&](float u) { return sigmoid_gate ? __fdividef(1.f, 1.f + __expf(-u)) : silu_f(u); };
   auto load = [&](int i, float (&a)[V], float (&b)[V]) {
     if constexpr (V == 4) {
       const float4 x = *reinterpret_cast<const float4*>(yr + i), u = ld_any4(zr, i, dt);
-      a[0] = x.x; a[1] = x.y; a[2] = x.z; a[3] = x.w;
-      b[0] = silu_f(u.x); b[1] = silu_f(u.y); b[2] = silu_f(u.z); b[3] = silu_f(u.w);
+      a[0] = x.x * f; a[1] = x.y * f; a[2] = x.z * f; a[3] = x.w * f;
+      b[0] = gate(u.x); b[1] = gate(u.y); b[2] = gate(u.z); b[3] = gate(u.w);
     } else {
-      a[0] = yr[i];
-      b[0] = silu_f(to_f32(zr[i]));
+      a[0] = yr[i] * f;
+      b[0] = gate(to_f32(zr[i]));
     }
   };
   float a[GN_NV][V], b[GN_NV][V], ss = 0.f;
@@ -529,7 +647,7 @@ template <int NP, int L, int SNP, int SL, int MODE, int Q, int TB, int PRODUCERS
 int scan_launch(ScanParams& p, int num_reqs, int warps, cudaStream_t st) {
   static_assert(NP * L == SNP * SL, "one state layout");
   constexpr int RP = 2 * NP * L, CW = 32 / L * 4 * Q;
-  const int CT = warps * CW, per_tok = (MODE == DECAY_HEAD ? 2 : 3) * RP + 2 * CT + 4;
+  const int CT = warps * CW, per_tok = (head_decay(MODE) ? 2 : 3) * RP + 2 * CT + 4;
   const size_t smem = (size_t)(2 * TB * (per_tok + CT)) * 4;
   if (smem > 200 * 1024) return -4;
   auto kern = state_scan_kernel<NP, L, SNP, SL, MODE, Q, TB, PRODUCERS>;
@@ -559,6 +677,7 @@ int scan_shape(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t 
     const int w = many ? cta_warps(Q2 * (32 / SL), 1) : cta_warps(32 / SL, SMS);
 #define DECODE(M) (many ? scan_launch<SNP, SL, SNP, SL, M, Q2, 1, 4>(p, num_reqs, w, st) : scan_launch<SNP, SL, SNP, SL, M, 1, 1, 4>(p, num_reqs, w, st))
     if (mode == DECAY_HEAD) return DECODE(DECAY_HEAD);
+    if (mode == DECAY_GATES) return DECODE(DECAY_GATES);
     if (mode == DECAY_GIVEN) return DECODE(DECAY_GIVEN);
     return DECODE(DECAY_LOWRANK);
 #undef DECODE
@@ -566,20 +685,22 @@ int scan_shape(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t 
   if (mode == DECAY_LOWRANK) return -5;                                 // prompts bring their decays
   constexpr int TB = 8;
   constexpr int64_t CTAS = SMS * 3 / 4, WARPS = SMS * 3;                // measured: where the next form begins to win
-  const bool head = mode == DECAY_HEAD;
+  // PH: producer warps of the forms with one decay per head; the widest rows of those let two CTAs share an SM
+#define PROMPT(NP, L, PH)                                                                                \
+  (mode == DECAY_HEAD    ? scan_launch<NP, L, SNP, SL, DECAY_HEAD, 1, TB, PH>(p, num_reqs, w, st)        \
+   : mode == DECAY_GATES ? scan_launch<NP, L, SNP, SL, DECAY_GATES, 1, TB, PH>(p, num_reqs, w, st)       \
+                         : scan_launch<NP, L, SNP, SL, DECAY_GIVEN, 1, TB, 4>(p, num_reqs, w, st))
   if (quads / (32 / L2) >= WARPS) {
     const int w = cta_warps(32 / L2, CTAS);
-    return head ? scan_launch<NP2, L2, SNP, SL, DECAY_HEAD, 1, TB, 2>(p, num_reqs, w, st)      // two CTAs fit on an SM
-                : scan_launch<NP2, L2, SNP, SL, DECAY_GIVEN, 1, TB, 4>(p, num_reqs, w, st);
+    return PROMPT(NP2, L2, 2);
   }
   if (quads / (32 / L1) >= WARPS) {
     const int w = cta_warps(32 / L1, CTAS);
-    return head ? scan_launch<NP1, L1, SNP, SL, DECAY_HEAD, 1, TB, 4>(p, num_reqs, w, st)
-                : scan_launch<NP1, L1, SNP, SL, DECAY_GIVEN, 1, TB, 4>(p, num_reqs, w, st);
+    return PROMPT(NP1, L1, 4);
   }
   const int w = cta_warps(32 / SL, CTAS);
-  return head ? scan_launch<SNP, SL, SNP, SL, DECAY_HEAD, 1, TB, 4>(p, num_reqs, w, st)
-              : scan_launch<SNP, SL, SNP, SL, DECAY_GIVEN, 1, TB, 4>(p, num_reqs, w, st);
+  return PROMPT(SNP, SL, 4);
+#undef PROMPT
 }
 
 inline bool al(const void* p, int64_t n) { return p == nullptr || (reinterpret_cast<uintptr_t>(p) % (size_t)n) == 0; }
@@ -588,11 +709,12 @@ inline int esz(int dt) { return dt == DT_F32 ? 4 : 2; }
 int scan(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t st) {
   if (num_reqs == 0) return 0;
   if (p.R < 1 || p.C < 1 || p.groups < 1 || p.H % p.groups || (mode != DECAY_HEAD && p.groups != p.H)) return -1;
+  if (mode != DECAY_GATES) p.CV = p.CO = p.C;
   if (p.state_stride % 4 || p.state_off % 4 || !al(p.state, 16)) return -2;
   p.vec = p.R % 4 == 0 && p.q_stride % 4 == 0 && p.k_stride % 4 == 0 && al(p.q, 4 * esz(p.q_dt)) && al(p.k, 4 * esz(p.k_dt)) &&
           al(p.alpha, 16);
-  p.vec_v = p.C % 4 == 0 && p.v_stride % 4 == 0 && al(p.v, 4 * esz(p.v_dt));
-  p.vec_o = p.C % 4 == 0 && al(p.out, 16);
+  p.vec_v = p.CV % 4 == 0 && p.v_stride % 4 == 0 && al(p.v, 4 * esz(p.v_dt));
+  p.vec_o = p.CO % 4 == 0 && al(p.out, 16);
   p.vec_a = p.rank % 4 == 0 && p.a1_stride % 4 == 0 && al(p.a1, 4 * esz(p.a_dt)) && al(p.a2, 4 * esz(p.a_dt));
   const int rp = p.R <= 16 ? 16 : p.R <= 32 ? 32 : p.R <= 64 ? 64 : p.R <= 128 ? 128 : p.R <= 256 ? 256 : 512;
   if (p.R > 512) return -3;
@@ -649,6 +771,40 @@ EXPORT int vb_ssd_scan(const float* xbc, int64_t xbc_stride, const void* dt, int
   return lattn::scan(p, lattn::DECAY_HEAD, num_reqs, max_len, st);
 }
 
+// Matrix memory.  q, k [T, H * R], v [T, H * C] (token strides free); gates [T, H] float4 of vb_memory_gates.  out [T, H, CO] fp32,
+// CO = C rounded up to four, plus four: column CO - 4 is n . q.  A head's state has CO columns (vb_state_scan_elems(R, CO)).
+EXPORT int vb_memory_scan(const void* q, const void* k, const void* v, int64_t q_stride, int64_t k_stride, int64_t v_stride,
+                          float q_scale, const float* gates, float* out, float* state, int64_t state_stride, int64_t state_off,
+                          const int* qsl, const int* seq_lens, const int* rows, int64_t rows_stride, int num_reqs, int max_len,
+                          int H, int R, int C, int dtype, cudaStream_t st) {
+  lattn::ScanParams p = {};
+  if (!lattn::al(gates, 16)) return -2;
+  p.q = q; p.k = k; p.v = v; p.q_stride = q_stride; p.k_stride = k_stride; p.v_stride = v_stride;
+  p.q_dt = p.k_dt = p.v_dt = dtype; p.q_scale = q_scale; p.gates = reinterpret_cast<const float4*>(gates);
+  p.out = out; p.state = state; p.state_stride = state_stride; p.state_off = state_off;
+  p.qsl = qsl; p.seq_lens = seq_lens; p.rows = rows; p.rows_stride = rows_stride;
+  p.H = H; p.groups = H; p.R = R; p.CV = C; p.C = p.CO = (C + 3) / 4 * 4 + 4;
+  return lattn::scan(p, lattn::DECAY_GATES, num_reqs, max_len, st);
+}
+
+// h [T, W] (token stride free), w [2 H, W] (input gates, then forget gates), bias [2 H]; logits [T, 2 H] fp32 without the bias, or
+// null where every request has one token.  gates [T, H] float4; the maxima at m_off of the slots advance in place.
+EXPORT int vb_memory_gates(const void* h, int64_t h_stride, const void* w, int W, const float* logits, const float* bias, float cap,
+                           float* gates, float* state, int64_t state_stride, int64_t m_off, const int* qsl, const int* seq_lens,
+                           const int* rows, int64_t rows_stride, int num_reqs, int max_len, int H, int dtype, cudaStream_t st) {
+  using namespace lattn;
+  if (num_reqs == 0) return 0;
+  if (!al(gates, 16) || (!logits && max_len != 1)) return -1;
+  GateParams p = {h, h_stride, w, W, logits, bias, cap, reinterpret_cast<float4*>(gates), state, state_stride, m_off, qsl, seq_lens,
+                  rows, rows_stride, H};
+  const bool vec = W % 4 == 0 && h_stride % 4 == 0 && al(h, 4 * esz(dtype)) && al(w, 4 * esz(dtype));
+  DISPATCH_DTYPE(dtype, T, {
+    if (vec) vb_launch(memory_gates_kernel<T, 4>, dim3(num_reqs, H), dim3(GATE_T), 0, st, p);
+    else vb_launch(memory_gates_kernel<T, 1>, dim3(num_reqs, H), dim3(GATE_T), 0, st, p);
+  });
+  return (int)cudaGetLastError();
+}
+
 EXPORT int vb_gla_decay(const void* a1, int64_t a1_stride, const void* a2, const void* b, float* out, int T_, int CH, int rank,
                         float inv_tau, int dtype, cudaStream_t st) {
   using namespace lattn;
@@ -662,14 +818,17 @@ EXPORT int vb_gla_decay(const void* a1, int64_t a1_stride, const void* a2, const
 }
 
 // y [T, groups * W] fp32, z [T, groups * W] (token stride free), w [w_len] repeated along the channels (w_len a multiple or
-// a divisor of W); out [T, groups * W] in the model dtype (token stride free)
-EXPORT int vb_gated_norm(const float* y, const void* z, int64_t z_stride, const void* w, int w_len, void* out,
-                         int64_t out_stride, int T_, int groups, int W, int gate_first, float eps, float scale, int dtype,
+// a divisor of W); out [T, groups * W] in the model dtype (token stride free).  flags: bit0 gate first, bit1 sigmoid gate (else
+// silu).  gates not null: y holds the rows [T, groups, CO] of vb_memory_scan and gates its gates.
+EXPORT int vb_gated_norm(const float* y, const float* gates, const void* z, int64_t z_stride, const void* w, int w_len, void* out,
+                         int64_t out_stride, int T_, int groups, int W, int flags, float eps, float scale, int dtype,
                          cudaStream_t st) {
   using namespace lattn;
   if (T_ == 0) return 0;
   const int64_t rows = (int64_t)T_ * groups;
   const int e = esz(dtype);
+  const int n_col = (W + 3) / 4 * 4, y_row = gates ? n_col + 4 : W;
+  const RowDivisor by = {reinterpret_cast<const float4*>(gates), n_col};
   const bool vec = W % 4 == 0 && w_len % 4 == 0 && z_stride % 4 == 0 && out_stride % 4 == 0 && al(y, 16) && al(z, 4 * e) &&
                    al(w, 4 * e) && al(out, 4 * e);
   const int per_warp = vec ? 32 * 4 * GN_NV : 32 * GN_NV;
@@ -677,9 +836,8 @@ EXPORT int vb_gated_norm(const float* y, const void* z, int64_t z_stride, const 
   while (wpg < 32 && wpg * per_warp < W) wpg *= 2;
   const int warps = wpg > 8 ? wpg : 8, per_cta = warps / wpg;
   dim3 grid((unsigned)((rows + per_cta - 1) / per_cta)), block(warps * 32);
-  DISPATCH_DTYPE(dtype, T, {
-    if (vec) vb_launch(gated_norm_kernel<T, 4>, grid, block, 0, st, y, (const T*)z, z_stride, (const T*)w, w_len, (T*)out, out_stride, rows, groups, W, gate_first, eps, scale, wpg);
-    else vb_launch(gated_norm_kernel<T, 1>, grid, block, 0, st, y, (const T*)z, z_stride, (const T*)w, w_len, (T*)out, out_stride, rows, groups, W, gate_first, eps, scale, wpg);
-  });
+#define GO(V) vb_launch(gated_norm_kernel<T, V>, grid, block, 0, st, y, y_row, (const T*)z, z_stride, (const T*)w, w_len, (T*)out, out_stride, rows, groups, W, flags & 1, flags >> 1 & 1, by, eps, scale, wpg)
+  DISPATCH_DTYPE(dtype, T, { if (vec) GO(4); else GO(1); });
+#undef GO
   return (int)cudaGetLastError();
 }

@@ -65,13 +65,13 @@ __global__ void topk_softmax_kernel(const T* __restrict__ logits, float* __restr
 // Router with sigmoid or softmax scores, a selection bias and group-limited choice; one CTA per token, fp32 throughout.
 //   logits: given ([T, E] fp32), or computed here from x [T, H] and w [E, H] (one warp per expert, decode batches)
 //   choice score = score + bias;  a group (one of n_group contiguous runs) is ranked by the sum of its two best choice
-//   scores (with a bias) or by its best (without);  the k best experts of the `keep` best groups are taken, the lowest
+//   scores (group_top2) or by its best;  the k best experts of the `keep` best groups are taken, the lowest
 //   index winning ties;  weight = score WITHOUT the bias (optionally renormalised) * scale
 template <typename TX, typename TW>
 __global__ void __launch_bounds__(512)
 grouped_topk_kernel(const float* __restrict__ logits, const TX* __restrict__ x, const TW* __restrict__ w, int H,
                     const float* __restrict__ bias, float* __restrict__ out_w, int* __restrict__ out_ids, int E, int k,
-                    int n_group, int keep, int softmax, int renorm, float scale) {
+                    int n_group, int keep, int group_top2, int softmax, int renorm, float scale) {
   extern __shared__ float smf[];
   float* score = smf;               // [E]
   float* choice = score + E;        // [E]
@@ -156,7 +156,7 @@ grouped_topk_kernel(const float* __restrict__ logits, const TX* __restrict__ x, 
         const float c = choice[g * gsz + i];
         if (c > a) { b = a; a = c; } else if (c > b) { b = c; }
       }
-      gs[g] = bias && gsz > 1 ? a + b : a;
+      gs[g] = group_top2 && gsz > 1 ? a + b : a;
     }
     __syncwarp();
     // drop the worst groups: what the keep-th best leaves behind.  A taken group is marked by -inf.
@@ -400,15 +400,15 @@ EXPORT int vb_moe_topk_softmax(const void* logits, float* out_w, int* out_ids, i
 
 // x / w null: `logits` are given.  dtypes: x fp32 or the model dtype (x_f32), w the model dtype.
 EXPORT int vb_moe_grouped_topk(const float* logits, const void* x, int x_f32, const void* w, int H, const float* bias,
-                               float* out_w, int* out_ids, int n_tokens, int E, int k, int n_group, int keep, int softmax,
-                               int renorm, float scale, int dtype, cudaStream_t st) {
+                               float* out_w, int* out_ids, int n_tokens, int E, int k, int n_group, int keep, int group_top2,
+                               int softmax, int renorm, float scale, int dtype, cudaStream_t st) {
   if (n_tokens == 0) return 0;
   if (E < 1 || E > 4096 || k < 1 || k > E || n_group < 1 || E % n_group || keep < 1 || keep > n_group) return -1;
   if (!logits && (!x || !w)) return -1;
   const size_t smem = (size_t)(2 * E + n_group + (logits ? 0 : H)) * sizeof(float);
   if (smem > 48 * 1024) return -3;
   const int thr = logits ? (E > 128 ? 256 : 64) : (E > 32 ? 512 : 256);
-#define GO(TX, TW) vb_launch(moe::grouped_topk_kernel<TX, TW>, dim3(n_tokens), dim3(thr), smem, st, logits, (const TX*)x, (const TW*)w, H, bias, out_w, out_ids, E, k, n_group, keep, softmax, renorm, scale)
+#define GO(TX, TW) vb_launch(moe::grouped_topk_kernel<TX, TW>, dim3(n_tokens), dim3(thr), smem, st, logits, (const TX*)x, (const TW*)w, H, bias, out_w, out_ids, E, k, n_group, keep, group_top2, softmax, renorm, scale)
   DISPATCH_DTYPE(dtype, T, {
     if (x_f32) GO(float, T); else GO(T, T);
   });

@@ -181,6 +181,40 @@ __global__ void act_kernel(T* __restrict__ out, const T* __restrict__ x, int64_t
   }
 }
 
+// y[t, c] = x[t, c] * sigmoid(g[t, c]), row strides free; x may be y
+template <typename T, int V>
+__global__ void sigmoid_mul_kernel(const T* __restrict__ x, int64_t x_stride, const T* __restrict__ g, int64_t g_stride,
+                                   T* __restrict__ y, int64_t y_stride, int n, int64_t total) {
+  pdl_trigger();
+  pdl_wait();
+  const int per_row = n / V;
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = i / per_row;
+    const int c = (int)(i - t * per_row) * V;
+    if constexpr (V == 1) {
+      y[t * y_stride + c] = from_f32<T>(__fdividef(to_f32(x[t * x_stride + c]), 1.f + __expf(-to_f32(g[t * g_stride + c]))));
+    } else {
+      const Vec16<T> a = ld16(x + t * x_stride + c), b = ld16(g + t * g_stride + c);
+      Vec16<T> o;
+#pragma unroll
+      for (int j = 0; j < V; ++j) o.e[j] = from_f32<T>(__fdividef(to_f32(a.e[j]), 1.f + __expf(-to_f32(b.e[j]))));
+      st16(y + t * y_stride + c, o);
+    }
+  }
+}
+
+// x[t, c] = cap tanh(x[t, c] / cap) in place, rows of n at any stride
+template <typename T>
+__global__ void soft_cap_kernel(T* __restrict__ x, int64_t stride, int n, int64_t total, float cap) {
+  pdl_trigger();
+  pdl_wait();
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = i / n;
+    T* p = x + t * stride + (i - t * n);
+    *p = from_f32<T>(cap * tanhf(to_f32(*p) / cap));
+  }
+}
+
 int norm_threads(int H, int vecN) {
   int nvec = H / vecN;
   int t = (nvec + MAXV - 1) / MAXV;
@@ -288,5 +322,32 @@ EXPORT int vb_activation(void* out, const void* x, int64_t n, int act, int dtype
     const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
     ACT_SWITCH(act_kernel, <<<blocks, 256, 0, st>>>((TT*)out, (const TT*)x, total));
   });
+  return (int)cudaGetLastError();
+}
+
+EXPORT int vb_sigmoid_mul(const void* x, int64_t x_stride, const void* g, int64_t g_stride, void* y, int64_t y_stride, int64_t T, int n,
+                          int dtype, cudaStream_t st) {
+  if (T == 0) return 0;
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+#define GO(V)                                                                                                       \
+  do {                                                                                                              \
+    const int64_t total = T * (n / (V));                                                                            \
+    const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);                      \
+    vb_launch(sigmoid_mul_kernel<TT, V>, blocks, 256, 0, st, (const TT*)x, x_stride, (const TT*)g, g_stride, (TT*)y, y_stride, n, total); \
+  } while (0)
+  DISPATCH_DTYPE(dtype, TT, {
+    constexpr int N = Vec16<TT>::N;
+    if (n % N == 0 && x_stride % N == 0 && g_stride % N == 0 && y_stride % N == 0 && al(x) && al(g) && al(y)) GO(N);
+    else GO(1);
+  });
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+EXPORT int vb_soft_cap(void* x, int64_t stride, int64_t T, int n, float cap, int dtype, cudaStream_t st) {
+  if (T == 0 || n == 0) return 0;
+  const int64_t total = T * n;
+  const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+  DISPATCH_DTYPE(dtype, TT, { vb_launch(soft_cap_kernel<TT>, blocks, 256, 0, st, (TT*)x, stride, n, total, cap); });
   return (int)cudaGetLastError();
 }

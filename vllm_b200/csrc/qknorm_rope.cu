@@ -220,6 +220,101 @@ __global__ void __launch_bounds__(ANY_WARPS * 32) qknorm_rope_any_kernel(const P
   }
 }
 
+// The norms over the WHOLE projections (all heads of q at once, all of k at once) instead of per head, then rotation and cache write,
+// 32-bit in between.  CTA = one token's q, or its k and v; weights [H * D].  V elements per access.  k null: queries alone.
+template <typename T, int V> VB_DEVICE void load_v(const T* p, float (&f)[V]) {
+  if constexpr (V == 1) f[0] = to_f32(p[0]);
+  else {
+    const Vec16<T> x = ld16(p);
+#pragma unroll
+    for (int j = 0; j < V; ++j) f[j] = to_f32(x.e[j]);
+  }
+}
+template <typename T, int V> VB_DEVICE void store_v(T* p, const float (&f)[V]) {
+  if constexpr (V == 1) p[0] = from_f32<T>(f[0]);
+  else {
+    Vec16<T> x;
+#pragma unroll
+    for (int j = 0; j < V; ++j) x.e[j] = from_f32<T>(f[j]);
+    st16(p, x);
+  }
+}
+template <typename T, int V>
+__global__ void __launch_bounds__(512) qknorm_rope_row_kernel(const Params p, int DV, int DC) {
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, D = p.D, half = p.rot / 2;
+  const bool is_k = blockIdx.y == 1;
+  const int heads = is_k ? p.Hkv : p.Hq, n = heads * D;
+  T* base = is_k ? reinterpret_cast<T*>(p.k) + t * p.k_stride : reinterpret_cast<T*>(p.q) + t * p.q_stride;
+  const T* w = reinterpret_cast<const T*>(is_k ? p.k_w : p.q_w);
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < n; i += blockDim.x * V) {
+    float f[V];
+    load_v<T, V>(base + i, f);
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += f[j] * f[j];
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)n + p.eps);
+  const int64_t slot = is_k && p.slot_mapping ? p.slot_mapping[t] : -1;
+  const bool do_cache = is_k && p.kv_cache != nullptr && slot >= 0;
+  const int64_t blk = do_cache ? slot / p.BS : 0;
+  const int off = do_cache ? (int)(slot % p.BS) : 0;
+  T* cache = reinterpret_cast<T*>(p.kv_cache);
+  const float* cs = p.rot > 0 ? p.cos_sin + p.positions[t] * p.rot : nullptr;
+  const int turning = half / V, per_head = turning + (D - p.rot) / V;
+  auto normed = [&](int at, float (&f)[V]) {
+    float g[V];
+    load_v<T, V>(base + at, f);
+    load_v<T, V>(w + at, g);
+#pragma unroll
+    for (int j = 0; j < V; ++j) f[j] *= inv * (g[j] + (p.gemma ? 1.f : 0.f));
+  };
+  for (int it = threadIdx.x; it < heads * per_head; it += blockDim.x) {
+    const int h = it / per_head, c = it - h * per_head;
+    T* dst = do_cache ? cache + ((blk * 2 * p.Hkv + h) * p.BS + off) * (int64_t)DC : nullptr;
+    float a[V];
+    if (c >= turning) {
+      const int e = p.rot + (c - turning) * V;
+      normed(h * D + e, a);
+      store_v<T, V>(base + h * D + e, a);
+      if (dst) store_v<T, V>(dst + e, a);
+      continue;
+    }
+    const int e0 = p.neox ? c * V : 2 * c, e1 = p.neox ? half + c * V : 2 * c + 1;      // neighbours turn together: V = 1
+    float b[V];
+    normed(h * D + e0, a);
+    normed(h * D + e1, b);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float co = cs[c * V + j], si = cs[half + c * V + j], x = a[j], y = b[j];
+      a[j] = x * co - y * si;
+      b[j] = y * co + x * si;
+    }
+    store_v<T, V>(base + h * D + e0, a);
+    store_v<T, V>(base + h * D + e1, b);
+    if (dst) { store_v<T, V>(dst + e0, a); store_v<T, V>(dst + e1, b); }
+  }
+  if (!do_cache || p.v == nullptr) return;
+  const T* v = reinterpret_cast<const T*>(p.v) + t * p.v_stride;
+  for (int it = threadIdx.x; it < p.Hkv * (DV / V); it += blockDim.x) {
+    const int h = it / (DV / V), d = (it - h * (DV / V)) * V;
+    T* dst = cache + ((blk * 2 + 1) * p.Hkv + h) * p.BS * (int64_t)DC;
+    if constexpr (V == 1) {
+      dst[p.vt ? (int64_t)d * p.BS + off : (int64_t)off * DC + d] = v[h * DV + d];
+    } else {
+      const Vec16<T> x = ld16(v + h * DV + d);
+      if (p.vt) {
+#pragma unroll
+        for (int j = 0; j < V; ++j) dst[(int64_t)(d + j) * p.BS + off] = x.e[j];
+      } else {
+        st16(dst + (int64_t)off * DC + d, x);
+      }
+    }
+  }
+}
+
 }  // namespace
 
 // q, k: [T, H*D] views of the fused qkv buffer (rotated / normalised in place); v may be null (no cache write of V);
@@ -276,5 +371,30 @@ EXPORT int vb_qknorm_rope_any(const int64_t* positions, void* q, void* k, const 
   const int64_t warps = (int64_t)T * (Hq + 2 * Hkv);
   dim3 grid((unsigned)((warps + ANY_WARPS - 1) / ANY_WARPS));
   DISPATCH_DTYPE(dtype, TT, vb_launch(qknorm_rope_any_kernel<TT>, grid, dim3(ANY_WARPS * 32), 0, st, p, DV, DC));
+  return (int)cudaGetLastError();
+}
+
+// Norms over whole rows: q_w [Hq * D], k_w [Hkv * D].  Hkv 0: queries alone (a layer that reads another layer's keys).  The cache
+// holds the model dtype, rows DC wide.
+EXPORT int vb_qknorm_rope_row(const int64_t* positions, void* q, void* k, const void* v, const void* q_w, const void* k_w,
+                              const float* cos_sin, int rot, int T, int Hq, int Hkv, int D, int DV, int DC, int64_t q_stride,
+                              int64_t k_stride, int64_t v_stride, void* kv_cache, const int64_t* slot_mapping, int BS, int neox,
+                              int gemma, int vt, float eps, int dtype, cudaStream_t st) {
+  if (T == 0) return 0;
+  if (!q_w || (Hkv && !k_w) || rot > D || rot % 2 || (kv_cache && (DC < D || DC < DV))) return -1;
+  Params p = {};
+  p.positions = positions; p.q = q; p.k = k; p.v = v; p.q_w = q_w; p.k_w = k_w; p.cos_sin = cos_sin;
+  p.kv_cache = kv_cache; p.slot_mapping = slot_mapping; p.q_stride = q_stride; p.k_stride = k_stride; p.v_stride = v_stride;
+  p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.rot = rot; p.BS = BS; p.neox = neox; p.gemma = gemma; p.vt = vt; p.eps = eps;
+  DISPATCH_DTYPE(dtype, TT, {
+    constexpr int N = Vec16<TT>::N;
+    auto ok = [](const void* a, int64_t stride) { return !a || ((reinterpret_cast<uintptr_t>(a) & 15) == 0 && stride % N == 0); };
+    const bool vec = (neox || rot == 0) && D % N == 0 && rot % (2 * N) == 0 && DV % N == 0 && DC % N == 0 && ok(q, q_stride) &&
+                     ok(k, k_stride) && ok(v, v_stride) && ok(q_w, 0) && ok(k_w, 0) && ok(kv_cache, 0);
+    const int items = Hq * D / (vec ? N : 1), want = (items + 31) / 32 * 32;
+    const dim3 grid(T, Hkv ? 2 : 1), block(want < 64 ? 64 : want > 512 ? 512 : want);
+    if (vec) vb_launch(qknorm_rope_row_kernel<TT, N>, grid, block, 0, st, p, DV, DC);
+    else vb_launch(qknorm_rope_row_kernel<TT, 1>, grid, block, 0, st, p, DV, DC);
+  });
   return (int)cudaGetLastError();
 }

@@ -8,7 +8,9 @@
 //                     x += rmsnorm(y) * w;   out = T(x)  |  T(rmsnorm(x) * w_next)
 //   norm_add          the same step for blocks with a norm on either side of a sublayer, layer norms or RMS norms:
 //                     x += m norm(y + bias);   out = T(norm_next(x))       (or x = table[id] at the model's entry)
-// The combine of the expert layer is the load of post_norm_add: expert outputs are read once, summed in slot order in
+//   add_norm          the same step for pre-norm blocks:  x += y + routed sum;   out = T(norm_next(x)).  The routed sum may have
+//                     identity experts: slots whose expert number is past the last one add w_j times the layer's input
+// The combine of the expert layer is the load of post_norm_add and add_norm: expert outputs are read once, summed in slot order in
 // fp32 (deterministic) and never written back.
 #include "common.cuh"
 
@@ -230,6 +232,58 @@ norm_add_kernel(const int* __restrict__ ids, int vocab, const T* __restrict__ y,
   }
 }
 
+// x += y + sum_s w_s (a row of `rows`, or of `h` for identity experts);  out = norm(x), or x where w2 is null.  y, rows, h may be null
+struct Routed {
+  const void* rows; int64_t stride;
+  const int* inv; const float* w; const int* ids;       // [T, k]; inv < 0: no row (identity expert, or another rank's)
+  int k, experts;                                       // ids from `experts` on are identities
+  const void* h; int64_t h_stride;
+};
+template <typename T, int V, int NV, bool LN>
+__global__ void __launch_bounds__(1024)
+add_norm_kernel(const T* __restrict__ y, int64_t y_stride, const Routed r, float* __restrict__ x, const T* __restrict__ w2,
+                const T* __restrict__ b2, int w_off, T* __restrict__ out, int H, float eps) {
+  __shared__ float red[32];
+  pdl_trigger();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  const int step = blockDim.x * V;
+  float id_w = 0.f;
+  if (r.h)
+    for (int s = 0; s < r.k; ++s)
+      if (r.ids[row * r.k + s] >= r.experts) id_w += r.w[row * r.k + s];
+  float v[NV][V];
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * step;
+    if (i >= H) continue;
+    load_f32<float, V>(x + row * H + i, v[n]);
+    auto add = [&](const T* src, float ws) {
+      float u[V];
+      load_f32<T, V>(src + i, u);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[n][j] += ws * u[j];
+    };
+    if (y) add(y + row * y_stride, 1.f);
+    if (r.rows) {
+#pragma unroll 4
+      for (int s = 0; s < r.k; ++s) {
+        const int p = r.inv[row * r.k + s];
+        if (p >= 0) add(reinterpret_cast<const T*>(r.rows) + (int64_t)p * r.stride, r.w[row * r.k + s]);
+      }
+    }
+    if (id_w != 0.f) add(reinterpret_cast<const T*>(r.h) + row * r.h_stride, id_w);
+    store_f32<float, V>(x + row * H + i, v[n]);
+  }
+  if (!out) return;
+  if (w2) normalise<T, V, NV, LN>(v, w2, b2, w_off, H, eps, red);
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * step;
+    if (i < H) store_f32<T, V>(out + row * H + i, v[n]);
+  }
+}
+
 template <typename T> constexpr int vec_of() { return sizeof(T) == 4 ? 4 : 8; }
 static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
@@ -293,6 +347,35 @@ EXPORT int vb_norm_add(const int* ids, int vocab, const void* y, int64_t y_strid
     constexpr int V = vec_of<T>();
     auto ok = [](const void* p) { return !p || al16(p); };
     const bool vec = H % V == 0 && y_stride % V == 0 && ok(y) && ok(y_bias) && ok(w1) && ok(b1) && ok(x) && ok(w2) && ok(b2) && ok(out);
+    const int items = vec ? H / V : H;
+    const int thr = items >= 1024 ? 1024 : ((items + 31) / 32) * 32;
+    const int nv = (items + thr - 1) / thr;
+    if (vec) { if (nv <= 1) GO(V, 1); else if (nv <= 4) GO(V, 4); else return -1; }
+    else { if (nv <= 1) GO(1, 1); else if (nv <= 16) GO(1, 16); else return -1; }
+  });
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+// x += y + routed sum, out = norm2(x) in the model dtype (x where w2 is null).  y [T, H] or null; rows null: nothing routed, else
+// inv / pair_w / ids [T, k]; h [T, H]: the input that identity experts (ids >= experts) pass on, or null.  ln, w_off as in vb_norm_add.
+EXPORT int vb_add_norm(const void* y, int64_t y_stride, const void* rows, int64_t rows_stride, const int* inv, const float* pair_w,
+                       const int* ids, int k, int experts, const void* h, int64_t h_stride, float* x, const void* w2, const void* b2,
+                       int w_off, int ln, void* out, int T_, int H, float eps, int dtype, cudaStream_t st) {
+  using namespace stream;
+  if (T_ == 0) return 0;
+  if ((rows && (!inv || !pair_w)) || (h && (!ids || !pair_w))) return -1;
+  const Routed r = {rows, rows_stride, inv, pair_w, ids, k, experts, h, h_stride};
+#define GO(VV, NVV)                                                                                                          \
+  do {                                                                                                                       \
+    if (ln) vb_launch(add_norm_kernel<T, VV, NVV, true>, dim3(T_), dim3(thr), 0, st, (const T*)y, y_stride, r, x, (const T*)w2, (const T*)b2, w_off, (T*)out, H, eps); \
+    else vb_launch(add_norm_kernel<T, VV, NVV, false>, dim3(T_), dim3(thr), 0, st, (const T*)y, y_stride, r, x, (const T*)w2, (const T*)b2, w_off, (T*)out, H, eps); \
+  } while (0)
+  DISPATCH_DTYPE(dtype, T, {
+    constexpr int V = vec_of<T>();
+    auto ok = [](const void* p) { return !p || al16(p); };
+    const bool vec = H % V == 0 && (!y || y_stride % V == 0) && (!rows || rows_stride % V == 0) && (!h || h_stride % V == 0) && ok(y) &&
+                     ok(rows) && ok(h) && ok(x) && ok(w2) && ok(b2) && ok(out);
     const int items = vec ? H / V : H;
     const int thr = items >= 1024 ? 1024 : ((items + 31) / 32) * 32;
     const int nv = (items + thr - 1) / thr;

@@ -36,11 +36,14 @@ class Attention(nn.Module):
                  causal: bool = True, rope: Optional[nn.Module] = None,
                  alibi_slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
                  chunk_size: int = 0, v_head_size: Optional[int] = None, fused_prologue: bool = False,
-                 out_scale: float = 1.0) -> None:
+                 out_scale: float = 1.0, whole_qk_norm: bool = False, kv_sharing_target: Optional[str] = None) -> None:
         """``v_head_size``: value width where it is not ``head_size`` (cache rows are as wide as the wider one).
         ``fused_prologue``: q/k norms, rotation and cache write are one kernel for whatever shape and dtype, 32-bit between norm
-        and rotation.  ``out_scale``: factor of the output, applied in 32-bit."""
+        and rotation.  ``out_scale``: factor of the output, applied in 32-bit.  ``whole_qk_norm``: the q/k norms go over all heads of
+        the projection at once (weights as long).  ``kv_sharing_target``: name of an earlier layer whose cache this one reads (it owns
+        none, writes nothing and is called without keys and values)."""
         super().__init__()
+        self.whole_qk_norm, self.kv_sharing_target, self.cache_name = whole_qk_norm, kv_sharing_target, kv_sharing_target or prefix
         self.v_head_size = v_head_size or head_size
         self.cache_head_size = max(head_size, self.v_head_size)
         self.fused_prologue, self.out_scale = fused_prologue, float(out_scale)
@@ -55,6 +58,13 @@ class Attention(nn.Module):
         self.causal = causal
         self.layer_name = prefix
         self.rope = rope
+        if kv_sharing_target is not None:
+            owner = _LAYER_REGISTRY.get(kv_sharing_target)
+            if not isinstance(owner, Attention) or (owner.num_heads, owner.num_kv_heads, owner.head_size, owner.v_head_size) != (
+                    self.num_heads, self.num_kv_heads, head_size, self.v_head_size):
+                raise ValueError(f"layer {prefix!r} shares the cache of {kv_sharing_target!r}, which is not an earlier attention layer "
+                                 "of the same head shapes on this rank")
+            return
         assert prefix not in _LAYER_REGISTRY, f"duplicate attention layer name {prefix}"
         _LAYER_REGISTRY[prefix] = self
 
@@ -62,6 +72,8 @@ class Attention(nn.Module):
         from vllm_b200.parallel.state import get_dcp_group
         d = get_dcp_group().world_size
         if d > 1:
+            if self.whole_qk_norm:
+                raise NotImplementedError("decode context parallelism does not cover norms over whole projections")
             if self.sliding_window or self.alibi_slopes is not None or self.sinks is not None or self.chunk_size:
                 raise NotImplementedError("decode context parallelism covers full causal attention (no sliding window / "
                                           "ALiBi / sinks / chunked-local layers)")
@@ -126,22 +138,30 @@ class Attention(nn.Module):
 
     def forward(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
                 positions: Optional[torch.Tensor] = None, qk_norm: Optional[tuple] = None,
-                out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                out: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``_attend``, then times sigmoid(``gate``) [T, Hq*DV] where given."""
+        o = self._attend(q, k, v, positions, qk_norm, out)
+        return o if gate is None else ops.sigmoid_mul_(o, gate)
+
+    def _attend(self, q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], positions: Optional[torch.Tensor],
+                qk_norm: Optional[tuple], out: Optional[torch.Tensor]) -> torch.Tensor:
         """q: [T, Hq*D], k: [T, Hkv*D], v: [T, Hkv*DV] → [T, Hq*DV] (``out``: a buffer for it, any token stride). If the layer has a ``rope``,
         rotation and the KV write happen in one fused kernel.  ``qk_norm`` = (q_norm, k_norm) per-head RMSNorm modules
-        (Qwen3 / Gemma-3 / OLMo-2 style): on CUDA they are fused with the rotation and the cache insert into ONE launch
-        (csrc/qknorm_rope.cu), otherwise applied here before the rotation."""
+        (Qwen3 / Gemma-3 / OLMo-2 style; over the whole projections with ``whole_qk_norm``): on CUDA they are fused with the rotation
+        and the cache insert into ONE launch (csrc/qknorm_rope.cu), otherwise applied here before the rotation.  k and v are None (and
+        so is k_norm) in a layer that reads another layer's cache."""
         ctx = get_forward_context()
         T = q.shape[0]
         D = self.head_size
-        md = ctx.metadata_for(self.layer_name)
-        kv_cache = ctx.kv_caches.get(self.layer_name)
+        md = ctx.metadata_for(self.cache_name)
+        kv_cache = ctx.kv_caches.get(self.cache_name)
+        shared = self.kv_sharing_target is not None
         if md is not None and kv_cache is None:
             raise RuntimeError(f"attention layer {self.layer_name!r} has no KV cache bound (KV-cache config does not "
                                "cover this worker's layers)")
         if md is None or kv_cache is None:
             # memory-profiling run: no cache; keep the data flow (and the GEMM shapes) intact
-            if self.v_head_size != D or out is not None:
+            if self.v_head_size != D or out is not None or self.fused_prologue:
                 return (q.new_empty(T, self.num_heads * self.v_head_size) if out is None else out).zero_()
             if self.rope is not None and positions is not None:
                 q, k = self.rope(positions, q, k)
@@ -154,30 +174,39 @@ class Attention(nn.Module):
                 k = kn(k.reshape(T, -1, D)).reshape(T, -1)
             return self._forward_dcp(q, k, v, positions, md, kv_cache)
         pcp = ctx.extra.get("pcp")
+        if pcp is not None and (shared or self.whole_qk_norm):
+            raise NotImplementedError("prefill context parallelism does not cover shared caches and norms over whole projections")
         mpos = ctx.extra.get("mrope_positions") if (self.rope is not None and self.rope.mrope_section) else None
         if qk_norm is not None:
             qn, kn = qk_norm
             fused = (md is not None and kv_cache is not None and q.is_cuda and pcp is None and mpos is None
                      and self.rope is not None and positions is not None
-                     and kv_cache.dtype == q.dtype and getattr(qn, "gemma", False) == getattr(kn, "gemma", False)
-                     and qn.eps == kn.eps and not envs.VLLM_B200_FORCE_REF_OPS
+                     and kv_cache.dtype == q.dtype
+                     and (shared or (getattr(qn, "gemma", False) == getattr(kn, "gemma", False) and qn.eps == kn.eps)) and not envs.VLLM_B200_FORCE_REF_OPS
                      and (self.fused_prologue or (q.dtype in (torch.bfloat16, torch.float16) and ops.cuda_ops().qknorm_rope_ok(
                          D, self.rope.cos_sin_cache.shape[-1], self.rope.is_neox_style))))
             if fused:
-                ops.cuda_ops().fused_qk_norm_rope(positions, q, k, qn.weight, kn.weight, self.rope.cos_sin_cache, D, qn.eps,
-                                                  self.rope.is_neox_style, v=v, kv_cache=kv_cache,
+                ops.cuda_ops().fused_qk_norm_rope(positions, q, k, qn.weight, None if shared else kn.weight, self.rope.cos_sin_cache,
+                                                  D, qn.eps, self.rope.is_neox_style, v=v, kv_cache=None if shared else kv_cache,
                                                   slot_mapping=md.slot_mapping, gemma=getattr(qn, "gemma", False),
-                                                  vt=md.kv_vt, v_head_dim=self.v_head_size, keep32=self.fused_prologue)
+                                                  vt=md.kv_vt, v_head_dim=self.v_head_size, keep32=self.fused_prologue,
+                                                  whole=self.whole_qk_norm)
                 positions = None            # rotation and cache insert are done: skip them below
                 skip_cache_write = True
             else:
-                q = qn(q.reshape(T, -1, D)).reshape(T, -1)
-                k = kn(k.reshape(T, -1, D)).reshape(T, -1)
+                whole = self.whole_qk_norm
+                q = qn(q.reshape(T, -1, q.shape[-1] if whole else D)).reshape(T, -1)
+                k = k if shared else kn(k.reshape(T, -1, k.shape[-1] if whole else D)).reshape(T, -1)
                 skip_cache_write = False
         else:
             skip_cache_write = False
         if skip_cache_write:
             pass
+        elif shared:
+            if mpos is not None:
+                raise NotImplementedError("shared caches with M-RoPE")
+            if self.rope is not None and positions is not None:
+                q, _ = self.rope(positions, q, None)
         elif self.v_head_size != D:
             if pcp is not None or mpos is not None:
                 raise NotImplementedError("unequal key and value widths with prefill context parallelism or M-RoPE")

@@ -170,7 +170,7 @@ class LogitsProcessor(nn.Module):
             logits = get_tp_group().all_gather(logits, -1)
         logits = logits[..., :self.vocab_size]
         if self.soft_cap:
-            logits = torch.tanh(logits / self.soft_cap) * self.soft_cap
+            logits = ops.soft_cap(logits, self.soft_cap)
         if self.scale != 1.0:
             logits = logits * self.scale
         return logits

@@ -28,9 +28,11 @@ class FusedMoE(nn.Module):
                  renormalize: bool = True, use_grouped_topk: bool = False, n_group: int = 1, topk_group: int = 1,
                  scoring_func: str = "softmax", routed_scaling_factor: float = 1.0, e_score_bias: bool = False,
                  act: str = "silu", enable_ep: bool = False, reduce_results: bool = True, prefix: str = "",
-                 quant_config=None, gated: bool = True) -> None:
+                 quant_config=None, gated: bool = True, identity_experts: int = 0) -> None:
+        """``identity_experts``: expert numbers from ``num_experts`` on (as many as this) return their input and have no weights."""
         super().__init__()
         g = get_tp_group()
+        self.identity_experts = identity_experts
         # ``gated`` False: an expert is up → act → down and ``w13_weight`` holds the up projection alone
         self.gated = gated
         if not gated and quant_config is not None and getattr(quant_config, "name", "") == "fp8_block":
@@ -73,6 +75,8 @@ class FusedMoE(nn.Module):
                 if (num_experts + R) % ep_size:
                     raise ValueError(f"num_experts + num_redundant_experts ({num_experts}+{R}) must divide by EP size {ep_size}")
                 self.eplb, self.num_physical = True, num_experts + R
+        if identity_experts and (self.wide_ep or self.eplb):
+            raise NotImplementedError("identity experts with wide expert parallelism or expert load balancing")
         if self.eplb:
             P, per = self.num_physical, self.num_physical // ep_size
             self.ep_rank, self.ep_size = ep_rank, ep_size
@@ -88,13 +92,18 @@ class FusedMoE(nn.Module):
             self.e_start = min(num_experts, ep_rank * per)
             self.e_end = min(num_experts, self.e_start + per)
             self.local_experts = self.e_end - self.e_start
-            emap = torch.full((num_experts,), -1, dtype=torch.int32)
+            emap = torch.full((num_experts + identity_experts,), -1, dtype=torch.int32)
             emap[self.e_start:self.e_end] = torch.arange(self.local_experts, dtype=torch.int32)
             self.register_buffer("expert_map", emap, persistent=False)
             self.inter_per_rank = intermediate_size
         else:
             self.e_start, self.e_end, self.local_experts = 0, num_experts, num_experts
-            self.expert_map = None
+            if identity_experts:
+                emap = torch.full((num_experts + identity_experts,), -1, dtype=torch.int32)
+                emap[:num_experts] = torch.arange(num_experts, dtype=torch.int32)
+                self.register_buffer("expert_map", emap, persistent=False)
+            else:
+                self.expert_map = None
             self.inter_per_rank = divide(intermediate_size, self.tp_size)
         I = self.inter_per_rank
         self.w13_weight = nn.Parameter(torch.empty(max(self.local_experts, 1), (2 if gated else 1) * I, hidden_size, dtype=dt),
@@ -150,13 +159,27 @@ class FusedMoE(nn.Module):
         out = self._local_experts(x2, w.to(torch.float32), ids)
         if self.reduce_results and self.tp_size > 1:
             out = get_tp_group().all_reduce(out)
+        if self.identity_experts:
+            out = out + ops.ref.identity_experts(x2, w, ids, self.num_experts)
         return out.reshape(shape)
+
+    def forward_add_norm(self, x: torch.Tensor, routing: tuple, stream: torch.Tensor, y: Optional[torch.Tensor], next_norm) -> torch.Tensor:
+        """In place on the fp32 residual stream: stream += moe(x) + y (``y``: a shared expert's output, or None).  Returns the next
+        GEMM's input, ``next_norm`` (a LayerNorm, or None) of the stream.  On one rank the top-k combine and the identity experts are
+        part of the norm kernel's load."""
+        w, ids = routing
+        nn_, eps = (None, 0.0) if next_norm is None else ((next_norm.weight, next_norm.bias), next_norm.eps)
+        if self.tp_size == 1 and not (self.ep or self.wide_ep or self.eplb or self.fp8_block):
+            return ops.fused_moe_add_norm(stream, x, self.w13_weight, self.w2_weight, w, ids, self.act, self.expert_map, self.gated,
+                                          self.num_experts, y, nn_, eps)
+        out = self.forward(x, routing=routing)
+        return ops.add_norm(stream, out if y is None else out + y, nn_, eps)
 
     def forward_post_norm(self, x: torch.Tensor, routing: tuple, stream: torch.Tensor, norm, next_norm=None) -> torch.Tensor:
         """In place on the fp32 residual stream: stream += norm(moe(x)).  Returns the next GEMM's input (the stream in x's
         dtype, or ``next_norm`` of it).  On one rank the top-k combine is part of the norm kernel's load."""
         nw, ng = (None, False) if next_norm is None else (next_norm.weight, next_norm.gemma)
-        if self.tp_size == 1 and not (self.gated or self.ep or self.wide_ep or self.eplb):
+        if self.tp_size == 1 and not (self.gated or self.identity_experts or self.ep or self.wide_ep or self.eplb):
             w, ids = routing
             return ops.fused_moe_post_norm(stream, x, self.w13_weight, self.w2_weight, w, ids, self.act, self.expert_map,
                                            norm.weight, norm.eps, norm.gemma, nw, ng)
@@ -168,7 +191,7 @@ class FusedMoE(nn.Module):
         epilogue red.adds every weighted row into the accumulator of the rank that owns the token.  None = not covered
         (wide EP, EPLB, fp8 experts, prefill-sized batches, CPU) → the caller uses the unfused sequence."""
         if (not x.is_cuda or self.wide_ep or self.eplb or self.fp8_block or norm is None or not self.gated
-                or x.dtype not in (torch.bfloat16, torch.float16) or self.w13_weight.dtype != x.dtype):
+                or self.identity_experts or x.dtype not in (torch.bfloat16, torch.float16) or self.w13_weight.dtype != x.dtype):
             return None
         from vllm_b200 import envs
         if envs.VLLM_B200_FORCE_REF_OPS or not envs.VLLM_B200_FUSED_MOE:
@@ -344,8 +367,11 @@ class GroupedRouter(nn.Module):
 
     def __init__(self, hidden_size: int, num_experts: int, top_k: int, dtype=None, n_group: int = 1, topk_group: int = 1,
                  scoring_func: str = "sigmoid", renormalize: bool = False, routed_scaling_factor: float = 1.0,
-                 selection_bias: bool = True) -> None:
+                 selection_bias: bool = True, group_score: Optional[str] = None) -> None:
+        """``group_score``: groups are ranked by their two best choice scores ("top2") or by their best ("max"); None: by two where
+        there is a selection bias."""
         super().__init__()
+        self.group_score = group_score
         if not 1 <= top_k <= num_experts or num_experts % n_group or not 1 <= topk_group <= n_group:
             raise ValueError(f"router: top {top_k} of {num_experts} experts, {topk_group} of {n_group} groups")
         if top_k > topk_group * (num_experts // n_group):
@@ -358,7 +384,7 @@ class GroupedRouter(nn.Module):
 
     def forward(self, x: torch.Tensor, x_half: Optional[torch.Tensor] = None) -> tuple[torch.Tensor, torch.Tensor]:
         return ops.router_topk(x, self.weight, self.top_k, self.n_group, self.topk_group, self.renormalize, self.scoring_func,
-                               self.bias, self.routed_scaling_factor, x_half)
+                               self.bias, self.routed_scaling_factor, x_half, self.group_score)
 
 
 def make_expert_params_mapping(gate_name: str, down_name: str, up_name: str, num_experts: int,

@@ -17,8 +17,8 @@ import torch.nn as nn
 from vllm_b200 import ops
 
 
-def _inv_freq(base: float, rot_dim: int) -> torch.Tensor:
-    return 1.0 / (base ** (torch.arange(0, rot_dim, 2, dtype=torch.float32) / rot_dim))
+def _inv_freq(base: float, rot_dim: int, dtype=torch.float32) -> torch.Tensor:
+    return 1.0 / (base ** (torch.arange(0, rot_dim, 2, dtype=dtype) / rot_dim))
 
 
 def _yarn_find_dim(num_rot: float, dim: int, base: float, max_pos: int) -> float:
@@ -32,10 +32,10 @@ def _yarn_range(low_rot: float, high_rot: float, dim: int, base: float, max_pos:
     return max(low, 0), min(high, dim - 1)
 
 
-def _yarn_ramp(low: float, high: float, n: int) -> torch.Tensor:
+def _yarn_ramp(low: float, high: float, n: int, dtype=torch.float32) -> torch.Tensor:
     if low == high:
         high += 0.001
-    return ((torch.arange(n, dtype=torch.float32) - low) / (high - low)).clamp(0, 1)
+    return ((torch.arange(n, dtype=dtype) - low) / (high - low)).clamp(0, 1)
 
 
 def yarn_mscale(scale: float = 1.0, mscale: float = 1.0) -> float:
@@ -58,7 +58,9 @@ class RotaryEmbedding(nn.Module):
         rs = self.rope_scaling
         kind = rs.get("rope_type", rs.get("type", "default"))
         d, base, max_pos = self.rotary_dim, self.base, self.max_position
-        inv = _inv_freq(base, d)
+        # ``exact``: the table is evaluated in 64 bits and rounded once (angles of far positions keep all of their 32-bit digits)
+        dt = torch.float64 if rs.get("exact") else torch.float32
+        inv = _inv_freq(base, d, dt)
         scale_pos = 1.0
         if kind in ("default", "mrope"):
             pass
@@ -82,9 +84,12 @@ class RotaryEmbedding(nn.Module):
             orig = rs.get("original_max_position_embeddings", max_pos)
             lo, hi = _yarn_range(rs.get("beta_fast", 32), rs.get("beta_slow", 1), d, base, orig,
                                  bool(rs.get("truncate", True)))
-            mask = (1 - _yarn_ramp(lo, hi, d // 2)) * rs.get("extrapolation_factor", 1.0)
+            if rs.get("ordered_ramp"):                   # ramp ends that cross (a short original context): a step at the lower one
+                hi = max(hi, lo)
+            mask = (1 - _yarn_ramp(lo, hi, d // 2, dt)) * rs.get("extrapolation_factor", 1.0)
             inv = inv / f * (1 - mask) + inv * mask
-            max_pos = max(max_pos, int(orig * f))
+            if not rs.get("fixed_length"):               # the table may stay as long as the model's positions
+                max_pos = max(max_pos, int(orig * f))
             if kind == "deepseek_yarn" or "mscale_all_dim" in rs:
                 # DeepSeek: cos/sin carry mscale(mscale)/mscale(mscale_all_dim); the attention layer multiplies its
                 # softmax scale by mscale(mscale_all_dim)^2 (reference: rotary_embedding/deepseek_scaling_rope.py)
@@ -101,9 +106,9 @@ class RotaryEmbedding(nn.Module):
         else:
             raise ValueError(f"unsupported rope scaling type {kind!r}")
         self.max_position = max_pos
-        t = torch.arange(max_pos, dtype=torch.float32) * scale_pos
+        t = torch.arange(max_pos, dtype=dt) * scale_pos
         freqs = torch.outer(t, inv)
-        return torch.cat((freqs.cos() * self.mscale, freqs.sin() * self.mscale), dim=-1).contiguous()
+        return torch.cat((freqs.cos() * self.mscale, freqs.sin() * self.mscale), dim=-1).float().contiguous()
 
     def forward_mrope(self, positions: torch.Tensor, q: torch.Tensor, k: torch.Tensor):
         """positions [3, T] (temporal, height, width ids): channel section i of the rotary dims takes its angle from

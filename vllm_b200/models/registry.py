@@ -16,6 +16,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "MistralForCausalLM": ("llama", "MistralForCausalLM"),
     "PomipelForCausalLM": ("pomipel", "PomipelForCausalLM"),
     "LegelixForCausalLM": ("legelix", "LegelixForCausalLM"),
+    "KopadraForCausalLM": ("kopadra", "KopadraForCausalLM"),
     "Qwen2ForCausalLM": ("llama", "Qwen2ForCausalLM"),
     "Qwen3ForCausalLM": ("llama", "Qwen3ForCausalLM"),
     "GemmaForCausalLM": ("llama", "GemmaForCausalLM"),

@@ -94,6 +94,20 @@ def activation(x: torch.Tensor, name: str) -> torch.Tensor:
     return ref.ACT_FNS[name](x)
 
 
+def sigmoid_mul_(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
+    """x *= sigmoid(gate) in place, rows of any stride."""
+    if _use_cuda(x):
+        return cuda_ops().sigmoid_mul_(x, gate)
+    return x.copy_(x.float() * torch.sigmoid(gate.float()))
+
+
+def soft_cap(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    """cap tanh(logits / cap) in 32-bit; in place on CUDA."""
+    if _use_cuda(logits):
+        return cuda_ops().soft_cap_(logits, cap)
+    return (torch.tanh(logits.float() / cap) * cap).to(logits.dtype)
+
+
 _HALF = (torch.bfloat16, torch.float16)
 
 
@@ -240,6 +254,14 @@ def norm_add(x, y, y_bias, norm, mult: float, next_norm, eps: float):
     return ref.norm_add(x, y, y_bias, norm, mult, next_norm, eps)
 
 
+def add_norm(x, y, next_norm, eps: float, dtype=None):
+    """In place on the fp32 stream: x += y.  Returns the next GEMM's input in y's dtype: the layer norm ``next_norm`` (weight, bias or
+    None) of x, or x where that is None."""
+    if _use_cuda(x):
+        return cuda_ops().add_norm(x, y, next_norm, eps)
+    return ref.add_norm(x, y, next_norm, eps)
+
+
 def embed_norm(ids, table, next_norm, eps: float):
     """Entry of an fp32 stream in front of a normed sublayer: (table[ids] fp32, next_norm of it in the table's dtype)."""
     if _use_cuda(table):
@@ -257,11 +279,11 @@ def scan_state_elems(R: int, C: int) -> int:
     return -(-C // 4) * 4 * rows
 
 
-def gated_norm(y, z, weight, groups: int, eps: float, gate_first: bool, out=None, scale: float = 1.0):
-    """RMS norm of y (fp32) over equal parts with the gate silu(z) before or behind it; in z's dtype."""
+def gated_norm(y, z, weight, groups: int, eps: float, gate_first: bool, out=None, scale: float = 1.0, gate: str = "silu"):
+    """RMS norm of y (fp32) over equal parts with the gate silu(z) or sigmoid(z) before or behind it; in z's dtype."""
     if _use_cuda(y):
-        return cuda_ops().gated_norm(y, z, weight, groups, eps, gate_first, out, scale)
-    o = ref.gated_norm(y, z, weight, groups, eps, gate_first) * scale
+        return cuda_ops().gated_norm(y, z, weight, groups, eps, gate_first, out, scale, gate)
+    o = ref.gated_norm(y, z, weight, groups, eps, gate_first, gate) * scale
     return o.to(z.dtype) if out is None else out.copy_(o)
 
 
@@ -285,20 +307,22 @@ def topk_softmax(gating, k, renormalize):
 
 
 def grouped_topk(scores, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None,
-                 routed_scaling_factor=1.0):
+                 routed_scaling_factor=1.0, group_score=None):
+    """``group_score``: a group is ranked by its two best choice scores ("top2") or its best ("max"); None: by two where there is a bias."""
     if _use_cuda(scores):
         return cuda_ops().grouped_topk(scores, k, n_group, topk_group, renormalize, scoring, bias,
-                                       routed_scaling_factor)
-    return ref.grouped_topk(scores, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor)
+                                       routed_scaling_factor, group_score)
+    return ref.grouped_topk(scores, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor, group_score)
 
 
 def router_topk(x, gate, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None, routed_scaling_factor=1.0,
-                x_half=None):
+                x_half=None, group_score=None):
     """Router with 32-bit logits: (weights fp32 [T, k], ids [T, k]) of x [T, H] (fp32 stream or model dtype) with gate [E, H]."""
     if _use_cuda(x):
-        return cuda_ops().router_topk(x, gate, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor, x_half)
+        return cuda_ops().router_topk(x, gate, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor, x_half,
+                                      group_score)
     return ref.grouped_topk(x.float() @ gate.float().t(), k, n_group, topk_group, renormalize, scoring, bias,
-                            routed_scaling_factor)
+                            routed_scaling_factor, group_score)
 
 
 def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None, gated: bool = True):
@@ -318,6 +342,19 @@ def fused_moe_post_norm(stream, x, w_up, w_down, topk_w, topk_ids, act, expert_m
                                         topk_w.to(torch.float32).contiguous())
     return ref.post_norm_add(stream, ref.fused_moe(x, w_up, w_down, topk_w, topk_ids, act, expert_map, False), weight, eps, gemma,
                              next_weight, next_gemma)
+
+
+def fused_moe_add_norm(stream, x, w13, w2, topk_w, topk_ids, act, expert_map, gated: bool, experts: int, y, next_norm, eps: float):
+    """add_norm of the routed sum (identity experts: numbers from ``experts`` on add their weight times x) plus ``y`` (or None); on CUDA
+    the combine is the load of that kernel."""
+    if _use_cuda(x):
+        from vllm_b200.ops.moe import expert_rows
+        ids = topk_ids if topk_ids.dtype == torch.int32 else topk_ids.to(torch.int32)
+        rows, inv = expert_rows(x, w13, w2, ids, act, expert_map, gated)
+        return cuda_ops().add_norm(stream, y, next_norm, eps, x.dtype, rows, inv, topk_w.to(torch.float32).contiguous(), ids, experts,
+                                   x if expert_map is not None and expert_map.numel() > experts else None)
+    out = ref.fused_moe(x, w13, w2, topk_w, topk_ids, act, expert_map, gated) + ref.identity_experts(x, topk_w, topk_ids, experts)
+    return ref.add_norm(stream, out if y is None else out + y, next_norm, eps)
 
 
 def block_fp8_linear(x, wq, w_scale, block=128, bias=None):

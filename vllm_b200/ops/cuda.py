@@ -200,6 +200,25 @@ def silu_and_mul_interleaved(x):
     return out
 
 
+_sigmoid_mul = _sig("vb_sigmoid_mul", _vp, _i64, _vp, _i64, _vp, _i64, _i64, _i, _i, _vp)
+_soft_cap = _sig("vb_soft_cap", _vp, _i64, _i64, _i, _f, _i, _vp)
+
+
+def sigmoid_mul_(x, g):
+    """x *= sigmoid(g) in place; rows of any stride."""
+    assert x.dim() == 2 and x.shape == g.shape and x.dtype == g.dtype and x.stride(1) == g.stride(1) == 1
+    _check(_sigmoid_mul(x.data_ptr(), x.stride(0), g.data_ptr(), g.stride(0), x.data_ptr(), x.stride(0), x.shape[0], x.shape[1],
+                        _DT[x.dtype], _st()), "sigmoid_mul")
+    return x
+
+
+def soft_cap_(x, cap: float):
+    """x = cap tanh(x / cap) in place; rows of any stride."""
+    assert x.dim() == 2 and x.stride(1) == 1
+    _check(_soft_cap(x.data_ptr(), x.stride(0), x.shape[0], x.shape[1], cap, _DT[x.dtype], _st()), "soft_cap")
+    return x
+
+
 def activation(x, name: str):
     xc = _rows(x)
     out = torch.empty_like(xc)
@@ -677,6 +696,27 @@ def norm_add(x, y, y_bias, norm, mult: float, next_norm, eps: float, ids=None):
     return x if out is None else out
 
 
+_add_norm = _sig("vb_add_norm", _vp, _i64, _vp, _i64, _vp, _vp, _vp, _i, _i, _vp, _i64, _vp, _vp, _vp, _i, _i, _vp, _i, _i, _f, _i, _vp)
+
+
+def add_norm(x, y, next_norm, eps: float, dtype=None, rows=None, inv=None, pair_w=None, ids=None, experts: int = 0, h=None):
+    """In place on the fp32 stream: x += y + routed sum (``rows`` of the experts by ``inv``, weights ``pair_w``, and ``h`` for expert
+    numbers from ``experts`` on).  ``next_norm``: (weight, bias or None) of a layer norm.  Returns next_norm(x) — or x — in ``dtype``
+    (y's)."""
+    T, H = x.shape
+    dtype = dtype or y.dtype
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    assert all(t is None or (t.dtype == dtype and t.stride(-1) == 1) for t in (y, rows, h)) and (ids is None or ids.dtype == torch.int32)
+    w2, b2 = next_norm if next_norm is not None else (None, None)
+    out = torch.empty((T, H), dtype=dtype, device=x.device) if w2 is not None or dtype != torch.float32 else None
+
+    def st(t):
+        return 0 if t is None else t.stride(0)
+    _check(_add_norm(_p(y), st(y), _p(rows), st(rows), _p(inv), _p(pair_w), _p(ids), 0 if pair_w is None else pair_w.shape[1], experts,
+                     _p(h), st(h), x.data_ptr(), _p(w2), _p(b2), 0, 1, _p(out), T, H, eps, _DT[dtype], _st()), "add_norm")
+    return x if out is None else out
+
+
 # ------------------------------------------------------------------ GEMM
 class _GemmWorkspace:
     def __init__(self) -> None:
@@ -880,7 +920,7 @@ _moe_combine = _sig("vb_moe_combine", _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp)
 _moe_gather = _sig("vb_moe_gather", _vp, _vp, _vp, _i, _i, _i, _vp)
 _gemm_grouped = _sig("vb_gemm_tc_grouped2", _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp)
 _grouped_simt = _sig("vb_moe_grouped_simt", _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp)
-_grouped_topk = _sig("vb_moe_grouped_topk", _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp)
+_grouped_topk = _sig("vb_moe_grouped_topk", _vp, _vp, _i, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp)
 _GROUPED_ACT = {None: 0, "none": 0, "relu2": 2}
 
 
@@ -986,22 +1026,27 @@ def grouped_simt(x: torch.Tensor, w: torch.Tensor, offs: torch.Tensor, R: int, r
     return y
 
 
-def grouped_topk(scores, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None, routed_scaling_factor=1.0):
+def grouped_topk(scores, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None, routed_scaling_factor=1.0, group_score=None):
     T, E = scores.shape
     lg = scores.float().contiguous()
     w = torch.empty((T, k), dtype=torch.float32, device=scores.device)
     ids = torch.empty((T, k), dtype=torch.int32, device=scores.device)
     b = None if bias is None else bias.float().contiguous()
     _check(_grouped_topk(lg.data_ptr(), None, 0, None, 0, _p(b), w.data_ptr(), ids.data_ptr(), T, E, k, n_group,
-                         topk_group if n_group > 1 else 1, int(scoring != "sigmoid"), int(renormalize), float(routed_scaling_factor),
-                         2, _st()), f"grouped_topk(E={E},k={k})")
+                         topk_group if n_group > 1 else 1, _group_top2(group_score, bias), int(scoring != "sigmoid"), int(renormalize),
+                         float(routed_scaling_factor), 2, _st()), f"grouped_topk(E={E},k={k})")
     return w, ids
+
+
+def _group_top2(group_score: Optional[str], bias) -> int:
+    return int(bias is not None if group_score is None else group_score == "top2")
 
 
 ROUTER_FUSED_TOKENS = 256       # above this the logits come from one tensor-core product with fp32 output
 
 
-def router_topk(x, gate, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None, routed_scaling_factor=1.0, x_half=None):
+def router_topk(x, gate, k, n_group, topk_group, renormalize, scoring="sigmoid", bias=None, routed_scaling_factor=1.0, x_half=None,
+                group_score=None):
     """Routing of x [T, H] (fp32 stream or model dtype) with gate [E, H]: 32-bit logits, scores, choice and weights.
     ``x_half``: the 16-bit copy of x for the large-batch product."""
     T, H = x.shape
@@ -1012,14 +1057,14 @@ def router_topk(x, gate, k, n_group, topk_group, renormalize, scoring="sigmoid",
             lg = x.float() @ gate.float().t()
         else:
             lg = torch.mm(xh, gate.t(), out_dtype=torch.float32)
-        return grouped_topk(lg, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor)
+        return grouped_topk(lg, k, n_group, topk_group, renormalize, scoring, bias, routed_scaling_factor, group_score)
     w = torch.empty((T, k), dtype=torch.float32, device=x.device)
     ids = torch.empty((T, k), dtype=torch.int32, device=x.device)
     assert x.is_contiguous() and gate.is_contiguous() and (x.dtype == torch.float32 or x.dtype == gate.dtype)
     assert bias is None or bias.dtype == torch.float32
     _check(_grouped_topk(None, x.data_ptr(), int(x.dtype == torch.float32), gate.data_ptr(), H, _p(bias), w.data_ptr(),
-                         ids.data_ptr(), T, E, k, n_group, topk_group if n_group > 1 else 1, int(scoring != "sigmoid"),
-                         int(renormalize), float(routed_scaling_factor), _DT[gate.dtype], _st()), f"router_topk(E={E},k={k},H={H})")
+                         ids.data_ptr(), T, E, k, n_group, topk_group if n_group > 1 else 1, _group_top2(group_score, bias),
+                         int(scoring != "sigmoid"), int(renormalize), float(routed_scaling_factor), _DT[gate.dtype], _st()), f"router_topk(E={E},k={k},H={H})")
     return w, ids
 
 
@@ -1282,15 +1327,29 @@ _qknorm_rope_any = _sig("vb_qknorm_rope_any", _vp, _vp, _vp, _vp, _vp, _vp, _vp,
                         _vp, _i, _i, _i, _i, _f, _i, _vp)
 
 
+_qknorm_rope_row = _sig("vb_qknorm_rope_row", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i64, _i64, _i64, _vp,
+                        _vp, _i, _i, _i, _i, _f, _i, _vp)
+
+
 def fused_qk_norm_rope(positions, q, k, q_weight, k_weight, cos_sin_cache, head_dim, eps, is_neox=True, *, v=None,
                        kv_cache=None, slot_mapping=None, gemma: bool = False, k_scale: float = 1.0, v_scale: float = 1.0,
-                       vt: bool = False, v_head_dim: Optional[int] = None, keep32: bool = False):
+                       vt: bool = False, v_head_dim: Optional[int] = None, keep32: bool = False, whole: bool = False):
     """In place: per-head RMSNorm(q), RMSNorm(k) → RoPE → (optionally) K/V insert into the paged cache; one launch.
-    ``keep32``: no rounding to the model dtype between the norm and the rotation."""
+    ``keep32``: no rounding to the model dtype between the norm and the rotation.  ``whole``: one norm over all heads (weights as
+    long); ``k`` may be None."""
     T = q.shape[0]
-    Hq, Hkv = q.shape[-1] // head_dim, k.shape[-1] // head_dim
+    Hq, Hkv = q.shape[-1] // head_dim, 0 if k is None else k.shape[-1] // head_dim
     rot = cos_sin_cache.shape[-1] if cos_sin_cache is not None else 0
-    assert q.stride(-1) == 1 and k.stride(-1) == 1
+    assert q.stride(-1) == 1 and (k is None or k.stride(-1) == 1)
+    if whole:
+        dv = v_head_dim or head_dim
+        BS, dc = (kv_cache.shape[3], kv_cache.shape[4]) if kv_cache is not None else (1, max(head_dim, dv))
+        assert kv_cache is None or kv_cache.dtype == q.dtype, "whole-projection norms write caches of the model dtype"
+        _check(_qknorm_rope_row(_p(positions), q.data_ptr(), _p(k), _p(v), _p(q_weight), _p(k_weight), _p(cos_sin_cache), rot, T, Hq, Hkv,
+                                head_dim, dv, dc, q.stride(0), 0 if k is None else k.stride(0), 0 if v is None else v.stride(0),
+                                _p(kv_cache), _p(slot_mapping), BS, int(is_neox), int(gemma), int(vt), eps, _DT[q.dtype], _st()),
+               "qknorm_rope_row")
+        return q, k
     flags = 4 if keep32 else 0
     BS = 1
     dv = v_head_dim or head_dim
@@ -1317,7 +1376,7 @@ def fused_qk_norm_rope(positions, q, k, q_weight, k_weight, cos_sin_cache, head_
 # ------------------------------------------------------------------ cache maintenance (csrc/cache_ops.cu)
 _copy_blocks = _sig("vb_copy_blocks", _vp, _vp, _vp, _i, _i64, _vp)
 _gather_cache = _sig("vb_gather_cache", _vp, _vp, _vp, _i64, _vp, _vp, _i, _i, _i, _i, _i64, _i64, _f, _i, _i, _vp)
-_convert_fp8 = _sig("vb_convert_fp8", _vp, _vp, _i64, _f, _i, _i, _vp)
+_convert_fp8 = _sig("vb_convert_fp8", _vp, _vp, _i64, _f, _i, _i, _i, _vp)
 
 
 def swap_blocks(src: torch.Tensor, dst: torch.Tensor, mapping) -> None:
@@ -1378,7 +1437,10 @@ _ssd_scan = _sig("vb_ssd_scan", _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _
 _gla_scan = _sig("vb_gla_scan", _vp, _vp, _vp, _i64, _i64, _i64, _f, _vp, _vp, _i64, _vp, _vp, _i, _f, _vp, _vp, _i64, _i64, _vp, _vp,
                  _vp, _i64, _i, _i, _i, _i, _i, _i, _vp)
 _gla_decay = _sig("vb_gla_decay", _vp, _i64, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp)
-_gated_norm = _sig("vb_gated_norm", _vp, _vp, _i64, _vp, _i, _vp, _i64, _i, _i, _i, _i, _f, _f, _i, _vp)
+_gated_norm = _sig("vb_gated_norm", _vp, _vp, _vp, _i64, _vp, _i, _vp, _i64, _i, _i, _i, _i, _f, _f, _i, _vp)
+_memory_scan = _sig("vb_memory_scan", _vp, _vp, _vp, _i64, _i64, _i64, _f, _vp, _vp, _vp, _i64, _i64, _vp, _vp, _vp, _i64, _i, _i, _i, _i,
+                    _i, _i, _vp)
+_memory_gates = _sig("vb_memory_gates", _vp, _i64, _vp, _i, _vp, _vp, _f, _vp, _vp, _i64, _i64, _vp, _vp, _vp, _i64, _i, _i, _i, _i, _vp)
 _gdn_scan = _sig("vb_gdn_scan", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _vp, _vp, _vp, _i64, _i, _i, _i, _i, _vp)
 
 
@@ -1459,17 +1521,51 @@ def gla_scan(q, k, v, a1, a2, a2_bias, tau: float, q_scale: float, cache, md, H:
     return o
 
 
-def gated_norm(y, z, weight, groups: int, eps: float, gate_first: bool, out=None, scale: float = 1.0):
-    """y fp32 [T, n]: RMS norm over ``groups`` equal parts, silu(z) before (``gate_first``) or behind it, times the weight
-    (repeated along the parts where it is shorter) and ``scale``; in z's dtype."""
-    T, n = y.shape
+def memory_gates(h, w, bias, cap: float, cache, m_off: int, md):
+    """Gates of a matrix memory: h [T, W] (row stride free), w [2 heads, W] (input gates, forget gates), bias fp32 → [T, heads, 4] fp32
+    (decay, input factor, exp(-m), -); the slots' running maxima at ``m_off`` advance in place.  32-bit throughout."""
+    T, H = h.shape[0], w.shape[0] // 2
+    st = _state_view(cache)
+    bt = md.block_table
+    assert h.stride(1) == 1 and w.is_contiguous() and w.dtype == h.dtype and bias.dtype == torch.float32
+    gates = _scan_out(T, H * 4, md, h.device)
+    logits = None
+    if not md.decode_only:
+        logits = torch.mm(h, w.t(), out_dtype=torch.float32) if h.dtype != torch.float32 else h @ w.t()
+    _check(_memory_gates(h.data_ptr(), h.stride(0), w.data_ptr(), h.shape[1], _p(logits), bias.data_ptr(), cap, gates.data_ptr(),
+                         st.data_ptr(), st.stride(0), m_off, md.query_start_loc.data_ptr(), md.seq_lens.data_ptr(), bt.data_ptr(),
+                         bt.stride(0), md.num_reqs, md.max_query_len, H, _DT[h.dtype], _st()), "memory_gates")
+    return gates.view(T, H, 4)
+
+
+def memory_scan(q, k, v, gates, q_scale: float, cache, md, H: int, R: int, C: int, state_off: int = 0):
+    """Matrix memory: q, k [T, H*R], v [T, H*C] (row strides free) → [T, H, C rounded up to four + 4] fp32, n . q in the last quad's
+    first column; the slots' states advance in place."""
+    T = q.shape[0]
+    st = _state_view(cache)
+    cols = -(-C // 4) * 4 + 4
+    o = _scan_out(T, H * cols, md, q.device)
+    bt = md.block_table
+    assert all(t.stride(1) == 1 and t.dtype == q.dtype for t in (q, k, v)) and gates.is_contiguous()
+    _check(_memory_scan(q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), k.stride(0), v.stride(0), q_scale, gates.data_ptr(),
+                        o.data_ptr(), st.data_ptr(), st.stride(0), state_off, md.query_start_loc.data_ptr(), md.seq_lens.data_ptr(),
+                        bt.data_ptr(), bt.stride(0), md.num_reqs, md.max_query_len, H, R, C, _DT[q.dtype], _st()), "memory_scan")
+    return o.view(T, H, cols)
+
+
+def gated_norm(y, z, weight, groups: int, eps: float, gate_first: bool, out=None, scale: float = 1.0, gate: str = "silu", gates=None):
+    """y fp32 [T, n]: RMS norm over ``groups`` equal parts, silu(z) (``gate`` "sigmoid": sigmoid(z)) before (``gate_first``) or behind it,
+    times the weight (repeated along the parts where it is shorter) and ``scale``; in z's dtype.  ``gates``: y is the result of
+    ``memory_scan`` with these gates, divided by its normaliser first."""
+    T, n = z.shape
     if out is None:
         out = torch.empty((T, n), dtype=z.dtype, device=z.device)
     W = n // groups
     wl = weight.numel()
     assert y.is_contiguous() and z.stride(1) == 1 and out.stride(1) == 1 and weight.dtype == z.dtype and n % groups == 0 and n % wl == 0
-    _check(_gated_norm(y.data_ptr(), z.data_ptr(), z.stride(0), weight.data_ptr(), wl, out.data_ptr(), out.stride(0), T, groups, W,
-                       int(gate_first), eps, scale, _DT[z.dtype], _st()), "gated_norm")
+    assert y.numel() == T * groups * (W if gates is None else -(-W // 4) * 4 + 4)
+    _check(_gated_norm(y.data_ptr(), _p(gates), z.data_ptr(), z.stride(0), weight.data_ptr(), wl, out.data_ptr(), out.stride(0), T, groups,
+                       W, int(gate_first) | 2 * int(gate == "sigmoid"), eps, scale, _DT[z.dtype], _st()), "gated_norm")
     return out
 
 

@@ -56,6 +56,27 @@ def _tile_width(R: int, E: int) -> int:
     return bn
 
 
+def expert_rows(x, w13, w2, topk_ids, act, expert_map, gated: bool):
+    """(rows [R, H] of expert outputs sorted by expert, inv [R]: (token, slot) pair → row, or -1), on the device at every batch size."""
+    return expert_rows_gated(x, w13, w2, topk_ids, act, expert_map) if gated else expert_rows_plain(x, w13, w2, topk_ids, act, expert_map)
+
+
+def expert_rows_gated(x, w13, w2, topk_ids, act, expert_map):
+    """Experts act(gate) * up → down; ``expert_rows_plain`` with the activation as a kernel between the two grouped GEMMs."""
+    from vllm_b200.ops import cuda as cu
+    T, k = topk_ids.shape
+    R, E, (N, K) = T * k, w13.shape[0], w13.shape[1:]
+    ids = topk_ids if topk_ids.dtype == torch.int32 else topk_ids.to(torch.int32)
+    sorted_tok, inv, offs = cu.moe_align(ids.contiguous(), E, expert_map)
+    x = x.contiguous()
+    if x.dtype in (torch.bfloat16, torch.float16) and w13.dtype == x.dtype and K % 8 == 0 and N % 16 == 0:
+        bn = _tile_width(R, E)
+        h = cu.gemm_tc_grouped(cu.moe_gather(x, sorted_tok), w13, offs, bn, flat=True)
+        return cu.gemm_tc_grouped(cu.act_and_mul(h, act), w2, offs, bn, flat=True), inv
+    h = cu.grouped_simt(x, w13, offs, R, sorted_tok)
+    return cu.grouped_simt(cu.act_and_mul(h, act), w2, offs, R), inv
+
+
 def expert_rows_plain(x, w_up, w_down, topk_ids, act, expert_map):
     """Experts without a gate, up → act → down: (rows [R, H] sorted by expert, inv [R]: (token, slot) pair → row).
 
@@ -83,10 +104,14 @@ def expert_rows_plain(x, w_up, w_down, topk_ids, act, expert_map):
     return cu.grouped_simt(a, w_down, offs, R), inv
 
 
-def fused_moe_plain(x, w_up, w_down, topk_w, topk_ids, act, expert_map):
+def combine_rows(rows, inv, topk_w, T: int):
     from vllm_b200.ops import cuda as cu
+    return cu.moe_combine(rows, inv, topk_w.to(torch.float32).contiguous(), T)
+
+
+def fused_moe_plain(x, w_up, w_down, topk_w, topk_ids, act, expert_map):
     rows, inv = expert_rows_plain(x, w_up, w_down, topk_ids, act, expert_map)
-    return cu.moe_combine(rows, inv, topk_w.to(torch.float32).contiguous(), x.shape[0])
+    return combine_rows(rows, inv, topk_w, x.shape[0])
 
 
 def fused_moe_fp8_grouped(x, w13q, w13_scale, w2q, w2_scale, topk_w, topk_ids, expert_map):
@@ -180,6 +205,9 @@ def fused_moe_cuda(x, w13, w2, topk_w, topk_ids, act="silu", expert_map: Optiona
     T, H = x.shape
     E = w13.shape[0]
     k = topk_ids.shape[1]
+    if T * k <= GROUPED_MAX_ROWS and w13.dtype == x.dtype and w13.is_contiguous() and w2.is_contiguous():
+        rows, inv = expert_rows_gated(x, w13, w2, topk_ids, act, expert_map)      # sizes off the 128-byte grid, fp32: no host sync
+        return combine_rows(rows, inv, topk_w, T)
     ids = topk_ids.long()
     if expert_map is not None:
         ids = expert_map[ids].long()
@@ -198,7 +226,7 @@ def fused_moe_cuda(x, w13, w2, topk_w, topk_ids, act="silu", expert_map: Optiona
         if n == 0:
             continue
         h = ops.linear(xs[off:off + n], w13[e])
-        h = ops.silu_and_mul(h) if act == "silu" else ops.gelu_and_mul(h)
+        h = ops.cuda_ops().act_and_mul(h, act)
         y = ops.linear(h, w2[e]).float() * ws[off:off + n, None]
         out.index_add_(0, tok[off:off + n], y)
         off += n

@@ -95,7 +95,8 @@ def fused_qk_norm_rope(positions: torch.Tensor, q: torch.Tensor, k: torch.Tensor
 
 ACT_FNS = {
     "relu": F.relu, "gelu": F.gelu, "gelu_new": gelu_new, "gelu_fast": gelu_fast,
-    "gelu_pytorch_tanh": lambda x: F.gelu(x, approximate="tanh"), "quick_gelu": quick_gelu,
+    "gelu_pytorch_tanh": lambda x: F.gelu(x, approximate="tanh"), "gelu_tanh": lambda x: F.gelu(x, approximate="tanh"),
+    "quick_gelu": quick_gelu,
     "silu": F.silu, "relu2": lambda x: F.relu(x).square(),
 }
 
@@ -336,9 +337,17 @@ def norm_add(x: torch.Tensor, y: torch.Tensor, y_bias: Optional[torch.Tensor], n
     return (x if next_norm is None else layer_norm(x, *next_norm, eps)).to(y.dtype)
 
 
-def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, gate_first: bool) -> torch.Tensor:
-    """fp32: rms norm of y over ``groups`` equal parts, times the weight (repeated along the parts), silu(z) first or last."""
-    gate = F.silu(z.float())
+def add_norm(x: torch.Tensor, y: torch.Tensor, next_norm, eps: float) -> torch.Tensor:
+    """In place: x (fp32) += y.  Returns x in y's dtype, or its layer norm with ``next_norm``."""
+    x += y.float()
+    return (x if next_norm is None else layer_norm(x, *next_norm, eps)).to(y.dtype)
+
+
+def gated_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, gate_first: bool, gate: str = "silu"
+               ) -> torch.Tensor:
+    """fp32: rms norm of y over ``groups`` equal parts, times the weight (repeated along the parts), silu(z) or sigmoid(z) first or
+    last."""
+    gate = F.silu(z.float()) if gate == "silu" else torch.sigmoid(z.float())
     y = y.float() * gate if gate_first else y.float()
     g = y.reshape(y.shape[0], groups, -1)
     y = (g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)).reshape(y.shape)
@@ -355,6 +364,21 @@ def gated_linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, alpha: 
         state = alpha[t][..., None] * state + k[t][..., None] * v[t][:, None]
         o[t] = (state * q[t][..., None]).sum(1)
     return o, state
+
+
+def matrix_memory_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Tensor, f: torch.Tensor, S: torch.Tensor,
+                       n: torch.Tensor, m: torch.Tensor):
+    """One sequence.  q, k [T, H, R], v [T, H, C], log input and forget gates i, f [T, H]; S [H, R, C], n [H, R], m [H] fp32 →
+    (o [T, H, C], S, n, m):  S = exp(f + m' - m) S + exp(i - m) k v^T (n with k alone), m the running maximum of f + m' and i."""
+    o = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        top = torch.maximum(f[t] + m, i[t])
+        keep, new = torch.exp(f[t] + m - top)[:, None], torch.exp(i[t] - top)[:, None] * k[t]
+        m = top
+        S = keep[..., None] * S + new[..., None] * v[t][:, None]
+        n = keep * n + new
+        o[t] = (S * q[t][..., None]).sum(1) / (torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6)[:, None]
+    return o, S, n, m
 
 
 # -------------------------------------------------------------- sampling
@@ -439,14 +463,15 @@ def topk_softmax(gating: torch.Tensor, k: int, renormalize: bool) -> tuple[torch
 
 def grouped_topk(scores_in: torch.Tensor, k: int, n_group: int, topk_group: int, renormalize: bool,
                  scoring: str = "sigmoid", bias: Optional[torch.Tensor] = None,
-                 routed_scaling_factor: float = 1.0) -> tuple[torch.Tensor, torch.Tensor]:
-    """DeepSeek group-limited routing."""
+                 routed_scaling_factor: float = 1.0, group_score: Optional[str] = None) -> tuple[torch.Tensor, torch.Tensor]:
+    """DeepSeek group-limited routing (``group_score`` "max": a group counts by its best choice score)."""
     s = scores_in.float().sigmoid() if scoring == "sigmoid" else scores_in.float().softmax(-1)
     T, E = s.shape
     sel = s + bias.float()[None] if bias is not None else s
     if n_group > 1:
         g = sel.view(T, n_group, E // n_group)
-        gs = g.topk(min(2, E // n_group), dim=-1).values.sum(-1) if bias is not None else g.max(-1).values
+        gs = g.topk(min(2, E // n_group), dim=-1).values.sum(-1) if (
+            bias is not None if group_score is None else group_score == "top2") else g.max(-1).values
         gi = gs.topk(topk_group, dim=-1).indices
         gm = torch.zeros_like(gs).scatter_(1, gi, 1.0)
         mask = gm[:, :, None].expand(T, n_group, E // n_group).reshape(T, E)
@@ -478,11 +503,16 @@ def fused_moe(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torc
             out.index_add_(0, tok, y * topk_w[tok, slot].float()[:, None])
             continue
         I = h.shape[-1] // 2
-        a = F.silu(h[:, :I]) if act == "silu" else F.gelu(h[:, :I])
+        a = ACT_FNS[act](h[:, :I])
         h = (a * h[:, I:]).to(x.dtype).float()
         y = h @ w2[e].float().t()
         out.index_add_(0, tok, y * topk_w[tok, slot].float()[:, None])
     return out.to(x.dtype)
+
+
+def identity_experts(x: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor, experts: int) -> torch.Tensor:
+    """What expert numbers from ``experts`` on contribute: their weights times the input."""
+    return (x.float() * (topk_w.float() * (topk_ids >= experts)).sum(-1, keepdim=True)).to(x.dtype)
 
 
 # ---------------------------------------------------------- cache maintenance
