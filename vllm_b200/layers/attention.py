@@ -253,7 +253,7 @@ class Attention(nn.Module):
                                 self.sliding_window, self.logits_soft_cap, self.causal, out=buf,
                                 alibi_slopes=self.alibi_slopes, sinks=self.sinks, chunk_size=self.chunk_size,
                                 v_head_size=self.v_head_size, out_scale=self.out_scale)
-        return o.view(T, self.num_heads * self.v_head_size) if out is None else out
+        return o.reshape(T, self.num_heads * self.v_head_size) if out is None else out
 
 
 class MLAAttentionCore(nn.Module):
