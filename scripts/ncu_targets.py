@@ -91,3 +91,32 @@ if which in ("scan", "all"):
         a2, a2b = torch.randn(GH * 128, 16, device="cuda").to(dt), torch.randn(GH * 128, device="cuda").to(dt)
         pool2 = torch.zeros(n + 1, GH * scan_state_elems(128, 256), device="cuda")
         rep(lambda: cu.gla_scan(qq, kk, vv, a1, a2, a2b, 16.0, 0.09, pool2, md, GH, 128, 256))
+if which in ("memory", "all"):
+    # Kopadra: gates, scan and norm of a matrix memory (prompts of 1024 tokens each, a decode batch), experts of a prompt step with
+    # identity experts and the step that combines them, at the sizes of a 2048-wide model
+    from vllm_b200.forward_context import AttentionMetadata
+    from vllm_b200.ops import moe, scan_state_elems
+    MH, R, C, W, i32 = 8, 128, 256, 2048, dict(dtype=torch.int32, device="cuda")
+    m_off = MH * scan_state_elems(R, C + 4)
+    for n, q in ((4, 1024), (64, 1)):
+        T = n * q
+        md = AttentionMetadata(num_reqs=n, num_actual_tokens=T, max_query_len=q, max_seq_len=q, query_start_loc=torch.arange(0, T + 1, q, **i32),
+                               seq_lens=torch.full((n,), q + (q == 1), **i32), block_table=(torch.arange(n, **i32) + 1).view(-1, 1),
+                               slot_mapping=None, decode_only=q == 1)
+        h, w, b = (torch.randn(T, W, device="cuda") * 0.3).to(dt), (torch.randn(2 * MH, W, device="cuda") * 0.02).to(dt), torch.randn(2 * MH, device="cuda")
+        x, nw = (torch.randn(T, MH * (2 * R + 2 * C), device="cuda") * 0.3).to(dt), torch.ones(MH * C, device="cuda", dtype=dt)
+        qq, kk, vv, gg = x.split([MH * R, MH * R, MH * C, MH * C], -1)
+        pool3 = torch.zeros(n + 1, m_off + MH, device="cuda")
+        rep(lambda: cu.gated_norm(cu.memory_scan(qq, kk, vv, cu.memory_gates(h, w, b, 15.0, pool3, m_off, md), 0.09, pool3, md, MH, R, C),
+                                  gg, nw, MH, 1e-6, False, gate="sigmoid",
+                                  gates=cu.memory_gates(h, w, b, 15.0, pool3, m_off, md)))
+    x = torch.randn(4096, W, device="cuda", dtype=dt) * 0.1
+    w13, w2 = (torch.randn(*s, device="cuda", dtype=dt) * 0.02 for s in ((48, 2 * 768, W), (48, W, 768)))
+    ids = torch.rand(4096, 64, device="cuda").topk(8, -1).indices.int()
+    pw, emap = torch.rand(4096, 8, device="cuda"), torch.cat([torch.arange(48, **i32), torch.full((16,), -1, **i32)])
+    stream, nw = torch.zeros(4096, W, device="cuda"), torch.ones(W, device="cuda", dtype=dt)
+
+    def experts():
+        rows, inv = moe.expert_rows_gated(x, w13, w2, ids, "silu", emap)
+        cu.add_norm(stream, x, (nw, None), 1e-6, dt, rows, inv, pw, ids, 48, x)
+    rep(experts)

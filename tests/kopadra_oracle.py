@@ -266,7 +266,13 @@ def only_memory():
     return config(64, 96, [(memory(2, 16, 24), dense(40)), (memory(4, 24, 8, cap=2.0), moe(24, 4, 2, 2, (3, 2), 24))])
 
 
-MODELS = dict(small=small, uneven=uneven, wide=wide, middling=middling, only_memory=only_memory)
+def only_attention():
+    """No recurrent layer, hence no state slots; finished prompts stay in the prefix cache, for the layers that share keys too."""
+    return config(64, 96, [(attn(4, 1, 16, 16, 8), dense(40)), (attn(4, 1, 16, 16, 16, scale=0.4, kv_from=0), moe(24, 5, 1, 3, (3, 2))),
+                           (attn(4, 1, 16, 16, 4, kv_from=0), None)])
+
+
+MODELS = dict(small=small, uneven=uneven, wide=wide, middling=middling, only_memory=only_memory, only_attention=only_attention)
 
 
 def make_weights(cfg, seed=0, steady=False, lasting=False, input_bias=0.0):

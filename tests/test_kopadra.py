@@ -437,7 +437,7 @@ def test_logits_are_capped(tmp_path, place):
 
 
 # ------------------------------------------------------------------------------------------------ generation
-@pytest.mark.parametrize("name", ["small", "wide", "only_memory"])
+@pytest.mark.parametrize("name", ["small", "wide", "only_memory", "only_attention"])
 def test_greedy_generation(tmp_path, place, name):
     """Through LLM.generate: chunked prompts (64 tokens a step), decode steps beside them, several requests."""
     cfg = ko.MODELS[name]()

@@ -478,9 +478,9 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ a1
 
 // Gates of a matrix memory, one CTA per request and head.  z = W h + b, capped: z' = cap tanh(z / cap); log input gate i = z'_i, log
 // forget gate f = log sigmoid(z'_f);  m_t = max(m_{t-1} + f_t, i_t), m before the first token 0;  out = (exp(f + m_{t-1} - m_t),
-// exp(i - m_t), exp(-m_t), 0).  A token maps m to max(m + F, M) with (F, M) = (f, i), and so does a run of tokens: blocks of GATE_T
-// tokens are scanned in parallel.  logits null: one token per request, and the two products are computed here.
-constexpr int GATE_T = 256;
+// exp(i - m_t), exp(-m_t), 0).  A token maps m to max(m + F, M) with (F, M) = (f, i), and so does a run of tokens: blocks of
+// blockDim tokens are scanned in parallel.  logits null: one token per request, and the two products are computed here.
+constexpr int GATE_T = 256, GATE_MAX_T = 1024;
 struct GateParams {
   const void* h; int64_t h_stride; const void* w; int W;
   const float* logits;                       // [T, 2 H], before the bias
@@ -493,13 +493,13 @@ struct GateParams {
 VB_DEVICE float2 compose(float2 a, float2 b) { return make_float2(a.x + b.x, fmaxf(a.y + b.x, b.y)); }      // a, then b
 
 template <typename T, int V>
-__global__ void __launch_bounds__(GATE_T) memory_gates_kernel(const GateParams p) {
+__global__ void __launch_bounds__(GATE_MAX_T) memory_gates_kernel(const GateParams p) {
   __shared__ float red[32];
-  __shared__ float2 runs[GATE_T / 32];
-  __shared__ float ms[GATE_T];
+  __shared__ float2 runs[32];
+  __shared__ float ms[GATE_MAX_T];
   pdl_trigger();
   pdl_wait();
-  const int req = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int req = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, width = blockDim.x;
   const int t0 = p.qsl[req], n = p.qsl[req + 1] - t0;
   if (n <= 0) return;
   float* slot = p.state + (int64_t)p.rows[req * p.rows_stride] * p.state_stride + p.m_off + hd;
@@ -515,7 +515,7 @@ __global__ void __launch_bounds__(GATE_T) memory_gates_kernel(const GateParams p
     const T* wi = reinterpret_cast<const T*>(p.w) + (int64_t)hd * p.W;
     const T* wf = wi + (int64_t)p.H * p.W;
     float zi = 0.f, zf = 0.f;
-    for (int c = tid * V; c < p.W; c += GATE_T * V) {
+    for (int c = tid * V; c < p.W; c += width * V) {
       if constexpr (V == 4) {
         constexpr int dt = DTypeOf<T>::v;
         const float4 x = ld_any4(h, c, dt), a = ld_any4(wi, c, dt), b = ld_any4(wf, c, dt);
@@ -535,7 +535,15 @@ __global__ void __launch_bounds__(GATE_T) memory_gates_kernel(const GateParams p
     }
     return;
   }
-  for (int b0 = 0; b0 < n; b0 += GATE_T) {
+  auto scan = [&](float2 run) {                                 // of the warp's lanes, each with those before it
+#pragma unroll
+    for (int d = 1; d < 32; d *= 2) {
+      const float2 o = make_float2(__shfl_up_sync(0xffffffffu, run.x, d), __shfl_up_sync(0xffffffffu, run.y, d));
+      if (lane >= d) run = compose(o, run);
+    }
+    return run;
+  };
+  for (int b0 = 0; b0 < n; b0 += width) {
     const int t = b0 + tid;
     float i = -INFINITY, f = 0.f;                               // behind the last token: m stays
     if (t < n) {
@@ -543,21 +551,20 @@ __global__ void __launch_bounds__(GATE_T) memory_gates_kernel(const GateParams p
       i = capped(z[0] + bi);
       f = log_sigmoid(capped(z[p.H] + bf));
     }
-    float2 run = make_float2(f, i);
-#pragma unroll
-    for (int d = 1; d < 32; d *= 2) {
-      const float2 o = make_float2(__shfl_up_sync(0xffffffffu, run.x, d), __shfl_up_sync(0xffffffffu, run.y, d));
-      if (lane >= d) run = compose(o, run);
-    }
+    const float2 run = scan(make_float2(f, i));
     if (lane == 31) runs[warp] = run;
     __syncthreads();
-    float before = m;                                           // m in front of this warp's tokens
-    for (int w = 0; w < warp; ++w) before = fmaxf(before + runs[w].x, runs[w].y);
+    if (warp == 0) {
+      const float2 all = scan(lane < width / 32 ? runs[lane] : make_float2(0.f, -INFINITY));
+      runs[lane] = all;
+    }
+    __syncthreads();
+    const float before = warp ? fmaxf(m + runs[warp - 1].x, runs[warp - 1].y) : m;
     const float after = fmaxf(before + run.x, run.y);
     ms[tid] = after;
     __syncthreads();
     if (t < n) p.out[(int64_t)(t0 + t) * p.H + hd] = gates(f, i, tid ? ms[tid - 1] : m, after);
-    m = ms[GATE_T - 1];
+    m = ms[width - 1];
     __syncthreads();
   }
   if (tid == 0) *slot = m;
@@ -691,7 +698,12 @@ int scan_shape(ScanParams& p, int mode, int num_reqs, int max_len, cudaStream_t 
    : mode == DECAY_GATES ? scan_launch<NP, L, SNP, SL, DECAY_GATES, 1, TB, PH>(p, num_reqs, w, st)       \
                          : scan_launch<NP, L, SNP, SL, DECAY_GIVEN, 1, TB, 4>(p, num_reqs, w, st))
   if (quads / (32 / L2) >= WARPS) {
-    const int w = cta_warps(32 / L2, CTAS);
+    constexpr int per = 32 / L2;
+    int w = cta_warps(per, CTAS);
+    if (mode == DECAY_GATES && w >= 4) {                                // the normaliser's quad: one more warp, not one more CTA
+      const int tiles = (head_quads - 1 + w * per - 1) / (w * per), need = (head_quads + tiles * per - 1) / (tiles * per);
+      if (need == w + 1) w = need;
+    }
     return PROMPT(NP2, L2, 2);
   }
   if (quads / (32 / L1) >= WARPS) {
@@ -798,9 +810,10 @@ EXPORT int vb_memory_gates(const void* h, int64_t h_stride, const void* w, int W
   GateParams p = {h, h_stride, w, W, logits, bias, cap, reinterpret_cast<float4*>(gates), state, state_stride, m_off, qsl, seq_lens,
                   rows, rows_stride, H};
   const bool vec = W % 4 == 0 && h_stride % 4 == 0 && al(h, 4 * esz(dtype)) && al(w, 4 * esz(dtype));
+  const dim3 block(max_len > 2 * GATE_T ? GATE_MAX_T : GATE_T);
   DISPATCH_DTYPE(dtype, T, {
-    if (vec) vb_launch(memory_gates_kernel<T, 4>, dim3(num_reqs, H), dim3(GATE_T), 0, st, p);
-    else vb_launch(memory_gates_kernel<T, 1>, dim3(num_reqs, H), dim3(GATE_T), 0, st, p);
+    if (vec) vb_launch(memory_gates_kernel<T, 4>, dim3(num_reqs, H), block, 0, st, p);
+    else vb_launch(memory_gates_kernel<T, 1>, dim3(num_reqs, H), block, 0, st, p);
   });
   return (int)cudaGetLastError();
 }
