@@ -271,7 +271,8 @@ class FusedMoE(nn.Module):
         """Contribution of the experts this rank owns (ids are global; the expert map drops the others)."""
         if self.fp8_block and self.w13_weight.dtype == torch.float8_e4m3fn:
             return self._forward_fp8(x2, w, ids)
-        return ops.fused_moe(x2, self.w13_weight, self.w2_weight, w, ids, self.act, self.expert_map, self.gated)
+        return ops.fused_moe(x2, self.w13_weight, self.w2_weight, w, ids, self.act, self.expert_map, self.gated,
+                             bool(self.identity_experts))
 
     def _dequant(self, wq: torch.Tensor, scale: torch.Tensor) -> torch.Tensor:
         blk = self.fp8_block

@@ -325,10 +325,10 @@ def router_topk(x, gate, k, n_group, topk_group, renormalize, scoring="sigmoid",
                             routed_scaling_factor, group_score)
 
 
-def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None, gated: bool = True):
-    """``gated`` False: w13 is the plain up projection [E, I, H]."""
+def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None, gated: bool = True, on_device: bool = False):
+    """``gated`` False: w13 is the plain up projection [E, I, H].  ``on_device``: never synchronise with the host, at any batch size."""
     if _use_cuda(x):
-        return cuda_ops().fused_moe(x, w13, w2, topk_w, topk_ids, act, expert_map, gated)
+        return cuda_ops().fused_moe(x, w13, w2, topk_w, topk_ids, act, expert_map, gated, on_device)
     return ref.fused_moe(x, w13, w2, topk_w, topk_ids, act, expert_map, gated)
 
 

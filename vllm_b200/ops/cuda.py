@@ -1068,10 +1068,10 @@ def router_topk(x, gate, k, n_group, topk_group, renormalize, scoring="sigmoid",
     return w, ids
 
 
-def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None, gated: bool = True):
+def fused_moe(x, w13, w2, topk_w, topk_ids, act="silu", expert_map=None, gated: bool = True, on_device: bool = False):
     from vllm_b200.ops import moe
-    if not gated:
-        return moe.fused_moe_plain(x, w13, w2, topk_w, topk_ids, act, expert_map)
+    if not gated or on_device:
+        return moe.fused_moe_rows(x, w13, w2, topk_w, topk_ids, act, expert_map, gated)
     return moe.fused_moe_cuda(x, w13, w2, topk_w, topk_ids, act, expert_map)
 
 

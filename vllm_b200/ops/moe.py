@@ -109,8 +109,9 @@ def combine_rows(rows, inv, topk_w, T: int):
     return cu.moe_combine(rows, inv, topk_w.to(torch.float32).contiguous(), T)
 
 
-def fused_moe_plain(x, w_up, w_down, topk_w, topk_ids, act, expert_map):
-    rows, inv = expert_rows_plain(x, w_up, w_down, topk_ids, act, expert_map)
+def fused_moe_rows(x, w13, w2, topk_w, topk_ids, act, expert_map, gated: bool):
+    """The weighted sum of ``expert_rows``: no host sync at any batch size."""
+    rows, inv = expert_rows(x, w13, w2, topk_ids, act, expert_map, gated)
     return combine_rows(rows, inv, topk_w, x.shape[0])
 
 
@@ -205,9 +206,6 @@ def fused_moe_cuda(x, w13, w2, topk_w, topk_ids, act="silu", expert_map: Optiona
     T, H = x.shape
     E = w13.shape[0]
     k = topk_ids.shape[1]
-    if T * k <= GROUPED_MAX_ROWS and w13.dtype == x.dtype and w13.is_contiguous() and w2.is_contiguous():
-        rows, inv = expert_rows_gated(x, w13, w2, topk_ids, act, expert_map)      # sizes off the 128-byte grid, fp32: no host sync
-        return combine_rows(rows, inv, topk_w, T)
     ids = topk_ids.long()
     if expert_map is not None:
         ids = expert_map[ids].long()
