@@ -249,7 +249,7 @@ def uneven():
 def wide():
     """Head sizes of the tensor-core attention kernels, states of real sizes."""
     return config(128, 160, [
-        (attn(8, 2, 128, 128, 64), moe(64, 8, 4, 4, (3, 1), 72, 2.2)),
+        (attn(8, 2, 128, 128, 64), moe(64, 9, 3, 4, (3, 1), 72, 2.2)),
         (memory(4, 64, 96, cap=15.0), dense(136)),
         (attn(8, 2, 128, 128, 128, scale=0.06, kv_from=0), moe(96, 6, 6, 6, (2, 2), 64)),
         (memory(2, 128, 128), dense(64))])

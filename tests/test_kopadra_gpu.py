@@ -87,7 +87,7 @@ def test_experts_with_identities(T, H, ff, E, ident, k, shared, dtype):
 
 
 @pytest.mark.parametrize("T", [7, 400])                      # fused logits, and logits of one product
-@pytest.mark.parametrize("E,k,count,keep", [(12, 4, 2, 1), (12, 3, 4, 2), (9, 5, 3, 2), (6, 1, 6, 1), (8, 8, 1, 1), (1, 1, 1, 1), (96, 8, 8, 3)])
+@pytest.mark.parametrize("E,k,count,keep", [(14, 5, 2, 1), (12, 3, 4, 2), (9, 5, 3, 2), (6, 1, 6, 1), (8, 8, 1, 1), (1, 1, 1, 1), (96, 8, 8, 3)])
 @pytest.mark.parametrize("dtype", [BF, F32])
 def test_router(E, k, count, keep, T, dtype):
     from vllm_b200 import ops

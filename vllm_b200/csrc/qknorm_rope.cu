@@ -2,7 +2,7 @@
 // attention prologues).
 //
 // Reference ops: csrc/libtorch_stable/fused_qknorm_rope_kernel.cu:563-686 (q/k norm + rope over the fused qkv
-// buffer) and the model-specific q-norm / rope / KV-insert fusions listed in SURVEY §2.3.  Ours goes one step
+// buffer) and the model-specific q-norm / rope / KV-insert fusions.  Ours goes one step
 // further than the generic reference op: the rotated K head is written to its cache page from the registers that
 // produced it and the V head is copied by a sibling warp of the same CTA, so a layer's attention prologue is ONE
 // launch instead of norm(q), norm(k), rope, reshape_and_cache.

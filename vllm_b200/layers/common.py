@@ -78,7 +78,7 @@ def get_act_and_mul(name: str) -> nn.Module:
 
 class VocabParallelEmbedding(nn.Module):
     """Embedding table sharded over the vocab dim; lookup of out-of-shard ids gives 0
-    and the TP all-reduce restores the full embedding (collective C2 in SURVEY §2.4)."""
+    and the TP all-reduce restores the full embedding."""
 
     def __init__(self, num_embeddings: int, embedding_dim: int, dtype=None, padding_size: int = 64,
                  prefix: str = "", replicate: bool = False) -> None:
