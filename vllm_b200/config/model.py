@@ -800,7 +800,29 @@ def kopadra_config(*, vocab: int, width: int, layers: list[str], heads: int, kv_
     return dict(dict(architecture="Kopadra", vocab=vocab, width=width, layers=out, norm=dict(eps=1e-6), logit_softcap=30.0), **kw)
 
 
+def gizilorn_config(*, vocab: int, width: int, layers: list[str], heads: int, kv_heads: int, dim: int, latent_heads: int, latent_dim: int,
+                    rot_dim: int, latent_vdim: int, kv_rank: int, window: int, latent_window: int, ff: int, streams: int, **kw) -> dict[str, Any]:
+    """A Gizilorn config.json.  Layers are "attention", "latent", or "reuse" (latent attention over the cache of the "latent" before it);
+    layers of a kind are alike."""
+    attn = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, softcap=50.0, mask=dict(size=window),
+                rot=dict(base=10000.0, dims=dim))
+    lat = dict(heads=latent_heads, dim=latent_dim, rot_dim=rot_dim, vdim=latent_vdim, kv_rank=kv_rank, scale=(latent_dim + rot_dim) ** -0.5,
+               mask=dict(size=latent_window), rot=dict(base=100000.0, dims=rot_dim))
+    out, owner = [], None
+    for i, kind in enumerate(layers):
+        m = attn if kind == "attention" else dict(lat, **(dict(kv_from=owner) if kind == "reuse" else {}))
+        owner = i if kind == "latent" else owner
+        out.append(dict(type="attention" if kind == "attention" else "latent_attention", mixer=copy.deepcopy(m), mlp=dict(kind="dense", ff=ff)))
+    return dict(dict(architecture="Gizilorn", vocab=vocab, width=width, layers=out, norm=dict(eps=1e-6), streams=streams), **kw)
+
+
 PRESETS.update({
+    "gizilorn-tiny": gizilorn_config(vocab=320, width=80, layers=["attention", "latent", "reuse"], heads=4, kv_heads=2, dim=24, latent_heads=2,
+                                     latent_dim=16, rot_dim=8, latent_vdim=24, kv_rank=48, window=72, latent_window=100, ff=120, streams=2,
+                                     max_position_embeddings=1024, torch_dtype="float32"),
+    "gizilorn-small": gizilorn_config(vocab=4096, width=1024, layers=["attention", "latent", "reuse", "attention"], heads=8, kv_heads=2, dim=128,
+                                      latent_heads=8, latent_dim=128, rot_dim=64, latent_vdim=128, kv_rank=512, window=1024,
+                                      latent_window=1024, ff=4096, streams=4, max_position_embeddings=8192, torch_dtype="bfloat16"),
     "kopadra-tiny": kopadra_config(vocab=320, width=80, layers=["attention+dense", "mlstm+moe", "reuse+moe"], heads=4, kv_heads=2, dim=24,
                                    mem_heads=2, mem_dim=20, mem_vdim=28, ff=120, expert_ff=40, experts=6, identity=3, top=2, groups=3, keep=2,
                                    shared_ff=56, max_position_embeddings=1024, torch_dtype="float32"),
@@ -939,6 +961,35 @@ def _flatten_nested_config(c: dict) -> None:
         if moes:
             c.setdefault("num_experts", max(r["experts"] for r in moes))
             c.setdefault("num_experts_per_tok", max(r["top"] for r in moes))
+    if c.get("architecture") == "Gizilorn":
+        layers = c["layers"]
+        attn = [l["mixer"] for l in layers if l["type"] == "attention"]
+        latent = [l["mixer"] for l in layers if l["type"] == "latent_attention"]
+        for i, l in enumerate(layers):
+            m, rot, j = l["mixer"], l["mixer"]["rot"], l["mixer"].get("kv_from")
+            if m["mask"]["size"] < 1:
+                raise ValueError(f"layer {i}: a window holds a position at least")
+            if l["type"] == "attention" and (m["heads"] % m["kv_heads"] or rot["dims"] % 2 or rot["dims"] > m["dim"] or m["vdim"] % 2):
+                raise ValueError(f"layer {i}: heads must divide into kv_heads, rotated dimensions be even and within the head, values even")
+            if l["type"] == "latent_attention" and (m["rot_dim"] % 2 or rot["dims"] != m["rot_dim"]):
+                raise ValueError(f"layer {i}: the rotated part must be even and rotated as a whole")
+            if j is not None and not (0 <= j < i and l["type"] == layers[j]["type"] == "latent_attention"
+                                      and layers[j]["mixer"].get("kv_from") is None
+                                      and all(layers[j]["mixer"][k] == m[k] for k in ("kv_rank", "rot_dim", "rot"))):
+                raise ValueError(f"layer {i}: kv_from {j} must name an earlier latent layer with a latent of its own, of the same kv_rank, "
+                                 "rot_dim and rotation")
+        if c["streams"] < 1:
+            raise ValueError("streams must be positive")
+        c.setdefault("architectures", ["GizilornForCausalLM"])
+        c.setdefault("model_type", "gizilorn")
+        c.setdefault("vocab_size", c["vocab"])
+        c.setdefault("hidden_size", c["width"])
+        c.setdefault("num_hidden_layers", len(layers))
+        c.setdefault("max_position_embeddings", OPEN_MAX_LEN)
+        # tensor parallelism splits the heads of latent layers; attention layers mix theirs and are replicated
+        c.setdefault("num_attention_heads", math.gcd(*(m["heads"] for m in latent or attn)))
+        c.setdefault("num_key_value_heads", math.gcd(*(m["heads"] for m in latent)) if latent else attn[0]["kv_heads"])
+        c.setdefault("head_dim", max((max(a["dim"], a["vdim"]) for a in attn), default=128))
     if c.get("model_type") == "dbrx":
         a, f = c.get("attn_config") or {}, c.get("ffn_config") or {}
         c.setdefault("hidden_size", c.get("d_model"))

@@ -73,11 +73,25 @@ class MLAAttentionSpec(KVCacheSpec):
         return self.phys_block_size * self.head_size * self.dtype_size
 
 
+def _window_pages(spec, max_model_len: int) -> int:
+    """Pages of a request whose tokens are kept for ``spec.sliding_window`` positions (one more where the window is not aligned)."""
+    n = min(max_model_len, (spec.sliding_window or max_model_len) - 1 + 16384)
+    return min(cdiv(n, spec.block_size) + 1, cdiv(max_model_len, spec.block_size))
+
+
 @dataclass(frozen=True)
 class SlidingWindowSpec(FullAttentionSpec):
     def max_memory_usage_bytes(self, max_model_len: int) -> int:
-        n = min(max_model_len, (self.sliding_window or max_model_len) - 1 + 16384)
-        return (cdiv(n, self.block_size) + 1) * self.page_size_bytes
+        return _window_pages(self, max_model_len) * self.page_size_bytes
+
+
+@dataclass(frozen=True)
+class SlidingWindowMLASpec(MLAAttentionSpec):
+    """Latents that no later token reads once they are ``sliding_window`` positions back."""
+    sliding_window: Optional[int] = None
+
+    def max_memory_usage_bytes(self, max_model_len: int) -> int:
+        return _window_pages(self, max_model_len) * self.page_size_bytes
 
 
 @dataclass(frozen=True)
@@ -133,7 +147,10 @@ def group_specs(layer_specs: dict[str, KVCacheSpec]) -> list[KVCacheGroupSpec]:
     groups: dict[KVCacheSpec, list[str]] = {}
     for name, spec in layer_specs.items():
         key = spec
-        if isinstance(spec, MLAAttentionSpec):
+        if isinstance(spec, (SlidingWindowSpec, SlidingWindowMLASpec)) and spec.dcp == 1:
+            # keys and latents alike: what a page holds is decided by the window
+            key = SlidingWindowMLASpec(spec.block_size, head_size=0, dtype_size=spec.dtype_size, sliding_window=spec.sliding_window)
+        elif isinstance(spec, MLAAttentionSpec):
             key = replace(spec, head_size=0)
         elif isinstance(spec, FullAttentionSpec):
             key = replace(spec, num_kv_heads=0, head_size=0)
@@ -341,7 +358,7 @@ class MambaManager(SingleTypeManager):
 def _manager_for(spec: KVCacheSpec, pool: BlockPool, gid: int) -> SingleTypeManager:
     if isinstance(spec, MambaSpec):
         return MambaManager(spec, pool, gid)
-    if isinstance(spec, SlidingWindowSpec):
+    if isinstance(spec, (SlidingWindowSpec, SlidingWindowMLASpec)):
         return SlidingWindowManager(spec, pool, gid)
     return FullAttentionManager(spec, pool, gid)
 

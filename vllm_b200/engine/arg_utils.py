@@ -171,7 +171,7 @@ class EngineArgs:
             # ALiBi / sinks / soft-cap) use the 32-token page it is tuned for
             special = any(mc.hf_config.get(k) for k in ("attn_logit_softcapping", "alibi")) or \
                 mc.hf_config.get("model_type") in ("bloom", "mpt", "gpt_oss")
-            any_page = mc.hf_config.get("model_type") in ("legelix", "kopadra")          # kernels that take every page size
+            any_page = mc.hf_config.get("model_type") in ("legelix", "kopadra", "gizilorn")          # kernels that take every page size
             block_size = 64 if (self.device == "cpu" or mc.is_mla or any_page or (mc.head_dim == 128 and not special)) else 32
         cc = CacheConfig(
             block_size=block_size, gpu_memory_utilization=self.gpu_memory_utilization,

@@ -14,7 +14,8 @@ import torch
 import torch.nn as nn
 
 from vllm_b200 import envs, ops
-from vllm_b200.core.kv_cache_manager import FullAttentionSpec, KVCacheSpec, MLAAttentionSpec, SlidingWindowSpec
+from vllm_b200.core.kv_cache_manager import (FullAttentionSpec, KVCacheSpec, MLAAttentionSpec, SlidingWindowMLASpec,
+                                            SlidingWindowSpec)
 from vllm_b200.forward_context import get_forward_context
 
 _LAYER_REGISTRY: dict[str, "Attention"] = {}
@@ -36,13 +37,21 @@ class Attention(nn.Module):
                  causal: bool = True, rope: Optional[nn.Module] = None,
                  alibi_slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
                  chunk_size: int = 0, v_head_size: Optional[int] = None, fused_prologue: bool = False,
-                 out_scale: float = 1.0, whole_qk_norm: bool = False, kv_sharing_target: Optional[str] = None) -> None:
+                 out_scale: float = 1.0, whole_qk_norm: bool = False, kv_sharing_target: Optional[str] = None,
+                 talk: Optional[torch.Tensor] = None, v_rope: Optional[nn.Module] = None, cache_window: Optional[int] = None) -> None:
         """``v_head_size``: value width where it is not ``head_size`` (cache rows are as wide as the wider one).
         ``fused_prologue``: q/k norms, rotation and cache write are one kernel for whatever shape and dtype, 32-bit between norm
         and rotation.  ``out_scale``: factor of the output, applied in 32-bit.  ``whole_qk_norm``: the q/k norms go over all heads of
         the projection at once (weights as long).  ``kv_sharing_target``: name of an earlier layer whose cache this one reads (it owns
-        none, writes nothing and is called without keys and values)."""
+        none, writes nothing and is called without keys and values).  ``talk`` [Hq, Hq]: the heads' weights are mixed by it behind the
+        softmax, head h then applies sum_g talk[h, g] weights_g to the values of its own KV head (a parameter of the model).  ``v_rope``:
+        values are rotated by their position before they are cached, outputs turned back by that of the query.  ``cache_window``: pages
+        stay for this many tokens (layers of different windows then share pages and a block table), at least ``sliding_window``."""
         super().__init__()
+        self.talk, self.v_rope = talk, v_rope
+        self.cache_window = max(cache_window or 0, sliding_window) if sliding_window else None
+        if (talk is not None or v_rope is not None) and (kv_sharing_target is not None or not causal or not fused_prologue):
+            raise NotImplementedError("mixed heads and rotated values take the fused prologue, causal masks and a cache of their own")
         self.whole_qk_norm, self.kv_sharing_target, self.cache_name = whole_qk_norm, kv_sharing_target, kv_sharing_target or prefix
         self.v_head_size = v_head_size or head_size
         self.cache_head_size = max(head_size, self.v_head_size)
@@ -50,7 +59,11 @@ class Attention(nn.Module):
         self.chunk_size = int(chunk_size or 0)        # chunked-local attention (Llama-4 rope layers)
         # ALiBi slopes / attention-sink logits of THIS rank's heads (buffers follow the module's device)
         self.register_buffer("alibi_slopes", None if alibi_slopes is None else alibi_slopes.float(), persistent=False)
-        self.sinks = sinks                       # nn.Parameter owned by the model (loaded from the checkpoint) or None
+        # nn.Parameter owned by the model (loaded from the checkpoint), or constants
+        if sinks is None or isinstance(sinks, nn.Parameter):
+            self.sinks = sinks
+        else:
+            self.register_buffer("sinks", sinks.float(), persistent=False)
         self.num_heads, self.head_size, self.scale = num_heads, head_size, scale
         self.num_kv_heads = num_kv_heads or num_heads
         self.sliding_window = sliding_window
@@ -72,8 +85,9 @@ class Attention(nn.Module):
         from vllm_b200.parallel.state import get_dcp_group
         d = get_dcp_group().world_size
         if d > 1:
-            if self.whole_qk_norm:
-                raise NotImplementedError("decode context parallelism does not cover norms over whole projections")
+            if self.whole_qk_norm or self.talk is not None or self.v_rope is not None:
+                raise NotImplementedError("decode context parallelism does not cover norms over whole projections, mixed heads and "
+                                          "rotated values")
             if self.sliding_window or self.alibi_slopes is not None or self.sinks is not None or self.chunk_size:
                 raise NotImplementedError("decode context parallelism covers full causal attention (no sliding window / "
                                           "ALiBi / sinks / chunked-local layers)")
@@ -174,29 +188,37 @@ class Attention(nn.Module):
                 k = kn(k.reshape(T, -1, D)).reshape(T, -1)
             return self._forward_dcp(q, k, v, positions, md, kv_cache)
         pcp = ctx.extra.get("pcp")
-        if pcp is not None and (shared or self.whole_qk_norm):
-            raise NotImplementedError("prefill context parallelism does not cover shared caches and norms over whole projections")
+        if pcp is not None and (shared or self.whole_qk_norm or self.talk is not None or self.v_rope is not None):
+            raise NotImplementedError("prefill context parallelism does not cover shared caches, norms over whole projections, mixed heads "
+                                      "and rotated values")
         mpos = ctx.extra.get("mrope_positions") if (self.rope is not None and self.rope.mrope_section) else None
-        if qk_norm is not None:
-            qn, kn = qk_norm
+        first = positions
+        if qk_norm is not None or self.fused_prologue:
+            qn, kn = qk_norm or (None, None)
             fused = (md is not None and kv_cache is not None and q.is_cuda and pcp is None and mpos is None
                      and self.rope is not None and positions is not None
                      and kv_cache.dtype == q.dtype
-                     and (shared or (getattr(qn, "gemma", False) == getattr(kn, "gemma", False) and qn.eps == kn.eps)) and not envs.VLLM_B200_FORCE_REF_OPS
+                     and (shared or qn is None or (getattr(qn, "gemma", False) == getattr(kn, "gemma", False) and qn.eps == kn.eps))
+                     and not envs.VLLM_B200_FORCE_REF_OPS
                      and (self.fused_prologue or (q.dtype in (torch.bfloat16, torch.float16) and ops.cuda_ops().qknorm_rope_ok(
                          D, self.rope.cos_sin_cache.shape[-1], self.rope.is_neox_style))))
             if fused:
-                ops.cuda_ops().fused_qk_norm_rope(positions, q, k, qn.weight, None if shared else kn.weight, self.rope.cos_sin_cache,
-                                                  D, qn.eps, self.rope.is_neox_style, v=v, kv_cache=None if shared else kv_cache,
+                ops.cuda_ops().fused_qk_norm_rope(positions, q, k, None if qn is None else qn.weight, None if shared or kn is None else
+                                                  kn.weight, self.rope.cos_sin_cache, D, 0.0 if qn is None else qn.eps,
+                                                  self.rope.is_neox_style, v=v, kv_cache=None if shared else kv_cache,
                                                   slot_mapping=md.slot_mapping, gemma=getattr(qn, "gemma", False),
                                                   vt=md.kv_vt, v_head_dim=self.v_head_size, keep32=self.fused_prologue,
-                                                  whole=self.whole_qk_norm)
+                                                  whole=self.whole_qk_norm,
+                                                  v_cos_sin=None if self.v_rope is None else self.v_rope.cos_sin_cache)
                 positions = None            # rotation and cache insert are done: skip them below
                 skip_cache_write = True
             else:
                 whole = self.whole_qk_norm
-                q = qn(q.reshape(T, -1, q.shape[-1] if whole else D)).reshape(T, -1)
-                k = k if shared else kn(k.reshape(T, -1, k.shape[-1] if whole else D)).reshape(T, -1)
+                if self.v_rope is not None:
+                    v, _ = self.v_rope(positions, v, None)
+                if qn is not None:
+                    q = qn(q.reshape(T, -1, q.shape[-1] if whole else D)).reshape(T, -1)
+                    k = k if shared else kn(k.reshape(T, -1, k.shape[-1] if whole else D)).reshape(T, -1)
                 skip_cache_write = False
         else:
             skip_cache_write = False
@@ -249,6 +271,10 @@ class Attention(nn.Module):
             Attention.cascade_calls += 1
             return out.view(T, self.num_heads * D)
         buf = None if out is None else out.view(T, self.num_heads, self.v_head_size)
+        if self.talk is not None or self.v_rope is not None:
+            o = ops.talking_attention(q.view(T, self.num_heads, D), kv_cache, md, self.scale, self.sliding_window, self.logits_soft_cap,
+                                      self.talk, self.sinks, self.v_head_size, self.v_rope, first, out=buf)
+            return o.reshape(T, self.num_heads * self.v_head_size) if out is None else out
         o = ops.paged_attention(q.view(T, self.num_heads, D), kv_cache, md, self.scale,
                                 self.sliding_window, self.logits_soft_cap, self.causal, out=buf,
                                 alibi_slopes=self.alibi_slopes, sinks=self.sinks, chunk_size=self.chunk_size,
@@ -263,15 +289,19 @@ class MLAAttentionCore(nn.Module):
     decode kernel in the reference does."""
 
     def __init__(self, num_heads: int, kv_lora_rank: int, qk_rope_head_dim: int, scale: float,
-                 prefix: str = "", kv_sharing_target: Optional[str] = None) -> None:
-        """``kv_sharing_target``: name of an earlier layer whose cache this one reads (it owns none and writes nothing)."""
+                 prefix: str = "", kv_sharing_target: Optional[str] = None, sliding_window: Optional[int] = None,
+                 cache_window: Optional[int] = None) -> None:
+        """``kv_sharing_target``: name of an earlier layer whose cache this one reads (it owns none and writes nothing).
+        ``sliding_window``: a query sees that many tokens; pages stay for ``cache_window`` tokens (at least the windows of all layers
+        that read them)."""
         super().__init__()
         self.num_heads, self.kv_lora_rank, self.qk_rope_head_dim = num_heads, kv_lora_rank, qk_rope_head_dim
         self.scale = scale
         self.layer_name = prefix
         self.head_size = kv_lora_rank + qk_rope_head_dim
         self.num_kv_heads = 1
-        self.sliding_window = None
+        self.sliding_window = sliding_window
+        self.cache_window = max(cache_window or 0, sliding_window) if sliding_window else None
         self.kv_sharing_target = kv_sharing_target
         self.cache_name = kv_sharing_target or prefix
         if kv_sharing_target is None:
@@ -281,10 +311,17 @@ class MLAAttentionCore(nn.Module):
         if not isinstance(owner, MLAAttentionCore) or owner.head_size != self.head_size:
             raise ValueError(f"layer {prefix!r} shares the cache of {kv_sharing_target!r}, which is not an earlier latent "
                              f"cache of width {self.head_size} on this rank")
+        if owner.cache_window is not None and (self.cache_window is None or self.cache_window > owner.cache_window):
+            raise ValueError(f"layer {prefix!r} reads further back than {kv_sharing_target!r} keeps its pages")
 
     def get_kv_cache_spec(self, block_size: int, dtype_size: int) -> KVCacheSpec:
         from vllm_b200.parallel.state import get_dcp_group
         d = get_dcp_group().world_size
+        if self.cache_window is not None:
+            if d > 1:
+                raise NotImplementedError("decode context parallelism with windows over latents")
+            return SlidingWindowMLASpec(block_size=block_size, head_size=self.head_size, dtype_size=dtype_size,
+                                        sliding_window=self.cache_window)
         return MLAAttentionSpec(block_size=block_size * d, head_size=self.head_size, dtype_size=dtype_size, dcp=d)
 
     def _forward_dcp(self, q_nope_abs, q_pe, kv_c, k_pe, md, kv_cache) -> torch.Tensor:

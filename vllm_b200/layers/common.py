@@ -68,6 +68,22 @@ class Activation(nn.Module):
         return ops.activation(x, self.name)
 
 
+class XIELU(nn.Module):
+    """a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below, with a = softplus(p), b = 1/2 + softplus(q) of two learned numbers p, q.
+    ``coef`` holds (a, b) in 32-bit."""
+
+    def __init__(self) -> None:
+        super().__init__()
+        self.coef = nn.Parameter(torch.ones(2, dtype=torch.float32), requires_grad=False)
+
+    def weight_loader(self, param: nn.Parameter, w: torch.Tensor, shard_id=None) -> None:
+        assert w.shape == (2,), w.shape
+        param.data.copy_(torch.nn.functional.softplus(w.double().cpu(), threshold=50.0) + torch.tensor([0.0, 0.5], dtype=torch.float64, device="cpu"))
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.xielu(x, self.coef)
+
+
 def get_act_and_mul(name: str) -> nn.Module:
     if name == "silu":
         return SiluAndMul()

@@ -112,6 +112,22 @@ class MergedReplicatedLinear(ReplicatedLinear):
         dst.copy_(w)
 
 
+class MergedMixedLinear(MergedReplicatedLinear):
+    """MergedReplicatedLinear some of whose parts (``sharded``) are split over the ranks."""
+
+    def __init__(self, input_size, output_sizes: list[int], sharded: list[bool], bias=False, dtype=None, quant_config=None, prefix="",
+                 align: int = 1) -> None:
+        self.tp_rank, self.tp_size = _tp()
+        self.sharded = list(sharded)
+        super().__init__(input_size, [divide(n, self.tp_size) if s else n for n, s in zip(output_sizes, sharded)], bias, dtype,
+                         quant_config, prefix, align)
+
+    def weight_loader(self, param: nn.Parameter, w: torch.Tensor, shard_id=None) -> None:
+        if shard_id is not None and shard_id < len(self.sharded) and self.sharded[shard_id]:
+            w = w.chunk(self.tp_size)[self.tp_rank]
+        super().weight_loader(param, w, shard_id)
+
+
 class SummedReplicatedLinear(ReplicatedLinear):
     """sum_i W_i x_i over inputs of their own as one GEMM: the inputs lie side by side in ``buffer``, part i at a multiple of
     ``align`` elements."""

@@ -17,6 +17,7 @@ _MODELS: dict[str, tuple[str, str]] = {
     "PomipelForCausalLM": ("pomipel", "PomipelForCausalLM"),
     "LegelixForCausalLM": ("legelix", "LegelixForCausalLM"),
     "KopadraForCausalLM": ("kopadra", "KopadraForCausalLM"),
+    "GizilornForCausalLM": ("gizilorn", "GizilornForCausalLM"),
     "Qwen2ForCausalLM": ("llama", "Qwen2ForCausalLM"),
     "Qwen3ForCausalLM": ("llama", "Qwen3ForCausalLM"),
     "GemmaForCausalLM": ("llama", "GemmaForCausalLM"),

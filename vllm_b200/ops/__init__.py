@@ -189,38 +189,66 @@ def paged_attention(q, kv_cache, md, scale, sliding_window=None, logits_soft_cap
     return (o, lse) if return_lse else o
 
 
-def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank):
+def talking_attention(q, kv_cache, md, scale, sliding_window, soft_cap, talk, sinks, v_head_size: int, v_rope=None, positions=None,
+                      out: Optional[torch.Tensor] = None):
+    """paged_attention whose heads' weights are mixed by ``talk`` [Hq, Hq] behind the softmax (None: not mixed), outputs turned back by
+    their position (``v_rope``: the rotation of the cached values)."""
+    if _use_cuda(q):
+        return cuda_ops().talking_attention(q, kv_cache, md, scale, sliding_window, soft_cap, talk, sinks, v_head_size, v_rope, positions, out)
+    if talk is None:
+        o = paged_attention(q, kv_cache, md, scale, sliding_window, soft_cap, sinks=sinks, v_head_size=v_head_size).float()
+    else:
+        sl = md.seq_lens_cpu if md.seq_lens_cpu is not None else md.seq_lens.cpu()
+        qsl = md.query_start_loc_cpu if md.query_start_loc_cpu is not None else md.query_start_loc.cpu()
+        o = ref.talking_attention(q, kv_cache, md.block_table, sl, qsl, scale, sliding_window, soft_cap, talk, sinks, v_head_size)
+    if v_rope is not None:
+        half = v_rope.cos_sin_cache.shape[-1] // 2
+        back = torch.cat((v_rope.cos_sin_cache[:, :half], -v_rope.cos_sin_cache[:, half:]), dim=-1)
+        o = ref.rotary_embedding(positions, o.reshape(o.shape[0], -1), None, back, v_head_size, v_rope.is_neox_style)[0].view(o.shape)
+    return o.to(q.dtype) if out is None else out.copy_(o)
+
+
+def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank, sliding_window: Optional[int] = None):
     """``q_pe`` None: no rope part."""
     if _use_cuda(q_nope_abs):
-        return cuda_ops().mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank)
+        return cuda_ops().mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank, sliding_window)
     sl = md.seq_lens_cpu if md.seq_lens_cpu is not None else md.seq_lens.cpu()
     qsl = md.query_start_loc_cpu if md.query_start_loc_cpu is not None else md.query_start_loc.cpu()
     if q_pe is None:
         q_pe = q_nope_abs[..., :0]
-    return ref.mla_decode_attention(q_nope_abs, q_pe, kv_cache, md.block_table, sl, qsl, scale, kv_lora_rank)
+    return ref.mla_decode_attention(q_nope_abs, q_pe, kv_cache, md.block_table, sl, qsl, scale, kv_lora_rank, sliding_window)
 
 
-def mla_attention_rows(q_abs, q_pe, kv_cache, block_table, seq_lens, max_len: int, scale):
-    """Attention over the latent cache for rows with a block table and a number of visible keys each (CUDA)."""
+def mla_attention_rows(q_abs, q_pe, kv_cache, block_table, seq_lens, max_len: int, scale, sliding_window: Optional[int] = None):
+    """Attention over the latent cache for rows with a block table and a number of visible keys each (CUDA); with a window, of its last
+    ones."""
     cu = cuda_ops()
     if cu._mla_tc_ok(q_abs, q_pe, kv_cache):
-        return cu.mla_decode_tc(q_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_len)
-    return cu.mla_simt(q_abs, q_pe, kv_cache, block_table, seq_lens, None, scale)
+        return cu.mla_decode_tc(q_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_len, sliding_window=sliding_window)
+    return cu.mla_simt(q_abs, q_pe, kv_cache, block_table, seq_lens, None, scale, sliding_window)
 
 
-def latent_expand_ok(q, v_dim: int, kv_rank: int) -> bool:
+def latent_expand_ok(q, dim: int, rot: int, v_dim: int, kv_rank: int) -> bool:
     """Can prompt portions run over expanded keys and values (csrc/mla_prefill.cu)?"""
-    return _use_cuda(q) and cuda_ops().mla_prefill_ok(q, v_dim, kv_rank)
+    return _use_cuda(q) and cuda_ops().mla_prefill_ok(q, dim, rot, v_dim, kv_rank)
 
 
-def gather_latents(kv_cache, block_table, cu_kv, num_kv: int, max_kv: int):
-    """Cached rows of a batch of sequences, contiguous [num_kv, R] (CUDA)."""
+def gather_latents(kv_cache, block_table, cu_kv, num_kv: int, max_kv: int, starts=None):
+    """Cached rows of a batch of sequences (from position ``starts`` on), contiguous [num_kv, R] (CUDA)."""
     out = torch.empty((num_kv, kv_cache.shape[-1]), dtype=kv_cache.dtype, device=kv_cache.device)
-    return cuda_ops().gather_cache(kv_cache, block_table, cu_kv, out, max_kv)
+    return cuda_ops().gather_cache(kv_cache, block_table, cu_kv, out, max_kv, starts)
 
 
-def mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0: int, max_q: int, scale) -> None:
-    cuda_ops().mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0, max_q, scale)
+def mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0: int, max_q: int, scale, k_pe=None, window: int = 0) -> None:
+    cuda_ops().mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0, max_q, scale, k_pe, window)
+
+
+def latent_rope_cache(proj, q_off, heads, dim, rot, kv_off, kv_rank, kv_weight, eps, positions, cos_sin, neox, cache=None, slots=None) -> None:
+    """On the columns of a merged projection [T, ...], in place: rotates the last ``rot`` dimensions of every query head, norms the latent,
+    rotates the key part behind it and writes both into their cache rows (``kv_rank`` 0: queries alone)."""
+    if _use_cuda(proj):
+        return cuda_ops().latent_rope_cache(proj, q_off, heads, dim, rot, kv_off, kv_rank, kv_weight, eps, positions, cos_sin, neox, cache, slots)
+    return ref.latent_rope_cache(proj, q_off, heads, dim, rot, kv_off, kv_rank, kv_weight, eps, positions, cos_sin, neox, cache, slots)
 
 
 def latent_norm_cache(lat, q_rank, q_weight, kv_rank, kv_weight, eps, cache=None, slots=None):
@@ -252,6 +280,36 @@ def norm_add(x, y, y_bias, norm, mult: float, next_norm, eps: float):
     if _use_cuda(x):
         return cuda_ops().norm_add(x, y, y_bias, norm, mult, next_norm, eps)
     return ref.norm_add(x, y, y_bias, norm, mult, next_norm, eps)
+
+
+def hyper_entry(ids, table, streams: int, embed_weight, into, weight, eps: float):
+    """Entry of ``streams`` equal fp32 streams: (x [T, S, H], rms norm of sum(into) e in the table's dtype), e the rms norm of table[ids],
+    or a row of ``table`` where ``ids`` is None."""
+    if _use_cuda(table):
+        return cuda_ops().hyper_entry(ids, table, streams, embed_weight, into, weight, eps)
+    return ref.hyper_entry(ids, table, streams, embed_weight, into, weight, eps)
+
+
+def hyper_step(x, y, coef, into, weight, eps: float, dtype=None):
+    """Hyper-connections, one step of S fp32 streams x [T, S, H] between sublayers: in place x_t = sum_s mix[s, t] x_s + out[t] y (``coef``:
+    out [S] and mix [S, S], fp32; y None: unchanged).  Returns the rms norm of sum_s into[s] x_s in ``dtype`` (y's)."""
+    if _use_cuda(x):
+        return cuda_ops().hyper_step(x, y, coef, into, weight, eps, dtype or y.dtype)
+    return ref.hyper_step(x, y, coef, into, weight, eps, dtype or y.dtype)
+
+
+def xielu(x, coef):
+    """a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below, (a, b) = ``coef`` (fp32)."""
+    if _use_cuda(x):
+        return cuda_ops().xielu(x, coef)
+    return ref.xielu(x, coef)
+
+
+def linear_xielu(x, weight, bias, coef):
+    """xielu(x W^T + b); one kernel for decode batches on CUDA."""
+    if _use_cuda(x):
+        return cuda_ops().linear_xielu(x, weight, bias, coef)
+    return ref.xielu(linear(x, weight, bias), coef)
 
 
 def add_norm(x, y, next_norm, eps: float, dtype=None):

@@ -217,6 +217,34 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.
     return (out, lse) if return_lse else out
 
 
+def talking_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_table: torch.Tensor, seq_lens: torch.Tensor,
+                      query_start_loc: torch.Tensor, scale: float, sliding_window: Optional[int], soft_cap: float,
+                      talk: torch.Tensor, sinks: Optional[torch.Tensor], v_dim: int) -> torch.Tensor:
+    """Attention whose heads' weights are mixed behind the softmax: out_h = sum_g talk[h, g] (weights_g V_kv(h)).  q [T, Hq, D] →
+    fp32 [T, Hq, v_dim]."""
+    T, Hq, D = q.shape
+    Hkv = kv_cache.shape[2]
+    G = Hq // Hkv
+    out = torch.zeros(T, Hq, v_dim, dtype=torch.float32, device=q.device)
+    for i, (s, e, sl) in enumerate(zip(query_start_loc.tolist(), query_start_loc.tolist()[1:], seq_lens.tolist())):
+        if e == s:
+            continue
+        k, v = gather_kv(kv_cache, block_table[i], sl)
+        att = torch.einsum("qhgd,hkd->hgqk", q[s:e].float().view(e - s, Hkv, G, D), k[..., :D].float()).reshape(Hq, e - s, sl) * scale
+        if soft_cap > 0:
+            att = soft_cap * torch.tanh(att / soft_cap)
+        qpos = torch.arange(sl - (e - s), sl, device=q.device)[:, None]
+        kpos = torch.arange(sl, device=q.device)[None]
+        ok = (kpos <= qpos) & (kpos > qpos - (sliding_window or sl))
+        att = att.masked_fill(~ok[None], float("-inf"))
+        lse = torch.logsumexp(att, dim=-1)
+        if sinks is not None:
+            lse = torch.logaddexp(lse, sinks.float()[:, None].expand_as(lse))
+        p = torch.einsum("hg,gqk->hqk", talk.float(), torch.exp(att - lse[..., None]))
+        out[s:e] = torch.einsum("hgqk,hkd->qhgd", p.view(Hkv, G, e - s, sl), v[..., :v_dim].float()).reshape(e - s, Hq, v_dim)
+    return out
+
+
 def merge_attn_states(o1: torch.Tensor, lse1: torch.Tensor, o2: torch.Tensor, lse2: torch.Tensor
                       ) -> tuple[torch.Tensor, torch.Tensor]:
     """LSE-weighted merge of two partial attention results. o: [T,H,D], lse: [T,H]."""
@@ -230,7 +258,7 @@ def merge_attn_states(o1: torch.Tensor, lse1: torch.Tensor, o2: torch.Tensor, ls
 
 def mla_decode_attention(q_nope_abs: torch.Tensor, q_pe: torch.Tensor, kv_cache: torch.Tensor,
                          block_table: torch.Tensor, seq_lens: torch.Tensor, query_start_loc: torch.Tensor,
-                         scale: float, kv_lora_rank: int) -> torch.Tensor:
+                         scale: float, kv_lora_rank: int, sliding_window: Optional[int] = None) -> torch.Tensor:
     """MLA as MQA over the latent cache. q_nope_abs: [T,H,R] (already multiplied by W_UK),
     q_pe: [T,H,P]; kv_cache: [nb, bs, R+P]; returns latent-space output [T,H,R]."""
     T, H, R = q_nope_abs.shape
@@ -249,7 +277,10 @@ def mla_decode_attention(q_nope_abs: torch.Tensor, q_pe: torch.Tensor, kv_cache:
                + torch.einsum("qhp,kp->hqk", q_pe[s:e].float(), kp)) * scale
         qpos = torch.arange(sl - ql, sl, device=att.device)[:, None]
         kpos = torch.arange(sl, device=att.device)[None, :]
-        att = att.masked_fill(~(kpos <= qpos)[None], float("-inf"))
+        ok = kpos <= qpos
+        if sliding_window:
+            ok &= kpos > qpos - sliding_window
+        att = att.masked_fill(~ok[None], float("-inf"))
         p = torch.softmax(att, dim=-1)
         out[s:e] = torch.einsum("hqk,kr->qhr", p, kc).to(out.dtype)
     return out
@@ -310,6 +341,49 @@ def latent_norm_cache(lat: torch.Tensor, q_rank: int, q_weight, kv_rank: int, kv
     if cache is not None:
         concat_and_cache_mla(ckv, ckv[:, :0], cache, slots)
     return cq, ckv
+
+
+def latent_rope_cache(proj: torch.Tensor, q_off: int, heads: int, dim: int, rot: int, kv_off: int, kv_rank: int, kv_weight, eps: float,
+                      positions: torch.Tensor, cos_sin: torch.Tensor, neox: bool, cache=None, slots=None):
+    """Columns of a merged projection, in place: the last ``rot`` of every query head (heads of dim + rot at ``q_off``) are rotated; with
+    ``kv_rank``, the latent at ``kv_off`` is RMS-normed, the key part behind it rotated, and both go into their cache rows."""
+    T = proj.shape[0]
+    q = proj[:, q_off:q_off + heads * (dim + rot)].view(T, heads, dim + rot)
+    if rot:
+        q[..., dim:] = rotary_embedding(positions, q[..., dim:].reshape(T, -1), None, cos_sin, rot, neox)[0].view(T, heads, rot)
+    if kv_rank:
+        c = rms_norm(proj[:, kv_off:kv_off + kv_rank], kv_weight, eps)
+        pe = proj[:, kv_off + kv_rank:kv_off + kv_rank + rot]
+        if rot:
+            pe = rotary_embedding(positions, pe.contiguous(), None, cos_sin, rot, neox)[0]
+        if cache is not None:
+            concat_and_cache_mla(c, pe, cache, slots)
+
+
+def hyper_step(x: torch.Tensor, y: Optional[torch.Tensor], coef: Optional[torch.Tensor], into: torch.Tensor, weight: torch.Tensor,
+               eps: float, dtype) -> torch.Tensor:
+    """x [T, S, H] fp32.  With ``y`` [T, H], in place: x_t = sum_s mix[s, t] x_s + out[t] y (``coef`` fp32: out [S], then mix [S, S]).
+    Returns rms_norm(sum_s into[s] x_s)."""
+    S = x.shape[1]
+    if y is not None:
+        x.copy_(torch.einsum("st,nsh->nth", coef[S:].view(S, S), x) + coef[:S, None] * y.float()[:, None])
+    return rms_norm(torch.einsum("s,nsh->nh", into, x), weight, eps).to(dtype)
+
+
+def hyper_entry(ids: Optional[torch.Tensor], table: torch.Tensor, streams: int, embed_weight, into: torch.Tensor, weight, eps: float
+                ) -> tuple[torch.Tensor, torch.Tensor]:
+    """Entry of ``streams`` equal fp32 streams: e = rms_norm(table[ids]) (e = table [T, H] as it is where ``ids`` is None).  Returns
+    (x [T, S, H], rms_norm(sum(into) e) in the table's dtype)."""
+    e = table.float() if ids is None else rms_norm(F.embedding(ids, table).float(), embed_weight, eps)
+    x = e[:, None].repeat(1, streams, 1)
+    return x, rms_norm(into.sum() * e, weight, eps).to(table.dtype)
+
+
+def xielu(x: torch.Tensor, coef: torch.Tensor) -> torch.Tensor:
+    """coef fp32 (a, b): a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below."""
+    z = x.float()
+    m = z.clamp(max=0.0)
+    return (torch.where(z > 0, coef[0] * z * z, coef[1] * (torch.expm1(m) - m)) + 0.5 * z).to(x.dtype)
 
 
 def embed_stream(ids: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, pos_table: Optional[torch.Tensor],

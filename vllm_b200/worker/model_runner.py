@@ -313,14 +313,16 @@ class ModelRunner:
         self.kv_vt = []
         for gid, g in enumerate(cfg.kv_cache_groups):
             s = g.spec
+            key_specs = [ls for ls in map(g.spec_of, g.layer_names) if not isinstance(ls, MLAAttentionSpec)]   # layers that store keys
             # tensor-core cache layout (V pages transposed) whenever the tcgen05 attention kernel applies
             self.kv_vt.append(bool(
                 self.is_cuda and not envs.VLLM_B200_FORCE_REF_OPS and envs.VLLM_B200_ATTN != "simt"
-                and not isinstance(s, MLAAttentionSpec) and getattr(s, "head_size", 0) == 128
+                and key_specs and all(getattr(ls, "head_size", 0) == 128 for ls in key_specs)
                 and s.block_size == 64 and getattr(s, "dcp", 1) == 1 and kvd in (torch.bfloat16, torch.float16)
                 and self.dtype in (torch.bfloat16, torch.float16)
                 # head shapes and features only the generic kernels implement keep the whole group on the standard layout
-                and all(self._tensor_core_layer(attention_layers().get(n)) for n in g.layer_names)))
+                and all(self._tensor_core_layer(attention_layers().get(n)) for n in g.layer_names
+                        if not isinstance(g.spec_of(n), MLAAttentionSpec))))
             for name in g.layer_names:
                 self.layer_to_group[name] = gid
                 ls = g.spec_of(name)
@@ -328,7 +330,7 @@ class ModelRunner:
                     self.kv_caches[name] = torch.zeros((cfg.num_state_slots, ls.state_bytes // 4), dtype=torch.float32,
                                                        device=self.device)
                     continue
-                if isinstance(s, MLAAttentionSpec):
+                if isinstance(ls, MLAAttentionSpec):
                     shape = (cfg.num_blocks, ls.phys_block_size, ls.head_size)
                 else:
                     shape = (cfg.num_blocks, 2, ls.num_kv_heads, getattr(ls, "phys_block_size", ls.block_size), ls.head_size)
@@ -351,7 +353,7 @@ class ModelRunner:
         if layer is None:
             return True
         d, hq, hkv = layer.head_size, getattr(layer, "num_heads", 1), layer.num_kv_heads
-        return (not getattr(layer, "logits_soft_cap", 0.0) and getattr(layer, "alibi_slopes", None) is None
+        return (getattr(layer, "alibi_slopes", None) is None
                 and cuda_ops().tc_attention_ok(d, getattr(layer, "v_head_size", d), max(hq // max(hkv, 1), 1)))
 
     def _init_gpu_prep(self) -> None:
@@ -1467,6 +1469,8 @@ class ModelRunner:
         sizes = self.vllm_config.compilation_config.mixed_sizes(self.max_num_tokens)
         if not sizes or not self.gpu_prep or not all(self.kv_vt) or self.has_mm or self.drafter is not None:
             return
+        if any(c.dim() == 3 for c in self.kv_caches.values()) or any(getattr(l, "talk", None) is not None for l in attention_layers().values()):
+            return                          # latents beside keys, mixed heads: the split of a mixed batch is planned on the host
         from vllm_b200.worker.cudagraph import MixedGraph
         t0 = time.perf_counter()
         try:
