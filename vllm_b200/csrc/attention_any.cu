@@ -3,6 +3,9 @@
 // sinks, soft cap, ALiBi.  The tensor-core kernels (attention_tc*.cu) take head size 128, attention_simt.cu the 16-bit sizes it
 // is tuned for; this one takes the rest, prompts and decode steps alike.
 //
+// FOLD: every query head attends to the values of several KV heads (its scores are with the keys of its own), one result each in
+// 32-bit: what a mix of the heads' weights behind the softmax needs (attention_talk.cu).
+//
 // CTA = 16 query rows (tokens x heads of one KV head) of one request.  Tiles of 32 keys and values are staged in shared
 // memory as fp32; in the scores a lane is a key (rows padded to an odd number of 16-byte units: conflict-free), in P.V a lane
 // is an output column.  Only the keys that some row of the tile can see are visited.
@@ -22,6 +25,7 @@ struct Params {
   int window, chunk, causal;
   float scale_log2, soft_cap, out_scale;
   const float* alibi; const float* sinks;
+  int c0, nc;                                   // FOLD: value heads c0 .. c0 + nc - 1; out fp32 [T, Hq, nc, DV]
 };
 
 VB_HOST_DEVICE int padded(int d) {               // floats of a staged row: 16-byte units, an odd number of them
@@ -29,7 +33,7 @@ VB_HOST_DEVICE int padded(int d) {               // floats of a staged row: 16-b
   return (u | 1) * 4;
 }
 
-template <typename T, int NVD>
+template <typename T, int NVD, bool FOLD>
 __global__ void __launch_bounds__(WARPS * 32) any_attn_kernel(const Params p) {
   extern __shared__ __align__(16) float sm[];
   const int DP = padded(p.D), D4 = (p.D + 3) / 4, DV = p.DV;
@@ -39,7 +43,8 @@ __global__ void __launch_bounds__(WARPS * 32) any_attn_kernel(const Params p) {
   float* ps = vs + KEYS * DV;                    // WARPS x KEYS x RPW (KEYS * DV is a multiple of four)
   pdl_trigger();
   pdl_wait();
-  const int b = blockIdx.z, hk = blockIdx.y, G = p.Hq / p.Hkv;
+  const int b = blockIdx.z, hk = FOLD ? blockIdx.y / p.nc : blockIdx.y, G = p.Hq / p.Hkv;
+  const int hv = FOLD ? p.c0 + blockIdx.y % p.nc : hk;
   const int q0 = p.qsl ? p.qsl[b] : b, q_len = p.qsl ? p.qsl[b + 1] - q0 : 1;
   const int row0 = blockIdx.x * ROWS, n_rows = min(ROWS, q_len * G - row0);
   if (n_rows <= 0) return;
@@ -81,7 +86,7 @@ __global__ void __launch_bounds__(WARPS * 32) any_attn_kernel(const Params p) {
         const int pos = t0 + k;
         const int64_t blk = bt[pos / p.BS];
         kr = cache + (((blk * 2) * p.Hkv + hk) * p.BS + pos % p.BS) * (int64_t)p.DC;
-        vr = kr + (int64_t)p.Hkv * p.BS * p.DC;
+        vr = kr + (int64_t)(p.Hkv + hv - hk) * p.BS * p.DC;
       }
       for (int d = lane; d < DP; d += 32) ks[k * DP + d] = in && d < p.D ? to_f32(kr[d]) : 0.f;
       for (int d = lane; d < DV; d += 32) vs[k * DV + d] = in ? to_f32(vr[d]) : 0.f;
@@ -145,6 +150,13 @@ __global__ void __launch_bounds__(WARPS * 32) any_attn_kernel(const Params p) {
     if (p.sinks) sum += exp2f(p.sinks[head[j]] * LOG2E - tu);
     const float inv = sum > 0.f ? f / sum * p.out_scale : 0.f;
     const int64_t tok = q0 + (row0 + w * RPW + j) / G;
+    if constexpr (FOLD) {
+      float* o = reinterpret_cast<float*>(p.out) + ((tok * p.Hq + head[j]) * p.nc + (hv - p.c0)) * DV;
+#pragma unroll
+      for (int i = 0; i < NVD; ++i)
+        if (lane + i * 32 < DV) o[lane + i * 32] = acc[j][i] * inv;
+      continue;
+    }
     T* o = reinterpret_cast<T*>(p.out) + tok * p.out_stride + (int64_t)head[j] * DV;
 #pragma unroll
     for (int i = 0; i < NVD; ++i) {
@@ -155,6 +167,26 @@ __global__ void __launch_bounds__(WARPS * 32) any_attn_kernel(const Params p) {
   }
 }
 
+}  // namespace anyattn
+
+namespace anyattn {
+template <bool FOLD>
+static int launch(const Params& p, int B, int max_rows, int dtype, cudaStream_t st) {
+  dim3 grid((max_rows + ROWS - 1) / ROWS, FOLD ? p.Hkv * p.nc : p.Hkv, B);
+  const size_t smem = ((size_t)(ROWS + KEYS) * padded(p.D) + (size_t)KEYS * p.DV + WARPS * KEYS * RPW) * 4;
+#define GO(N)                                                                                                   \
+  do {                                                                                                          \
+    auto k = any_attn_kernel<T, N, FOLD>;                                                                       \
+    static bool set = false;                                                                                    \
+    if (!set) { cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); set = true; } \
+    vb_launch(k, grid, dim3(WARPS * 32), smem, st, p);                                                          \
+  } while (0)
+  DISPATCH_DTYPE(dtype, T, {
+    if (p.DV <= 64) GO(2); else if (p.DV <= 128) GO(4); else if (p.DV <= 256) GO(8); else GO(16);
+  });
+#undef GO
+  return (int)cudaGetLastError();
+}
 }  // namespace anyattn
 
 // kv_cache [blocks, 2, Hkv, BS, DC] (not the transposed-value layout); q [T, Hq * D], out [T, Hq * DV] (token strides free).
@@ -170,20 +202,22 @@ EXPORT int vb_any_attention(const void* q, const void* kv_cache, const int* bloc
   p.q = q; p.kv_cache = kv_cache; p.out = out; p.lse_out = lse_out; p.block_table = block_table; p.seq_lens = seq_lens; p.qsl = qsl;
   p.q_stride = q_stride; p.out_stride = out_stride; p.bt_stride = bt_stride; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.DV = DV; p.DC = DC;
   p.BS = BS; p.window = window; p.chunk = chunk; p.causal = causal; p.scale_log2 = scale * LOG2E; p.soft_cap = soft_cap;
-  p.out_scale = out_scale; p.alibi = alibi; p.sinks = sinks;
-  const int rows = (qsl ? max_q_len : 1) * (Hq / Hkv);
-  dim3 grid((rows + ROWS - 1) / ROWS, Hkv, B);
-  const size_t smem = ((size_t)(ROWS + KEYS) * padded(D) + (size_t)KEYS * DV + WARPS * KEYS * RPW) * 4;
-#define GO(N)                                                                                                   \
-  do {                                                                                                          \
-    auto k = any_attn_kernel<T, N>;                                                                             \
-    static bool set = false;                                                                                    \
-    if (!set) { cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); set = true; } \
-    vb_launch(k, grid, dim3(WARPS * 32), smem, st, p);                                                          \
-  } while (0)
-  DISPATCH_DTYPE(dtype, T, {
-    if (DV <= 64) GO(2); else if (DV <= 128) GO(4); else if (DV <= 256) GO(8); else GO(16);
-  });
-#undef GO
-  return (int)cudaGetLastError();
+  p.out_scale = out_scale; p.alibi = alibi; p.sinks = sinks; p.c0 = 0; p.nc = 1;
+  return launch<false>(p, B, (qsl ? max_q_len : 1) * (Hq / Hkv), dtype, st);
+}
+
+// Causal attention of every query head with the values of KV heads c0 .. c0 + nc - 1: out fp32 [T, Hq, nc, DV].
+EXPORT int vb_any_attention_fold(const void* q, const void* kv_cache, const int* block_table, const int* seq_lens, const int* qsl,
+                                 float* out, int B, int max_q_len, int Hq, int Hkv, int D, int DV, int DC, int BS, int64_t q_stride,
+                                 int bt_stride, int window, float scale, float soft_cap, const float* sinks, int c0, int nc, int dtype,
+                                 cudaStream_t st) {
+  using namespace anyattn;
+  if (B == 0) return 0;
+  if (D < 1 || DV < 1 || D > MAX_D || DV > MAX_D || DC < D || DC < DV || Hq % Hkv || c0 < 0 || nc < 1 || c0 + nc > Hkv) return -1;
+  Params p;
+  p.q = q; p.kv_cache = kv_cache; p.out = out; p.lse_out = nullptr; p.block_table = block_table; p.seq_lens = seq_lens; p.qsl = qsl;
+  p.q_stride = q_stride; p.out_stride = 0; p.bt_stride = bt_stride; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.DV = DV; p.DC = DC; p.BS = BS;
+  p.window = window; p.chunk = 0; p.causal = 1; p.scale_log2 = scale * LOG2E; p.soft_cap = soft_cap; p.out_scale = 1.f;
+  p.alibi = nullptr; p.sinks = sinks; p.c0 = c0; p.nc = nc;
+  return launch<true>(p, B, (qsl ? max_q_len : 1) * (Hq / Hkv), dtype, st);
 }

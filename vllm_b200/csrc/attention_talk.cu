@@ -1,0 +1,439 @@
+// Attention whose heads talk to one another: the weights of all heads are mixed behind the softmax,
+//
+//   out_h(i) = sum_j ( sum_g T[h, g] w_g(i, j) ) V_c(h)(j)  =  sum_g T[h, g]  O_{g, c(h)}(i),      O_{g, c}(i) = sum_j w_g(i, j) V_c(j)
+//
+// (c(h): the KV head of h).  The mix is linear, so it can wait until the keys are summed up: the attention kernels produce O_{g, c}, every
+// query head with the values of every KV head ("fold"), in one pass over the keys, and talk_mix applies T to H x vdim numbers per token
+// instead of H x H numbers per key.  (Mixing the weights themselves needs the denominators first, hence a second pass over the scores, and
+// H multiplications per weight on the CUDA cores: more time than the tensor cores take for the additional values.)
+//
+//   talk_fold   prompts: tcgen05, 128 rows (tokens x heads of one KV head), two value heads per CTA
+//   talk_mix    T, split-KV sums and denominators, the turn back of rotated values, 16-bit output
+// Decode steps: attention_talk_decode.cu; other head shapes and dtypes: attention_any.cu.
+//
+// Scores are capped, cap tanh(s / cap), with cap <= 60: e^s then fits into fp32 (and bf16) whatever the score is, and the softmax needs no
+// running maximum: one pass over S, no rescaling, and partial sums of different key ranges simply add up.
+#include "common.cuh"
+#include "talk.cuh"
+
+namespace talk {
+
+constexpr int D = 128, BS = 64, TM = 128, TN = 128;
+constexpr int NUM_THREADS = 192;
+constexpr int K_STAGES = 2, V_SLOTS = 4;
+constexpr int TILE_BYTES = TN * D * 2;          // 32 KB: a tile of keys, or of one head's values
+
+struct Params {
+  const int* block_table; const int* seq_lens; const int* qsl;
+  void* out;                    // [T, Hq, nc, D], normalised
+  const float* sinks;           // optional [Hq]
+  int bt_stride, Hq, Hkv, G, TQ, window, c0, nc;
+  Cap cap;
+  int* error;
+};
+
+VB_DEVICE void tma_load_3d(void* dst, const void* tmap, int c0, int c1, int c2, uint64_t* bar) {
+  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+               ::"r"(smem_u32(dst)), "l"(tmap), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2) : "memory");
+}
+VB_DEVICE void tmem_st_32x32(uint32_t taddr, const uint32_t* r) {
+  asm volatile(
+      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
+      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
+      "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};"
+      ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+        "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]),
+        "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]),
+        "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31]) : "memory");
+}
+VB_DEVICE void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+// D[tmem] (+)= A[tmem: row = lane, two 16-bit values per column] * B[smem desc]
+VB_DEVICE void umma_f16_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+               "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+               ::"r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
+}
+
+// CTA = (query tile, KV head of the scores x pair of value heads, request).  Warp roles: 0 TMA producer, 1 MMA issuer + TMEM owner, 2..5
+// softmax / epilogue (thread = query row = TMEM lane).  TMEM: S double-buffered (2 x 128 columns), two accumulators (2 x 128).  P
+// overwrites the S it came from (bf16, 64 columns) and is the PV product's A operand there, so it is double-buffered too: the softmax of
+// tile j runs under the PV products of tile j - 1.
+__global__ void __launch_bounds__(NUM_THREADS, 1)
+talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
+                 const __grid_constant__ CUtensorMap tmap_v, const Params p) {
+  using T = __nv_bfloat16;
+  extern __shared__ __align__(1024) unsigned char smem_raw[];
+  unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  unsigned char* q_smem = smem;
+  unsigned char* k_smem = q_smem + TILE_BYTES;
+  unsigned char* v_smem = k_smem + K_STAGES * TILE_BYTES;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_smem + V_SLOTS * TILE_BYTES);
+  uint64_t* q_full = bars;
+  uint64_t* k_full = bars + 1;                 // [K_STAGES]
+  uint64_t* k_empty = k_full + K_STAGES;
+  uint64_t* v_full = k_empty + K_STAGES;       // [V_SLOTS]
+  uint64_t* v_empty = v_full + V_SLOTS;
+  uint64_t* s_full = v_empty + V_SLOTS;        // [2]
+  uint64_t* p_full = s_full + 2;               // [2]
+  uint64_t* pv_done = p_full + 2;              // [2]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 2);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int budget = MBAR_BUDGET;
+  const int b = blockIdx.z, groups = (p.nc + 1) / 2;
+  const int h = blockIdx.y / groups, cv = blockIdx.y % groups * 2;       // KV head of the scores, first value head (behind c0)
+  const int nv = min(2, p.nc - cv);
+  pdl_trigger();
+  pdl_wait();
+  const int q0 = p.qsl[b], q_len = p.qsl[b + 1] - q0;
+  const int tok0 = blockIdx.x * p.TQ;
+  if (tok0 >= q_len) return;                                             // uniform across the CTA
+  const int n_tok = min(p.TQ, q_len - tok0);
+  const int pos0 = p.seq_lens[b] - q_len + tok0;
+  const int kv_end = pos0 + n_tok, kv_begin = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  const int tile_lo = kv_begin / TN, n_tiles = (kv_end + TN - 1) / TN - tile_lo;
+  const int n_pages = (kv_end + BS - 1) / BS;
+
+  if (warp == 0 && lane == 0) {
+    tma_prefetch_desc(&tmap_q); tma_prefetch_desc(&tmap_k); tma_prefetch_desc(&tmap_v);
+    mbar_init(q_full, 1);
+    for (int s = 0; s < K_STAGES; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
+    for (int s = 0; s < V_SLOTS; ++s) { mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
+    for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&p_full[s], 128); mbar_init(&pv_done[s], 1); }
+    mbar_fence_init();
+  }
+  if (warp == 1) tmem_alloc(tmem_slot, 512);
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot, tmem_o = tmem_base + 256;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      // ===== TMA producer.  Tiles are always whole: pages past the sequence are read from the null page (finite, masked)
+      mbar_expect_tx(q_full, TILE_BYTES);
+      tma_load_3d(q_smem, &tmap_q, 0, h * p.G, q0 + tok0, q_full);
+      tma_load_3d(q_smem + TM * 128, &tmap_q, 64, h * p.G, q0 + tok0, q_full);
+      const int* bt = p.block_table + (int64_t)b * p.bt_stride;
+      for (int j = 0; j < n_tiles && budget >= 0; ++j) {
+        const int s = j % K_STAGES;
+        int blk[2];
+        for (int u = 0; u < 2; ++u) {
+          const int page = (tile_lo + j) * 2 + u;
+          blk[u] = page < n_pages ? bt[page] : 0;
+        }
+        mbar_wait_lim(&k_empty[s], ((j / K_STAGES) & 1) ^ 1, budget);
+        if (budget < 0) break;
+        unsigned char* ks = k_smem + s * TILE_BYTES;
+        mbar_expect_tx(&k_full[s], TILE_BYTES);
+        for (int u = 0; u < 2; ++u) {
+          const int row = (blk[u] * 2 * p.Hkv + h) * BS;
+          tma_load_2d(ks + u * (BS * 128), &tmap_k, 0, row, &k_full[s]);
+          tma_load_2d(ks + TN * 128 + u * (BS * 128), &tmap_k, 64, row, &k_full[s]);
+        }
+        for (int v = 0; v < nv; ++v) {
+          const int n = j * nv + v, sl = n % V_SLOTS;
+          mbar_wait_lim(&v_empty[sl], ((n / V_SLOTS) & 1) ^ 1, budget);
+          if (budget < 0) break;
+          unsigned char* vs = v_smem + sl * TILE_BYTES;
+          mbar_expect_tx(&v_full[sl], TILE_BYTES);
+          for (int u = 0; u < 2; ++u)
+            tma_load_2d(vs + u * (D * 128), &tmap_v, 0, ((blk[u] * 2 + 1) * p.Hkv + p.c0 + cv + v) * D, &v_full[sl]);
+        }
+      }
+      if (budget < 0) {                         // let the copies in flight land before the block gives up its memory
+        for (int s = 0; s < K_STAGES; ++s)
+          for (int n = 0; n < 4096 && !(mbar_try_wait(&k_full[s], 0) || mbar_try_wait(&k_full[s], 1)); ++n) {}
+        for (int s = 0; s < V_SLOTS; ++s)
+          for (int n = 0; n < 4096 && !(mbar_try_wait(&v_full[s], 0) || mbar_try_wait(&v_full[s], 1)); ++n) {}
+      }
+    }
+  } else if (warp == 1) {
+    // ===== MMA issuer
+    const uint32_t idesc = umma_idesc_f16(TM, TN, true);
+    const uint64_t d_q = umma_desc_sw128(q_smem), d_k = umma_desc_sw128(k_smem), d_v = umma_desc_sw128(v_smem);
+    mbar_wait_lim(q_full, 0, budget);
+    __syncwarp();
+    for (int j = 0; j <= n_tiles; ++j) {
+      if (j < n_tiles) {
+        const int s = j % K_STAGES;
+        mbar_wait_lim(&k_full[s], (j / K_STAGES) & 1, budget);
+        if (j >= 2) mbar_wait_lim(&pv_done[j & 1], ((j >> 1) & 1) ^ 1, budget);      // PV of tile j - 2 has read the P in this buffer
+        tc_fence_after();
+        if (lane == 0) {
+#pragma unroll
+          for (int kb = 0; kb < 2; ++kb)
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+              umma_f16(tmem_base + (j & 1) * 128, d_q + (uint64_t)(((kb * TM * 128) >> 4) + k * 2),
+                       d_k + (uint64_t)(((s * TILE_BYTES + kb * TN * 128) >> 4) + k * 2), idesc, (kb | k) != 0);
+          umma_commit(&s_full[j & 1]);
+          umma_commit(&k_empty[s]);
+        }
+        __syncwarp();
+      }
+      if (j > 0) {
+        const int jj = j - 1;
+        mbar_wait_lim(&p_full[jj & 1], (jj >> 1) & 1, budget);
+        for (int v = 0; v < nv; ++v) {
+          const int n = jj * nv + v, sl = n % V_SLOTS;
+          mbar_wait_lim(&v_full[sl], (n / V_SLOTS) & 1, budget);
+          tc_fence_after();
+          if (lane == 0) {
+#pragma unroll
+            for (int kk = 0; kk < 8; ++kk)
+              umma_f16_ta(tmem_o + v * 128, tmem_base + (jj & 1) * 128 + kk * 8,
+                          d_v + (uint64_t)(((sl * TILE_BYTES + (kk / 4) * D * 128) >> 4) + (kk & 3) * 2), idesc, (jj | kk) != 0);
+            umma_commit(&v_empty[sl]);
+            if (v == nv - 1) umma_commit(&pv_done[jj & 1]);
+          }
+          __syncwarp();
+        }
+      }
+    }
+  } else {
+    // ===== softmax / epilogue
+    const int qd = warp & 3, r = qd * 32 + lane;
+    const uint32_t t_lane = (uint32_t)(qd * 32) << 16;
+    const int tq = r / p.G, g = r % p.G;
+    const bool row_valid = tq < n_tok;
+    const int qpos = pos0 + tq;
+    float l_run = 0.f;
+    for (int j = 0; j < n_tiles; ++j) {
+      const uint32_t t_s = tmem_base + (j & 1) * 128 + t_lane;
+      mbar_wait_lim(&s_full[j & 1], (j >> 1) & 1, budget);
+      __syncwarp();
+      tc_fence_after();
+      const int hi = row_valid ? qpos + 1 - (tile_lo + j) * TN : 0;      // keys [lo, hi) of this tile are visible to the row
+      const int lo = p.window > 0 ? hi - p.window : 0;
+      const bool full = __all_sync(0xffffffffu, hi >= TN && lo <= 0) != 0;
+      uint32_t v[4][32], pk[64];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) tmem_ld_32x32(t_s + c * 32, v[c]);
+      tmem_ld_wait();
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        float s[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) s[i] = __uint_as_float(v[c][i]);
+        cap_exp<32>(s, p.cap);
+        if (!full) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i >= hi || c * 32 + i < lo) s[i] = 0.f;
+        }
+        float l0 = 0.f, l1 = 0.f;
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+          l0 += s[i];
+          l1 += s[i + 1];
+          pk[c * 16 + i / 2] = pack2<T>(s[i], s[i + 1]);
+        }
+        l_run += l0 + l1;
+      }
+      tmem_st_32x32(t_s, pk);
+      tmem_st_32x32(t_s + 32, pk + 32);
+      tmem_st_wait();
+      tc_fence_before();
+      mbar_arrive(&p_full[j & 1]);
+    }
+    mbar_wait_lim(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, budget);
+    __syncwarp();
+    tc_fence_after();
+    const int hq = h * p.G + g;
+    float inv = 0.f;
+    if (row_valid) {
+      const float den = l_run + (p.sinks ? ex2(p.sinks[hq] * 1.4426950408889634f) : 0.f);
+      inv = den > 0.f ? 1.f / den : 0.f;
+    }
+    for (int u = 0; u < nv; ++u) {
+      T* orow = reinterpret_cast<T*>(p.out) + (((int64_t)(q0 + tok0 + tq) * p.Hq + hq) * p.nc + cv + u) * D;
+#pragma unroll
+      for (int c = 0; c < D; c += 32) {
+        uint32_t o[32];
+        tmem_ld_32x32(tmem_o + u * 128 + t_lane + c, o);
+        tmem_ld_wait();
+        if (row_valid) {
+#pragma unroll
+          for (int i = 0; i < 32; i += 8) {
+            uint4 w;
+            w.x = pack2<T>(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
+            w.y = pack2<T>(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
+            w.z = pack2<T>(__uint_as_float(o[i + 4]) * inv, __uint_as_float(o[i + 5]) * inv);
+            w.w = pack2<T>(__uint_as_float(o[i + 6]) * inv, __uint_as_float(o[i + 7]) * inv);
+            *reinterpret_cast<uint4*>(orow + c + i) = w;
+          }
+        }
+      }
+    }
+    tc_fence_before();
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) tmem_dealloc(tmem_base, 512);
+  if (budget < 0 && p.error) *p.error = 1;
+}
+
+// out[t, h, :] = turn_back( sum_g T[h, g] / den_g * sum_s o[s, t, g, c(h) - c0, :] ).  CTA = token x some value heads; thread = VP pairs of
+// one value head, all heads of that KV head in tiles of four.  den null sums: o is normalised.
+struct MixParams {
+  const void* o; const float* l; const float* sinks; const float* talk;
+  const int64_t* positions; const float* cos_sin;        // optional [positions, DV]: pair m turns by minus its angle
+  void* out; int64_t out_stride;
+  int T, H, G, DV, S, c0, nc, neox;
+};
+template <typename TO, int N> VB_DEVICE void load_n(const TO* p, float (&f)[N]) {
+  if constexpr (N == 1) {
+    f[0] = to_f32(p[0]);
+  } else if constexpr (sizeof(TO) == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    f[0] = x.x; f[1] = x.y; f[2] = x.z; f[3] = x.w;
+  } else {
+    const uint2 x = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack2<TO>(x.x), c = unpack2<TO>(x.y);
+    f[0] = a.x; f[1] = a.y; f[2] = c.x; f[3] = c.y;
+  }
+}
+template <typename TO, typename T, int VP>
+__global__ void __launch_bounds__(256) talk_mix_kernel(const MixParams p) {
+  extern __shared__ float w[];                           // [nc here * G][H], then 1 / den [H]
+  pdl_trigger();
+  const int cpb = (p.nc + gridDim.y - 1) / gridDim.y, cb = blockIdx.y * cpb, ncb = min(cpb, p.nc - cb);
+  if (ncb <= 0) return;
+  const int rows = ncb * p.G, t = blockIdx.x, H = p.H;
+  float* inv = w + cpb * p.G * H;
+  pdl_wait();
+  for (int g = threadIdx.x; g < H; g += blockDim.x) {
+    float den = 1.f;
+    if (p.l) {
+      den = p.sinks ? expf(p.sinks[g]) : 0.f;
+      for (int s = 0; s < p.S; ++s) den += p.l[((int64_t)s * p.T + t) * H + g];
+    }
+    inv[g] = den > 0.f ? 1.f / den : 0.f;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < rows * H; i += blockDim.x) w[i] = p.talk[(int64_t)(p.c0 + cb) * p.G * H + i] * inv[i % H];
+  __syncthreads();
+  const int half = p.DV / 2, per = half / VP;
+  const float* cs = p.cos_sin ? p.cos_sin + p.positions[t] * p.DV : nullptr;
+  const int64_t split = (int64_t)p.T * H * p.nc * p.DV;
+  for (int it = threadIdx.x; it < ncb * per; it += blockDim.x) {
+    const int c = it / per, m = (it - c * per) * VP;
+    // VP > 1: pairs (m, m + half), also where nothing turns; else the layout of the rotation
+    const bool halves = VP > 1 || p.neox;
+    const int e0 = halves ? m : 2 * m, e1 = halves ? m + half : 2 * m + 1;
+    const TO* o = reinterpret_cast<const TO*>(p.o) + ((int64_t)t * H * p.nc + cb + c) * p.DV;
+    for (int j0 = 0; j0 < p.G; j0 += 4) {
+      const int nj = min(4, p.G - j0);
+      float a[4][VP], bq[4][VP];
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int q = 0; q < VP; ++q) { a[j][q] = 0.f; bq[j][q] = 0.f; }
+      const float* wj = w + (c * p.G + j0) * H;
+      for (int s = 0; s < p.S; ++s) {
+#pragma unroll 4
+        for (int g = 0; g < H; ++g) {
+          float x[VP], y[VP];
+          const TO* src = o + s * split + (int64_t)g * p.nc * p.DV;
+          load_n<TO, VP>(src + e0, x);
+          load_n<TO, VP>(src + e1, y);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float k = wj[(j < nj ? j : 0) * H + g];
+#pragma unroll
+            for (int q = 0; q < VP; ++q) { a[j][q] += k * x[q]; bq[j][q] += k * y[q]; }
+          }
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        if (j >= nj) break;
+        T* dst = reinterpret_cast<T*>(p.out) + t * p.out_stride + (int64_t)((p.c0 + cb + c) * p.G + j0 + j) * p.DV;
+        if (cs) {
+#pragma unroll
+          for (int q = 0; q < VP; ++q) {
+            const float co = cs[m + q], si = cs[half + m + q], x = a[j][q], y = bq[j][q];
+            a[j][q] = x * co + y * si;
+            bq[j][q] = y * co - x * si;
+          }
+        }
+        if constexpr (VP == 1) {
+          dst[e0] = from_f32<T>(a[j][0]);
+          dst[e1] = from_f32<T>(bq[j][0]);
+        } else if constexpr (sizeof(T) == 4) {
+          *reinterpret_cast<float4*>(dst + e0) = make_float4(a[j][0], a[j][1], a[j][2], a[j][3]);
+          *reinterpret_cast<float4*>(dst + e1) = make_float4(bq[j][0], bq[j][1], bq[j][2], bq[j][3]);
+        } else {
+          *reinterpret_cast<uint2*>(dst + e0) = make_uint2(pack2<T>(a[j][0], a[j][1]), pack2<T>(a[j][2], a[j][3]));
+          *reinterpret_cast<uint2*>(dst + e1) = make_uint2(pack2<T>(bq[j][0], bq[j][1]), pack2<T>(bq[j][2], bq[j][3]));
+        }
+      }
+    }
+  }
+}
+
+template <typename TO, typename T>
+static int launch_mix(const MixParams& p, cudaStream_t st) {
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  // decode batches: one value head per CTA, so that there are enough of them
+  const bool few = p.T <= 512;
+  const bool vec = !few && (p.neox || !p.cos_sin) && p.DV % 8 == 0 && p.out_stride % 8 == 0 && al(p.o) && al(p.out);
+  const int cpb = few ? 1 : p.nc, per = p.DV / 2 / (vec ? 4 : 1), items = cpb * per;
+  const int thr = items >= 256 ? 256 : (items < 64 ? 64 : (items + 31) / 32 * 32);
+  const size_t smem = ((size_t)cpb * p.G + 1) * p.H * 4;
+  if (smem > 200 * 1024) return -3;
+  const dim3 grid(p.T, (p.nc + cpb - 1) / cpb);
+#define GO(N)                                                                                                   \
+  do {                                                                                                          \
+    auto k = talk_mix_kernel<TO, T, N>;                                                                         \
+    static bool set = false;                                                                                    \
+    if (!set) { cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); set = true; } \
+    vb_launch(k, grid, dim3(thr), smem, st, p);                                                                 \
+  } while (0)
+  if (vec) GO(4); else GO(1);
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+}  // namespace talk
+
+// q [T, Hq * 128] (token stride free), kv_cache [nb, 2, Hkv, 64 x 128] with transposed value pages, bf16; out [T, Hq, nc, 128]: the
+// normalised attention of every query head with the values of KV heads c0 .. c0 + nc - 1.  0 < soft_cap <= 60.
+EXPORT int vb_talk_fold(const void* q, const void* kv_cache, int64_t num_blocks, const int* block_table, const int* seq_lens,
+                        const int* qsl, void* out, int* error, int B, int T_total, int max_q_len, int Hq, int Hkv, int64_t q_stride,
+                        int bt_stride, int window, float scale, float soft_cap, const float* sinks, int c0, int nc, cudaStream_t st) {
+  using namespace talk;
+  if (B == 0 || max_q_len <= 0) return 0;
+  const int G = Hq / Hkv;
+  if (G < 1 || G > 128 || 128 % G || Hq % Hkv || c0 < 0 || nc < 1 || c0 + nc > Hkv || q_stride % 8) return -4;
+  if (!(soft_cap > 0.f && soft_cap <= MAX_CAP)) return -5;
+  Params p;
+  p.block_table = block_table; p.seq_lens = seq_lens; p.qsl = qsl; p.out = out; p.sinks = sinks; p.bt_stride = bt_stride; p.Hq = Hq;
+  p.Hkv = Hkv; p.G = G; p.TQ = TM / G; p.window = window; p.c0 = c0; p.nc = nc; p.cap = make_cap(scale, soft_cap); p.error = error;
+  CUtensorMap tq, tk, tv;
+  int rc;
+  if ((rc = map_queries(&tq, q, Hq, T_total, q_stride, G, p.TQ))) return rc;
+  if ((rc = map_pages(&tk, &tv, kv_cache, num_blocks, Hkv))) return rc;
+  const int smem = (1 + K_STAGES + V_SLOTS) * TILE_BYTES + 32 * 8 + 16 + 1024;
+  static bool a = false;
+  if (!a) { cudaFuncSetAttribute(talk_fold_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); a = true; }
+  const dim3 grid((max_q_len + p.TQ - 1) / p.TQ, Hkv * ((nc + 1) / 2), B);
+  vb_launch(talk_fold_kernel, grid, dim3(NUM_THREADS), (size_t)smem, st, tq, tk, tv, p);
+  return (int)cudaGetLastError();
+}
+
+// o [S, T, H, nc, DV] in fp32 (o_dtype DT_F32) or bf16; l [S, T, H]: sums of the weights (the denominators but for the sinks [H]) where o
+// is not normalised yet; talk [H, H] fp32; writes heads c0 * G .. (c0 + nc) * G - 1 of out [T, H, DV] (token stride free).
+EXPORT int vb_talk_mix(const void* o, int o_dtype, const float* l, const float* sinks, const float* talk_w, const int64_t* positions,
+                       const float* cos_sin, int neox, void* out, int64_t out_stride, int T_, int H, int G, int DV, int S, int c0, int nc,
+                       int dtype, cudaStream_t st) {
+  using namespace talk;
+  if (T_ == 0) return 0;
+  if (DV < 2 || DV % 2 || H % G || S < 1 || nc < 1 || (c0 + nc) * G > H || (cos_sin && !positions)) return -1;
+  MixParams p = {o, l, sinks, talk_w, positions, cos_sin, out, out_stride, T_, H, G, DV, S, c0, nc, neox};
+  if (o_dtype == DT_BF16) return dtype == DT_BF16 ? launch_mix<__nv_bfloat16, __nv_bfloat16>(p, st) : -2;
+  if (o_dtype != DT_F32) return -2;
+  DISPATCH_DTYPE(dtype, T, return (launch_mix<float, T>(p, st)));
+  return 0;
+}

@@ -108,6 +108,11 @@ VB_DEVICE bool elect_one() {
 }
 VB_DEVICE float ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
+// a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below
+VB_DEVICE float xielu(float z, float a, float b) {
+  return 0.5f * z + (z > 0.f ? a * z * z : b * (expm1f(z) - z));
+}
+
 // -------------------------------------------------------------- PTX: mbarrier
 VB_DEVICE void mbar_init(uint64_t* bar, uint32_t count) {
   asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(bar)), "r"(count));

@@ -33,7 +33,8 @@ struct Params {
   int M, N, K;
   int k_blocks_per_split;  // BK blocks handled by one CTA
   int splits;
-  int act;                 // 0 none, 1 silu-mul over interleaved (gate,up) feature pairs (SWAP only), 2 squared ReLU (grouped)
+  int act;                 // 0 none, 1 silu-mul over interleaved (gate,up) feature pairs (SWAP only), 2 squared ReLU (grouped), 3 xIELU (SWAP)
+  const float* act_coef;   // its two numbers
   int pf;                  // L2 prefetch ahead of the smem ring (SWAP)
   // grouped (MoE) mode, SWAP only: grid.y = n_experts * chunks; expert e multiplies the rows
   // [expert_offs[e], expert_offs[e+1]) of X (tokens sorted by expert) with W[e] = rows [e*N, (e+1)*N) of the weight
@@ -291,6 +292,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
               if (c + j < m_lim) {
                 float o = v[j] + bias;
                 if (p.act == 2) { o = fmaxf(o, 0.f); o *= o; }
+                if (p.act == 3) o = xielu(o, p.act_coef[0], p.act_coef[1]);
                 y[(size_t)(m0 + j) * p.N + n] = from_f32<T>(o);
               }
           }
@@ -361,7 +363,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
               if (r < p.splits) { acc.x += x[h][r].x; acc.y += x[h][r].y; acc.z += x[h][r].z; acc.w += x[h][r].w; }
             const int n = a_tile * TM + rq * 4;
             float o[4] = {acc.x, acc.y, acc.z, acc.w};
-            if (p.act) {      // (gate, up) pairs are adjacent features: two outputs per unit
+            if (p.act == 1) {      // (gate, up) pairs are adjacent features: two outputs per unit
               if (n + 4 <= p.N) {
                 T* ya = y + (size_t)(m_base + col) * (p.N >> 1) + (n >> 1);
                 const uint32_t pk = pack2<T>((o[0] / (1.f + __expf(-o[0]))) * o[1], (o[2] / (1.f + __expf(-o[2]))) * o[3]);
@@ -373,6 +375,10 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
             if (p.bias) {
 #pragma unroll
               for (int e = 0; e < 4; ++e) if (n + e < p.N) o[e] += to_f32(reinterpret_cast<const T*>(p.bias)[n + e]);
+            }
+            if (p.act == 3) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e) o[e] = xielu(o[e], p.act_coef[0], p.act_coef[1]);
             }
             if (n + 4 <= p.N && (p.N & 3) == 0) {
               uint2 pk;
@@ -502,17 +508,20 @@ EXPORT int vb_gemm_tc_plan(int M, int N, int K, int num_sms, int* swap, int* bn,
 }
 
 EXPORT int vb_gemm_tc2(const void* x, const void* w, const void* bias, void* y, int M, int N, int K, int64_t x_stride,
-                       int swap, int bn, int splits, float* ws, unsigned* counters, int act, int dtype, cudaStream_t st);
+                       int swap, int bn, int splits, float* ws, unsigned* counters, int act, const float* act_coef, int dtype,
+                       cudaStream_t st);
 EXPORT int vb_gemm_tc(const void* x, const void* w, const void* bias, void* y, int M, int N, int K, int64_t x_stride,
                       int swap, int bn, int splits, float* ws, unsigned* counters, int dtype, cudaStream_t st) {
-  return vb_gemm_tc2(x, w, bias, y, M, N, K, x_stride, swap, bn, splits, ws, counters, 0, dtype, st);
+  return vb_gemm_tc2(x, w, bias, y, M, N, K, x_stride, swap, bn, splits, ws, counters, 0, nullptr, dtype, st);
 }
-// act = 1: W rows interleave (gate_i, up_i); y is [M, N/2] = silu(gate) * up (swap-AB shapes only, N % 4 == 0, no bias)
+// act = 1: W rows interleave (gate_i, up_i); y is [M, N/2] = silu(gate) * up (swap-AB shapes only, N % 4 == 0, no bias).
+// act = 3: xIELU of the biased product, its two numbers in act_coef (swap-AB shapes only)
 EXPORT int vb_gemm_tc2(const void* x, const void* w, const void* bias, void* y, int M, int N, int K, int64_t x_stride,
-                       int swap, int bn, int splits, float* ws, unsigned* counters, int act, int dtype, cudaStream_t st) {
+                       int swap, int bn, int splits, float* ws, unsigned* counters, int act, const float* act_coef, int dtype,
+                       cudaStream_t st) {
   using namespace gemm;
   if (dtype == DT_F32 || K % 8 != 0) return -1;
-  if (act && (act != 1 || !swap || bias || (N & 3))) return -1;
+  if (act && (!swap || !(act == 1 ? !bias && !(N & 3) : act == 3 && act_coef))) return -1;
   const bool bf16 = dtype == DT_BF16;
   CUtensorMap ta, tb;
   Params p;
@@ -520,6 +529,7 @@ EXPORT int vb_gemm_tc2(const void* x, const void* w, const void* bias, void* y, 
   p.expert_offs = nullptr; p.n_experts = 0; p.flat = 0; p.red_acc = nullptr; p.row_pair = nullptr; p.pair_w = nullptr; p.red_k = 1; p.red_H = 0; p.red_world = 1; p.red_per = 1;
   { static int pf = -1; if (pf < 0) { const char* e = std::getenv("VLLM_B200_GEMM_PF"); pf = (e && e[0] == '1') ? 1 : 0; } p.pf = pf; }
   p.y = y; p.bias = bias; p.ws = ws; p.counters = counters; p.M = M; p.N = N; p.K = K; p.splits = splits; p.act = act;
+  p.act_coef = act_coef;
   const int kb = (K + BK - 1) / BK;
   p.k_blocks_per_split = (kb + splits - 1) / splits;
   int rc;
@@ -604,7 +614,7 @@ static int grouped_impl(const void* x, const void* w, void* y, const int* offs, 
   CUtensorMap ta, tb;
   Params p;
   p.trace = nullptr; p.pf = 0;
-  p.y = y; p.bias = nullptr; p.ws = nullptr; p.counters = nullptr; p.M = R; p.N = N; p.K = K; p.splits = 1; p.act = act;
+  p.y = y; p.bias = nullptr; p.ws = nullptr; p.counters = nullptr; p.M = R; p.N = N; p.K = K; p.splits = 1; p.act = act; p.act_coef = nullptr;
   p.expert_offs = offs; p.n_experts = E; p.flat = flat;
   p.red_acc = red_acc; p.row_pair = row_pair; p.pair_w = pair_w; p.red_k = red_k; p.red_H = red_H;
   p.red_world = red_world; p.red_per = red_per < 1 ? 1 : red_per;

@@ -1,7 +1,7 @@
 // Multi-head latent attention (MLA) decode on tcgen05: MQA over the paged latent cache, the latent tile shared by all
 // heads of the CTA and by BOTH matrix products.
 //
-//   cache row (one per token, all heads share it):  [ c_kv : R | k_rope : 0 or 64 ]  (bf16 / fp16)
+//   cache row (one per token, all heads share it):  [ c_kv : R | k_rope : up to 64 ]  (bf16 / fp16)
 //   S^T[tok, h] = Kc[tok, :] · Q[h, :]^T              A = latent tile [128 tok x 64-dim k-blocks] K-major (TMA, SW128)
 //                                                     B = Q           [N heads x (R + rope)]
 //   O^T[d, h]  += Kc[tok, d]^T · P^T[tok, h]          A = THE SAME shared-memory bytes read as an MN-major operand
@@ -30,7 +30,7 @@
 
 namespace mla {
 
-constexpr int DR = 64;                // width of the rope part, where there is one
+constexpr int DR = 64;                // block of the rope part, where there is one (TMA zero-fills a narrower one)
 constexpr int TILE = 64;
 constexpr int KB_BYTES = TILE * 128;  // 8 KB: one k-block [64 tok x 64 dims]
 // tile geometry of a latent of NL 64-dim blocks with (ROPE = 1) or without a rope block behind it
@@ -53,6 +53,7 @@ struct Params {
   int64_t out_stride;   // elements between batch rows of out
   int bt_stride;
   int H, BS, num_splits, R;
+  int window;           // > 0: a query sees its last `window` keys
   int* error;           // raised when a wait ran into its limit
   float scale_log2;
 };
@@ -126,10 +127,11 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
   pdl_trigger();
   pdl_wait();
   const int seq_len = p.seq_lens[b];
-  int tile_lo = 0, tile_hi = (seq_len + TILE - 1) / TILE;
+  const int kv_begin = p.window > 0 ? max(0, seq_len - p.window) : 0;
+  int tile_lo = kv_begin / TILE, tile_hi = (seq_len + TILE - 1) / TILE;
   {
-    const int per = (tile_hi + p.num_splits - 1) / p.num_splits;
-    tile_lo = split * per;
+    const int per = (tile_hi - tile_lo + p.num_splits - 1) / p.num_splits;
+    tile_lo += split * per;
     tile_hi = min(tile_hi, tile_lo + per);
   }
   const int n_tiles = max(tile_hi - tile_lo, 0);
@@ -208,7 +210,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
           mbar_expect_tx(&kv_full[slot], bytes);
           for (int u = 0; u < ppt; ++u)
             if (row[u] >= 0)
-              tma_load_2d_hint(stp + kb * KB_BYTES + u * rows * 128, &tmap_kv, kb * 64, row[u], &kv_full[slot], L2_EVICT_FIRST);
+              tma_load_2d_hint(stp + kb * KB_BYTES + u * rows * 128, &tmap_kv, kb == NL ? R : kb * 64, row[u], &kv_full[slot], L2_EVICT_FIRST);
         }
       }
       if (budget < 0) {                         // let the copies in flight land before the block gives up its memory
@@ -301,7 +303,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmap_qn, const __grid_cons
       tc_fence_before();
       mbar_arrive(&s_empty[sb]);
       const int kpos = (tile_lo + j) * TILE + t;
-      const bool ok = t < TILE && kpos < seq_len;        // TMEM lanes 64..127 are the QK padding rows
+      const bool ok = t < TILE && kpos < seq_len && kpos >= kv_begin;        // TMEM lanes 64..127 are the QK padding rows
 #pragma unroll
       for (int g = 0; g < N; ++g) {
         s[g] = ok ? s[g] * p.scale_log2 : -INFINITY;
@@ -460,18 +462,19 @@ static int launch(const CUtensorMap& tqn, const CUtensorMap& tqr, const CUtensor
 
 }  // namespace mla
 
-// q_nope: [B, H, R] (absorbed W_UK), q_pe: [B, H, 64] or null, cache: [num_blocks, BS, R (+ 64)]; out: [B, H, R].
-// bf16 covers every R (a multiple of 8 up to 512) without a rope part and R = 512 with one; fp16 the latter only.
+// q_nope: [B, H, R] (absorbed W_UK), q_pe: [B, H, rope] or null, cache: [num_blocks, BS, R + rope]; out: [B, H, R].
+// bf16 covers every R (a multiple of 8 up to 512) and rope part (none, or a multiple of 8 up to 64); fp16 R = 512 with 64 only.
+// window > 0: row b sees keys seq_lens[b] - window .. seq_lens[b] - 1.
 // `error` (device int, may be null) becomes 1 when a wait inside the kernel ran into its limit.
 EXPORT int vb_mla_decode(const void* q_nope, const void* q_pe, const void* cache, int64_t num_blocks, const int* block_table,
                          const int* seq_lens, void* out, float* part_out, float* part_lse, float* lse_out, int* error, int B,
                          int H, int R, int rope, int BS, int64_t qn_stride_b, int64_t qn_stride_h, int64_t qr_stride_b,
-                         int64_t qr_stride_h, int64_t out_stride, int bt_stride, int num_splits, float scale, int dtype,
+                         int64_t qr_stride_h, int64_t out_stride, int bt_stride, int num_splits, int window, float scale, int dtype,
                          cudaStream_t st) {
   using namespace mla;
   if (B == 0) return 0;
   if (dtype == DT_F32 || R < 8 || R > 512 || R % 8) return -1;
-  if (rope ? (rope != DR || R != 512) : dtype != DT_BF16) return -2;
+  if (rope < 0 || rope > DR || rope % 8 || (dtype != DT_BF16 && (rope != DR || R != 512))) return -2;
   if (BS != 16 && BS != 32 && BS != 64 && BS != 128) return -4;
   auto enc = get_encode();
   if (!enc) return -10;
@@ -482,7 +485,7 @@ EXPORT int vb_mla_decode(const void* q_nope, const void* q_pe, const void* cache
   Params p;
   p.block_table = block_table; p.seq_lens = seq_lens; p.out = out; p.part_out = part_out; p.part_lse = part_lse;
   p.lse_out = lse_out; p.out_stride = out_stride; p.bt_stride = bt_stride; p.H = H; p.BS = BS; p.num_splits = num_splits;
-  p.R = R; p.error = error;
+  p.R = R; p.error = error; p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
   CUtensorMap tqn, tqr, tkv;
   const int gbox = H < N ? H : N;
@@ -495,7 +498,7 @@ EXPORT int vb_mla_decode(const void* q_nope, const void* q_pe, const void* cache
                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
   };
   if (enc_q(&tqn, q_nope, R, qn_stride_b, qn_stride_h) != CUDA_SUCCESS) return -11;
-  if (rope && enc_q(&tqr, q_pe, DR, qr_stride_b, qr_stride_h) != CUDA_SUCCESS) return -12;
+  if (rope && enc_q(&tqr, q_pe, rope, qr_stride_b, qr_stride_h) != CUDA_SUCCESS) return -12;
   if (!rope) tqr = tqn;
   {
     cuuint64_t dims[2] = {(cuuint64_t)DK, (cuuint64_t)num_blocks * BS};
@@ -510,14 +513,20 @@ EXPORT int vb_mla_decode(const void* q_nope, const void* q_pe, const void* cache
   int rc;
 #define GO(TT, NL, RP, FL) rc = N == 16 ? launch<TT, 16, NL, RP, FL>(tqn, tqr, tkv, p, grid, st) : launch<TT, 32, NL, RP, FL>(tqn, tqr, tkv, p, grid, st)
   const int nl = (R + 63) / 64;
-  if (rope) { if (bf16) GO(__nv_bfloat16, 8, 1, true); else GO(__half, 8, 1, true); }
-  else if (R == 512) GO(__nv_bfloat16, 8, 0, true);
-  else if (nl <= 1) GO(__nv_bfloat16, 1, 0, false);
-  else if (nl == 2) GO(__nv_bfloat16, 2, 0, false);
-  else if (nl == 3) GO(__nv_bfloat16, 3, 0, false);
-  else if (nl == 4) GO(__nv_bfloat16, 4, 0, false);
-  else if (nl <= 6) GO(__nv_bfloat16, 6, 0, false);
-  else GO(__nv_bfloat16, 8, 0, false);
+#define WIDTHS(RP)                                                                                            \
+  do {                                                                                                        \
+    if (R == 512) GO(__nv_bfloat16, 8, RP, true);                                                             \
+    else if (nl <= 1) GO(__nv_bfloat16, 1, RP, false);                                                        \
+    else if (nl == 2) GO(__nv_bfloat16, 2, RP, false);                                                        \
+    else if (nl == 3) GO(__nv_bfloat16, 3, RP, false);                                                        \
+    else if (nl == 4) GO(__nv_bfloat16, 4, RP, false);                                                        \
+    else if (nl <= 6) GO(__nv_bfloat16, 6, RP, false);                                                        \
+    else GO(__nv_bfloat16, 8, RP, false);                                                                     \
+  } while (0)
+  if (!bf16) GO(__half, 8, 1, true);
+  else if (rope) WIDTHS(1);
+  else WIDTHS(0);
+#undef WIDTHS
 #undef GO
   if (rc) return rc;
   if (num_splits > 1) {

@@ -9,6 +9,9 @@
 //   S = Q · K^T    both operands K-major (dims contiguous), 128 x 128 tile, dim in 64-wide k-blocks
 //   O += P · V     V is read as an MN-major B operand: a 128-byte swizzle row holds 64 dims of ONE token
 // dim and vdim are multiples of 8 up to 128; TMA zero-fills the tail of a 64-wide block, so odd widths cost nothing else.
+// A rotated part of the score (up to 64 wide, one key part for all heads) is one more k-block: its queries are columns of the query
+// heads, its keys columns of the gathered cache rows, so nothing is copied together.  With a window, the request's key rows start at
+// the first one that its portion sees.
 //
 // CTA = (request, head, 128 query tokens), heaviest (latest) query tiles first.  Warp roles: 0 TMA producer, 1 MMA
 // issuer + TMEM owner, 2..5 softmax / rescale / epilogue with one thread per query row (row max and sum are
@@ -31,6 +34,7 @@ struct Params {
   int64_t out_st, out_sh;
   int h0;                  // first head of this launch in q / out (K and V hold the launch's heads only)
   int vdim;
+  int window;              // > 0: a query sees its last `window` keys
   float scale_log2;
   int* error;
 };
@@ -64,17 +68,20 @@ VB_DEVICE uint64_t desc_mn(const void* smem_tile) {
   return d;
 }
 
-template <typename T, int NQ, int NV>
+// NN blocks of unrotated and NR of rotated dimensions; VS stages of values
+template <typename T, int NN, int NR, int NV, int VS>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
-                   const __grid_constant__ CUtensorMap tmap_v, const Params p) {
+                   const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_qr,
+                   const __grid_constant__ CUtensorMap tmap_kr, const Params p) {
+  constexpr int NQ = NN + NR;
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   unsigned char* q_smem = smem;                             // NQ blocks
   unsigned char* p_smem = q_smem + NQ * BLK;                // 2 blocks: [128 rows x 128 keys]
   unsigned char* k_smem = p_smem + 2 * BLK;                 // STAGES x NQ blocks
-  unsigned char* v_smem = k_smem + STAGES * NQ * BLK;       // STAGES x NV blocks
-  uint64_t* bars = reinterpret_cast<uint64_t*>(v_smem + STAGES * NV * BLK);
+  unsigned char* v_smem = k_smem + STAGES * NQ * BLK;       // VS x NV blocks
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_smem + VS * NV * BLK);
   uint64_t* q_full = bars;
   uint64_t* k_full = bars + 1;                 // [STAGES]
   uint64_t* v_full = k_full + STAGES;          // [STAGES]
@@ -100,7 +107,8 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
   const int kv0 = p.kv_start[b];
   const int pos0 = p.seq_len[b] - q_len + tok0;             // position of the tile's first query
   const int kv_end = pos0 + n_tok;                          // keys any query of the tile can see
-  const int n_tiles = (kv_end + TN - 1) / TN;
+  const int tile_lo = p.window > 0 ? max(0, pos0 - p.window + 1) / TN : 0;
+  const int n_tiles = (kv_end + TN - 1) / TN - tile_lo;
 
   if (warp == 0 && lane == 0) {
     tma_prefetch_desc(&tmap_q); tma_prefetch_desc(&tmap_k); tma_prefetch_desc(&tmap_v);
@@ -126,26 +134,28 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       // masked by the softmax (finite values times a weight of 0).
       mbar_expect_tx(q_full, NQ * BLK);
 #pragma unroll
-      for (int i = 0; i < NQ; ++i) tma_load_3d(q_smem + i * BLK, &tmap_q, i * 64, p.h0 + h, q0, q_full);
+      for (int i = 0; i < NN; ++i) tma_load_3d(q_smem + i * BLK, &tmap_q, i * 64, p.h0 + h, q0, q_full);
+      if (NR) tma_load_3d(q_smem + NN * BLK, &tmap_qr, 0, p.h0 + h, q0, q_full);
       for (int j = 0; j < n_tiles; ++j) {
-        const int s = j % STAGES;
-        const uint32_t par = ((j / STAGES) & 1) ^ 1;
-        const int row = kv0 + j * TN;
+        const int s = j % STAGES, vs = j % VS;
+        const uint32_t par = ((j / STAGES) & 1) ^ 1, v_par = ((j / VS) & 1) ^ 1;
+        const int row = kv0 + (tile_lo + j) * TN;
         mbar_wait_lim(&k_empty[s], par, budget);
         if (budget < 0) break;
         mbar_expect_tx(&k_full[s], NQ * BLK);
 #pragma unroll
-        for (int i = 0; i < NQ; ++i) tma_load_3d(k_smem + (s * NQ + i) * BLK, &tmap_k, i * 64, h, row, &k_full[s]);
-        mbar_wait_lim(&v_empty[s], par, budget);
+        for (int i = 0; i < NN; ++i) tma_load_3d(k_smem + (s * NQ + i) * BLK, &tmap_k, i * 64, h, row, &k_full[s]);
+        if (NR) tma_load_3d(k_smem + (s * NQ + NN) * BLK, &tmap_kr, 0, 0, row, &k_full[s]);
+        mbar_wait_lim(&v_empty[vs], v_par, budget);
         if (budget < 0) break;
-        mbar_expect_tx(&v_full[s], NV * BLK);
+        mbar_expect_tx(&v_full[vs], NV * BLK);
 #pragma unroll
-        for (int i = 0; i < NV; ++i) tma_load_3d(v_smem + (s * NV + i) * BLK, &tmap_v, i * 64, h, row, &v_full[s]);
+        for (int i = 0; i < NV; ++i) tma_load_3d(v_smem + (vs * NV + i) * BLK, &tmap_v, i * 64, h, row, &v_full[vs]);
       }
       if (budget < 0) {                         // let the copies in flight land before the block gives up its memory
         for (int s = 0; s < STAGES; ++s)
           for (int n = 0; n < 4096 && !(mbar_try_wait(&k_full[s], 0) || mbar_try_wait(&k_full[s], 1)); ++n) {}
-        for (int s = 0; s < STAGES; ++s)
+        for (int s = 0; s < VS; ++s)
           for (int n = 0; n < 4096 && !(mbar_try_wait(&v_full[s], 0) || mbar_try_wait(&v_full[s], 1)); ++n) {}
       }
     }
@@ -178,8 +188,8 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         __syncwarp();
       }
       if (j > 0) {
-        const int jj = j - 1, s = jj % STAGES;
-        mbar_wait_lim(&v_full[s], (jj / STAGES) & 1, budget);
+        const int jj = j - 1, s = jj % VS;
+        mbar_wait_lim(&v_full[s], (jj / VS) & 1, budget);
         mbar_wait_lim(p_full, jj & 1, budget);
         tc_fence_after();
         if (lane == 0) {
@@ -208,8 +218,9 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
       mbar_wait_lim(&s_full[sb], (j >> 1) & 1, budget);
       __syncwarp();
       tc_fence_after();
-      const int hi = row_valid ? pos0 + r + 1 - j * TN : 0;     // keys [0, hi) of this tile are visible to the row
-      const bool full = __all_sync(0xffffffffu, hi >= TN) != 0; // tiles below the diagonal: no masks
+      const int hi = row_valid ? pos0 + r + 1 - (tile_lo + j) * TN : 0;     // keys [lo, hi) of this tile are visible to the row
+      const int lo = p.window > 0 ? hi - p.window : 0;
+      const bool full = __all_sync(0xffffffffu, hi >= TN && lo <= 0) != 0;  // tiles inside every row's range: no masks
       // ---- pass 1: row max
       float mx = -INFINITY;
 #pragma unroll
@@ -223,7 +234,7 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (c + i < hi) mx = fmaxf(mx, __uint_as_float(v[i]) * p.scale_log2);
+            if (c + i < hi && c + i >= lo) mx = fmaxf(mx, __uint_as_float(v[i]) * p.scale_log2);
         }
       }
       // keep the old reference maximum unless the new one is more than 2^8 above it
@@ -260,8 +271,8 @@ mla_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_cons
         for (int i = 0; i < 32; i += 2) {
           float p0 = ex2(__uint_as_float(v[i]) * p.scale_log2 - m_ref), p1 = ex2(__uint_as_float(v[i + 1]) * p.scale_log2 - m_ref);
           if (!full) {
-            if (c + i >= hi) p0 = 0.f;
-            if (c + i + 1 >= hi) p1 = 0.f;
+            if (c + i >= hi || c + i < lo) p0 = 0.f;
+            if (c + i + 1 >= hi || c + i + 1 < lo) p1 = 0.f;
           }
           l_run += p0 + p1;
           pk[i / 2] = pack2<T>(p0, p1);
@@ -324,12 +335,12 @@ static EncodeTiledFn get_encode() {
   return fn;
 }
 
-// [rows, heads, width] with row stride `rs` elements, heads `width` apart; box = 128 rows of 64 values of one head
-static int tmap(CUtensorMap* m, const void* ptr, int width, int heads, int64_t rows, int64_t rs, bool bf16) {
+// [rows, heads, width] with row stride `rs` and head stride `hs` elements; box = 128 rows of 64 values of one head
+static int tmap(CUtensorMap* m, const void* ptr, int width, int heads, int64_t rows, int64_t rs, int64_t hs, bool bf16) {
   auto enc = get_encode();
   if (!enc) return -10;
   cuuint64_t dims[3] = {(cuuint64_t)width, (cuuint64_t)heads, (cuuint64_t)rows};
-  cuuint64_t strides[2] = {(cuuint64_t)width * 2, (cuuint64_t)rs * 2};
+  cuuint64_t strides[2] = {(cuuint64_t)hs * 2, (cuuint64_t)rs * 2};
   cuuint32_t box[3] = {64, 1, 128};
   cuuint32_t es[3] = {1, 1, 1};
   return enc(m, bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 3, const_cast<void*>(ptr), dims,
@@ -337,41 +348,52 @@ static int tmap(CUtensorMap* m, const void* ptr, int width, int heads, int64_t r
              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS ? 0 : -11;
 }
 
-template <typename T, int NQ, int NV>
-static int launch(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const Params& p, dim3 grid, cudaStream_t st) {
-  const int smem = (NQ + 2 + STAGES * (NQ + NV)) * BLK + 32 * 8 + 16 + 1024;
-  auto k = mla_prefill_kernel<T, NQ, NV>;
+struct Maps { CUtensorMap q, k, v, qr, kr; };
+
+template <typename T, int NN, int NR, int NV>
+static int launch(const Maps& m, const Params& p, dim3 grid, cudaStream_t st) {
+  constexpr int NQ = NN + NR;
+  constexpr int VS = NQ + 2 + STAGES * (NQ + NV) <= 13 ? STAGES : 1;         // what fits into shared memory
+  const int smem = (NQ + 2 + STAGES * NQ + VS * NV) * BLK + 32 * 8 + 16 + 1024;
+  auto k = mla_prefill_kernel<T, NN, NR, NV, VS>;
   static bool a = false;
   if (!a) { cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); a = true; }
-  vb_launch(k, grid, dim3(NUM_THREADS), (size_t)smem, st, tq, tk, tv, p);
+  vb_launch(k, grid, dim3(NUM_THREADS), (size_t)smem, st, m.q, m.k, m.v, m.qr, m.kr, p);
   return (int)cudaGetLastError();
 }
 
 }  // namespace mlap
 
-// q [T, H, dim] and out [T, H, vdim] (row strides q_st / out_st); k [KV, hl, dim], v [KV, hl, vdim] hold the heads
-// h0 .. h0 + hl - 1.  Request b owns query rows q_start[b] .. + q_len[b] and key rows kv_start[b] .. + seq_len[b].
-EXPORT int vb_mla_prefill(const void* q, const void* k, const void* v, void* out, const int* q_start, const int* q_len,
+// q [T, H, dim + rot] and out [T, H, vdim] (row strides q_st / out_st); k [KV, hl, dim], v [KV, hl, vdim] hold the heads
+// h0 .. h0 + hl - 1; k_pe [KV, rot] (row stride kr_st; rot = 0: none) is the rotated key part of all heads.  Request b owns query rows
+// q_start[b] .. + q_len[b] and key rows kv_start[b] .. + seq_len[b], of which its portion is the tail.
+EXPORT int vb_mla_prefill(const void* q, const void* k, const void* v, const void* k_pe, void* out, const int* q_start, const int* q_len,
                           const int* seq_len, const int* kv_start, int* error, int B, int T_, int64_t KV, int H, int h0, int hl,
-                          int dim, int vdim, int64_t q_st, int64_t k_st, int64_t v_st, int64_t out_st, int max_q, float scale,
-                          int dtype, cudaStream_t st) {
+                          int dim, int rot, int vdim, int64_t q_st, int64_t k_st, int64_t v_st, int64_t kr_st, int64_t out_st, int max_q,
+                          int window, float scale, int dtype, cudaStream_t st) {
   using namespace mlap;
   if (B == 0 || T_ == 0 || max_q <= 0) return 0;
-  if (dtype == DT_F32 || dim < 8 || dim > 128 || dim % 8 || vdim < 8 || vdim > 128 || vdim % 8) return -1;
-  if (q_st % 8 || k_st % 8 || v_st % 8 || out_st % 8 || h0 < 0 || h0 + hl > H) return -2;
+  if (dtype == DT_F32 || dim < 8 || dim > 128 || dim % 8 || vdim < 8 || vdim > 128 || vdim % 8 || rot < 0 || rot > 64 || rot % 8) return -1;
+  if (q_st % 8 || k_st % 8 || v_st % 8 || out_st % 8 || h0 < 0 || h0 + hl > H || (rot && (!k_pe || kr_st % 8))) return -2;
   const bool bf16 = dtype == DT_BF16;
-  CUtensorMap tq, tk, tv;
+  Maps m;
   int rc;
-  if ((rc = tmap(&tq, q, dim, H, T_, q_st, bf16))) return rc;
-  if ((rc = tmap(&tk, k, dim, hl, KV, k_st, bf16))) return rc;
-  if ((rc = tmap(&tv, v, vdim, hl, KV, v_st, bf16))) return rc;
+  if ((rc = tmap(&m.q, q, dim, H, T_, q_st, dim + rot, bf16))) return rc;
+  if ((rc = tmap(&m.k, k, dim, hl, KV, k_st, dim, bf16))) return rc;
+  if ((rc = tmap(&m.v, v, vdim, hl, KV, v_st, vdim, bf16))) return rc;
+  m.qr = m.q; m.kr = m.k;
+  if (rot) {
+    if ((rc = tmap(&m.qr, reinterpret_cast<const char*>(q) + (int64_t)dim * 2, rot, H, T_, q_st, dim + rot, bf16))) return rc;
+    if ((rc = tmap(&m.kr, k_pe, rot, 1, KV, kr_st, kr_st, bf16))) return rc;
+  }
   Params p;
   p.q_start = q_start; p.q_len = q_len; p.seq_len = seq_len; p.kv_start = kv_start; p.out = out; p.out_st = out_st;
-  p.out_sh = vdim; p.h0 = h0; p.vdim = vdim; p.scale_log2 = scale * 1.4426950408889634f; p.error = error;
+  p.out_sh = vdim; p.h0 = h0; p.vdim = vdim; p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.error = error;
   const dim3 grid((max_q + TM - 1) / TM, hl, B);
   const int nq = (dim + 63) / 64, nv = (vdim + 63) / 64;
-#define GO(TT) (nq == 1 ? (nv == 1 ? launch<TT, 1, 1>(tq, tk, tv, p, grid, st) : launch<TT, 1, 2>(tq, tk, tv, p, grid, st)) \
-                        : (nv == 1 ? launch<TT, 2, 1>(tq, tk, tv, p, grid, st) : launch<TT, 2, 2>(tq, tk, tv, p, grid, st)))
+#define GV(TT, N, R) (nv == 1 ? launch<TT, N, R, 1>(m, p, grid, st) : launch<TT, N, R, 2>(m, p, grid, st))
+#define GO(TT) (rot ? (nq == 1 ? GV(TT, 1, 1) : GV(TT, 2, 1)) : (nq == 1 ? GV(TT, 1, 0) : GV(TT, 2, 0)))
   return bf16 ? GO(__nv_bfloat16) : GO(__half);
 #undef GO
+#undef GV
 }

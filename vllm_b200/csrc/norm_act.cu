@@ -325,6 +325,38 @@ EXPORT int vb_activation(void* out, const void* x, int64_t n, int act, int dtype
   return (int)cudaGetLastError();
 }
 
+// y = a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below; y may be x
+template <typename T, int V>
+__global__ void __launch_bounds__(256) xielu_kernel(const T* __restrict__ x, T* __restrict__ y, const float* __restrict__ coef, int64_t total) {
+  pdl_trigger();
+  const float a = coef[0], b = coef[1];
+  pdl_wait();
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+    if constexpr (V == 1) {
+      y[i] = from_f32<T>(xielu(to_f32(x[i]), a, b));
+    } else {
+      Vec16<T> v = ld16(x + i * V);
+#pragma unroll
+      for (int j = 0; j < V; ++j) v.e[j] = from_f32<T>(xielu(to_f32(v.e[j]), a, b));
+      st16(y + i * V, v);
+    }
+  }
+}
+
+EXPORT int vb_xielu(const void* x, void* y, const float* coef, int64_t n, int dtype, cudaStream_t st) {
+  if (n == 0) return 0;
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  DISPATCH_DTYPE(dtype, TT, {
+    constexpr int N = Vec16<TT>::N;
+    const bool vec = n % N == 0 && al(x) && al(y);
+    const int64_t total = vec ? n / N : n;
+    const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+    if (vec) vb_launch(xielu_kernel<TT, N>, blocks, 256, 0, st, (const TT*)x, (TT*)y, coef, total);
+    else vb_launch(xielu_kernel<TT, 1>, blocks, 256, 0, st, (const TT*)x, (TT*)y, coef, total);
+  });
+  return (int)cudaGetLastError();
+}
+
 EXPORT int vb_sigmoid_mul(const void* x, int64_t x_stride, const void* g, int64_t g_stride, void* y, int64_t y_stride, int64_t T, int n,
                           int dtype, cudaStream_t st) {
   if (T == 0) return 0;

@@ -51,6 +51,7 @@ struct Params {
   int64_t q_stride, k_stride, v_stride;
   int T, Hq, Hkv, D, rot, BS;
   int neox, gemma, kv_fp8, vt;
+  const float* v_cos_sin;                  // optional [max_pos, value width]: values are rotated too, in the layout of the keys
   int keep32;                              // the normalised head stays in 32 bits on its way to the rotation
   float eps, k_inv_scale, v_inv_scale;
 };
@@ -71,12 +72,51 @@ __global__ void __launch_bounds__(256) qknorm_rope_cache_kernel(const Params p) 
   const int64_t blk = do_cache ? slot / p.BS : 0;
   const int off = do_cache ? (int)(slot % p.BS) : 0;
 
+  // NeoX pairs sit in lanes `span` apart (a power of two, checked on the host), GPT-J pairs inside the lane
+  auto rotate = [&](float (&f)[E], const float* cs, int rot) {
+    const int half = rot / 2;
+    if (p.neox) {
+      const int span = half / E;                       // lanes per half
+      const bool rot_lane = lane < 2 * span;
+      const bool first = (lane & span) == 0;
+#pragma unroll
+      for (int j = 0; j < E; ++j) {
+        const float other = __shfl_xor_sync(0xffffffffu, f[j], span);
+        if (rot_lane) {
+          const int i = (lane & (span - 1)) * E + j;   // index inside the half
+          const float co = cs[i], si = cs[half + i];
+          f[j] = first ? f[j] * co - other * si : f[j] * co + other * si;
+        }
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < E; j += 2) {
+        const int e0 = lane * E + j;
+        if (e0 < rot) {
+          const int i = e0 >> 1;
+          const float co = cs[i], si = cs[half + i];
+          const float x1 = f[j], x2 = f[j + 1];
+          f[j] = x1 * co - x2 * si;
+          f[j + 1] = x2 * co + x1 * si;
+        }
+      }
+    }
+  };
+
   if (it >= p.Hq + p.Hkv) {
     // ---- V head → cache page
     if (!do_cache || p.v == nullptr) return;
     const int h = it - p.Hq - p.Hkv;
     LaneVec<T, E> a;
     a.load(reinterpret_cast<const T*>(p.v) + t * p.v_stride + (int64_t)h * D + lane * E);
+    if (p.v_cos_sin) {
+      float f[E];
+#pragma unroll
+      for (int j = 0; j < E; ++j) f[j] = to_f32(a.e[j]);
+      rotate(f, p.v_cos_sin + p.positions[t] * D, D);
+#pragma unroll
+      for (int j = 0; j < E; ++j) a.e[j] = from_f32<T>(f[j]);
+    }
     const size_t page = (((size_t)blk * 2 + 1) * p.Hkv + h) * p.BS * D;
     if (p.vt) {            // tensor-core layout: V pages transposed [D, BS]
       T* vc = reinterpret_cast<T*>(p.kv_cache) + page + off;
@@ -118,36 +158,7 @@ __global__ void __launch_bounds__(256) qknorm_rope_cache_kernel(const Params p) 
       if (!p.keep32) f[j] = to_f32(from_f32<T>(f[j]));     // round through T like the unfused norm does
     }
   }
-  if (p.rot > 0) {
-    const int half = p.rot / 2;
-    const float* cs = p.cos_sin + p.positions[t] * p.rot;
-    if (p.neox) {
-      const int span = half / E;                       // lanes per half (power of two, checked on the host)
-      const bool rot_lane = lane < 2 * span;
-      const bool first = (lane & span) == 0;
-#pragma unroll
-      for (int j = 0; j < E; ++j) {
-        const float other = __shfl_xor_sync(0xffffffffu, f[j], span);
-        if (rot_lane) {
-          const int i = (lane & (span - 1)) * E + j;   // index inside the half
-          const float co = cs[i], si = cs[half + i];
-          f[j] = first ? f[j] * co - other * si : f[j] * co + other * si;
-        }
-      }
-    } else {
-#pragma unroll
-      for (int j = 0; j < E; j += 2) {
-        const int e0 = lane * E + j;
-        if (e0 < p.rot) {
-          const int i = e0 >> 1;
-          const float co = cs[i], si = cs[half + i];
-          const float x1 = f[j], x2 = f[j + 1];
-          f[j] = x1 * co - x2 * si;
-          f[j + 1] = x2 * co + x1 * si;
-        }
-      }
-    }
-  }
+  if (p.rot > 0) rotate(f, p.cos_sin + p.positions[t] * p.rot, p.rot);
 #pragma unroll
   for (int j = 0; j < E; ++j) a.e[j] = from_f32<T>(f[j]);
   a.store(base + lane * E);
@@ -187,7 +198,18 @@ __global__ void __launch_bounds__(ANY_WARPS * 32) qknorm_rope_any_kernel(const P
     const int h = it - p.Hq - p.Hkv;
     const T* v = reinterpret_cast<const T*>(p.v) + t * p.v_stride + (int64_t)h * DV;
     T* dst = cache + ((blk * 2 + 1) * p.Hkv + h) * p.BS * (int64_t)DC + (p.vt ? off : off * DC);
-    for (int d = lane; d < DV; d += 32) dst[p.vt ? (int64_t)d * p.BS : d] = v[d];
+    const float* cs = p.v_cos_sin ? p.v_cos_sin + p.positions[t] * DV : nullptr;
+    const int half = DV / 2;
+    for (int d = lane; d < DV; d += 32) {
+      T y = v[d];
+      if (cs) {
+        const int i = p.neox ? d % half : d >> 1;
+        const bool first = p.neox ? d < half : (d & 1) == 0;
+        const float x = to_f32(y), o = to_f32(v[p.neox ? (first ? d + half : d - half) : d ^ 1]), co = cs[i], si = cs[half + i];
+        y = from_f32<T>(first ? x * co - o * si : x * co + o * si);
+      }
+      dst[p.vt ? (int64_t)d * p.BS : d] = y;
+    }
     return;
   }
   const bool is_k = it >= p.Hq;
@@ -317,11 +339,12 @@ __global__ void __launch_bounds__(512) qknorm_rope_row_kernel(const Params p, in
 
 }  // namespace
 
-// q, k: [T, H*D] views of the fused qkv buffer (rotated / normalised in place); v may be null (no cache write of V);
+// q, k: [T, H*D] views of the fused qkv buffer (rotated / normalised in place); v may be null (no cache write of V), and is rotated on
+// its way into the cache where there is v_cos_sin [positions, value width];
 // kv_cache may be null (norm + rope only).  flags: bit0 fp8 cache, bit1 transposed V pages, bit2 no rounding to T between the
 // norm and the rotation.
 EXPORT int vb_qknorm_rope_cache(const int64_t* positions, void* q, void* k, const void* v, const void* q_w, const void* k_w,
-                                const float* cos_sin, int rot, int T, int Hq, int Hkv, int D, int64_t q_stride,
+                                const float* cos_sin, const float* v_cos_sin, int rot, int T, int Hq, int Hkv, int D, int64_t q_stride,
                                 int64_t k_stride, int64_t v_stride, void* kv_cache, const int64_t* slot_mapping, int BS,
                                 int neox, int gemma, int flags, float eps, float k_scale, float v_scale, int dtype,
                                 cudaStream_t st) {
@@ -339,6 +362,7 @@ EXPORT int vb_qknorm_rope_cache(const int64_t* positions, void* q, void* k, cons
     } else if (E % 2) return -1;
   }
   Params p;
+  p.v_cos_sin = v_cos_sin;
   p.positions = positions; p.q = q; p.k = k; p.v = v; p.q_w = q_w; p.k_w = k_w; p.cos_sin = cos_sin;
   p.kv_cache = kv_cache; p.slot_mapping = slot_mapping; p.q_stride = q_stride; p.k_stride = k_stride; p.v_stride = v_stride;
   p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.rot = rot; p.BS = BS; p.neox = neox; p.gemma = gemma;
@@ -359,12 +383,13 @@ EXPORT int vb_qknorm_rope_cache(const int64_t* positions, void* q, void* k, cons
 
 // Every other shape and dtype.  The cache holds the model dtype.
 EXPORT int vb_qknorm_rope_any(const int64_t* positions, void* q, void* k, const void* v, const void* q_w, const void* k_w,
-                              const float* cos_sin, int rot, int T, int Hq, int Hkv, int D, int DV, int DC, int64_t q_stride,
+                              const float* cos_sin, const float* v_cos_sin, int rot, int T, int Hq, int Hkv, int D, int DV, int DC, int64_t q_stride,
                               int64_t k_stride, int64_t v_stride, void* kv_cache, const int64_t* slot_mapping, int BS, int neox,
                               int gemma, int vt, float eps, int dtype, cudaStream_t st) {
   if (T == 0) return 0;
-  if (D > ANY_MAX_D || rot > D || rot % 2 || DC < D || DC < DV) return -1;
+  if (D > ANY_MAX_D || rot > D || rot % 2 || DC < D || DC < DV || (v_cos_sin && DV % 2)) return -1;
   Params p = {};
+  p.v_cos_sin = v_cos_sin;
   p.positions = positions; p.q = q; p.k = k; p.v = v; p.q_w = q_w; p.k_w = k_w; p.cos_sin = cos_sin;
   p.kv_cache = kv_cache; p.slot_mapping = slot_mapping; p.q_stride = q_stride; p.k_stride = k_stride; p.v_stride = v_stride;
   p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.rot = rot; p.BS = BS; p.neox = neox; p.gemma = gemma; p.vt = vt; p.eps = eps;

@@ -10,6 +10,8 @@
 //                     x += m norm(y + bias);   out = T(norm_next(x))       (or x = table[id] at the model's entry)
 //   add_norm          the same step for pre-norm blocks:  x += y + routed sum;   out = T(norm_next(x)).  The routed sum may have
 //                     identity experts: slots whose expert number is past the last one add w_j times the layer's input
+//   hyper_step        hyper-connections, S streams per token:  x_t = sum_s mix[s, t] x_s + out[t] y;   out = T(rmsnorm(sum_s in[s] x_s))
+//                     (or x_s = rmsnorm(table[id]) for all s at the model's entry); one read and one write of every stream
 // The combine of the expert layer is the load of post_norm_add and add_norm: expert outputs are read once, summed in slot order in
 // fp32 (deterministic) and never written back.
 #include "common.cuh"
@@ -284,6 +286,92 @@ add_norm_kernel(const T* __restrict__ y, int64_t y_stride, const Routed r, float
   }
 }
 
+// S streams per token (x [T, S, H]).  ids: entry, x_s = rmsnorm(y[id]) * w_e;  entry rows (no coef): x_s = y;  coef (out [S], mix [S, S]):
+// x_t = sum_s mix[s, t] x_s + out[t] y;  y null: x is read only.  out = rmsnorm(sum_s into[s] x_s) * w.  SM: S, or a bound of it (V = 1).
+constexpr int MAX_STREAMS = 16;
+template <typename T, int V, int NV, int SM, bool EXACT>
+__global__ void __launch_bounds__(512)
+hyper_kernel(const int* __restrict__ ids, int vocab, const T* __restrict__ y, int64_t y_stride, const T* __restrict__ w_e,
+             const float* __restrict__ coef, const float* __restrict__ into, float* __restrict__ x, int S_, const T* __restrict__ w,
+             T* __restrict__ out, int H, float eps) {
+  __shared__ float red[32];
+  __shared__ float cf[2 * MAX_STREAMS + MAX_STREAMS * MAX_STREAMS];        // into, out, mix
+  pdl_trigger();
+  const int S = EXACT ? SM : S_;
+  const bool step = coef != nullptr;
+  // weights are never written by a predecessor: they may be fetched before it ends
+  for (int i = threadIdx.x; i < S; i += blockDim.x) cf[i] = into[i];
+  if (step)
+    for (int i = threadIdx.x; i < S + S * S; i += blockDim.x) cf[S + i] = coef[i];
+  __syncthreads();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  const int stride = blockDim.x * V;
+  const float* in_ = cf;
+  const float* out_ = cf + S;
+  const float* mix = cf + 2 * S;
+  float* xr = x + row * S * H;
+  float u[NV][V];
+  if (y && !step) {
+    const T* src = y + (ids ? (int64_t)min(max(ids[row], 0), vocab - 1) * H : row * y_stride);
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+      if (threadIdx.x * V + n * stride < H) load_f32<T, V>(src + threadIdx.x * V + n * stride, u[n]);
+    if (w_e) normalise<T, V, NV, false>(u, w_e, nullptr, 0, H, eps, red);
+    float total = 0.f;
+    for (int s = 0; s < S; ++s) total += in_[s];
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = threadIdx.x * V + n * stride;
+      if (i >= H) continue;
+      for (int s = 0; s < S; ++s) store_f32<float, V>(xr + (int64_t)s * H + i, u[n]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) u[n][j] *= total;
+    }
+  } else {
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      const int i = threadIdx.x * V + n * stride;
+      if (i >= H) continue;
+      float xs[SM][V], yv[V];
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (EXACT || s < S) load_f32<float, V>(xr + (int64_t)s * H + i, xs[s]);
+      if (step) load_f32<T, V>(y + row * y_stride + i, yv);
+#pragma unroll
+      for (int j = 0; j < V; ++j) u[n][j] = 0.f;
+#pragma unroll
+      for (int t = 0; t < SM; ++t) {
+        if (!EXACT && t >= S) break;
+        float v[V];
+        if (step) {
+#pragma unroll
+          for (int j = 0; j < V; ++j) v[j] = out_[t] * yv[j];
+#pragma unroll
+          for (int s = 0; s < SM; ++s)
+            if (EXACT || s < S) {
+              const float m = mix[s * S + t];
+#pragma unroll
+              for (int j = 0; j < V; ++j) v[j] += m * xs[s][j];
+            }
+          store_f32<float, V>(xr + (int64_t)t * H + i, v);
+        } else {
+#pragma unroll
+          for (int j = 0; j < V; ++j) v[j] = xs[t][j];
+        }
+#pragma unroll
+        for (int j = 0; j < V; ++j) u[n][j] += in_[t] * v[j];
+      }
+    }
+  }
+  normalise<T, V, NV, false>(u, w, nullptr, 0, H, eps, red);
+#pragma unroll
+  for (int n = 0; n < NV; ++n) {
+    const int i = threadIdx.x * V + n * stride;
+    if (i < H) store_f32<T, V>(out + row * H + i, u[n]);
+  }
+}
+
 template <typename T> constexpr int vec_of() { return sizeof(T) == 4 ? 4 : 8; }
 static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
@@ -383,5 +471,34 @@ EXPORT int vb_add_norm(const void* y, int64_t y_stride, const void* rows, int64_
     else { if (nv <= 1) GO(1, 1); else if (nv <= 16) GO(1, 16); else return -1; }
   });
 #undef GO
+  return (int)cudaGetLastError();
+}
+
+// S streams x [T, S, H] (see hyper_kernel).  coef null and y given: the model's entry (ids null: rows of y as they are).
+EXPORT int vb_hyper_step(const int* ids, int vocab, const void* y, int64_t y_stride, const void* w_e, const float* coef, const float* into,
+                         float* x, int S, const void* w, void* out, int T_, int H, float eps, int dtype, cudaStream_t st) {
+  using namespace stream;
+  if (T_ == 0) return 0;
+  if (S < 1 || S > MAX_STREAMS || !into || !x || !w || !out || (coef && !y) || (ids && !y)) return -1;
+#define RUN(VV, NVV, SS, EX) vb_launch(hyper_kernel<T, VV, NVV, SS, EX>, dim3(T_), dim3(thr), 0, st, ids, vocab, (const T*)y, y_stride, (const T*)w_e, coef, into, x, S, (const T*)w, (T*)out, H, eps)
+#define GO(VV, NVV)                                                                                                    \
+  do {                                                                                                                 \
+    if (S == 1) RUN(VV, NVV, 1, true); else if (S == 2) RUN(VV, NVV, 2, true); else if (S == 3) RUN(VV, NVV, 3, true);  \
+    else RUN(VV, NVV, 4, true);                                                                                        \
+  } while (0)
+  DISPATCH_DTYPE(dtype, T, {
+    constexpr int V = vec_of<T>();
+    auto ok = [](const void* p) { return !p || al16(p); };
+    const bool vec = S <= 4 && H % V == 0 && (ids || y_stride % V == 0) && ok(y) && ok(w_e) && ok(x) && ok(w) && ok(out);
+    const int items = vec ? H / V : H;
+    const int thr = items >= 512 ? 512 : ((items + 31) / 32) * 32;
+    const int nv = (items + thr - 1) / thr;
+    if (vec && nv <= 8) { if (nv <= 1) GO(V, 1); else if (nv <= 4) GO(V, 4); else GO(V, 8); }
+    else if (!vec && nv <= 1) { if (S <= 4) GO(1, 1); else RUN(1, 1, MAX_STREAMS, false); }
+    else if (!vec && nv <= 32) RUN(1, 32, MAX_STREAMS, false);
+    else return -1;
+  });
+#undef GO
+#undef RUN
   return (int)cudaGetLastError();
 }

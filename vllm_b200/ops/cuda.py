@@ -104,7 +104,12 @@ _topk_topp = _sig("vb_topk_topp", _vp, _i, _i, _vp, _vp, _vp, _vp)
 _row_lse = _sig("vb_row_lse", _vp, _i64, _i, _i, _vp, _i, _vp)
 _gemm_plan = _sig("vb_gemm_tc_plan", _i, _i, _i, _i, ctypes.POINTER(_i), ctypes.POINTER(_i), ctypes.POINTER(_i),
                   ctypes.POINTER(_i64), ctypes.POINTER(_i))
-_gemm_tc = _sig("vb_gemm_tc2", _vp, _vp, _vp, _vp, _i, _i, _i, _i64, _i, _i, _i, _vp, _vp, _i, _i, _vp)
+_gemm_tc = _sig("vb_gemm_tc2", _vp, _vp, _vp, _vp, _i, _i, _i, _i64, _i, _i, _i, _vp, _vp, _i, _vp, _i, _vp)
+_any_fold = _sig("vb_any_attention_fold", _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i64, _i, _i, _f, _f, _vp, _i, _i,
+                 _i, _vp)
+_talk_fold = _sig("vb_talk_fold", _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i64, _i, _i, _f, _f, _vp, _i, _i, _vp)
+_talk_decode = _sig("vb_talk_decode", _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i64, _i, _i, _i, _f, _f, _vp)
+_talk_mix = _sig("vb_talk_mix", _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _vp, _i64, _i, _i, _i, _i, _i, _i, _i, _i, _vp)
 
 
 def _st() -> int:
@@ -425,6 +430,86 @@ def paged_attention(q, kv_cache, md, scale, sliding_window=None, logits_soft_cap
     return (out, lse) if return_lse else out
 
 
+# bytes of unmixed head outputs held at a time; larger batches are done some value heads at a time
+TALK_BYTES = 1 << 30
+
+
+def tc_talk_ok(dtype, soft_cap: float) -> bool:
+    """Do the tensor-core kernels of mixed heads take these scores (head shapes: ``tc_attention_ok``)?  e^score must fit into 32 bits."""
+    return dtype == torch.bfloat16 and 0.0 < soft_cap <= 60.0
+
+
+def talk_decode_ok(H: int, Hkv: int) -> bool:
+    g = H // Hkv
+    return H <= 32 and Hkv <= 8 and g in (1, 2, 4, 8, 16) and (g > 2 or H <= 16)
+
+
+def talk_splits(B: int, max_seq_len: int, window: int) -> int:
+    """Key ranges per request in a decode step: one wave of CTAs, two tiles of 128 keys each at least."""
+    if batch_invariant():
+        return 1
+    keys = min(max_seq_len, window) if window else max_seq_len
+    return max(1, min(num_sms() // max(B, 1), (keys + 255) // 256, 16))
+
+
+def talking_attention(q, kv_cache, md, scale, sliding_window, soft_cap, talk, sinks, v_head_size: int, v_rope=None, positions=None,
+                      out=None):
+    """Attention whose heads' weights are mixed by ``talk`` (csrc/attention_talk.cu); q [T, Hq, D] → [T, Hq, DV]."""
+    T, Hq, D = q.shape
+    Hkv, BS = kv_cache.shape[2], kv_cache.shape[3]
+    DV, G, window, dev = v_head_size, Hq // Hkv, sliding_window or 0, q.device
+    back = None if v_rope is None else v_rope.cos_sin_cache
+    neox = v_rope is not None and v_rope.is_neox_style
+    if talk is None:
+        o = paged_attention(q, kv_cache, md, scale, sliding_window, soft_cap, sinks=sinks, v_head_size=DV)
+        if v_rope is not None:
+            half = back.shape[-1] // 2
+            from vllm_b200 import ops
+            o = ops.rotary_embedding(positions, o.view(T, Hq * DV), None, torch.cat((back[:, :half], -back[:, half:]), -1), DV, neox)[0]
+            o = o.view(T, Hq, DV)
+        return o if out is None else out.copy_(o)
+    if out is None:
+        out = torch.empty((T, Hq, DV), dtype=q.dtype, device=dev)
+    assert q.stride(2) == 1 and q.stride(1) == D and out.stride(2) == 1 and out.stride(1) == DV and kv_cache.dtype == q.dtype
+    assert talk.dtype == torch.float32 and talk.is_contiguous() and (sinks is None or sinks.dtype == torch.float32) and not md.flat
+    bt = md.block_table
+
+    def mix(o, l, S, c0, nc):
+        _check(_talk_mix(o.data_ptr(), _DT[o.dtype], _p(l), _p(sinks) if l is not None else None, talk.data_ptr(), _p(positions), _p(back),
+                         int(neox), out.data_ptr(), out.stride(0), T, Hq, G, DV, S, c0, nc, _DT[q.dtype], _st()), "talk_mix")
+    if md.kv_vt and md.decode_only and talk_decode_ok(Hq, Hkv):
+        S = talk_splits(md.num_reqs, md.max_seq_len, window)
+        o = torch.empty((S, T, Hq, Hkv, DV), dtype=torch.float32, device=dev)
+        l = torch.empty((S, T, Hq), dtype=torch.float32, device=dev)
+        _check(_talk_decode(q.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0], bt.data_ptr(), md.seq_lens.data_ptr(), o.data_ptr(),
+                            l.data_ptr(), kernel_error_flag(dev).data_ptr(), md.num_reqs, Hq, Hkv, q.stride(0), bt.stride(0), S, window,
+                            scale, soft_cap, _st()), f"talk_decode(H={Hq}, Hkv={Hkv})")
+        mix(o, l, S, 0, Hkv)
+        return out
+    tc = md.kv_vt
+    if tc:
+        assert tc_attention_ok(D, DV, G) and BS == 64 and tc_talk_ok(q.dtype, soft_cap), "tensor-core layout with another head shape"
+    per_head = T * Hq * DV * (2 if tc else 4)
+    step = max(2 if tc else 1, min(Hkv, TALK_BYTES // max(per_head, 1) // 2 * 2))
+    qsl = md.query_start_loc
+    for c0 in range(0, Hkv, step):
+        nc = min(step, Hkv - c0)
+        # (padding rows are written by no CTA: keep them finite)
+        o = (torch.empty if md.num_actual_tokens == T else torch.zeros)((T, Hq, nc, DV), dtype=torch.bfloat16 if tc else torch.float32, device=dev)
+        if tc:
+            _check(_talk_fold(q.data_ptr(), kv_cache.data_ptr(), kv_cache.shape[0], bt.data_ptr(), md.seq_lens.data_ptr(), qsl.data_ptr(),
+                              o.data_ptr(), kernel_error_flag(dev).data_ptr(), md.num_reqs, T, 1 if md.decode_only else md.max_query_len,
+                              Hq, Hkv, q.stride(0), bt.stride(0), window, scale, soft_cap, _p(sinks), c0, nc, _st()),
+                   f"talk_fold(H={Hq}, Hkv={Hkv})")
+        else:
+            _check(_any_fold(q.data_ptr(), kv_cache.data_ptr(), bt.data_ptr(), md.seq_lens.data_ptr(),
+                             None if md.decode_only else qsl.data_ptr(), o.data_ptr(), md.num_reqs,
+                             1 if md.decode_only else md.max_query_len, Hq, Hkv, D, DV, kv_cache.shape[4], BS, q.stride(0), bt.stride(0),
+                             window, scale, soft_cap, _p(sinks), c0, nc, _DT[q.dtype], _st()), f"any_attention_fold(D={D}, DV={DV})")
+        mix(o, None, 1, c0, nc)
+    return out
+
+
 def merge_attn_states(o1, lse1, o2, lse2):
     T, H, D = o1.shape
     out = torch.empty_like(o1)
@@ -435,11 +520,12 @@ def merge_attn_states(o1, lse1, o2, lse2):
 
 
 _mla_decode = _sig("vb_mla_decode", _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i64, _i64,
-                   _i64, _i64, _i64, _i, _i, _f, _i, _vp)
-_mla_prefill = _sig("vb_mla_prefill", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i64, _i, _i, _i, _i, _i, _i64, _i64,
-                    _i64, _i64, _i, _f, _i, _vp)
+                   _i64, _i64, _i64, _i, _i, _i, _f, _i, _vp)
+_mla_prefill = _sig("vb_mla_prefill", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i64, _i, _i, _i, _i, _i, _i, _i64, _i64,
+                    _i64, _i64, _i64, _i, _i, _f, _i, _vp)
 _mla_simt = _sig("vb_mla_simt", _vp, _vp, _vp, _vp, _vp, _i64, _vp, _vp, _i, _i, _i, _i, _i, _i, _i64, _i64, _i64, _i64, _i64,
-                 _i64, _f, _i, _vp)
+                 _i64, _i, _f, _i, _vp)
+_latent_rope = _sig("vb_latent_rope_cache", _vp, _vp, _i64, _i, _i, _i, _i, _vp, _f, _vp, _vp, _i, _vp, _i64, _vp, _i, _i, _vp)
 _latent_norm = _sig("vb_latent_norm_cache", _vp, _i64, _i, _vp, _vp, _i, _vp, _vp, _vp, _i64, _vp, _i, _f, _i, _vp)
 _mla_ws: dict[int, tuple] = {}
 _kernel_error: dict[int, torch.Tensor] = {}
@@ -477,13 +563,13 @@ def mla_decode_splits(B: int, H: int, max_seq_len: int) -> int:
 
 
 def mla_decode_tc(q_nope_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_seq_len: int, num_splits: int = 0,
-                  return_lse: bool = False):
-    """tcgen05 MLA decode (csrc/mla_decode.cu): q_nope_abs [B, H, R], q_pe [B, H, 64] or None, cache [blocks, BS, R (+64)]."""
+                  return_lse: bool = False, sliding_window: Optional[int] = None):
+    """tcgen05 MLA decode (csrc/mla_decode.cu): q_nope_abs [B, H, R], q_pe [B, H, P] or None, cache [blocks, BS, R + P]."""
     B, H, R = q_nope_abs.shape
     P = 0 if q_pe is None else q_pe.shape[-1]
     assert kv_cache.shape[-1] == R + P and q_nope_abs.stride(-1) == 1 and (q_pe is None or q_pe.stride(-1) == 1)
     dev = q_nope_abs.device
-    splits = num_splits or mla_decode_splits(B, H, max_seq_len)
+    splits = num_splits or mla_decode_splits(B, H, min(max_seq_len, sliding_window) if sliding_window else max_seq_len)
     out = torch.empty((B, H, R), dtype=q_nope_abs.dtype, device=dev)
     lse = torch.empty((B, H), dtype=torch.float32, device=dev) if return_lse else None
     po = pl = None
@@ -503,7 +589,7 @@ def mla_decode_tc(q_nope_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_
                        block_table.data_ptr(), seq_lens.data_ptr(), out.data_ptr(), _p(po), _p(pl), _p(lse), err.data_ptr(), B,
                        H, R, P, kv_cache.shape[1], q_nope_abs.stride(0), q_nope_abs.stride(1),
                        q_pe.stride(0) if P else 0, q_pe.stride(1) if P else 0,
-                       out.stride(0), block_table.stride(0), splits, scale, _DT[q_nope_abs.dtype], _st()),
+                       out.stride(0), block_table.stride(0), splits, sliding_window or 0, scale, _DT[q_nope_abs.dtype], _st()),
            f"mla_decode(B={B},H={H},R={R})", 2 if splits > 1 else 1)
     return (out, lse) if return_lse else out
 
@@ -513,7 +599,9 @@ def _mla_tc_ok(q_nope_abs, q_pe, kv_cache) -> bool:
     if q_pe is None:
         shape_ok = q_nope_abs.dtype == torch.bfloat16 and R % 8 == 0 and R <= 512 and kv_cache.shape[-1] == R
     else:
-        shape_ok = (q_nope_abs.dtype in _HALF_DTYPES and R == 512 and q_pe.shape[-1] == 64 and kv_cache.shape[-1] == 576
+        P = q_pe.shape[-1]
+        widths = (R == 512 and P == 64) or (q_nope_abs.dtype == torch.bfloat16 and R % 8 == 0 and R <= 512 and P % 8 == 0 and P <= 64)
+        shape_ok = (q_nope_abs.dtype in _HALF_DTYPES and widths and kv_cache.shape[-1] == R + P and q_pe.data_ptr() % 16 == 0
                     and q_pe.stride(-1) == 1 and (q_pe.stride(0) * 2) % 16 == 0 and (q_pe.stride(1) * 2) % 16 == 0)
     return (shape_ok and kv_cache.dtype == q_nope_abs.dtype and kv_cache.dim() == 3
             and kv_cache.shape[1] in (16, 32, 64, 128) and q_nope_abs.stride(-1) == 1
@@ -524,7 +612,7 @@ def _mla_tc_ok(q_nope_abs, q_pe, kv_cache) -> bool:
 _HALF_DTYPES = (torch.bfloat16, torch.float16)
 
 
-def mla_simt(q_abs, q_pe, kv_cache, block_table, seq_lens, qsl, scale):
+def mla_simt(q_abs, q_pe, kv_cache, block_table, seq_lens, qsl, scale, sliding_window: Optional[int] = None):
     """Variable-length attention over the latent cache for any width and dtype (csrc/latent.cu); fp32 arithmetic."""
     T, H, R = q_abs.shape
     P = 0 if q_pe is None else q_pe.shape[-1]
@@ -535,30 +623,45 @@ def mla_simt(q_abs, q_pe, kv_cache, block_table, seq_lens, qsl, scale):
     _check(_mla_simt(q_abs.data_ptr(), _p(q_pe), kv_cache.data_ptr(), out.data_ptr(), block_table.data_ptr(),
                      block_table.stride(0), seq_lens.data_ptr(), _p(qsl), seq_lens.numel(), T, H, R, P, kv_cache.shape[1],
                      q_abs.stride(0), q_abs.stride(1), q_pe.stride(0) if P else 0, q_pe.stride(1) if P else 0,
-                     out.stride(0), out.stride(1), scale, _DT[q_abs.dtype], _st()), f"mla_simt(T={T},H={H},R={R})")
+                     out.stride(0), out.stride(1), sliding_window or 0, scale, _DT[q_abs.dtype], _st()), f"mla_simt(T={T},H={H},R={R})")
     return out
 
 
-def mla_prefill_ok(q, v_dim: int, kv_lora_rank: int) -> bool:
-    D = q.shape[-1]
-    return (q.dtype in _HALF_DTYPES and D % 8 == 0 and 8 <= D <= 128 and v_dim % 8 == 0 and 8 <= v_dim <= 128
-            and kv_lora_rank % 8 == 0 and envs.VLLM_B200_ATTN != "simt")
+def mla_prefill_ok(q, dim: int, rot: int, v_dim: int, kv_lora_rank: int) -> bool:
+    return (q.dtype in _HALF_DTYPES and dim % 8 == 0 and 8 <= dim <= 128 and rot % 8 == 0 and rot <= 64 and v_dim % 8 == 0
+            and 8 <= v_dim <= 128 and kv_lora_rank % 8 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+            and envs.VLLM_B200_ATTN != "simt")
 
 
-def mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0: int, max_q: int, scale) -> None:
+def mla_prefill(q, k, v, out, q_start, q_len, seq_len, kv_start, h0: int, max_q: int, scale, k_pe=None, window: int = 0) -> None:
     """Causal attention of prompt portions over expanded keys and values (csrc/mla_prefill.cu), written into ``out``.
-    q [T, H, dim], out [T, H, vdim]; k [KV, hl, dim], v [KV, hl, vdim] hold heads h0 .. h0 + hl - 1."""
-    T, H, D = q.shape
-    KV, hl, _ = k.shape
-    VD = v.shape[-1]
-    assert q.stride(2) == 1 and q.stride(1) == D and k.stride(2) == 1 and k.stride(1) == D and v.stride(2) == 1 and v.stride(1) == VD
+    q [T, H, dim + rot], out [T, H, vdim]; k [KV, hl, dim], v [KV, hl, vdim] hold heads h0 .. h0 + hl - 1, k_pe [KV, rot] the rotated key
+    part of all heads (None: rot = 0)."""
+    T, H, DQ = q.shape
+    KV, hl, D = k.shape
+    VD, P = v.shape[-1], 0 if k_pe is None else k_pe.shape[-1]
+    assert DQ == D + P and (k_pe is None or (k_pe.stride(1) == 1 and k_pe.data_ptr() % 16 == 0))
+    assert q.stride(2) == 1 and q.stride(1) == DQ and k.stride(2) == 1 and k.stride(1) == D and v.stride(2) == 1 and v.stride(1) == VD
     assert out.shape == (T, H, VD) and out.stride(1) == VD and out.stride(2) == 1
     for t in (q, k, v, out):
         assert t.data_ptr() % 16 == 0
-    _check(_mla_prefill(q.data_ptr(), k.data_ptr(), v.data_ptr(), out.data_ptr(), q_start.data_ptr(), q_len.data_ptr(),
+    _check(_mla_prefill(q.data_ptr(), k.data_ptr(), v.data_ptr(), _p(k_pe), out.data_ptr(), q_start.data_ptr(), q_len.data_ptr(),
                         seq_len.data_ptr(), kv_start.data_ptr(), kernel_error_flag(q.device).data_ptr(), q_len.numel(), T, KV, H,
-                        h0, hl, D, VD, q.stride(0), k.stride(0), v.stride(0), out.stride(0), max_q, scale, _DT[q.dtype], _st()),
+                        h0, hl, D, P, VD, q.stride(0), k.stride(0), v.stride(0), 0 if k_pe is None else k_pe.stride(0), out.stride(0), max_q,
+                        window, scale, _DT[q.dtype], _st()),
            f"mla_prefill(T={T},KV={KV},H={H})")
+
+
+def latent_rope_cache(proj, q_off: int, heads: int, dim: int, rot: int, kv_off: int, kv_rank: int, kv_weight, eps: float, positions, cos_sin,
+                      neox: bool, cache=None, slots=None) -> None:
+    """On the columns of a merged projection, in place (csrc/latent.cu): see ops.latent_rope_cache."""
+    assert proj.dim() == 2 and proj.stride(1) == 1 and (cos_sin is None or cos_sin.shape[-1] == rot)
+    if cache is not None:
+        assert cache.shape[-1] == kv_rank + rot and cache.dtype == proj.dtype and cache.is_contiguous() and slots.dtype == torch.int64
+    es = proj.element_size()
+    _check(_latent_rope(proj.data_ptr() + q_off * es, proj.data_ptr() + kv_off * es if kv_rank else None, proj.stride(0), heads, dim, rot,
+                        kv_rank, _p(kv_weight), eps, _p(positions), _p(cos_sin), int(neox), _p(cache), kv_rank + rot,
+                        _p(slots) if cache is not None else None, proj.shape[0], _DT[proj.dtype], _st()), "latent_rope_cache")
 
 
 def latent_norm_cache(lat, q_rank: int, q_weight, kv_rank: int, kv_weight, eps: float, cache=None, slots=None, want_kv: bool = True):
@@ -575,7 +678,7 @@ def latent_norm_cache(lat, q_rank: int, q_weight, kv_rank: int, kv_weight, eps: 
     return cq, ckv
 
 
-def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank):
+def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank, sliding_window: Optional[int] = None):
     """MLA as MQA over the latent cache (K = latent (+ rope) row, V = the latent part of the same row).
 
     Decode batches run on the tcgen05 MLA kernel (csrc/mla_decode.cu: the latent tile is shared by all heads of the
@@ -585,10 +688,10 @@ def mla_attention(q_nope_abs, q_pe, kv_cache, md, scale, kv_lora_rank):
     R = q_nope_abs.shape[-1]
     if md.decode_only and R == kv_lora_rank and _mla_tc_ok(q_nope_abs, q_pe, kv_cache):
         return mla_decode_tc(q_nope_abs, q_pe, kv_cache, md.block_table, md.seq_lens, scale, md.max_seq_len,
-                             md.num_splits or 0)
+                             md.num_splits or 0, sliding_window=sliding_window)
     B = md.num_reqs
     return mla_simt(q_nope_abs, q_pe, kv_cache, md.block_table, md.seq_lens[:B],
-                    None if md.decode_only else md.query_start_loc, scale)
+                    None if md.decode_only else md.query_start_loc, scale, sliding_window)
 
 
 # ------------------------------------------------------------------ sampling
@@ -717,6 +820,47 @@ def add_norm(x, y, next_norm, eps: float, dtype=None, rows=None, inv=None, pair_
     return x if out is None else out
 
 
+_hyper = _sig("vb_hyper_step", _vp, _i, _vp, _i64, _vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _vp)
+_xielu = _sig("vb_xielu", _vp, _vp, _vp, _i64, _i, _vp)
+
+
+def _hyper_call(ids, vocab, y, embed_weight, coef, into, x, weight, eps, dtype):
+    T, S, H = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and into.dtype == torch.float32 and into.numel() == S
+    assert (coef is None or (coef.dtype == torch.float32 and coef.numel() == S + S * S)) and (ids is None or ids.dtype == torch.int32)
+    assert weight.dtype == dtype and (y is None or (y.dtype == dtype and y.stride(-1) == 1))
+    out = torch.empty((T, H), dtype=dtype, device=x.device)
+    _check(_hyper(_p(ids), vocab, _p(y), 0 if y is None else y.stride(0), _p(embed_weight), _p(coef), into.data_ptr(), x.data_ptr(), S,
+                  weight.data_ptr(), out.data_ptr(), T, H, eps, _DT[dtype], _st()), "hyper_step")
+    return out
+
+
+def hyper_entry(ids, table, streams: int, embed_weight, into, weight, eps: float):
+    T = table.shape[0] if ids is None else ids.numel()
+    x = torch.empty((T, streams, table.shape[1]), dtype=torch.float32, device=table.device)
+    return x, _hyper_call(ids, table.shape[0], table, embed_weight, None, into, x, weight, eps, table.dtype)
+
+
+def hyper_step(x, y, coef, into, weight, eps: float, dtype):
+    return _hyper_call(None, 0, y, None, coef if y is not None else None, into, x, weight, eps, dtype)
+
+
+def xielu(x, coef, out=None):
+    x = x.contiguous()
+    out = torch.empty_like(x) if out is None else out
+    _check(_xielu(x.data_ptr(), out.data_ptr(), coef.data_ptr(), x.numel(), _DT[x.dtype], _st()), "xielu")
+    return out
+
+
+def linear_xielu(x, weight, bias, coef):
+    """xielu(x W^T + b): in the epilogue of the decode GEMM, else one pass over its result in place."""
+    x2 = x.reshape(-1, x.shape[-1])
+    if 0 < x2.shape[0] <= 256 and _tc_ok(x2, weight) and _plan(x2.shape[0], weight.shape[0], x2.shape[1])[0]:
+        return gemm_tc(x2, weight, bias, act=3, act_coef=coef).view(x.shape[:-1] + (weight.shape[0],))
+    y = linear(x, weight, bias)
+    return xielu(y, coef, out=y)
+
+
 # ------------------------------------------------------------------ GEMM
 class _GemmWorkspace:
     def __init__(self) -> None:
@@ -742,9 +886,9 @@ def _plan(M: int, N: int, K: int):
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
-            out: Optional[torch.Tensor] = None, act: bool = False) -> torch.Tensor:
-    """Y = X W^T on our tcgen05 kernel. x: [M, K] (row stride free), w: [N, K] contiguous.  ``act`` (M <= 256): W's
-    rows interleave (gate_i, up_i) and the epilogue emits silu(gate) * up → [M, N/2]."""
+            out: Optional[torch.Tensor] = None, act: int = 0, act_coef: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Y = X W^T on our tcgen05 kernel. x: [M, K] (row stride free), w: [N, K] contiguous.  ``act`` 1 (M <= 256): W's
+    rows interleave (gate_i, up_i) and the epilogue emits silu(gate) * up → [M, N/2]; 3 (M <= 256): xIELU with ``act_coef``."""
     M, K = x.shape
     N = w.shape[0]
     swap, bn, splits, wsb, tiles = _plan(M, N, K)
@@ -756,9 +900,9 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = Non
                 raise RuntimeError("GEMM split-K workspace must be allocated before CUDA-graph capture")
             g.ws = torch.empty(max(wsb // 4, 16 << 20), dtype=torch.float32, device=x.device)
             g.counters = torch.zeros(max(tiles, 4096), dtype=torch.int32, device=x.device)
-    y = out if out is not None else torch.empty((M, N // 2 if act else N), dtype=x.dtype, device=x.device)
+    y = out if out is not None else torch.empty((M, N // 2 if act == 1 else N), dtype=x.dtype, device=x.device)
     _check(_gemm_tc(x.data_ptr(), w.data_ptr(), _p(bias), y.data_ptr(), M, N, K, x.stride(0), swap, bn, splits,
-                    _p(g.ws), _p(g.counters), int(act), _DT[x.dtype], _st()), f"gemm_tc(M={M},N={N},K={K})")
+                    _p(g.ws), _p(g.counters), int(act), _p(act_coef), _DT[x.dtype], _st()), f"gemm_tc(M={M},N={N},K={K})")
     return y
 
 
@@ -1304,7 +1448,7 @@ def scaled_fp4_quant(x, global_scale=None, mx: bool = False, swizzled: bool = Fa
 
 
 # ------------------------------------------------------------------ q/k norm + RoPE + cache (csrc/qknorm_rope.cu)
-_qknorm_rope = _sig("vb_qknorm_rope_cache", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i64, _i64, _i64, _vp,
+_qknorm_rope = _sig("vb_qknorm_rope_cache", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i64, _i64, _i64, _vp,
                     _vp, _i, _i, _i, _i, _f, _f, _f, _i, _vp)
 
 
@@ -1323,7 +1467,7 @@ def qknorm_rope_ok(head_dim: int, rot: int, is_neox: bool) -> bool:
     return True
 
 
-_qknorm_rope_any = _sig("vb_qknorm_rope_any", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i64, _i64, _i64, _vp,
+_qknorm_rope_any = _sig("vb_qknorm_rope_any", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i64, _i64, _i64, _vp,
                         _vp, _i, _i, _i, _i, _f, _i, _vp)
 
 
@@ -1333,11 +1477,12 @@ _qknorm_rope_row = _sig("vb_qknorm_rope_row", _vp, _vp, _vp, _vp, _vp, _vp, _vp,
 
 def fused_qk_norm_rope(positions, q, k, q_weight, k_weight, cos_sin_cache, head_dim, eps, is_neox=True, *, v=None,
                        kv_cache=None, slot_mapping=None, gemma: bool = False, k_scale: float = 1.0, v_scale: float = 1.0,
-                       vt: bool = False, v_head_dim: Optional[int] = None, keep32: bool = False, whole: bool = False):
+                       vt: bool = False, v_head_dim: Optional[int] = None, keep32: bool = False, whole: bool = False, v_cos_sin=None):
     """In place: per-head RMSNorm(q), RMSNorm(k) → RoPE → (optionally) K/V insert into the paged cache; one launch.
     ``keep32``: no rounding to the model dtype between the norm and the rotation.  ``whole``: one norm over all heads (weights as
-    long); ``k`` may be None."""
+    long); ``k`` may be None.  Weights None: no norms.  ``v_cos_sin``: values are rotated on their way into the cache."""
     T = q.shape[0]
+    assert v_cos_sin is None or (not whole and v_cos_sin.shape[-1] == (v_head_dim or head_dim))
     Hq, Hkv = q.shape[-1] // head_dim, 0 if k is None else k.shape[-1] // head_dim
     rot = cos_sin_cache.shape[-1] if cos_sin_cache is not None else 0
     assert q.stride(-1) == 1 and (k is None or k.stride(-1) == 1)
@@ -1359,15 +1504,16 @@ def fused_qk_norm_rope(positions, q, k, q_weight, k_weight, cos_sin_cache, head_
         BS, dc = kv_cache.shape[3], kv_cache.shape[4]
     step = min(head_dim // 32, 16 // q.element_size())          # elements of one vector access of the register kernel
     vec = all(t is None or (t.stride(0) % step == 0 and t.data_ptr() % (step * t.element_size()) == 0) for t in (q, k, v)) if step else False
-    if not (q.dtype in _HALF_DTYPES and dv == dc == head_dim and vec and qknorm_rope_ok(head_dim, rot, is_neox)):
+    if not (q.dtype in _HALF_DTYPES and dv == dc == head_dim and vec and qknorm_rope_ok(head_dim, rot, is_neox)
+            and (v_cos_sin is None or qknorm_rope_ok(head_dim, head_dim, is_neox))):
         assert not flags & 1, "this head shape needs a cache of the model dtype"
         _check(_qknorm_rope_any(_p(positions), q.data_ptr(), k.data_ptr(), _p(v), _p(q_weight), _p(k_weight), _p(cos_sin_cache),
-                                rot, T, Hq, Hkv, head_dim, dv, dc, q.stride(0), k.stride(0), v.stride(0) if v is not None else 0,
+                                _p(v_cos_sin), rot, T, Hq, Hkv, head_dim, dv, dc, q.stride(0), k.stride(0), v.stride(0) if v is not None else 0,
                                 _p(kv_cache), _p(slot_mapping), BS, int(is_neox), int(gemma), int(vt), eps, _DT[q.dtype], _st()),
                "qknorm_rope_any")
         return q, k
     _check(_qknorm_rope(_p(positions), q.data_ptr(), k.data_ptr(), _p(v), _p(q_weight), _p(k_weight), _p(cos_sin_cache),
-                        rot, T, Hq, Hkv, head_dim, q.stride(0), k.stride(0), v.stride(0) if v is not None else 0,
+                        _p(v_cos_sin), rot, T, Hq, Hkv, head_dim, q.stride(0), k.stride(0), v.stride(0) if v is not None else 0,
                         _p(kv_cache), _p(slot_mapping), BS, int(is_neox), int(gemma), flags, eps, k_scale, v_scale,
                         _DT[q.dtype], _st()), "qknorm_rope_cache")
     return q, k

@@ -321,7 +321,7 @@ class ModelRunner:
                 and s.block_size == 64 and getattr(s, "dcp", 1) == 1 and kvd in (torch.bfloat16, torch.float16)
                 and self.dtype in (torch.bfloat16, torch.float16)
                 # head shapes and features only the generic kernels implement keep the whole group on the standard layout
-                and all(self._tensor_core_layer(attention_layers().get(n)) for n in g.layer_names
+                and all(self._tensor_core_layer(attention_layers().get(n), self.dtype) for n in g.layer_names
                         if not isinstance(g.spec_of(n), MLAAttentionSpec))))
             for name in g.layer_names:
                 self.layer_to_group[name] = gid
@@ -348,12 +348,15 @@ class ModelRunner:
         self._init_gpu_prep()
 
     @staticmethod
-    def _tensor_core_layer(layer) -> bool:
+    def _tensor_core_layer(layer, dtype) -> bool:
         from vllm_b200.ops import cuda_ops
         if layer is None:
             return True
         d, hq, hkv = layer.head_size, getattr(layer, "num_heads", 1), layer.num_kv_heads
-        return (getattr(layer, "alibi_slopes", None) is None
+        if getattr(layer, "talk", None) is not None and not cuda_ops().tc_talk_ok(dtype, layer.logits_soft_cap):
+            return False
+        return ((getattr(layer, "talk", None) is not None or not getattr(layer, "logits_soft_cap", 0.0))
+                and getattr(layer, "alibi_slopes", None) is None
                 and cuda_ops().tc_attention_ok(d, getattr(layer, "v_head_size", d), max(hq // max(hkv, 1), 1)))
 
     def _init_gpu_prep(self) -> None:
