@@ -95,7 +95,7 @@ class Attention(nn.Module):
                                      dtype_size=dtype_size, dcp=d)
         cls = SlidingWindowSpec if self.sliding_window else FullAttentionSpec
         return cls(block_size=block_size, num_kv_heads=self.num_kv_heads, head_size=self.cache_head_size,
-                   dtype_size=dtype_size, sliding_window=self.sliding_window)
+                   dtype_size=dtype_size, sliding_window=self.cache_window)
 
     def _forward_dcp(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, positions, md, kv_cache) -> torch.Tensor:
         """Decode context parallelism for GQA / MQA caches (reference: config/parallel.py:342-388, v1/attention/ops/dcp.py:
