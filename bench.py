@@ -19,7 +19,7 @@ Both arms print the SAME ``metric`` string and measure the SAME thing:
            over R interleaved repetitions after a full warm-up generate; e2e = 64 * K / t_decode.  Every engine
            step inside copies its inputs host -> device from pinned memory and reads the sampled ids back.
 
-``--design pomipel|legelix|kopadra`` measures another workload: a few layers of that design beside the closest model.
+``--design pomipel|legelix|kopadra|gizilorn`` measures another workload: a few layers of that design beside the closest model.
 
 ``--impl reference`` runs the UNMODIFIED reference (baseline/_ref if the offline install worked, else the stock
 vLLM wheel of the image — DESIGN.md §0) on its DEFAULT engine: multiprocess engine core, async scheduling,
@@ -289,15 +289,15 @@ def main() -> None:
     ap.add_argument("--sync", action="store_true", help="disable async scheduling (host waits for every step)")
     ap.add_argument("--parallelism", default="tp", choices=["tp", "ep"],
                     help="MoE models: ep = experts sharded over the TP group with the fused all-to-all kernels")
-    ap.add_argument("--design", choices=["pomipel", "legelix", "kopadra"], help="instead of the headline workload: prefill and decode of this "
+    ap.add_argument("--design", choices=["pomipel", "legelix", "kopadra", "gizilorn"], help="instead of the headline workload: prefill and decode of this "
                     "design's layers and its kernels, beside the closest model at equal sizes (vllm_b200/benchmarks/latent_layers.py, "
-                    "hybrid_layers.py, memory_layers.py)")
+                    "hybrid_layers.py, memory_layers.py, talking_layers.py)")
     ap.add_argument("--design-part", default="all", choices=["all", "model", "kernels"])
     ap.add_argument("--design-sizes", default=None, help="comma-separated sizes (default: all)")
     args = ap.parse_args()
     if args.design:
         import importlib
-        module = {"pomipel": "latent_layers", "legelix": "hybrid_layers", "kopadra": "memory_layers"}[args.design]
+        module = {"pomipel": "latent_layers", "legelix": "hybrid_layers", "kopadra": "memory_layers", "gizilorn": "talking_layers"}[args.design]
         run_design = importlib.import_module(f"vllm_b200.benchmarks.{module}").run
         print(json.dumps(run_design(args.design_part, args.design_sizes.split(",") if args.design_sizes else None, args.steps)), flush=True)
         return

@@ -7,7 +7,7 @@
 // instead of H x H numbers per key.  (Mixing the weights themselves needs the denominators first, hence a second pass over the scores, and
 // H multiplications per weight on the CUDA cores: more time than the tensor cores take for the additional values.)
 //
-//   talk_fold   prompts: tcgen05, 128 rows (tokens x heads of one KV head), two value heads per CTA
+//   talk_fold   prompts: tcgen05 on pairs of CTAs (cta_group::2), 256 rows (tokens x heads of one KV head), two value heads
 //   talk_mix    T, split-KV sums and denominators, the turn back of rotated values, 16-bit output
 // Decode steps: attention_talk_decode.cu; other head shapes and dtypes: attention_any.cu.
 //
@@ -20,8 +20,10 @@ namespace talk {
 
 constexpr int D = 128, BS = 64, TM = 128, TN = 128;
 constexpr int NUM_THREADS = 192;
-constexpr int K_STAGES = 2, V_SLOTS = 4;
-constexpr int TILE_BYTES = TN * D * 2;          // 32 KB: a tile of keys, or of one head's values
+constexpr int K_STAGES = 4, V_STAGES = 3;
+constexpr int Q_BYTES = TM * D * 2;             // 32 KB: 2 k-blocks of [128 rows x 64]
+constexpr int K_BYTES = BS * D * 2;             // 16 KB: this CTA's page of a key tile, 2 k-blocks of [64 tokens x 64]
+constexpr int V_BYTES = 2 * 128 * 128;          // 32 KB: this CTA's value rows of a tile, 2 pages of [up to 128 rows x 64 tokens]
 
 struct Params {
   const int* block_table; const int* seq_lens; const int* qsl;
@@ -32,10 +34,6 @@ struct Params {
   int* error;
 };
 
-VB_DEVICE void tma_load_3d(void* dst, const void* tmap, int c0, int c1, int c2, uint64_t* bar) {
-  asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
-               ::"r"(smem_u32(dst)), "l"(tmap), "r"(smem_u32(bar)), "r"(c0), "r"(c1), "r"(c2) : "memory");
-}
 VB_DEVICE void tmem_st_32x32(uint32_t taddr, const uint32_t* r) {
   asm volatile(
       "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
@@ -47,17 +45,57 @@ VB_DEVICE void tmem_st_32x32(uint32_t taddr, const uint32_t* r) {
         "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31]) : "memory");
 }
 VB_DEVICE void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-// D[tmem] (+)= A[tmem: row = lane, two 16-bit values per column] * B[smem desc]
-VB_DEVICE void umma_f16_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+// ---- pairs of CTAs: one MMA over the rows of both, issued by the leader (rank 0).  Each CTA holds its own rows of A and D, and half of
+// the N rows of B.
+// D[tmem] (+)= A * B; A from shared memory, or from TMEM (row = lane, two 16-bit values per column)
+VB_DEVICE void umma2_f16(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
   asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-               "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+               "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+               ::"r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
+}
+VB_DEVICE void umma2_f16_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
+  asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+               "tcgen05.mma.cta_group::2.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
                ::"r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
 }
+// arrives on the barrier at this offset in both CTAs once the MMAs issued before have completed
+VB_DEVICE void umma2_commit(uint64_t* bar) {
+  asm volatile("tcgen05.commit.cta_group::2.mbarrier::arrive::one.shared::cluster.multicast::cluster.b64 [%0], %1;"
+               ::"r"(smem_u32(bar)), "h"((uint16_t)3) : "memory");
+}
+// loads into this CTA's shared memory and counts the bytes on a barrier of the pair (a shared::cluster address)
+VB_DEVICE void tma2_load_2d(void* dst, const void* tmap, int c0, int c1, uint32_t bar) {
+  asm volatile("cp.async.bulk.tensor.2d.cta_group::2.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4}], [%2];"
+               ::"r"(smem_u32(dst)), "l"(tmap), "r"(bar), "r"(c0), "r"(c1) : "memory");
+}
+VB_DEVICE void tma2_load_3d(void* dst, const void* tmap, int c0, int c1, int c2, uint32_t bar) {
+  asm volatile("cp.async.bulk.tensor.3d.cta_group::2.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+               ::"r"(smem_u32(dst)), "l"(tmap), "r"(bar), "r"(c0), "r"(c1), "r"(c2) : "memory");
+}
+VB_DEVICE void tmem2_alloc(uint32_t* smem_dst, uint32_t ncols) {
+  asm volatile("tcgen05.alloc.cta_group::2.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(smem_dst)), "r"(ncols) : "memory");
+  asm volatile("tcgen05.relinquish_alloc_permit.cta_group::2.sync.aligned;" ::: "memory");
+}
+VB_DEVICE void tmem2_dealloc(uint32_t taddr, uint32_t ncols) {
+  asm volatile("tcgen05.dealloc.cta_group::2.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(ncols) : "memory");
+}
+VB_DEVICE void arrive_cluster(uint32_t bar) {
+  asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(bar) : "memory");
+}
+VB_DEVICE void wait_cluster_lim(uint64_t* bar, uint32_t parity, int& budget) {      // what threads of the other CTA have arrived on
+  for (;;) {
+    uint32_t ok;
+    asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.acquire.cluster.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+                 : "=r"(ok) : "r"(smem_u32(bar)), "r"(parity) : "memory");
+    if (ok || --budget < 0) break;
+  }
+}
 
-// CTA = (query tile, KV head of the scores x pair of value heads, request).  Warp roles: 0 TMA producer, 1 MMA issuer + TMEM owner, 2..5
-// softmax / epilogue (thread = query row = TMEM lane).  TMEM: S double-buffered (2 x 128 columns), two accumulators (2 x 128).  P
-// overwrites the S it came from (bf16, 64 columns) and is the PV product's A operand there, so it is double-buffered too: the softmax of
-// tile j runs under the PV products of tile j - 1.
+// Pair of CTAs = two query tiles in a row x KV head of the scores x pair of value heads, one request.  Both tiles read the same keys and
+// values; each CTA fetches half of them (a page of the key tile; one value head, or half of a single one).  Warp roles: 0 TMA producer, 1
+// MMA issuer (leader) + TMEM owner, 2..5 softmax / epilogue (thread = query row = TMEM lane).  TMEM: S double-buffered (2 x 128
+// columns), two accumulators (2 x 128).  P overwrites the S it came from (bf16, 64 columns) and is the PV product's A operand there, so
+// it is double-buffered too: the softmax of tile j runs under the PV products of tile j - 1.
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                  const __grid_constant__ CUtensorMap tmap_v, const Params p) {
@@ -65,32 +103,32 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
   extern __shared__ __align__(1024) unsigned char smem_raw[];
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   unsigned char* q_smem = smem;
-  unsigned char* k_smem = q_smem + TILE_BYTES;
-  unsigned char* v_smem = k_smem + K_STAGES * TILE_BYTES;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(v_smem + V_SLOTS * TILE_BYTES);
-  uint64_t* q_full = bars;
-  uint64_t* k_full = bars + 1;                 // [K_STAGES]
+  unsigned char* k_smem = q_smem + Q_BYTES;
+  unsigned char* v_smem = k_smem + K_STAGES * K_BYTES;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_smem + V_STAGES * V_BYTES);
+  uint64_t* q_full = bars;                     // the leader's count the bytes of both CTAs
+  uint64_t* k_full = bars + 1;                 // [K_STAGES] (leader's)
   uint64_t* k_empty = k_full + K_STAGES;
-  uint64_t* v_full = k_empty + K_STAGES;       // [V_SLOTS]
-  uint64_t* v_empty = v_full + V_SLOTS;
-  uint64_t* s_full = v_empty + V_SLOTS;        // [2]
-  uint64_t* p_full = s_full + 2;               // [2]
+  uint64_t* v_full = k_empty + K_STAGES;       // [V_STAGES] (leader's)
+  uint64_t* v_empty = v_full + V_STAGES;
+  uint64_t* s_full = v_empty + V_STAGES;       // [2]
+  uint64_t* p_full = s_full + 2;               // [2] (leader's: the warps of both CTAs)
   uint64_t* pv_done = p_full + 2;              // [2]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 2);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int budget = MBAR_BUDGET;
-  const int b = blockIdx.z, groups = (p.nc + 1) / 2;
+  const int rank = (int)cluster_ctarank(), b = blockIdx.z, groups = (p.nc + 1) / 2;
   const int h = blockIdx.y / groups, cv = blockIdx.y % groups * 2;       // KV head of the scores, first value head (behind c0)
-  const int nv = min(2, p.nc - cv);
+  const int nv = min(2, p.nc - cv), v_rows = nv * 64;                    // rows of a value tile's B operand in this CTA
   pdl_trigger();
   pdl_wait();
   const int q0 = p.qsl[b], q_len = p.qsl[b + 1] - q0;
-  const int tok0 = blockIdx.x * p.TQ;
-  if (tok0 >= q_len) return;                                             // uniform across the CTA
-  const int n_tok = min(p.TQ, q_len - tok0);
-  const int pos0 = p.seq_lens[b] - q_len + tok0;
-  const int kv_end = pos0 + n_tok, kv_begin = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+  const int pair0 = ((int)blockIdx.x & ~1) * p.TQ, tok0 = blockIdx.x * p.TQ;
+  if (pair0 >= q_len) return;                                            // uniform across the pair
+  const int n_tok = min(p.TQ, q_len - tok0);                             // <= 0: the pair's second tile is empty
+  const int ctx = p.seq_lens[b] - q_len, pos0 = ctx + tok0;
+  const int kv_end = ctx + min(q_len, pair0 + 2 * p.TQ), kv_begin = p.window > 0 ? max(0, ctx + pair0 - p.window + 1) : 0;
   const int tile_lo = kv_begin / TN, n_tiles = (kv_end + TN - 1) / TN - tile_lo;
   const int n_pages = (kv_end + BS - 1) / BS;
 
@@ -98,94 +136,93 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     tma_prefetch_desc(&tmap_q); tma_prefetch_desc(&tmap_k); tma_prefetch_desc(&tmap_v);
     mbar_init(q_full, 1);
     for (int s = 0; s < K_STAGES; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
-    for (int s = 0; s < V_SLOTS; ++s) { mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
-    for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&p_full[s], 128); mbar_init(&pv_done[s], 1); }
+    for (int s = 0; s < V_STAGES; ++s) { mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
+    for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&p_full[s], 8); mbar_init(&pv_done[s], 1); }
     mbar_fence_init();
   }
-  if (warp == 1) tmem_alloc(tmem_slot, 512);
+  if (warp == 1) tmem2_alloc(tmem_slot, 512);
   tc_fence_before();
   __syncthreads();
+  cluster_sync();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot, tmem_o = tmem_base + 256;
 
   if (warp == 0) {
     if (lane == 0) {
-      // ===== TMA producer.  Tiles are always whole: pages past the sequence are read from the null page (finite, masked)
-      mbar_expect_tx(q_full, TILE_BYTES);
-      tma_load_3d(q_smem, &tmap_q, 0, h * p.G, q0 + tok0, q_full);
-      tma_load_3d(q_smem + TM * 128, &tmap_q, 64, h * p.G, q0 + tok0, q_full);
+      // ===== TMA producer of this CTA's halves.  Tiles are always whole: pages past the sequence are read from the null page (finite,
+      // masked)
+      const uint32_t bar_q = dsmem_addr(smem_u32(q_full), 0);
+      if (rank == 0) mbar_expect_tx(q_full, 2 * Q_BYTES);
+      tma2_load_3d(q_smem, &tmap_q, 0, h * p.G, q0 + tok0, bar_q);
+      tma2_load_3d(q_smem + TM * 128, &tmap_q, 64, h * p.G, q0 + tok0, bar_q);
       const int* bt = p.block_table + (int64_t)b * p.bt_stride;
       for (int j = 0; j < n_tiles && budget >= 0; ++j) {
-        const int s = j % K_STAGES;
         int blk[2];
         for (int u = 0; u < 2; ++u) {
           const int page = (tile_lo + j) * 2 + u;
           blk[u] = page < n_pages ? bt[page] : 0;
         }
+        const int s = j % K_STAGES, vs = j % V_STAGES;
         mbar_wait_lim(&k_empty[s], ((j / K_STAGES) & 1) ^ 1, budget);
         if (budget < 0) break;
-        unsigned char* ks = k_smem + s * TILE_BYTES;
-        mbar_expect_tx(&k_full[s], TILE_BYTES);
+        const uint32_t bar_k = dsmem_addr(smem_u32(&k_full[s]), 0);
+        if (rank == 0) mbar_expect_tx(&k_full[s], 2 * K_BYTES);
+        for (int kb = 0; kb < 2; ++kb)
+          tma2_load_2d(k_smem + s * K_BYTES + kb * (BS * 128), &tmap_k, kb * 64, ((rank ? blk[1] : blk[0]) * 2 * p.Hkv + h) * BS, bar_k);
+        mbar_wait_lim(&v_empty[vs], ((j / V_STAGES) & 1) ^ 1, budget);
+        if (budget < 0) break;
+        const uint32_t bar_v = dsmem_addr(smem_u32(&v_full[vs]), 0);
+        if (rank == 0) mbar_expect_tx(&v_full[vs], 2 * 2 * v_rows * 128);
         for (int u = 0; u < 2; ++u) {
-          const int row = (blk[u] * 2 * p.Hkv + h) * BS;
-          tma_load_2d(ks + u * (BS * 128), &tmap_k, 0, row, &k_full[s]);
-          tma_load_2d(ks + TN * 128 + u * (BS * 128), &tmap_k, 64, row, &k_full[s]);
-        }
-        for (int v = 0; v < nv; ++v) {
-          const int n = j * nv + v, sl = n % V_SLOTS;
-          mbar_wait_lim(&v_empty[sl], ((n / V_SLOTS) & 1) ^ 1, budget);
-          if (budget < 0) break;
-          unsigned char* vs = v_smem + sl * TILE_BYTES;
-          mbar_expect_tx(&v_full[sl], TILE_BYTES);
-          for (int u = 0; u < 2; ++u)
-            tma_load_2d(vs + u * (D * 128), &tmap_v, 0, ((blk[u] * 2 + 1) * p.Hkv + p.c0 + cv + v) * D, &v_full[sl]);
+          // two value heads: the CTA's own, 128 rows; one: half of its rows
+          const int row = ((blk[u] * 2 + 1) * p.Hkv + p.c0 + cv + (nv == 2 ? rank : 0)) * D + (nv == 2 ? 0 : rank * 64);
+          for (int r = 0; r < v_rows; r += 64) tma2_load_2d(v_smem + vs * V_BYTES + (u * v_rows + r) * 128, &tmap_v, 0, row + r, bar_v);
         }
       }
-      if (budget < 0) {                         // let the copies in flight land before the block gives up its memory
+      if (budget < 0 && rank == 0) {            // let the copies in flight land before the pair gives up its memory
         for (int s = 0; s < K_STAGES; ++s)
           for (int n = 0; n < 4096 && !(mbar_try_wait(&k_full[s], 0) || mbar_try_wait(&k_full[s], 1)); ++n) {}
-        for (int s = 0; s < V_SLOTS; ++s)
+        for (int s = 0; s < V_STAGES; ++s)
           for (int n = 0; n < 4096 && !(mbar_try_wait(&v_full[s], 0) || mbar_try_wait(&v_full[s], 1)); ++n) {}
       }
     }
   } else if (warp == 1) {
-    // ===== MMA issuer
-    const uint32_t idesc = umma_idesc_f16(TM, TN, true);
-    const uint64_t d_q = umma_desc_sw128(q_smem), d_k = umma_desc_sw128(k_smem), d_v = umma_desc_sw128(v_smem);
-    mbar_wait_lim(q_full, 0, budget);
-    __syncwarp();
-    for (int j = 0; j <= n_tiles; ++j) {
-      if (j < n_tiles) {
-        const int s = j % K_STAGES;
-        mbar_wait_lim(&k_full[s], (j / K_STAGES) & 1, budget);
-        if (j >= 2) mbar_wait_lim(&pv_done[j & 1], ((j >> 1) & 1) ^ 1, budget);      // PV of tile j - 2 has read the P in this buffer
-        tc_fence_after();
-        if (lane == 0) {
+    if (rank == 0) {
+      // ===== MMA issuer
+      const uint32_t idesc_s = umma_idesc_f16(2 * TM, TN, true), idesc_o = umma_idesc_f16(2 * TM, nv * 128, true);
+      const uint64_t d_q = umma_desc_sw128(q_smem), d_k = umma_desc_sw128(k_smem), d_v = umma_desc_sw128(v_smem);
+      mbar_wait_lim(q_full, 0, budget);
+      __syncwarp();
+      for (int j = 0; j <= n_tiles; ++j) {
+        if (j < n_tiles) {
+          const int s = j % K_STAGES;
+          mbar_wait_lim(&k_full[s], (j / K_STAGES) & 1, budget);
+          if (j >= 2) mbar_wait_lim(&pv_done[j & 1], ((j >> 1) & 1) ^ 1, budget);    // PV of tile j - 2 has read the P in this buffer
+          tc_fence_after();
+          if (lane == 0) {
 #pragma unroll
-          for (int kb = 0; kb < 2; ++kb)
+            for (int kb = 0; kb < 2; ++kb)
 #pragma unroll
-            for (int k = 0; k < 4; ++k)
-              umma_f16(tmem_base + (j & 1) * 128, d_q + (uint64_t)(((kb * TM * 128) >> 4) + k * 2),
-                       d_k + (uint64_t)(((s * TILE_BYTES + kb * TN * 128) >> 4) + k * 2), idesc, (kb | k) != 0);
-          umma_commit(&s_full[j & 1]);
-          umma_commit(&k_empty[s]);
+              for (int k = 0; k < 4; ++k)
+                umma2_f16(tmem_base + (j & 1) * 128, d_q + (uint64_t)(((kb * TM * 128) >> 4) + k * 2),
+                          d_k + (uint64_t)(((s * K_BYTES + kb * BS * 128) >> 4) + k * 2), idesc_s, (kb | k) != 0);
+            umma2_commit(&s_full[j & 1]);
+            umma2_commit(&k_empty[s]);
+          }
+          __syncwarp();
         }
-        __syncwarp();
-      }
-      if (j > 0) {
-        const int jj = j - 1;
-        mbar_wait_lim(&p_full[jj & 1], (jj >> 1) & 1, budget);
-        for (int v = 0; v < nv; ++v) {
-          const int n = jj * nv + v, sl = n % V_SLOTS;
-          mbar_wait_lim(&v_full[sl], (n / V_SLOTS) & 1, budget);
+        if (j > 0) {
+          const int jj = j - 1, vs = jj % V_STAGES;
+          mbar_wait_lim(&v_full[vs], (jj / V_STAGES) & 1, budget);
+          wait_cluster_lim(&p_full[jj & 1], (jj >> 1) & 1, budget);
           tc_fence_after();
           if (lane == 0) {
 #pragma unroll
             for (int kk = 0; kk < 8; ++kk)
-              umma_f16_ta(tmem_o + v * 128, tmem_base + (jj & 1) * 128 + kk * 8,
-                          d_v + (uint64_t)(((sl * TILE_BYTES + (kk / 4) * D * 128) >> 4) + (kk & 3) * 2), idesc, (jj | kk) != 0);
-            umma_commit(&v_empty[sl]);
-            if (v == nv - 1) umma_commit(&pv_done[jj & 1]);
+              umma2_f16_ta(tmem_o, tmem_base + (jj & 1) * 128 + kk * 8,
+                           d_v + (uint64_t)((vs * V_BYTES + (kk / 4) * v_rows * 128) >> 4) + (uint64_t)((kk & 3) * 2), idesc_o, (jj | kk) != 0);
+            umma2_commit(&v_empty[vs]);
+            umma2_commit(&pv_done[jj & 1]);
           }
           __syncwarp();
         }
@@ -195,6 +232,7 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     // ===== softmax / epilogue
     const int qd = warp & 3, r = qd * 32 + lane;
     const uint32_t t_lane = (uint32_t)(qd * 32) << 16;
+    const uint32_t bar_p = dsmem_addr(smem_u32(p_full), 0);
     const int tq = r / p.G, g = r % p.G;
     const bool row_valid = tq < n_tok;
     const int qpos = pos0 + tq;
@@ -222,20 +260,21 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
           for (int i = 0; i < 32; ++i)
             if (c * 32 + i >= hi || c * 32 + i < lo) s[i] = 0.f;
         }
-        float l0 = 0.f, l1 = 0.f;
+        float l[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          l0 += s[i];
-          l1 += s[i + 1];
+          l[i & 2] += s[i];
+          l[(i & 2) + 1] += s[i + 1];
           pk[c * 16 + i / 2] = pack2<T>(s[i], s[i + 1]);
         }
-        l_run += l0 + l1;
+        l_run += (l[0] + l[1]) + (l[2] + l[3]);
       }
       tmem_st_32x32(t_s, pk);
       tmem_st_32x32(t_s + 32, pk + 32);
       tmem_st_wait();
       tc_fence_before();
-      mbar_arrive(&p_full[j & 1]);
+      __syncwarp();
+      if (lane == 0) arrive_cluster(bar_p + (j & 1) * 8);
     }
     mbar_wait_lim(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, budget);
     __syncwarp();
@@ -268,9 +307,10 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     }
     tc_fence_before();
   }
+  __syncwarp();
   tc_fence_before();
-  __syncthreads();
-  if (warp == 1) tmem_dealloc(tmem_base, 512);
+  cluster_sync();                               // nobody leaves while the other CTA may still arrive on its barriers
+  if (warp == 1) tmem2_dealloc(tmem_base, 512);
   if (budget < 0 && p.error) *p.error = 1;
 }
 
@@ -414,12 +454,22 @@ EXPORT int vb_talk_fold(const void* q, const void* kv_cache, int64_t num_blocks,
   CUtensorMap tq, tk, tv;
   int rc;
   if ((rc = map_queries(&tq, q, Hq, T_total, q_stride, G, p.TQ))) return rc;
-  if ((rc = map_pages(&tk, &tv, kv_cache, num_blocks, Hkv))) return rc;
-  const int smem = (1 + K_STAGES + V_SLOTS) * TILE_BYTES + 32 * 8 + 16 + 1024;
+  if ((rc = map_pages(&tk, &tv, kv_cache, num_blocks, Hkv, 64))) return rc;
+  const int smem = Q_BYTES + K_STAGES * K_BYTES + V_STAGES * V_BYTES + 32 * 8 + 16 + 1024;
   static bool a = false;
   if (!a) { cudaFuncSetAttribute(talk_fold_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); a = true; }
-  const dim3 grid((max_q_len + p.TQ - 1) / p.TQ, Hkv * ((nc + 1) / 2), B);
-  vb_launch(talk_fold_kernel, grid, dim3(NUM_THREADS), (size_t)smem, st, tq, tk, tv, p);
+  const int pairs = (max_q_len + 2 * p.TQ - 1) / (2 * p.TQ);
+  if (B > 65535) return -6;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(2 * pairs, Hkv * ((nc + 1) / 2), B); cfg.blockDim = dim3(NUM_THREADS); cfg.dynamicSmemBytes = (size_t)smem; cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = 2; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;      // the pair is two neighbours along x
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = vb_pdl_enabled() ? 2 : 1;
+  cudaLaunchKernelEx(&cfg, talk_fold_kernel, tq, tk, tv, p);
   return (int)cudaGetLastError();
 }
 

@@ -292,7 +292,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
               if (c + j < m_lim) {
                 float o = v[j] + bias;
                 if (p.act == 2) { o = fmaxf(o, 0.f); o *= o; }
-                if (p.act == 3) o = xielu(o, p.act_coef[0], p.act_coef[1]);
+                if (p.act == 3) o = xielu16(o, p.act_coef[0], p.act_coef[1]);
                 y[(size_t)(m0 + j) * p.N + n] = from_f32<T>(o);
               }
           }
@@ -378,7 +378,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
             }
             if (p.act == 3) {
 #pragma unroll
-              for (int e = 0; e < 4; ++e) o[e] = xielu(o[e], p.act_coef[0], p.act_coef[1]);
+              for (int e = 0; e < 4; ++e) o[e] = xielu16(o[e], p.act_coef[0], p.act_coef[1]);
             }
             if (n + 4 <= p.N && (p.N & 3) == 0) {
               uint2 pk;

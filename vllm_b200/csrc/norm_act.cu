@@ -333,11 +333,11 @@ __global__ void __launch_bounds__(256) xielu_kernel(const T* __restrict__ x, T* 
   pdl_wait();
   for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
     if constexpr (V == 1) {
-      y[i] = from_f32<T>(xielu(to_f32(x[i]), a, b));
+      y[i] = from_f32<T>(sizeof(T) == 4 ? xielu(to_f32(x[i]), a, b) : xielu16(to_f32(x[i]), a, b));
     } else {
       Vec16<T> v = ld16(x + i * V);
 #pragma unroll
-      for (int j = 0; j < V; ++j) v.e[j] = from_f32<T>(xielu(to_f32(v.e[j]), a, b));
+      for (int j = 0; j < V; ++j) v.e[j] = from_f32<T>(sizeof(T) == 4 ? xielu(to_f32(v.e[j]), a, b) : xielu16(to_f32(v.e[j]), a, b));
       st16(y + i * V, v);
     }
   }

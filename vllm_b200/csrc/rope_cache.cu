@@ -28,7 +28,7 @@ __global__ void rope_cache_kernel(const int64_t* __restrict__ positions, T* __re
                                   const T* __restrict__ v, const float* __restrict__ cos_sin, int rot, int Hq,
                                   int Hkv, int D, int64_t q_stride, int64_t k_stride, int64_t v_stride,
                                   void* __restrict__ kv_cache, const int64_t* __restrict__ slot_mapping, int BS,
-                                  float k_inv_scale, float v_inv_scale, int vt) {
+                                  float k_inv_scale, float v_inv_scale, int vt, const float* __restrict__ v_cos_sin) {
   constexpr int N = 8;  // 16-bit dtypes only
   pdl_trigger();
   pdl_wait();
@@ -115,7 +115,30 @@ __global__ void rope_cache_kernel(const int64_t* __restrict__ positions, T* __re
     } else if (do_cache) {
       const int j = i - n_qk;
       const int h = j / (D / N), c = j % (D / N);
-      Vec16<T> a = ld16(v + t * v_stride + (int64_t)h * D + c * N);
+      const T* vr = v + t * v_stride + (int64_t)h * D;
+      Vec16<T> a = ld16(vr + c * N);
+      if (v_cos_sin) {              // values turn with their position too, all of their dims, in the layout of the keys
+        const float* vc = v_cos_sin + positions[t] * D;
+        const int vh = D / 2;
+        if (NEOX) {
+          const bool first = c * N < vh;
+          const Vec16<T> b = ld16(vr + c * N + (first ? vh : -vh));
+          const int i0 = first ? c * N : c * N - vh;
+#pragma unroll
+          for (int e = 0; e < N; ++e) {
+            const float x = to_f32(a.e[e]), o = to_f32(b.e[e]), co = vc[i0 + e], si = vc[vh + i0 + e];
+            a.e[e] = from_f32<T>(first ? x * co - o * si : x * co + o * si);
+          }
+        } else {
+#pragma unroll
+          for (int e = 0; e < N; e += 2) {
+            const int p0 = (c * N + e) / 2;
+            const float x1 = to_f32(a.e[e]), x2 = to_f32(a.e[e + 1]), co = vc[p0], si = vc[vh + p0];
+            a.e[e] = from_f32<T>(x1 * co - x2 * si);
+            a.e[e + 1] = from_f32<T>(x2 * co + x1 * si);
+          }
+        }
+      }
       if (vt) {
         // tensor-core layout: the V page is stored transposed [D, BS] (tokens contiguous) so that it is a
         // K-major B operand for O = P·V (see attention_tc.cu)
@@ -150,12 +173,14 @@ __global__ void concat_cache_mla_kernel(const T* __restrict__ kv_c, const T* __r
 
 }  // namespace
 
-// q may be null (cache write only, rot = 0); kv_cache may be null (rope only).
+// q may be null (cache write only, rot = 0); kv_cache may be null (rope only).  v_cos_sin [positions, D] (optional): values are rotated on
+// their way into the cache.
 EXPORT int vb_rope_and_cache(const int64_t* positions, void* q, void* k, const void* v, const float* cos_sin, int rot,
                              int T, int Hq, int Hkv, int D, int64_t q_stride, int64_t k_stride, int64_t v_stride,
                              void* kv_cache, const int64_t* slot_mapping, int BS, int neox, int kv_fp8,
-                             float k_scale, float v_scale, int dtype, cudaStream_t st) {
+                             float k_scale, float v_scale, const float* v_cos_sin, int dtype, cudaStream_t st) {
   if (T == 0) return 0;
+  if (v_cos_sin && ((D / 2) % 8 || !positions)) return -1;
   if (dtype == DT_F32 || D % 8 != 0 || (rot / 2) % 8 != 0 || (D - rot) % 8 != 0) return -1;
   const int items = (Hq + Hkv) * ((rot / 2 + (D - rot)) / 8) + Hkv * (D / 8);
   int thr = ((items + 31) / 32) * 32;
@@ -166,7 +191,7 @@ EXPORT int vb_rope_and_cache(const int64_t* positions, void* q, void* k, const v
 #define VB_ROPE_LAUNCH(NX, F8)                                                                                    \
   vb_launch(rope_cache_kernel<TT, NX, F8>, T, thr, 0, st, positions, (TT*)q, (TT*)k, (const TT*)v, cos_sin, rot, Hq, Hkv, \
                                                    D, q_stride, k_stride, v_stride, kv_cache, slot_mapping, BS,     \
-                                                   1.f / k_scale, 1.f / v_scale, vt)
+                                                   1.f / k_scale, 1.f / v_scale, vt, v_cos_sin)
   DISPATCH_HALF(dtype, TT, {
     if (neox) { if (kv_fp8) VB_ROPE_LAUNCH(true, true); else VB_ROPE_LAUNCH(true, false); }
     else { if (kv_fp8) VB_ROPE_LAUNCH(false, true); else VB_ROPE_LAUNCH(false, false); }

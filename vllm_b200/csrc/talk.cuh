@@ -24,9 +24,10 @@ VB_DEVICE float rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(
 // In place, for N scores of a thread; the whole warp takes part.  Where all scores of the warp are below a quarter of the cap the Taylor
 // series of tanh to the seventh power is exact to 3e-7 and needs no more special functions than a plain softmax.
 template <int N> VB_DEVICE void cap_exp(float (&s)[N], const Cap& c) {
-  float m = 0.f;
+  float m4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-  for (int i = 0; i < N; ++i) m = fmaxf(m, fabsf(s[i]));
+  for (int i = 0; i < N; ++i) m4[i & 3] = fmaxf(m4[i & 3], fabsf(s[i]));
+  const float m = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
   if (__all_sync(0xffffffffu, m * c.ku < 0.25f)) {
 #pragma unroll
     for (int i = 0; i < N; ++i) {
@@ -65,11 +66,11 @@ inline int map_queries(CUtensorMap* m, const void* q, int Hq, int T, int64_t str
   const cuuint32_t box[3] = {64, (cuuint32_t)G, (cuuint32_t)TQ};
   return encode(m, q, 3, dims, strides, box);
 }
-// key pages as rows of 128 dims (box 64 x 64 tokens), value pages as rows of 64 tokens (box 64 x 128 dims)
-inline int map_pages(CUtensorMap* k, CUtensorMap* v, const void* cache, int64_t blocks, int Hkv) {
+// key pages as rows of 128 dims (box 64 x 64 tokens), value pages as rows of 64 tokens (box 64 x v_rows dims)
+inline int map_pages(CUtensorMap* k, CUtensorMap* v, const void* cache, int64_t blocks, int Hkv, int v_rows) {
   const cuuint64_t kd[2] = {128, (cuuint64_t)blocks * 2 * Hkv * 64}, ks[1] = {256};
   const cuuint64_t vd[2] = {64, (cuuint64_t)blocks * 2 * Hkv * 128}, vs[1] = {128};
-  const cuuint32_t kb[2] = {64, 64}, vb[2] = {64, 128};
+  const cuuint32_t kb[2] = {64, 64}, vb[2] = {64, (cuuint32_t)v_rows};
   int rc = encode(k, cache, 2, kd, ks, kb);
   return rc ? rc : encode(v, cache, 2, vd, vs, vb);
 }

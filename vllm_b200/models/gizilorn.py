@@ -159,7 +159,7 @@ class GizilornForCausalLM(LlamaForCausalLM):
         attn = [l["mixer"] for l in cfg["layers"] if l["type"] == "attention"]
         latent = [l["mixer"] for l in cfg["layers"] if l["type"] == "latent_attention"]
         if attn:
-            out |= {"qknorm_rope", "attention_talk"}
+            out |= {"qknorm_rope", "rope_cache", "attention_talk"} if half else {"qknorm_rope", "attention_talk"}
             # one cache layout for all attention layers: the tensor-core kernels run where they take every layer's head shape
             if half and all(cu.tc_attention_ok(a["dim"], a["vdim"], a["heads"] // a["kv_heads"]) for a in attn):
                 out |= {"attention_tc", "attention_talk_decode"}

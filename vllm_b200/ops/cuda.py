@@ -85,7 +85,7 @@ _layer_norm = _sig("vb_layer_norm", _vp, _vp, _vp, _vp, _i, _i, _f, _i, _vp)
 _act_and_mul = _sig("vb_act_and_mul", _vp, _vp, _i64, _i, _i, _i, _vp)
 _activation = _sig("vb_activation", _vp, _vp, _i64, _i, _i, _vp)
 _rope_and_cache = _sig("vb_rope_and_cache", _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i64, _i64, _i64, _vp, _vp,
-                       _i, _i, _i, _f, _f, _i, _vp)
+                       _i, _i, _i, _f, _f, _vp, _i, _vp)
 _concat_mla = _sig("vb_concat_and_cache_mla", _vp, _vp, _vp, _vp, _i, _i, _i, _i64, _i64, _i, _i, _vp)
 _paged_attention = _sig("vb_paged_attention", _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
                         _i64, _i64, _i, _i, _i, _f, _f, _f, _i, _i, _i, _vp)
@@ -237,7 +237,7 @@ def _kv_fp8(kv_cache) -> int:
 
 
 def rope_and_cache(positions, q, k, v, cos_sin_cache, head_dim, is_neox, kv_cache, slot_mapping,
-                   k_scale: float = 1.0, v_scale: float = 1.0, vt: bool = False):
+                   k_scale: float = 1.0, v_scale: float = 1.0, vt: bool = False, v_cos_sin=None):
     T = q.shape[0]
     Hq, Hkv = q.shape[-1] // head_dim, k.shape[-1] // head_dim
     assert q.stride(-1) == 1 and k.stride(-1) == 1 and v.stride(-1) == 1
@@ -247,7 +247,7 @@ def rope_and_cache(positions, q, k, v, cos_sin_cache, head_dim, is_neox, kv_cach
     _check(_rope_and_cache(positions.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), cos_sin_cache.data_ptr(),
                            rot, T, Hq, Hkv, head_dim, q.stride(0), k.stride(0), v.stride(0), kv_cache.data_ptr(),
                            slot_mapping.data_ptr(), kv_cache.shape[3], int(is_neox), flags, k_scale,
-                           v_scale, _DT[q.dtype], _st()), "rope_and_cache")
+                           v_scale, _p(v_cos_sin), _DT[q.dtype], _st()), "rope_and_cache")
     return q, k
 
 
@@ -261,7 +261,7 @@ def rotary_embedding(positions, q, k, cos_sin_cache, head_dim, is_neox=True):
     rot = cos_sin_cache.shape[-1]
     _check(_rope_and_cache(positions.data_ptr(), q.data_ptr(), _p(k), None, cos_sin_cache.data_ptr(), rot, T, Hq,
                            Hkv, head_dim, q.stride(0), k.stride(0) if k is not None else 0, 0, None, None, 1,
-                           int(is_neox), 0, 1.0, 1.0, _DT[q.dtype], _st()), "rotary_embedding")
+                           int(is_neox), 0, 1.0, 1.0, None, _DT[q.dtype], _st()), "rotary_embedding")
     return q, k
 
 
@@ -271,7 +271,7 @@ def reshape_and_cache(key, value, kv_cache, slot_mapping, k_scale: float = 1.0, 
     key, value = _heads(key), _heads(value)
     _check(_rope_and_cache(None, None, key.data_ptr(), value.data_ptr(), None, 0, T, 0, Hkv, D, 0, key.stride(0),
                            value.stride(0), kv_cache.data_ptr(), slot_mapping.data_ptr(), kv_cache.shape[3], 1,
-                           _kv_fp8(kv_cache) | (2 if vt else 0), k_scale, v_scale, _DT[key.dtype], _st()),
+                           _kv_fp8(kv_cache) | (2 if vt else 0), k_scale, v_scale, None, _DT[key.dtype], _st()),
            "reshape_and_cache")
 
 
@@ -550,7 +550,7 @@ def check_kernel_error(device: torch.device) -> None:
         raise RuntimeError("a kernel gave up waiting for a copy or a matrix product; its outputs are not valid")
 
 
-def mla_decode_splits(B: int, H: int, max_seq_len: int) -> int:
+def mla_decode_splits(B: int, H: int, max_seq_len: int, least: int = 512) -> int:
     if batch_invariant():
         return 1
     forced = envs.VLLM_B200_ATTN_SPLITS
@@ -559,7 +559,7 @@ def mla_decode_splits(B: int, H: int, max_seq_len: int) -> int:
     groups = (H + 31) // 32 if H > 16 else 1
     ctas = max(B * groups, 1)
     s = max(1, min(16, num_sms() // ctas))           # one CTA per SM (170 KB smem): stay inside ONE wave
-    return max(1, min(s, max_seq_len // 512))       # every split should still stream >= 8 tiles
+    return max(1, min(s, max_seq_len // least))     # every split should still stream >= 8 tiles (windows: 4)
 
 
 def mla_decode_tc(q_nope_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_seq_len: int, num_splits: int = 0,
@@ -569,7 +569,8 @@ def mla_decode_tc(q_nope_abs, q_pe, kv_cache, block_table, seq_lens, scale, max_
     P = 0 if q_pe is None else q_pe.shape[-1]
     assert kv_cache.shape[-1] == R + P and q_nope_abs.stride(-1) == 1 and (q_pe is None or q_pe.stride(-1) == 1)
     dev = q_nope_abs.device
-    splits = num_splits or mla_decode_splits(B, H, min(max_seq_len, sliding_window) if sliding_window else max_seq_len)
+    splits = num_splits or (mla_decode_splits(B, H, min(max_seq_len, sliding_window), 256) if sliding_window else
+                            mla_decode_splits(B, H, max_seq_len))
     out = torch.empty((B, H, R), dtype=q_nope_abs.dtype, device=dev)
     lse = torch.empty((B, H), dtype=torch.float32, device=dev) if return_lse else None
     po = pl = None
@@ -1495,6 +1496,11 @@ def fused_qk_norm_rope(positions, q, k, q_weight, k_weight, cos_sin_cache, head_
                                 _p(kv_cache), _p(slot_mapping), BS, int(is_neox), int(gemma), int(vt), eps, _DT[q.dtype], _st()),
                "qknorm_rope_row")
         return q, k
+    if (q_weight is None and k_weight is None and kv_cache is not None and v is not None and (v_head_dim or head_dim) == head_dim == kv_cache.shape[4]
+            and q.dtype in _HALF_DTYPES and head_dim % 16 == 0 and rot % 16 == 0 and kv_cache.dtype == q.dtype
+            and all(t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 for t in (q, k, v))):
+        # nothing to norm: the row kernel
+        return rope_and_cache(positions, q, k, v, cos_sin_cache, head_dim, is_neox, kv_cache, slot_mapping, vt=vt, v_cos_sin=v_cos_sin)
     flags = 4 if keep32 else 0
     BS = 1
     dv = v_head_dim or head_dim
