@@ -19,7 +19,7 @@
 namespace talk {
 
 constexpr int D = 128, BS = 64, TM = 128, TN = 128;
-constexpr int NUM_THREADS = 192;
+constexpr int SOFTMAX_WARPS = 16, NUM_THREADS = 64 + SOFTMAX_WARPS * 32;
 constexpr int K_STAGES = 4, V_STAGES = 3;
 constexpr int Q_BYTES = TM * D * 2;             // 32 KB: 2 k-blocks of [128 rows x 64]
 constexpr int K_BYTES = BS * D * 2;             // 16 KB: this CTA's page of a key tile, 2 k-blocks of [64 tokens x 64]
@@ -30,37 +30,37 @@ struct Params {
   void* out;                    // [T, Hq, nc, D], normalised
   const float* sinks;           // optional [Hq]
   int bt_stride, Hq, Hkv, G, TQ, window, c0, nc;
+  int per_cta;                  // pairs of value heads that a pair of CTAs does one after the other
   Cap cap;
   int* error;
 };
 
-VB_DEVICE void tmem_st_32x32(uint32_t taddr, const uint32_t* r) {
+VB_DEVICE void tmem_st_32x16(uint32_t taddr, const uint32_t (&r)[16]) {
   asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
-      "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};"
+      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
+      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};"
       ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
-        "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]),
-        "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]),
-        "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31]) : "memory");
+        "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]) : "memory");
 }
 VB_DEVICE void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 // ---- pairs of CTAs: one MMA over the rows of both, issued by the leader (rank 0).  Each CTA holds its own rows of A and D, and half of
 // the N rows of B.
-// D[tmem] (+)= A * B; A from shared memory, or from TMEM (row = lane, two 16-bit values per column)
+// D[tmem] (+)= A * B; A from shared memory, or from TMEM (row = lane, two 16-bit values per column).  The whole warp calls these and one
+// lane is elected inside: descriptors stay in uniform registers, an MMA behind a lane test takes a hundred cycles to issue.
 VB_DEVICE void umma2_f16(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-  asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-               "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+  asm volatile("{\n\t.reg .pred p, q;\n\telect.sync _|q, 0xffffffff;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+               "@q tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n\t}"
                ::"r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
 }
 VB_DEVICE void umma2_f16_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-  asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-               "tcgen05.mma.cta_group::2.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+  asm volatile("{\n\t.reg .pred p, q;\n\telect.sync _|q, 0xffffffff;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+               "@q tcgen05.mma.cta_group::2.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
                ::"r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
 }
 // arrives on the barrier at this offset in both CTAs once the MMAs issued before have completed
 VB_DEVICE void umma2_commit(uint64_t* bar) {
-  asm volatile("tcgen05.commit.cta_group::2.mbarrier::arrive::one.shared::cluster.multicast::cluster.b64 [%0], %1;"
+  asm volatile("{\n\t.reg .pred q;\n\telect.sync _|q, 0xffffffff;\n\t"
+               "@q tcgen05.commit.cta_group::2.mbarrier::arrive::one.shared::cluster.multicast::cluster.b64 [%0], %1;\n\t}"
                ::"r"(smem_u32(bar)), "h"((uint16_t)3) : "memory");
 }
 // loads into this CTA's shared memory and counts the bytes on a barrier of the pair (a shared::cluster address)
@@ -80,7 +80,7 @@ VB_DEVICE void tmem2_dealloc(uint32_t taddr, uint32_t ncols) {
   asm volatile("tcgen05.dealloc.cta_group::2.sync.aligned.b32 %0, %1;" ::"r"(taddr), "r"(ncols) : "memory");
 }
 VB_DEVICE void arrive_cluster(uint32_t bar) {
-  asm volatile("mbarrier.arrive.release.cluster.shared::cluster.b64 _, [%0];" ::"r"(bar) : "memory");
+  asm volatile("mbarrier.arrive.shared::cluster.b64 _, [%0];" ::"r"(bar) : "memory");
 }
 VB_DEVICE void wait_cluster_lim(uint64_t* bar, uint32_t parity, int& budget) {      // what threads of the other CTA have arrived on
   for (;;) {
@@ -91,11 +91,13 @@ VB_DEVICE void wait_cluster_lim(uint64_t* bar, uint32_t parity, int& budget) {  
   }
 }
 
-// Pair of CTAs = two query tiles in a row x KV head of the scores x pair of value heads, one request.  Both tiles read the same keys and
-// values; each CTA fetches half of them (a page of the key tile; one value head, or half of a single one).  Warp roles: 0 TMA producer, 1
-// MMA issuer (leader) + TMEM owner, 2..5 softmax / epilogue (thread = query row = TMEM lane).  TMEM: S double-buffered (2 x 128
-// columns), two accumulators (2 x 128).  P overwrites the S it came from (bf16, 64 columns) and is the PV product's A operand there, so
-// it is double-buffered too: the softmax of tile j runs under the PV products of tile j - 1.
+// Pair of CTAs = two query tiles in a row x KV head of the scores x some pairs of value heads (one after the other), one request.  Both
+// tiles read the same keys and values; each CTA fetches half of them (a page of the key tile; one value head, or half of a single one).
+// Warp roles: 0 TMA producer, 1 MMA issuer (leader) + TMEM owner, 2..17 softmax / epilogue (thread = query row = TMEM lane, a quarter of
+// the columns: four warps per scheduler, since one alone waits for its own results most of the time).  TMEM: S double-buffered (2 x 128
+// columns), two accumulators (2 x 128).  P overwrites the S it came from (bf16, 16 of each 32 columns) and is the PV product's A operand
+// there, so it is double-buffered too: the softmax of tile n runs under the PV products of tile n - 1.  Tiles are numbered through over
+// the pairs of value heads: the first scores of the next pair are computed while the last results of this one are stored.
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                  const __grid_constant__ CUtensorMap tmap_v, const Params p) {
@@ -113,14 +115,18 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
   uint64_t* v_empty = v_full + V_STAGES;
   uint64_t* s_full = v_empty + V_STAGES;       // [2]
   uint64_t* p_full = s_full + 2;               // [2] (leader's: the warps of both CTAs)
-  uint64_t* pv_done = p_full + 2;              // [2]
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 2);
+  uint64_t* o_full = p_full + 2;
+  uint64_t* o_empty = o_full + 1;              // (leader's: the warps of both CTAs)
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_empty + 1);
+  float* sums = reinterpret_cast<float*>(tmem_slot + 2);        // 2 x [4][128] sums of the column quarters
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int budget = MBAR_BUDGET;
   const int rank = (int)cluster_ctarank(), b = blockIdx.z, groups = (p.nc + 1) / 2;
-  const int h = blockIdx.y / groups, cv = blockIdx.y % groups * 2;       // KV head of the scores, first value head (behind c0)
-  const int nv = min(2, p.nc - cv), v_rows = nv * 64;                    // rows of a value tile's B operand in this CTA
+  const int parts = (groups + p.per_cta - 1) / p.per_cta;
+  const int h = blockIdx.y / parts, g0 = blockIdx.y % parts * p.per_cta; // KV head of the scores, first pair of value heads
+  const int ng = min(p.per_cta, groups - g0);
+  auto heads_of = [&](int ci) { return min(2, p.nc - (g0 + ci) * 2); };  // value heads of pair ci: two, or one at the end
   pdl_trigger();
   pdl_wait();
   const int q0 = p.qsl[b], q_len = p.qsl[b + 1] - q0;
@@ -137,7 +143,9 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     mbar_init(q_full, 1);
     for (int s = 0; s < K_STAGES; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
     for (int s = 0; s < V_STAGES; ++s) { mbar_init(&v_full[s], 1); mbar_init(&v_empty[s], 1); }
-    for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&p_full[s], 8); mbar_init(&pv_done[s], 1); }
+    for (int s = 0; s < 2; ++s) { mbar_init(&s_full[s], 1); mbar_init(&p_full[s], 2 * SOFTMAX_WARPS); }
+    mbar_init(o_full, 1);
+    mbar_init(o_empty, 2 * SOFTMAX_WARPS);
     mbar_fence_init();
   }
   if (warp == 1) tmem2_alloc(tmem_slot, 512);
@@ -156,20 +164,22 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
       tma2_load_3d(q_smem, &tmap_q, 0, h * p.G, q0 + tok0, bar_q);
       tma2_load_3d(q_smem + TM * 128, &tmap_q, 64, h * p.G, q0 + tok0, bar_q);
       const int* bt = p.block_table + (int64_t)b * p.bt_stride;
-      for (int j = 0; j < n_tiles && budget >= 0; ++j) {
+      const int total = ng * n_tiles;
+      for (int n = 0, j = 0, ci = 0; n < total; ++n) {
+        const int cv = (g0 + ci) * 2, nv = heads_of(ci), v_rows = nv * 64;      // rows of a value tile's B operand in this CTA
         int blk[2];
         for (int u = 0; u < 2; ++u) {
           const int page = (tile_lo + j) * 2 + u;
           blk[u] = page < n_pages ? bt[page] : 0;
         }
-        const int s = j % K_STAGES, vs = j % V_STAGES;
-        mbar_wait_lim(&k_empty[s], ((j / K_STAGES) & 1) ^ 1, budget);
+        const int s = n % K_STAGES, vs = n % V_STAGES;
+        mbar_wait_lim(&k_empty[s], ((n / K_STAGES) & 1) ^ 1, budget);
         if (budget < 0) break;
         const uint32_t bar_k = dsmem_addr(smem_u32(&k_full[s]), 0);
         if (rank == 0) mbar_expect_tx(&k_full[s], 2 * K_BYTES);
         for (int kb = 0; kb < 2; ++kb)
           tma2_load_2d(k_smem + s * K_BYTES + kb * (BS * 128), &tmap_k, kb * 64, ((rank ? blk[1] : blk[0]) * 2 * p.Hkv + h) * BS, bar_k);
-        mbar_wait_lim(&v_empty[vs], ((j / V_STAGES) & 1) ^ 1, budget);
+        mbar_wait_lim(&v_empty[vs], ((n / V_STAGES) & 1) ^ 1, budget);
         if (budget < 0) break;
         const uint32_t bar_v = dsmem_addr(smem_u32(&v_full[vs]), 0);
         if (rank == 0) mbar_expect_tx(&v_full[vs], 2 * 2 * v_rows * 128);
@@ -178,6 +188,7 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
           const int row = ((blk[u] * 2 + 1) * p.Hkv + p.c0 + cv + (nv == 2 ? rank : 0)) * D + (nv == 2 ? 0 : rank * 64);
           for (int r = 0; r < v_rows; r += 64) tma2_load_2d(v_smem + vs * V_BYTES + (u * v_rows + r) * 128, &tmap_v, 0, row + r, bar_v);
         }
+        if (++j == n_tiles) { j = 0; ++ci; }
       }
       if (budget < 0 && rank == 0) {            // let the copies in flight land before the pair gives up its memory
         for (int s = 0; s < K_STAGES; ++s)
@@ -188,121 +199,139 @@ talk_fold_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     }
   } else if (warp == 1) {
     if (rank == 0) {
-      // ===== MMA issuer
-      const uint32_t idesc_s = umma_idesc_f16(2 * TM, TN, true), idesc_o = umma_idesc_f16(2 * TM, nv * 128, true);
+      // ===== MMA issuer.  MMAs of one thread execute in order, so QK of tile j may follow PV of tile j - 2, whose P it overwrites, at once:
+      // the tensor cores always have the next product queued while this thread waits
+      const uint32_t idesc_s = umma_idesc_f16(2 * TM, TN, true);
       const uint64_t d_q = umma_desc_sw128(q_smem), d_k = umma_desc_sw128(k_smem), d_v = umma_desc_sw128(v_smem);
       mbar_wait_lim(q_full, 0, budget);
-      __syncwarp();
-      for (int j = 0; j <= n_tiles; ++j) {
-        if (j < n_tiles) {
-          const int s = j % K_STAGES;
-          mbar_wait_lim(&k_full[s], (j / K_STAGES) & 1, budget);
-          if (j >= 2) mbar_wait_lim(&pv_done[j & 1], ((j >> 1) & 1) ^ 1, budget);    // PV of tile j - 2 has read the P in this buffer
-          tc_fence_after();
-          if (lane == 0) {
-#pragma unroll
-            for (int kb = 0; kb < 2; ++kb)
-#pragma unroll
-              for (int k = 0; k < 4; ++k)
-                umma2_f16(tmem_base + (j & 1) * 128, d_q + (uint64_t)(((kb * TM * 128) >> 4) + k * 2),
-                          d_k + (uint64_t)(((s * K_BYTES + kb * BS * 128) >> 4) + k * 2), idesc_s, (kb | k) != 0);
-            umma2_commit(&s_full[j & 1]);
-            umma2_commit(&k_empty[s]);
-          }
+      const int nt = __shfl_sync(0xffffffffu, n_tiles, 0), total = ng * nt;        // (uniform)
+      for (int n = 0, jj = 0, ci = 0; n <= total; ++n) {
+        if (n < total) {
+          const int s = n % K_STAGES;
+          mbar_wait_lim(&k_full[s], (n / K_STAGES) & 1, budget);
           __syncwarp();
+          tc_fence_after();
+#pragma unroll
+          for (int kb = 0; kb < 2; ++kb)
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+              umma2_f16(tmem_base + (n & 1) * 128, d_q + (uint64_t)(((kb * TM * 128) >> 4) + k * 2),
+                        d_k + (uint64_t)(((s * K_BYTES + kb * BS * 128) >> 4) + k * 2), idesc_s, (kb | k) != 0);
+          umma2_commit(&s_full[n & 1]);
+          umma2_commit(&k_empty[s]);
         }
-        if (j > 0) {
-          const int jj = j - 1, vs = jj % V_STAGES;
-          mbar_wait_lim(&v_full[vs], (jj / V_STAGES) & 1, budget);
-          wait_cluster_lim(&p_full[jj & 1], (jj >> 1) & 1, budget);
-          tc_fence_after();
-          if (lane == 0) {
-#pragma unroll
-            for (int kk = 0; kk < 8; ++kk)
-              umma2_f16_ta(tmem_o, tmem_base + (jj & 1) * 128 + kk * 8,
-                           d_v + (uint64_t)((vs * V_BYTES + (kk / 4) * v_rows * 128) >> 4) + (uint64_t)((kk & 3) * 2), idesc_o, (jj | kk) != 0);
-            umma2_commit(&v_empty[vs]);
-            umma2_commit(&pv_done[jj & 1]);
-          }
+        if (n > 0) {
+          const int m = n - 1, vs = m % V_STAGES, nv = heads_of(ci);     // tile jj of pair ci
+          const uint32_t idesc_o = umma_idesc_f16(2 * TM, nv * 128, true);
+          if (jj == 0 && ci > 0) wait_cluster_lim(o_empty, (ci - 1) & 1, budget);
+          mbar_wait_lim(&v_full[vs], (m / V_STAGES) & 1, budget);
+          wait_cluster_lim(&p_full[m & 1], (m >> 1) & 1, budget);
           __syncwarp();
+          tc_fence_after();
+#pragma unroll
+          for (int kk = 0; kk < 8; ++kk)
+            umma2_f16_ta(tmem_o, tmem_base + (m & 1) * 128 + (kk / 2) * 32 + (kk & 1) * 8,
+                         d_v + (uint64_t)((vs * V_BYTES + (kk / 4) * nv * 64 * 128) >> 4) + (uint64_t)((kk & 3) * 2), idesc_o, (jj | kk) != 0);
+          umma2_commit(&v_empty[vs]);
+          if (++jj == nt) { umma2_commit(o_full); jj = 0; ++ci; }
         }
       }
     }
   } else {
     // ===== softmax / epilogue
-    const int qd = warp & 3, r = qd * 32 + lane;
+    const int qd = warp & 3, r = qd * 32 + lane, quarter = (warp - 2) >> 2, c0 = quarter * 32;
     const uint32_t t_lane = (uint32_t)(qd * 32) << 16;
-    const uint32_t bar_p = dsmem_addr(smem_u32(p_full), 0);
-    const int tq = r / p.G, g = r % p.G;
+    const uint32_t bar_p = dsmem_addr(smem_u32(p_full), 0), bar_o = dsmem_addr(smem_u32(o_empty), 0);
+    const int tq = r / p.G, g = r % p.G, hq = h * p.G + g;
     const bool row_valid = tq < n_tok;
     const int qpos = pos0 + tq;
-    float l_run = 0.f;
-    for (int j = 0; j < n_tiles; ++j) {
-      const uint32_t t_s = tmem_base + (j & 1) * 128 + t_lane;
-      mbar_wait_lim(&s_full[j & 1], (j >> 1) & 1, budget);
+    const float sink = p.sinks && row_valid ? ex2(p.sinks[hq] * 1.4426950408889634f) : 0.f;
+    int n = 0;
+    for (int ci = 0; ci < ng; ++ci) {
+      float l_run = 0.f;
+      for (int j = 0; j < n_tiles; ++j, ++n) {
+        const uint32_t t_s = tmem_base + (n & 1) * 128 + c0 + t_lane;
+        const int first = (tile_lo + j) * TN + c0;
+        const int hi = row_valid ? qpos + 1 - first : 0;                 // keys [lo, hi) of these 32 are visible to the row
+        const int lo = p.window > 0 ? hi - p.window : 0;
+        const bool full = __all_sync(0xffffffffu, hi >= 32 && lo <= 0) != 0;
+        const bool none = __all_sync(0xffffffffu, hi <= 0 || lo >= 32) != 0;
+        mbar_wait_lim(&s_full[n & 1], (n >> 1) & 1, budget);
+        __syncwarp();
+        tc_fence_after();
+        uint32_t pk[16];
+        if (none) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) pk[i] = 0u;
+        } else {
+          uint32_t v[32];
+          tmem_ld_32x32(t_s, v);
+          tmem_ld_wait();
+          float s[32];
+#pragma unroll
+          for (int i = 0; i < 32; ++i) s[i] = __uint_as_float(v[i]);
+          cap_exp<32>(s, p.cap);
+          if (!full) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (i >= hi || i < lo) s[i] = 0.f;
+          }
+          uint64_t l[2] = {0ull, 0ull};
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) {
+            l[(i >> 1) & 1] = add2(l[(i >> 1) & 1], pair2(s[i], s[i + 1]));
+            pk[i / 2] = pack2<T>(s[i], s[i + 1]);
+          }
+          const float2 lt = split2(add2(l[0], l[1]));
+          l_run += lt.x + lt.y;
+        }
+        tmem_st_32x16(t_s, pk);
+        tmem_st_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) arrive_cluster(bar_p + (n & 1) * 8);
+      }
+      // ---- epilogue of a pair of value heads
+      float* sm = sums + (ci & 1) * 512;
+      sm[quarter * 128 + r] = l_run;
+      asm volatile("bar.sync 1, 512;" ::: "memory");
+      const float den = (sm[r] + sm[128 + r]) + (sm[256 + r] + sm[384 + r]) + sink;
+      const float inv = row_valid && den > 0.f ? 1.f / den : 0.f;
+      mbar_wait_lim(o_full, ci & 1, budget);
       __syncwarp();
       tc_fence_after();
-      const int hi = row_valid ? qpos + 1 - (tile_lo + j) * TN : 0;      // keys [lo, hi) of this tile are visible to the row
-      const int lo = p.window > 0 ? hi - p.window : 0;
-      const bool full = __all_sync(0xffffffffu, hi >= TN && lo <= 0) != 0;
-      uint32_t v[4][32], pk[64];
+      // two value heads: half of each per quarter of the warps; one: a quarter of it
+      const int cv = (g0 + ci) * 2;
+      T* orow = reinterpret_cast<T*>(p.out) + (((int64_t)(q0 + tok0 + tq) * p.Hq + hq) * p.nc + cv) * D;
+      auto store = [&](const uint32_t (&o)[32], int at) {               // 32 columns of the row, whole sectors
+        if (!row_valid) return;
 #pragma unroll
-      for (int c = 0; c < 4; ++c) tmem_ld_32x32(t_s + c * 32, v[c]);
-      tmem_ld_wait();
+        for (int i = 0; i < 32; i += 16) {
+          uint32_t w[8];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        float s[32];
-#pragma unroll
-        for (int i = 0; i < 32; ++i) s[i] = __uint_as_float(v[c][i]);
-        cap_exp<32>(s, p.cap);
-        if (!full) {
-#pragma unroll
-          for (int i = 0; i < 32; ++i)
-            if (c * 32 + i >= hi || c * 32 + i < lo) s[i] = 0.f;
+          for (int e = 0; e < 8; ++e) w[e] = pack2<T>(__uint_as_float(o[i + 2 * e]) * inv, __uint_as_float(o[i + 2 * e + 1]) * inv);
+          asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(orow + at + i), "r"(w[0]), "r"(w[1]), "r"(w[2]), "r"(w[3]),
+                       "r"(w[4]), "r"(w[5]), "r"(w[6]), "r"(w[7]) : "memory");
         }
-        float l[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll
-        for (int i = 0; i < 32; i += 2) {
-          l[i & 2] += s[i];
-          l[(i & 2) + 1] += s[i + 1];
-          pk[c * 16 + i / 2] = pack2<T>(s[i], s[i + 1]);
-        }
-        l_run += (l[0] + l[1]) + (l[2] + l[3]);
-      }
-      tmem_st_32x32(t_s, pk);
-      tmem_st_32x32(t_s + 32, pk + 32);
-      tmem_st_wait();
-      tc_fence_before();
-      __syncwarp();
-      if (lane == 0) arrive_cluster(bar_p + (j & 1) * 8);
-    }
-    mbar_wait_lim(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1, budget);
-    __syncwarp();
-    tc_fence_after();
-    const int hq = h * p.G + g;
-    float inv = 0.f;
-    if (row_valid) {
-      const float den = l_run + (p.sinks ? ex2(p.sinks[hq] * 1.4426950408889634f) : 0.f);
-      inv = den > 0.f ? 1.f / den : 0.f;
-    }
-    for (int u = 0; u < nv; ++u) {
-      T* orow = reinterpret_cast<T*>(p.out) + (((int64_t)(q0 + tok0 + tq) * p.Hq + hq) * p.nc + cv + u) * D;
-#pragma unroll
-      for (int c = 0; c < D; c += 32) {
-        uint32_t o[32];
-        tmem_ld_32x32(tmem_o + u * 128 + t_lane + c, o);
+      };
+      auto release = [&]() {                                            // the accumulators are in registers
         tmem_ld_wait();
-        if (row_valid) {
-#pragma unroll
-          for (int i = 0; i < 32; i += 8) {
-            uint4 w;
-            w.x = pack2<T>(__uint_as_float(o[i]) * inv, __uint_as_float(o[i + 1]) * inv);
-            w.y = pack2<T>(__uint_as_float(o[i + 2]) * inv, __uint_as_float(o[i + 3]) * inv);
-            w.z = pack2<T>(__uint_as_float(o[i + 4]) * inv, __uint_as_float(o[i + 5]) * inv);
-            w.w = pack2<T>(__uint_as_float(o[i + 6]) * inv, __uint_as_float(o[i + 7]) * inv);
-            *reinterpret_cast<uint4*>(orow + c + i) = w;
-          }
-        }
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) arrive_cluster(bar_o);
+      };
+      uint32_t o0[32];
+      if (heads_of(ci) == 2) {
+        uint32_t o1[32];
+        tmem_ld_32x32(tmem_o + quarter * 64 + t_lane, o0);
+        tmem_ld_32x32(tmem_o + quarter * 64 + 32 + t_lane, o1);
+        release();
+        store(o0, quarter * 64);
+        store(o1, quarter * 64 + 32);
+      } else {
+        tmem_ld_32x32(tmem_o + quarter * 32 + t_lane, o0);
+        release();
+        store(o0, quarter * 32);
       }
     }
     tc_fence_before();
@@ -454,14 +483,20 @@ EXPORT int vb_talk_fold(const void* q, const void* kv_cache, int64_t num_blocks,
   CUtensorMap tq, tk, tv;
   int rc;
   if ((rc = map_queries(&tq, q, Hq, T_total, q_stride, G, p.TQ))) return rc;
-  if ((rc = map_pages(&tk, &tv, kv_cache, num_blocks, Hkv, 64))) return rc;
-  const int smem = Q_BYTES + K_STAGES * K_BYTES + V_STAGES * V_BYTES + 32 * 8 + 16 + 1024;
+  if ((rc = map_pages(&tk, &tv, kv_cache, num_blocks, Hkv, BS, 64))) return rc;
+  const int smem = Q_BYTES + K_STAGES * K_BYTES + V_STAGES * V_BYTES + 32 * 8 + 16 + 4096 + 1024;
   static bool a = false;
   if (!a) { cudaFuncSetAttribute(talk_fold_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); a = true; }
-  const int pairs = (max_q_len + 2 * p.TQ - 1) / (2 * p.TQ);
+  const int pairs = (max_q_len + 2 * p.TQ - 1) / (2 * p.TQ), groups = (nc + 1) / 2;
+  static int n_sms = 0;
+  if (!n_sms) { int dv = 0; cudaGetDevice(&dv); cudaDeviceGetAttribute(&n_sms, cudaDevAttrMultiProcessorCount, dv); }
+  // all pairs of value heads in one CTA where that still makes a few waves
+  const int64_t ctas = (int64_t)2 * pairs * Hkv * B;
+  p.per_cta = groups;
+  while (p.per_cta > 1 && ctas * ((groups + p.per_cta - 1) / p.per_cta) < 4 * n_sms) p.per_cta = (p.per_cta + 1) / 2;
   if (B > 65535) return -6;
   cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(2 * pairs, Hkv * ((nc + 1) / 2), B); cfg.blockDim = dim3(NUM_THREADS); cfg.dynamicSmemBytes = (size_t)smem; cfg.stream = st;
+  cfg.gridDim = dim3(2 * pairs, Hkv * ((groups + p.per_cta - 1) / p.per_cta), B); cfg.blockDim = dim3(NUM_THREADS); cfg.dynamicSmemBytes = (size_t)smem; cfg.stream = st;
   cudaLaunchAttribute attr[2];
   attr[0].id = cudaLaunchAttributeClusterDimension;
   attr[0].val.clusterDim.x = 2; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;      // the pair is two neighbours along x

@@ -294,7 +294,7 @@ EXPORT int vb_talk_decode(const void* q, const void* kv_cache, int64_t num_block
   CUtensorMap tq, tk, tv;
   int rc;
   if ((rc = talk::map_queries(&tq, q, H, B, q_stride, GH, 1))) return rc;
-  if ((rc = talk::map_pages(&tk, &tv, kv_cache, num_blocks, Hkv, D))) return rc;
+  if ((rc = talk::map_pages(&tk, &tv, kv_cache, num_blocks, Hkv, BS, D))) return rc;
 #define GO(N) return H <= 16 ? launch<N, 16>(tq, tk, tv, p, st) : launch<N, 32>(tq, tk, tv, p, st)
   switch (GH) {
     case 1: return H <= 16 ? launch<1, 16>(tq, tk, tv, p, st) : -4;

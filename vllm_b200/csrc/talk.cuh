@@ -21,18 +21,37 @@ inline Cap make_cap(float scale, float cap) {
 }
 VB_DEVICE float rcp(float x) { float y; asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
 
+// pairs of floats: one instruction per pair
+VB_DEVICE uint64_t pair2(float a, float b) { uint64_t r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b)); return r; }
+VB_DEVICE float2 split2(uint64_t v) { float2 r; asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v)); return r; }
+VB_DEVICE uint64_t add2(uint64_t a, uint64_t b) { uint64_t r; asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+VB_DEVICE uint64_t mul2(uint64_t a, uint64_t b) { uint64_t r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+VB_DEVICE uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r;
+}
+
+VB_DEVICE float max3(float a, float b, float c) { float r; asm("max.f32 %0, %1, %2, %3;" : "=f"(r) : "f"(a), "f"(b), "f"(c)); return r; }
+
 // In place, for N scores of a thread; the whole warp takes part.  Where all scores of the warp are below a quarter of the cap the Taylor
 // series of tanh to the seventh power is exact to 3e-7 and needs no more special functions than a plain softmax.
 template <int N> VB_DEVICE void cap_exp(float (&s)[N], const Cap& c) {
-  float m4[4] = {0.f, 0.f, 0.f, 0.f};
+  uint64_t x[N / 2], q[N / 2];
+  float m4[4] = {0.f, 0.f, 0.f, 0.f};                      // (squares: no signs)
 #pragma unroll
-  for (int i = 0; i < N; ++i) m4[i & 3] = fmaxf(m4[i & 3], fabsf(s[i]));
+  for (int i = 0; i < N / 2; ++i) {
+    x[i] = pair2(s[2 * i], s[2 * i + 1]);
+    q[i] = mul2(x[i], x[i]);
+    const float2 f = split2(q[i]);
+    m4[i & 3] = max3(m4[i & 3], f.x, f.y);
+  }
   const float m = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
-  if (__all_sync(0xffffffffu, m * c.ku < 0.25f)) {
+  if (__all_sync(0xffffffffu, m * c.ku * c.ku < 0.0625f)) {
+    const uint64_t k0 = pair2(c.k0, c.k0), k1 = pair2(c.k1, c.k1), k2 = pair2(c.k2, c.k2), k3 = pair2(c.k3, c.k3);
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-      const float q = s[i] * s[i];
-      s[i] = ex2(s[i] * fmaf(q, fmaf(q, fmaf(q, c.k3, c.k2), c.k1), c.k0));
+    for (int i = 0; i < N / 2; ++i) {
+      const float2 f = split2(mul2(x[i], fma2(q[i], fma2(q[i], fma2(q[i], k3, k2), k1), k0)));
+      s[2 * i] = ex2(f.x);
+      s[2 * i + 1] = ex2(f.y);
     }
   } else {
 #pragma unroll
@@ -66,11 +85,11 @@ inline int map_queries(CUtensorMap* m, const void* q, int Hq, int T, int64_t str
   const cuuint32_t box[3] = {64, (cuuint32_t)G, (cuuint32_t)TQ};
   return encode(m, q, 3, dims, strides, box);
 }
-// key pages as rows of 128 dims (box 64 x 64 tokens), value pages as rows of 64 tokens (box 64 x v_rows dims)
-inline int map_pages(CUtensorMap* k, CUtensorMap* v, const void* cache, int64_t blocks, int Hkv, int v_rows) {
+// key pages as rows of 128 dims (box 64 x k_rows tokens), value pages as rows of 64 tokens (box 64 x v_rows dims)
+inline int map_pages(CUtensorMap* k, CUtensorMap* v, const void* cache, int64_t blocks, int Hkv, int k_rows, int v_rows) {
   const cuuint64_t kd[2] = {128, (cuuint64_t)blocks * 2 * Hkv * 64}, ks[1] = {256};
   const cuuint64_t vd[2] = {64, (cuuint64_t)blocks * 2 * Hkv * 128}, vs[1] = {128};
-  const cuuint32_t kb[2] = {64, 64}, vb[2] = {64, (cuuint32_t)v_rows};
+  const cuuint32_t kb[2] = {64, (cuuint32_t)k_rows}, vb[2] = {64, (cuuint32_t)v_rows};
   int rc = encode(k, cache, 2, kd, ks, kb);
   return rc ? rc : encode(v, cache, 2, vd, vs, vb);
 }
