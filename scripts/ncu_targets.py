@@ -120,3 +120,31 @@ if which in ("memory", "all"):
         rows, inv = moe.expert_rows_gated(x, w13, w2, ids, "silu", emap)
         cu.add_norm(stream, x, (nw, None), 1e-6, dt, rows, inv, pw, ids, 48, x)
     rep(experts)
+if which in ("talk", "all"):
+    # Gizilorn: attention with mixed heads (prompts, a decode batch), streams, latent attention with a rotated part and a window, at the
+    # sizes of a 2048-wide model
+    from vllm_b200.benchmarks.latent_layers import _pages
+    from vllm_b200.forward_context import AttentionMetadata
+    H, G, D, W, i32 = 16, 4, 128, 2048, dict(dtype=torch.int32, device="cuda")
+    talk, sinks = torch.randn(H, H, device="cuda") * 0.2, torch.zeros(H, device="cuda")
+    for n, q, seq, window in ((2, 4096, 4096, 2048), (64, 1, 4096, 4096)):
+        per = seq // 64
+        kv = (torch.randn(n * per + 1, 2, G, 64, D, device="cuda") * 0.3).to(dt)
+        md = AttentionMetadata(num_reqs=n, num_actual_tokens=n * q, max_query_len=q, max_seq_len=seq,
+                               query_start_loc=torch.arange(0, n * q + 1, q, **i32), seq_lens=torch.full((n,), seq, **i32),
+                               block_table=(torch.randperm(n * per, device="cuda").int() + 1).view(n, per), slot_mapping=None, kv_vt=True,
+                               decode_only=q == 1)
+        x = torch.randn(n * q, H, D, device="cuda").to(dt)
+        rep(lambda: cu.talking_attention(x, kv, md, D ** -0.5, window, 50.0, talk, sinks, D))
+        del kv
+    xs, y, w = torch.randn(8192, 4, W, device="cuda"), torch.randn(8192, W, device="cuda").to(dt), torch.ones(W, device="cuda", dtype=dt)
+    coef, into = torch.randn(20, device="cuda") * 0.3, torch.ones(4, device="cuda")
+    rep(lambda: cu.hyper_step(xs, y, coef, into, w, 1e-6, dt))
+    cache, bt, sl = _pages(64, 4096, 576)
+    qn, qp = (torch.randn(64, H, m, device="cuda") * 0.3 for m in (512, 64))
+    qn, qp = qn.to(dt), qp.to(dt)
+    rep(lambda: cu.mla_decode_tc(qn, qp, cache, bt, sl, 0.07, 4096, sliding_window=2048))
+    q, k, v = ((torch.randn(8192, H, m, device="cuda") * 0.3).to(dt) for m in (192, 128, 128))
+    lat, out = (torch.randn(8192, 576, device="cuda") * 0.3).to(dt), torch.empty(8192, H, 128, device="cuda", dtype=dt)
+    start, lens = torch.arange(0, 8192, 4096, **i32), torch.full((2,), 4096, **i32)
+    rep(lambda: cu.mla_prefill(q, k, v, out, start, lens, lens, start, 0, 4096, 0.07, lat[:, 512:], 2048))

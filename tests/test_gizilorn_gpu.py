@@ -103,6 +103,19 @@ def test_xielu(T, n, dtype):
     _close(got, want, 6e-3 if dtype != F32 else 1e-6)
 
 
+def test_apertus_runs_the_same_activation():
+    from vllm_b200.models.llama_variants import _XIELU
+    act = _XIELU(F32)
+    act.alpha_p.data.fill_(0.4)
+    act.alpha_n.data.fill_(-0.9)
+    x = _rand(7, 300, seed=1, size=3.0)
+    want = act(x)                                              # its plain operations, on the CPU
+    _close(act.cuda()(x.cuda()), want, 1e-6)
+    act.beta.data.fill_(0.25)
+    act.half = None
+    _close(act(x.cuda()), act.cpu()(x), 1e-6)
+
+
 @pytest.mark.parametrize("dtype", [BF, F16, F32])
 @pytest.mark.parametrize("M,N,K", [(1, 320, 192), (7, 4096, 1024), (64, 1000, 2048), (200, 512, 4096), (256, 22, 64), (300, 640, 256), (5, 36, 40)])
 def test_projection_with_xielu(M, N, K, dtype):

@@ -19,6 +19,7 @@ from typing import Iterable, Optional
 import torch
 import torch.nn as nn
 
+from vllm_b200 import ops
 from vllm_b200.config import VllmConfig
 from vllm_b200.layers.attention import Attention
 from vllm_b200.layers.common import Activation, LayerNorm, LogitsProcessor, ParallelLMHead, RMSNorm
@@ -87,9 +88,16 @@ class _XIELU(nn.Module):
         self.beta = nn.Parameter(torch.full((), 0.5, dtype=dtype), requires_grad=False)
         self.eps = nn.Parameter(torch.full((), -1e-6, dtype=dtype), requires_grad=False)
 
+        self.half: Optional[bool] = None             # is β a half, as the kernel has it?
+
     def forward(self, x):
         ap = torch.nn.functional.softplus(self.alpha_p)
         an = self.beta + torch.nn.functional.softplus(self.alpha_n)
+        if x.is_cuda:
+            if self.half is None:
+                self.half = float(self.beta) == 0.5
+            if self.half:                            # (ε only keeps expm1 away from zero, where it is exact)
+                return ops.xielu(x, torch.cat([ap, an]).float())
         return torch.where(x > 0, ap * x * x + self.beta * x, (torch.expm1(torch.min(x, self.eps)) - x) * an + self.beta * x)
 
 
