@@ -329,25 +329,26 @@ hyper_kernel(const int* __restrict__ ids, int vocab, const T* __restrict__ y, in
       for (int j = 0; j < V; ++j) u[n][j] *= total;
     }
   } else {
-#pragma unroll
+    constexpr int UN = EXACT ? NV : 1, US = EXACT ? SM : 1;              // many streams: loops, not eight thousand instructions
+#pragma unroll UN
     for (int n = 0; n < NV; ++n) {
       const int i = threadIdx.x * V + n * stride;
       if (i >= H) continue;
       float xs[SM][V], yv[V];
-#pragma unroll
+#pragma unroll US
       for (int s = 0; s < SM; ++s)
         if (EXACT || s < S) load_f32<float, V>(xr + (int64_t)s * H + i, xs[s]);
       if (step) load_f32<T, V>(y + row * y_stride + i, yv);
 #pragma unroll
       for (int j = 0; j < V; ++j) u[n][j] = 0.f;
-#pragma unroll
+#pragma unroll US
       for (int t = 0; t < SM; ++t) {
         if (!EXACT && t >= S) break;
         float v[V];
         if (step) {
 #pragma unroll
           for (int j = 0; j < V; ++j) v[j] = out_[t] * yv[j];
-#pragma unroll
+#pragma unroll US
           for (int s = 0; s < SM; ++s)
             if (EXACT || s < S) {
               const float m = mix[s * S + t];
